@@ -1,0 +1,90 @@
+/* nqb200_mixers -- C ABI of the sequence-mixing kernels (sm_100a): input convolution fused with RMS norm,
+ * partial rotary embedding with a paged K/V store, chunk-masked attention with a score cap and a sink,
+ * retention, minGRU, clamped GLU, and the skinny dense linears of decode steps with these steps inside.
+ *
+ * Conventions as in nqb200.h: plain device pointers, asynchronous on `stream`, status codes, nothing here
+ * allocates.  `dtype` is the type of activations, weights and K/V caches: NQB200_BF16, or NQB200_F32 where
+ * everything is computed and kept in 32 bits.  The residual stream, norm and convolution weights, gate biases
+ * and recurrent states are always float.
+ *
+ * Tokens of a step are flattened; sequence b owns tokens cu[b] .. cu[b+1]-1, the first of which stands at
+ * position pos0[b] of its sequence.  pos0[b] == 0 means that the sequence starts here: whatever its state slot
+ * holds is taken as zero.  K/V of position p live in row (table[b * table_width + p / block_size] * block_size
+ * + p % block_size) of the caches. */
+#ifndef NQB200_MIXERS_H
+#define NQB200_MIXERS_H
+
+#include "nqb200.h"
+
+#ifdef __cplusplus
+extern "C" {
+#endif
+
+enum { NQB200_F32 = 2 };
+
+typedef struct {
+  const int32_t* cu;      /* [batch + 1] */
+  const int32_t* pos0;    /* [batch] */
+  const int32_t* slot;    /* [batch] row of the recurrent-state pools */
+  const int32_t* table;   /* [batch, table_width] K/V blocks */
+  int32_t batch, tokens, max_len, table_width, block_size;
+} nqb200_batch;
+
+/* x[t] = (accumulate ? x[t] : 0) + embed[ids[t]] + step.  ids or step may be NULL (that term is left out).
+ * x float [tokens, width], embed [vocab, width] of `dtype`, step float [width]. */
+int nqb200_stream_add(float* x, const int64_t* ids, const void* embed, const float* step, int accumulate,
+                      int64_t tokens, int64_t width, int dtype, void* stream);
+
+/* out[r] = RMSnorm(x[rows ? rows[r] : r]) * weight, rounded to dtype. */
+int nqb200_rmsnorm_rows(const float* x, const int64_t* rows, const float* weight, void* out, int64_t n_rows,
+                        int64_t width, float eps, int dtype, void* stream);
+
+/* h = RMSnorm(x) * weight; out[t, c] = h[t, c] + sum_j conv[c * taps + j] h[t - taps + 1 + j, c], rounded to
+ * dtype.  state float [slots, taps - 1, width] holds each sequence's last taps - 1 rows of h and is updated. */
+int nqb200_rmsnorm_conv(const float* x, const float* weight, const float* conv, float* state, void* out,
+                        const nqb200_batch* b, int64_t width, int64_t taps, float eps, int dtype, void* stream);
+
+/* proj [tokens, stride] of dtype holds q (heads x dim at column q_off), k (kv_heads x dim at k_off) and v
+ * (kv_heads x vdim at v_off).  q and k are rotated (pairs i, i + rot/2 of the first rot dimensions, angle
+ * position * inv_freq[i]); q in place, k and v go to the caches [rows, kv_heads, dim | vdim]. */
+int nqb200_rope_store(void* proj, void* k_cache, void* v_cache, const float* inv_freq, const nqb200_batch* b,
+                      int64_t stride, int64_t q_off, int64_t k_off, int64_t v_off, int64_t heads, int64_t kv_heads,
+                      int64_t dim, int64_t vdim, int64_t rot, int dtype, void* stream);
+
+typedef struct {
+  int32_t heads, kv_heads, dim, vdim;
+  int32_t chunk;          /* a query sees keys j <= i with j / chunk == i / chunk; <= 0: no chunks */
+  float scale, softcap;   /* softcap <= 0: none */
+  const float* sink;      /* [heads] or NULL */
+  float out_scale;
+} nqb200_attention;
+
+/* Attention of rotated q (rows of `q`, row stride q_stride, head h at column h * dim) over the paged caches.
+ * out[t * out_stride + h * vdim + c] = out_scale * o, rounded to dtype. */
+int nqb200_chunk_attention(const void* q, int64_t q_stride, const void* k_cache, const void* v_cache, void* out,
+                           int64_t out_stride, const nqb200_attention* a, const nqb200_batch* b, int dtype, void* stream);
+
+/* Retention.  proj holds q and k (heads x dim at q_off, k_off) and v (heads x vdim at v_off).
+ * S <- decay[h] S + (dim^-1/2 k) v^T, o = S^T q, state float [slots, heads, dim, vdim].  o float [tokens, heads * vdim]. */
+int nqb200_retention(const void* proj, int64_t stride, int64_t q_off, int64_t k_off, int64_t v_off, const float* decay,
+                     float* state, float* o, int64_t heads, int64_t dim, int64_t vdim, const nqb200_batch* b, int dtype,
+                     void* stream);
+
+/* out[t * out_stride + h * vdim + c] = out_scale * o / rms(o over the head) * silu(gate[t * gate_stride + h * vdim + c]). */
+int nqb200_head_norm_gate(const float* o, const void* gate, int64_t gate_stride, void* out, int64_t out_stride,
+                          int64_t tokens, int64_t heads, int64_t vdim, float eps, float out_scale, int dtype, void* stream);
+
+/* minGRU over proj [tokens, stride]: z, x and gate pre-activations at columns z_off, x_off, g_off.
+ * z = sigmoid(zp + z_bias), u = xp + x_bias, candidate = u >= 0 ? u + 1/2 : sigmoid(u),
+ * S <- (1 - z) S + z candidate, out = S silu(g).  state float [slots, width]. */
+int nqb200_mingru(const void* proj, int64_t stride, int64_t z_off, int64_t x_off, int64_t g_off, const float* z_bias,
+                  const float* x_bias, float* state, void* out, int64_t width, const nqb200_batch* b, int dtype,
+                  void* stream);
+
+/* out[t, i] = g sigmoid(1.702 g) (u + 1), g = min(gate_up[t, i], limit), u = clamp(gate_up[t, ff + i], -limit, limit). */
+int nqb200_clamped_glu(const void* gate_up, void* out, int64_t tokens, int64_t ff, float limit, int dtype, void* stream);
+
+#ifdef __cplusplus
+}
+#endif
+#endif

@@ -13,8 +13,9 @@ import torch
 
 _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(_HERE, "lib", "libnqb200.so")
+MIXERS_PATH = os.path.join(_HERE, "lib", "libnqb200_mixers.so")
 
-F16, BF16 = 0, 1
+F16, BF16, F32 = 0, 1, 2
 _vp, _i64, _int, _sz = ctypes.c_void_p, ctypes.c_int64, ctypes.c_int, ctypes.c_size_t
 
 class DecodeFusion(ctypes.Structure):
@@ -64,7 +65,36 @@ SIGNATURES = {
     "nqb200_gemm_launch_count": (_int, [_i64, _i64, _i64, _i64, _int]),
 }
 
+
+class StepDesc(ctypes.Structure):
+    """nqb200_batch of include/nqb200_mixers.h."""
+    _fields_ = [("cu", _vp), ("pos0", _vp), ("slot", _vp), ("table", _vp), ("batch", ctypes.c_int32), ("tokens", ctypes.c_int32),
+                ("max_len", ctypes.c_int32), ("table_width", ctypes.c_int32), ("block_size", ctypes.c_int32)]
+
+
+class AttentionDesc(ctypes.Structure):
+    """nqb200_attention of include/nqb200_mixers.h."""
+    _fields_ = [("heads", ctypes.c_int32), ("kv_heads", ctypes.c_int32), ("dim", ctypes.c_int32), ("vdim", ctypes.c_int32),
+                ("chunk", ctypes.c_int32), ("scale", ctypes.c_float), ("softcap", ctypes.c_float), ("sink", _vp),
+                ("out_scale", ctypes.c_float)]
+
+
+_step, _att, _f32 = ctypes.POINTER(StepDesc), ctypes.POINTER(AttentionDesc), ctypes.c_float
+# mirrors include/nqb200_mixers.h one to one
+MIXER_SIGNATURES = {
+    "nqb200_stream_add": (_int, [_vp, _vp, _vp, _vp, _int, _i64, _i64, _int, _vp]),
+    "nqb200_rmsnorm_rows": (_int, [_vp, _vp, _vp, _vp, _i64, _i64, _f32, _int, _vp]),
+    "nqb200_rmsnorm_conv": (_int, [_vp, _vp, _vp, _vp, _vp, _step, _i64, _i64, _f32, _int, _vp]),
+    "nqb200_rope_store": (_int, [_vp, _vp, _vp, _vp, _step] + [_i64] * 9 + [_int, _vp]),
+    "nqb200_chunk_attention": (_int, [_vp, _i64, _vp, _vp, _vp, _i64, _att, _step, _int, _vp]),
+    "nqb200_retention": (_int, [_vp, _i64, _i64, _i64, _i64, _vp, _vp, _vp, _i64, _i64, _i64, _step, _int, _vp]),
+    "nqb200_head_norm_gate": (_int, [_vp, _vp, _i64, _vp, _i64, _i64, _i64, _i64, _f32, _f32, _int, _vp]),
+    "nqb200_mingru": (_int, [_vp, _i64, _i64, _i64, _i64, _vp, _vp, _vp, _vp, _i64, _step, _int, _vp]),
+    "nqb200_clamped_glu": (_int, [_vp, _vp, _i64, _i64, _f32, _int, _vp]),
+}
+
 _lib = None
+_mixers = None
 _lock = threading.Lock()
 
 
@@ -87,6 +117,40 @@ def load() -> ctypes.CDLL:
                 fn.argtypes = args
             _lib = lib
     return _lib
+
+
+def load_mixers() -> ctypes.CDLL:
+    """Load the library of sequence-mixing kernels once; raise if it has not been built."""
+    global _mixers
+    if _mixers is None:
+        with _lock:
+            if _mixers is None:
+                if not os.path.exists(MIXERS_PATH):
+                    raise RuntimeError(f"{MIXERS_PATH} is missing: build it with `python -m nanoquantization_b200.csrc.build` "
+                                       "(needs nvcc). There is no CPU or PyTorch fallback for these kernels.")
+                lib = ctypes.CDLL(MIXERS_PATH)
+                for name, (res, args) in MIXER_SIGNATURES.items():
+                    fn = getattr(lib, name)
+                    fn.restype, fn.argtypes = res, args
+                _mixers = lib
+    return _mixers
+
+
+_STATUS = ("ok", "bad shape", "bad dtype", "misaligned pointer", "null pointer", "workspace missing or too small",
+           "unsupported device", "CUDA launch failed", "a bounded device-side wait timed out", "size exceeds the supported maximum")
+
+
+def check_mixers(status: int) -> None:
+    if status != 0:
+        raise RuntimeError(f"nqb200_mixers: {_STATUS[status] if status < len(_STATUS) else 'unknown status'} (status {status})")
+
+
+def mixer_dtype_code(dtype: torch.dtype) -> int:
+    if dtype == torch.bfloat16:
+        return BF16
+    if dtype == torch.float32:
+        return F32
+    raise TypeError(f"the sequence-mixing kernels take bfloat16 or float32, got {dtype}")
 
 
 def check(status: int) -> None:
@@ -148,6 +212,8 @@ def workspace(dev: torch.device, nbytes: int) -> torch.Tensor | None:
 
 def check_workspaces() -> None:
     """Synchronise and raise if any kernel recorded a give-up (a bounded wait that ran out)."""
+    if not _workspaces:
+        return
     lib = load()
     for (_dev, stream), ws in list(_workspaces.items()):
         check(lib.nqb200_workspace_status(ws.data_ptr(), ws.numel(), stream))

@@ -1,0 +1,145 @@
+// Rotary embedding + paged K/V store, and chunk-masked attention with a score cap and a sink.  The kernels in
+// this file take any head sizes and both element types; the tensor-core kernels take over where they apply.
+#include "mixers.cuh"
+
+namespace nqb200 {
+
+// One CTA per token: the token's cos / sin once into shared memory, then every head of q, k and v.
+template <typename T>
+__global__ void __launch_bounds__(256) rope_store_kernel(T* __restrict__ proj, T* __restrict__ k_cache, T* __restrict__ v_cache,
+                                                         const float* __restrict__ inv_freq, const nqb200_batch bt, int stride, int q_off,
+                                                         int k_off, int v_off, int heads, int kv_heads, int dim, int vdim, int rot) {
+  extern __shared__ float cs[];  // [rot/2] cos, [rot/2] sin
+  grid_launch_dependents();
+  grid_dependency_wait();
+  const int b = blockIdx.y, i = blockIdx.x, t0 = bt.cu[b];
+  if (i >= bt.cu[b + 1] - t0) return;
+  const int p = bt.pos0[b] + i, half = rot / 2;
+  for (int f = threadIdx.x; f < half; f += blockDim.x) sincosf((float)p * inv_freq[f], &cs[half + f], &cs[f]);
+  __syncthreads();
+  T* row = proj + (size_t)(t0 + i) * stride;
+  const size_t slot = kv_row(bt, b, p);
+  T* kd = k_cache + slot * kv_heads * dim;
+  T* vd = v_cache + slot * kv_heads * vdim;
+  const int per = half + (dim - rot);  // rotation pairs, then the dimensions that pass
+  for (int e = threadIdx.x; e < (heads + kv_heads) * per; e += blockDim.x) {
+    const int hd = e / per, j = e - hd * per;
+    const bool isq = hd < heads;
+    const T* src = row + (isq ? q_off + hd * dim : k_off + (hd - heads) * dim);
+    T* dst = isq ? row + q_off + hd * dim : kd + (hd - heads) * dim;
+    if (j < half) {
+      const float u = to_f(src[j]), v = to_f(src[j + half]), c = cs[j], s = cs[half + j];
+      dst[j] = from_f<T>(u * c - v * s);
+      dst[j + half] = from_f<T>(v * c + u * s);
+    } else if (!isq) {
+      dst[j + half] = src[j + half];
+    }
+  }
+  for (int e = threadIdx.x; e < kv_heads * vdim; e += blockDim.x) vd[e] = row[v_off + e];
+}
+
+constexpr int kSimpleKeys = 128;   // keys per pass = threads
+constexpr int kSimpleVCols = 8;    // value columns per thread at most: vdim <= 1024
+
+// One CTA per (token, head): a thread scores one key per pass, then owns value columns.
+template <typename T>
+__global__ void __launch_bounds__(kSimpleKeys) attention_simple_kernel(const T* __restrict__ q, int64_t q_stride, const T* __restrict__ k_cache,
+                                                                       const T* __restrict__ v_cache, T* __restrict__ out, int64_t out_stride,
+                                                                       const nqb200_attention at, const nqb200_batch bt) {
+  extern __shared__ float qs[];  // [dim]
+  __shared__ float sc[kSimpleKeys];
+  __shared__ int rows[kSimpleKeys];
+  __shared__ float red[4];
+  grid_launch_dependents();
+  grid_dependency_wait();
+  const int b = blockIdx.z, h = blockIdx.y, i = blockIdx.x, tid = threadIdx.x, t0 = bt.cu[b];
+  if (i >= bt.cu[b + 1] - t0) return;
+  const int p = bt.pos0[b] + i, lo = at.chunk > 0 ? p / at.chunk * at.chunk : 0, g = h / (at.heads / at.kv_heads);
+  const T* qr = q + (size_t)(t0 + i) * q_stride + (size_t)h * at.dim;
+  for (int d = tid; d < at.dim; d += kSimpleKeys) qs[d] = to_f(qr[d]);
+  float m = at.sink ? at.sink[h] : -INFINITY, l = at.sink ? 1.f : 0.f;
+  float acc[kSimpleVCols] = {};
+  for (int j0 = lo; j0 <= p; j0 += kSimpleKeys) {
+    const int j = j0 + tid;
+    __syncthreads();
+    float s = -INFINITY;
+    if (j <= p) {
+      const size_t r = kv_row(bt, b, j);
+      rows[tid] = (int)r;
+      const T* kr = k_cache + (r * at.kv_heads + g) * at.dim;
+      float d = 0.f;
+      for (int c = 0; c < at.dim; ++c) d += qs[c] * to_f(kr[c]);
+      s = d * at.scale;
+      if (at.softcap > 0.f) s = at.softcap * tanhf(s / at.softcap);
+    }
+    const float wm = warp_max(s);
+    if ((tid & 31) == 0) red[tid >> 5] = wm;
+    __syncthreads();
+    const float m_new = fmaxf(m, fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3])));
+    const float corr = expf(m - m_new), e = expf(s - m_new);
+    sc[tid] = e;
+    const float ws = warp_sum(e);
+    __syncthreads();
+    if ((tid & 31) == 0) red[tid >> 5] = ws;
+    __syncthreads();
+    l = l * corr + (red[0] + red[1] + red[2] + red[3]);
+    m = m_new;
+    const int cnt = min(kSimpleKeys, p - j0 + 1);
+#pragma unroll
+    for (int c = 0; c < kSimpleVCols; ++c) {
+      const int col = tid + c * kSimpleKeys;
+      if (col >= at.vdim) break;
+      float a = acc[c] * corr;
+      for (int jj = 0; jj < cnt; ++jj) a += sc[jj] * to_f(v_cache[((size_t)rows[jj] * at.kv_heads + g) * at.vdim + col]);
+      acc[c] = a;
+    }
+  }
+  const float f = at.out_scale / l;
+#pragma unroll
+  for (int c = 0; c < kSimpleVCols; ++c) {
+    const int col = tid + c * kSimpleKeys;
+    if (col < at.vdim) out[(size_t)(t0 + i) * out_stride + (size_t)h * at.vdim + col] = from_f<T>(acc[c] * f);
+  }
+}
+
+}  // namespace nqb200
+
+using namespace nqb200;
+
+extern "C" int nqb200_rope_store(void* proj, void* k_cache, void* v_cache, const float* inv_freq, const nqb200_batch* b, int64_t stride,
+                                 int64_t q_off, int64_t k_off, int64_t v_off, int64_t heads, int64_t kv_heads, int64_t dim, int64_t vdim,
+                                 int64_t rot, int dtype, void* stream) {
+  const int st = check_batch(b, true);
+  if (st != NQB200_OK) return st;
+  if (heads <= 0 || kv_heads <= 0 || dim <= 0 || vdim <= 0 || rot < 0 || rot > dim || rot % 2 != 0 || stride <= 0) return NQB200_ERR_BAD_SHAPE;
+  if (!mixer_dtype(dtype)) return NQB200_ERR_BAD_DTYPE;
+  if (b->tokens == 0) return NQB200_OK;
+  if (!proj || !k_cache || !v_cache || (rot > 0 && !inv_freq)) return NQB200_ERR_NULL_POINTER;
+  const dim3 grid((unsigned)b->max_len, (unsigned)b->batch), block(256);
+  const size_t smem = (size_t)rot * sizeof(float);
+#define NQB200_ROPE(T)                                                                                                                   \
+  launch_overlapped(rope_store_kernel<T>, grid, block, smem, (cudaStream_t)stream, (T*)proj, (T*)k_cache, (T*)v_cache, inv_freq, *b,     \
+                    (int)stride, (int)q_off, (int)k_off, (int)v_off, (int)heads, (int)kv_heads, (int)dim, (int)vdim, (int)rot)
+  return dtype == NQB200_F32 ? NQB200_ROPE(float) : NQB200_ROPE(bf16);
+#undef NQB200_ROPE
+}
+
+extern "C" int nqb200_chunk_attention(const void* q, int64_t q_stride, const void* k_cache, const void* v_cache, void* out,
+                                      int64_t out_stride, const nqb200_attention* a, const nqb200_batch* b, int dtype, void* stream) {
+  const int st = check_batch(b, true);
+  if (st != NQB200_OK) return st;
+  if (!a) return NQB200_ERR_NULL_POINTER;
+  if (a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads != 0 || a->dim <= 0 || a->dim > 4096 || a->vdim <= 0 ||
+      a->vdim > kSimpleKeys * kSimpleVCols || a->heads > 65535)
+    return NQB200_ERR_BAD_SHAPE;
+  if (!mixer_dtype(dtype)) return NQB200_ERR_BAD_DTYPE;
+  if (b->tokens == 0) return NQB200_OK;
+  if (!q || !k_cache || !v_cache || !out) return NQB200_ERR_NULL_POINTER;
+  const dim3 grid((unsigned)b->max_len, (unsigned)a->heads, (unsigned)b->batch), block(kSimpleKeys);
+  const size_t smem = (size_t)a->dim * sizeof(float);
+#define NQB200_ATT(T)                                                                                                              \
+  launch_overlapped(attention_simple_kernel<T>, grid, block, smem, (cudaStream_t)stream, (const T*)q, q_stride, (const T*)k_cache, \
+                    (const T*)v_cache, (T*)out, out_stride, *a, *b)
+  return dtype == NQB200_F32 ? NQB200_ATT(float) : NQB200_ATT(bf16);
+#undef NQB200_ATT
+}

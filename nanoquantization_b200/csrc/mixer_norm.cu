@@ -1,0 +1,168 @@
+// The residual stream's own steps: embedding / loop entry, RMS norm, RMS norm + input convolution, and the
+// clamped GLU between the feed-forward's linears.  The stream is float; a norm reads it once and leaves the
+// 16-bit operand of the next linear.
+#include "mixers.cuh"
+
+namespace nqb200 {
+
+template <typename T>
+__global__ void __launch_bounds__(256) stream_add_kernel(float* __restrict__ x, const int64_t* __restrict__ ids,
+                                                         const T* __restrict__ embed, const float* __restrict__ step,
+                                                         int accumulate, int width) {
+  grid_launch_dependents();
+  grid_dependency_wait();
+  float* row = x + (size_t)blockIdx.x * width;
+  const T* e = ids ? embed + (size_t)ids[blockIdx.x] * width : nullptr;
+  for (int c = threadIdx.x; c < width; c += blockDim.x) {
+    float v = accumulate ? row[c] : 0.f;
+    if (e) v += to_f(e[c]);
+    if (step) v += step[c];
+    row[c] = v;
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) rmsnorm_rows_kernel(const float* __restrict__ x, const int64_t* __restrict__ rows,
+                                                           const float* __restrict__ weight, T* __restrict__ out, int width, float eps) {
+  __shared__ float red[8];
+  grid_launch_dependents();
+  grid_dependency_wait();
+  const float* row = x + (size_t)(rows ? rows[blockIdx.x] : blockIdx.x) * width;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < width; c += 256) ss += row[c] * row[c];
+  ss = warp_sum(ss);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+  __syncthreads();
+  float tot = 0.f;
+#pragma unroll
+  for (int w = 0; w < 8; ++w) tot += red[w];
+  const float inv = 1.f / sqrtf(tot / (float)width + eps);
+  for (int c = threadIdx.x; c < width; c += 256) out[(size_t)blockIdx.x * width + c] = from_f<T>(row[c] * inv * weight[c]);
+}
+
+// A CTA takes `tile` tokens of one sequence (tile >= taps - 1).  It needs 1/rms of those and of the taps - 1
+// tokens before them; rows from before this step come from the state, which only the first tile of a sequence
+// reaches.  That same CTA also writes the new state (it recomputes the norm of the step's last taps - 1 tokens),
+// so the state is read and written by one CTA and no order between CTAs matters.
+template <typename T>
+__global__ void __launch_bounds__(256) rmsnorm_conv_kernel(const float* __restrict__ x, const float* __restrict__ weight,
+                                                           const float* __restrict__ conv, float* state, T* __restrict__ out,
+                                                           const nqb200_batch bt, int width, int taps, int tile, float eps) {
+  extern __shared__ float inv_s[];  // [halo + tile] tokens around the tile, then [halo] last tokens of the step
+  grid_launch_dependents();
+  grid_dependency_wait();
+  const int b = blockIdx.y, t0 = bt.cu[b], n = bt.cu[b + 1] - t0, first = blockIdx.x * tile;
+  if (first >= n) return;
+  const int halo = taps - 1, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
+  const bool head = first == 0;
+  for (int r = warp; r < halo + tile + (head ? halo : 0); r += nwarps) {
+    const int tok = r < halo + tile ? first - halo + r : n - halo + (r - halo - tile);
+    if (tok < 0 || tok >= n) continue;
+    const float* row = x + (size_t)(t0 + tok) * width;
+    float ss = 0.f;
+    for (int c = lane; c < width; c += 32) ss += row[c] * row[c];
+    ss = warp_sum(ss);
+    if (lane == 0) inv_s[r] = 1.f / sqrtf(ss / (float)width + eps);
+  }
+  __syncthreads();
+  const bool fresh = bt.pos0[b] == 0;
+  float* st = state + (size_t)bt.slot[b] * halo * width;
+  const int cnt = min(tile, n - first);
+  for (int c = threadIdx.x; c < width; c += blockDim.x) {
+    const float w = weight[c];
+    const float* cw = conv + (size_t)c * taps;
+    for (int i = 0; i < cnt; ++i) {
+      const int tok = first + i;
+      const float h = x[(size_t)(t0 + tok) * width + c] * inv_s[halo + i] * w;
+      float acc = 0.f;
+      for (int j = 0; j < halo; ++j) {
+        const int src = tok - halo + j;
+        float hv = 0.f;
+        if (src >= 0) hv = x[(size_t)(t0 + src) * width + c] * inv_s[i + j] * w;
+        else if (!fresh) hv = st[(size_t)(src + halo) * width + c];
+        acc += cw[j] * hv;
+      }
+      acc += cw[halo] * h;
+      out[(size_t)(t0 + tok) * width + c] = from_f<T>(h + acc);
+    }
+    if (head) {
+      for (int r = 0; r < halo; ++r) {  // ascending: an old row that moves down is read before it is overwritten
+        const int src = n - halo + r;
+        float hv = 0.f;
+        if (src >= 0) hv = x[(size_t)(t0 + src) * width + c] * inv_s[halo + tile + r] * w;
+        else if (!fresh) hv = st[(size_t)(src + halo) * width + c];
+        st[(size_t)r * width + c] = hv;
+      }
+    }
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) clamped_glu_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int64_t tokens, int ff,
+                                                          float limit) {
+  grid_launch_dependents();
+  grid_dependency_wait();
+  const int64_t total = tokens * (int64_t)ff;
+  for (int64_t idx = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; idx < total; idx += (int64_t)gridDim.x * blockDim.x) {
+    const int64_t t = idx / ff, i = idx - t * ff;
+    const float g = fminf(to_f(gate_up[t * 2 * ff + i]), limit);
+    const float u = fminf(fmaxf(to_f(gate_up[t * 2 * ff + ff + i]), -limit), limit);
+    out[idx] = from_f<T>(g * sigmoid_f(1.702f * g) * (u + 1.f));
+  }
+}
+
+}  // namespace nqb200
+
+using namespace nqb200;
+
+extern "C" int nqb200_stream_add(float* x, const int64_t* ids, const void* embed, const float* step, int accumulate, int64_t tokens,
+                                 int64_t width, int dtype, void* stream) {
+  if (tokens < 0 || width <= 0 || tokens > INT32_MAX || width > INT32_MAX) return NQB200_ERR_BAD_SHAPE;
+  if (!mixer_dtype(dtype)) return NQB200_ERR_BAD_DTYPE;
+  if (tokens == 0) return NQB200_OK;
+  if (!x || (ids && !embed)) return NQB200_ERR_NULL_POINTER;
+  const dim3 grid((unsigned)tokens), block(256);
+  if (dtype == NQB200_F32)
+    return launch_overlapped(stream_add_kernel<float>, grid, block, 0, (cudaStream_t)stream, x, ids, (const float*)embed, step, accumulate, (int)width);
+  return launch_overlapped(stream_add_kernel<bf16>, grid, block, 0, (cudaStream_t)stream, x, ids, (const bf16*)embed, step, accumulate, (int)width);
+}
+
+extern "C" int nqb200_rmsnorm_rows(const float* x, const int64_t* rows, const float* weight, void* out, int64_t n_rows, int64_t width,
+                                   float eps, int dtype, void* stream) {
+  if (n_rows < 0 || width <= 0 || n_rows > INT32_MAX || width > INT32_MAX) return NQB200_ERR_BAD_SHAPE;
+  if (!mixer_dtype(dtype)) return NQB200_ERR_BAD_DTYPE;
+  if (n_rows == 0) return NQB200_OK;
+  if (!x || !weight || !out) return NQB200_ERR_NULL_POINTER;
+  const dim3 grid((unsigned)n_rows), block(256);
+  if (dtype == NQB200_F32)
+    return launch_overlapped(rmsnorm_rows_kernel<float>, grid, block, 0, (cudaStream_t)stream, x, rows, weight, (float*)out, (int)width, eps);
+  return launch_overlapped(rmsnorm_rows_kernel<bf16>, grid, block, 0, (cudaStream_t)stream, x, rows, weight, (bf16*)out, (int)width, eps);
+}
+
+extern "C" int nqb200_rmsnorm_conv(const float* x, const float* weight, const float* conv, float* state, void* out,
+                                   const nqb200_batch* b, int64_t width, int64_t taps, float eps, int dtype, void* stream) {
+  const int st = check_batch(b, false);
+  if (st != NQB200_OK) return st;
+  if (width <= 0 || width > INT32_MAX || taps <= 0 || taps > 1024) return NQB200_ERR_BAD_SHAPE;
+  if (!mixer_dtype(dtype)) return NQB200_ERR_BAD_DTYPE;
+  if (b->tokens == 0) return NQB200_OK;
+  if (!x || !weight || !conv || !out || (taps > 1 && !state)) return NQB200_ERR_NULL_POINTER;
+  const int halo = (int)taps - 1, tile = halo > 8 ? halo : 8;
+  const dim3 grid((unsigned)((b->max_len + tile - 1) / tile), (unsigned)b->batch), block(256);
+  const size_t smem = (size_t)(2 * halo + tile) * sizeof(float);
+  if (dtype == NQB200_F32)
+    return launch_overlapped(rmsnorm_conv_kernel<float>, grid, block, smem, (cudaStream_t)stream, x, weight, conv, state, (float*)out, *b, (int)width, (int)taps, tile, eps);
+  return launch_overlapped(rmsnorm_conv_kernel<bf16>, grid, block, smem, (cudaStream_t)stream, x, weight, conv, state, (bf16*)out, *b, (int)width, (int)taps, tile, eps);
+}
+
+extern "C" int nqb200_clamped_glu(const void* gate_up, void* out, int64_t tokens, int64_t ff, float limit, int dtype, void* stream) {
+  if (tokens < 0 || ff <= 0 || ff > INT32_MAX) return NQB200_ERR_BAD_SHAPE;
+  if (!mixer_dtype(dtype)) return NQB200_ERR_BAD_DTYPE;
+  if (tokens == 0) return NQB200_OK;
+  if (!gate_up || !out) return NQB200_ERR_NULL_POINTER;
+  const int64_t want = (tokens * ff + 255) / 256;
+  const dim3 grid((unsigned)(want < (int64_t)kNumSMs * 16 ? want : (int64_t)kNumSMs * 16)), block(256);
+  if (dtype == NQB200_F32)
+    return launch_overlapped(clamped_glu_kernel<float>, grid, block, 0, (cudaStream_t)stream, (const float*)gate_up, (float*)out, tokens, (int)ff, limit);
+  return launch_overlapped(clamped_glu_kernel<bf16>, grid, block, 0, (cudaStream_t)stream, (const bf16*)gate_up, (bf16*)out, tokens, (int)ff, limit);
+}

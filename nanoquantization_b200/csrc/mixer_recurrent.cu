@@ -1,0 +1,242 @@
+// Recurrences over tokens with a float state per sequence: retention (a matrix per head with a fixed decay) and
+// minGRU (an element-wise gated scan).  Kernels here take any sizes and both element types.
+#include "mixers.cuh"
+
+namespace nqb200 {
+
+constexpr int kRetCols = 32, kRetGroups = 8, kRetTokens = 16;
+
+// One CTA per (32 value columns, head, sequence), tokens in order.  Thread (group, column) keeps rows
+// group, group + 8, ... of its column of S in registers.
+template <typename T, int DPT>
+__global__ void __launch_bounds__(kRetCols* kRetGroups) retention_simple_kernel(const T* __restrict__ proj, int64_t stride, int q_off, int k_off,
+                                                                                int v_off, const float* __restrict__ decay, float* state,
+                                                                                float* __restrict__ o, int heads, int dim, int vdim,
+                                                                                const nqb200_batch bt) {
+  extern __shared__ float sm[];
+  float* qs = sm;                               // [tokens][dim]
+  float* ks = qs + kRetTokens * dim;            // [tokens][dim], scaled
+  float* vs = ks + kRetTokens * dim;            // [tokens][cols]
+  float* part = vs + kRetTokens * kRetCols;     // [tokens][groups][cols]
+  grid_launch_dependents();
+  grid_dependency_wait();
+  const int b = blockIdx.z, h = blockIdx.y, col = threadIdx.x % kRetCols, grp = threadIdx.x / kRetCols, tid = threadIdx.x;
+  const int c = blockIdx.x * kRetCols + col, t0 = bt.cu[b], n = bt.cu[b + 1] - t0;
+  if (n <= 0) return;
+  float* st = state + ((size_t)bt.slot[b] * heads + h) * dim * vdim;
+  const bool live = c < vdim, fresh = bt.pos0[b] == 0;
+  const float d = decay[h], kscale = 1.f / sqrtf((float)dim);
+  float S[DPT];
+#pragma unroll
+  for (int r = 0; r < DPT; ++r) {
+    const int row = r * kRetGroups + grp;
+    S[r] = (live && !fresh && row < dim) ? st[(size_t)row * vdim + c] : 0.f;
+  }
+  for (int base = 0; base < n; base += kRetTokens) {
+    const int cnt = min(kRetTokens, n - base);
+    __syncthreads();
+    for (int e = tid; e < cnt * dim; e += blockDim.x) {
+      const int i = e / dim, r = e - i * dim;
+      const T* row = proj + (size_t)(t0 + base + i) * stride + (size_t)h * dim + r;
+      qs[e] = to_f(row[q_off]);
+      ks[e] = to_f(row[k_off]) * kscale;
+    }
+    for (int e = tid; e < cnt * kRetCols; e += blockDim.x) {
+      const int i = e / kRetCols, cc = blockIdx.x * kRetCols + e % kRetCols;
+      vs[e] = cc < vdim ? to_f(proj[(size_t)(t0 + base + i) * stride + v_off + (size_t)h * vdim + cc]) : 0.f;
+    }
+    __syncthreads();
+    for (int i = 0; i < cnt; ++i) {
+      const float v = vs[i * kRetCols + col];
+      float acc = 0.f;
+#pragma unroll
+      for (int r = 0; r < DPT; ++r) {
+        const int row = r * kRetGroups + grp;
+        if (row < dim) {
+          S[r] = d * S[r] + ks[i * dim + row] * v;
+          acc += S[r] * qs[i * dim + row];
+        }
+      }
+      part[(i * kRetGroups + grp) * kRetCols + col] = acc;
+    }
+    __syncthreads();
+    for (int e = tid; e < cnt * kRetCols; e += blockDim.x) {
+      const int i = e / kRetCols, cc = blockIdx.x * kRetCols + e % kRetCols;
+      if (cc >= vdim) continue;
+      float acc = 0.f;
+#pragma unroll
+      for (int g = 0; g < kRetGroups; ++g) acc += part[(i * kRetGroups + g) * kRetCols + e % kRetCols];
+      o[((size_t)(t0 + base + i) * heads + h) * vdim + cc] = acc;
+    }
+  }
+  if (live) {
+#pragma unroll
+    for (int r = 0; r < DPT; ++r) {
+      const int row = r * kRetGroups + grp;
+      if (row < dim) st[(size_t)row * vdim + c] = S[r];
+    }
+  }
+}
+
+// One warp per (token, head).
+template <typename T>
+__global__ void __launch_bounds__(256) head_norm_gate_kernel(const float* __restrict__ o, const T* __restrict__ gate, int64_t gate_stride,
+                                                             T* __restrict__ out, int64_t out_stride, int64_t pairs, int heads, int vdim,
+                                                             float eps, float out_scale) {
+  grid_launch_dependents();
+  grid_dependency_wait();
+  const int64_t w = blockIdx.x * (int64_t)(blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (w >= pairs) return;
+  const int64_t t = w / heads;
+  const int h = (int)(w - t * heads), lane = threadIdx.x & 31;
+  const float* row = o + w * vdim;
+  float ss = 0.f;
+  for (int c = lane; c < vdim; c += 32) ss += row[c] * row[c];
+  const float inv = out_scale / sqrtf(warp_sum(ss) / (float)vdim + eps);
+  for (int c = lane; c < vdim; c += 32) {
+    const float g = to_f(gate[t * gate_stride + (int64_t)h * vdim + c]);
+    out[t * out_stride + (int64_t)h * vdim + c] = from_f<T>(row[c] * inv * (g * sigmoid_f(g)));
+  }
+}
+
+constexpr int kGruSegs = 32, kGruCols = 32, kGruLen = 4;  // 128 tokens per pass
+
+// One CTA per (32 channels, sequence).  Thread (segment, channel) folds its 4 tokens into S -> A S + B, a warp per
+// channel scans the 32 segments, and the thread replays its tokens from the state at its segment's start.
+template <typename T>
+__global__ void __launch_bounds__(kGruSegs* kGruCols) mingru_kernel(const T* __restrict__ proj, int64_t stride, int z_off, int x_off, int g_off,
+                                                                    const float* __restrict__ z_bias, const float* __restrict__ x_bias,
+                                                                    float* state, T* __restrict__ out, int width, const nqb200_batch bt) {
+  __shared__ float As[kGruSegs][kGruCols + 1], Bs[kGruSegs][kGruCols + 1], carry[kGruCols];
+  grid_launch_dependents();
+  grid_dependency_wait();
+  const int b = blockIdx.y, col = threadIdx.x % kGruCols, seg = threadIdx.x / kGruCols, c = blockIdx.x * kGruCols + col;
+  const int t0 = bt.cu[b], n = bt.cu[b + 1] - t0;
+  if (n <= 0) return;
+  const bool live = c < width;
+  float* st = state + (size_t)bt.slot[b] * width;
+  const float zb = live ? z_bias[c] : 0.f, xb = live ? x_bias[c] : 0.f;
+  if (seg == 0) carry[col] = live && bt.pos0[b] != 0 ? st[c] : 0.f;
+  for (int base = 0; base < n; base += kGruSegs * kGruLen) {
+    float a[kGruLen], v[kGruLen], A = 1.f, B = 0.f;
+#pragma unroll
+    for (int i = 0; i < kGruLen; ++i) {
+      const int tok = base + seg * kGruLen + i;
+      a[i] = 1.f; v[i] = 0.f;
+      if (live && tok < n) {
+        const T* row = proj + (size_t)(t0 + tok) * stride;
+        const float z = sigmoid_f(to_f(row[z_off + c]) + zb), u = to_f(row[x_off + c]) + xb;
+        a[i] = 1.f - z;
+        v[i] = z * (u >= 0.f ? u + 0.5f : sigmoid_f(u));
+      }
+      A *= a[i];
+      B = a[i] * B + v[i];
+    }
+    As[seg][col] = A;
+    Bs[seg][col] = B;
+    __syncthreads();
+    {
+      // warp `seg` scans channel `seg`; its lanes are the segments
+      const int ch = seg, lane = col;
+      float sa = As[lane][ch], sb = Bs[lane][ch];
+#pragma unroll
+      for (int off = 1; off < 32; off <<= 1) {
+        const float pa = __shfl_up_sync(0xFFFFFFFFu, sa, off), pb = __shfl_up_sync(0xFFFFFFFFu, sb, off);
+        if (lane >= off) { sb = sa * pb + sb; sa = sa * pa; }
+      }
+      const float s0 = carry[ch], end = sa * s0 + sb;
+      float begin = __shfl_up_sync(0xFFFFFFFFu, end, 1);
+      if (lane == 0) begin = s0;
+      Bs[lane][ch] = begin;
+      __syncwarp();
+      if (lane == 31) carry[ch] = end;
+    }
+    __syncthreads();
+    float S = Bs[seg][col];
+#pragma unroll
+    for (int i = 0; i < kGruLen; ++i) {
+      const int tok = base + seg * kGruLen + i;
+      S = a[i] * S + v[i];
+      if (live && tok < n) {
+        const float g = to_f(proj[(size_t)(t0 + tok) * stride + g_off + c]);
+        out[(size_t)(t0 + tok) * width + c] = from_f<T>(S * (g * sigmoid_f(g)));
+      }
+    }
+    __syncthreads();
+  }
+  if (seg == 0 && live) st[c] = carry[col];
+}
+
+}  // namespace nqb200
+
+using namespace nqb200;
+
+template <typename T, int DPT>
+static int retention_simple(const void* proj, int64_t stride, int64_t q_off, int64_t k_off, int64_t v_off, const float* decay, float* state,
+                            float* o, int64_t heads, int64_t dim, int64_t vdim, const nqb200_batch* b, cudaStream_t st) {
+  const dim3 grid((unsigned)((vdim + kRetCols - 1) / kRetCols), (unsigned)heads, (unsigned)b->batch), block(kRetCols * kRetGroups);
+  const size_t smem = (size_t)kRetTokens * (2 * dim + kRetCols + kRetGroups * kRetCols) * sizeof(float);
+  if (smem > 48 * 1024 &&
+      cudaFuncSetAttribute(retention_simple_kernel<T, DPT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+    cudaGetLastError();
+    return NQB200_ERR_LAUNCH;
+  }
+  return launch_overlapped(retention_simple_kernel<T, DPT>, grid, block, smem, st, (const T*)proj, stride, (int)q_off, (int)k_off, (int)v_off,
+                           decay, state, o, (int)heads, (int)dim, (int)vdim, *b);
+}
+
+extern "C" int nqb200_retention(const void* proj, int64_t stride, int64_t q_off, int64_t k_off, int64_t v_off, const float* decay,
+                                float* state, float* o, int64_t heads, int64_t dim, int64_t vdim, const nqb200_batch* b, int dtype,
+                                void* stream) {
+  const int s = check_batch(b, false);
+  if (s != NQB200_OK) return s;
+  if (heads <= 0 || heads > 65535 || dim <= 0 || dim > 1024 || vdim <= 0 || stride <= 0) return NQB200_ERR_BAD_SHAPE;
+  if (!mixer_dtype(dtype)) return NQB200_ERR_BAD_DTYPE;
+  if (b->tokens == 0) return NQB200_OK;
+  if (!proj || !decay || !state || !o) return NQB200_ERR_NULL_POINTER;
+  cudaStream_t st = (cudaStream_t)stream;
+#define NQB200_RET(T, D) return retention_simple<T, D>(proj, stride, q_off, k_off, v_off, decay, state, o, heads, dim, vdim, b, st)
+#define NQB200_RET_T(T)                                                                                       \
+  do {                                                                                                        \
+    if (dim <= 64) NQB200_RET(T, 8);                                                                          \
+    if (dim <= 128) NQB200_RET(T, 16);                                                                        \
+    if (dim <= 256) NQB200_RET(T, 32);                                                                        \
+    if (dim <= 512) NQB200_RET(T, 64);                                                                        \
+    NQB200_RET(T, 128);                                                                                       \
+  } while (0)
+  if (dtype == NQB200_F32) NQB200_RET_T(float);
+  NQB200_RET_T(bf16);
+#undef NQB200_RET_T
+#undef NQB200_RET
+}
+
+extern "C" int nqb200_head_norm_gate(const float* o, const void* gate, int64_t gate_stride, void* out, int64_t out_stride, int64_t tokens,
+                                     int64_t heads, int64_t vdim, float eps, float out_scale, int dtype, void* stream) {
+  if (tokens < 0 || heads <= 0 || vdim <= 0) return NQB200_ERR_BAD_SHAPE;
+  if (!mixer_dtype(dtype)) return NQB200_ERR_BAD_DTYPE;
+  if (tokens == 0) return NQB200_OK;
+  if (!o || !gate || !out) return NQB200_ERR_NULL_POINTER;
+  const int64_t pairs = tokens * heads;
+  const dim3 grid((unsigned)((pairs + 7) / 8)), block(256);
+  if (dtype == NQB200_F32)
+    return launch_overlapped(head_norm_gate_kernel<float>, grid, block, 0, (cudaStream_t)stream, o, (const float*)gate, gate_stride, (float*)out,
+                             out_stride, pairs, (int)heads, (int)vdim, eps, out_scale);
+  return launch_overlapped(head_norm_gate_kernel<bf16>, grid, block, 0, (cudaStream_t)stream, o, (const bf16*)gate, gate_stride, (bf16*)out,
+                           out_stride, pairs, (int)heads, (int)vdim, eps, out_scale);
+}
+
+extern "C" int nqb200_mingru(const void* proj, int64_t stride, int64_t z_off, int64_t x_off, int64_t g_off, const float* z_bias,
+                             const float* x_bias, float* state, void* out, int64_t width, const nqb200_batch* b, int dtype, void* stream) {
+  const int s = check_batch(b, false);
+  if (s != NQB200_OK) return s;
+  if (width <= 0 || width > INT32_MAX || stride <= 0) return NQB200_ERR_BAD_SHAPE;
+  if (!mixer_dtype(dtype)) return NQB200_ERR_BAD_DTYPE;
+  if (b->tokens == 0) return NQB200_OK;
+  if (!proj || !z_bias || !x_bias || !state || !out) return NQB200_ERR_NULL_POINTER;
+  const dim3 grid((unsigned)((width + kGruCols - 1) / kGruCols), (unsigned)b->batch), block(kGruSegs * kGruCols);
+  if (dtype == NQB200_F32)
+    return launch_overlapped(mingru_kernel<float>, grid, block, 0, (cudaStream_t)stream, (const float*)proj, stride, (int)z_off, (int)x_off,
+                             (int)g_off, z_bias, x_bias, state, (float*)out, (int)width, *b);
+  return launch_overlapped(mingru_kernel<bf16>, grid, block, 0, (cudaStream_t)stream, (const bf16*)proj, stride, (int)z_off, (int)x_off,
+                           (int)g_off, z_bias, x_bias, state, (bf16*)out, (int)width, *b);
+}

@@ -1,0 +1,45 @@
+// Helpers shared by the sequence-mixing kernels: element types and the flattened-batch descriptor.
+#pragma once
+#include "common.cuh"
+#include "nqb200_mixers.h"
+
+namespace nqb200 {
+
+using bf16 = __nv_bfloat16;
+
+__device__ __forceinline__ float to_f(float v) { return v; }
+__device__ __forceinline__ float to_f(bf16 v) { return __bfloat162float(v); }
+template <typename T> __device__ __forceinline__ T from_f(float v);
+template <> __device__ __forceinline__ float from_f<float>(float v) { return v; }
+template <> __device__ __forceinline__ bf16 from_f<bf16>(float v) { return __float2bfloat16_rn(v); }
+
+__device__ __forceinline__ float sigmoid_f(float v) { return 1.f / (1.f + expf(-v)); }
+
+__device__ __forceinline__ float warp_sum(float v) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xFFFFFFFFu, v, o);
+  return v;
+}
+__device__ __forceinline__ float warp_max(float v) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xFFFFFFFFu, v, o));
+  return v;
+}
+
+// Cache row of position p of sequence b.
+__device__ __forceinline__ size_t kv_row(const nqb200_batch& bt, int b, int p) {
+  return (size_t)bt.table[(size_t)b * bt.table_width + p / bt.block_size] * bt.block_size + p % bt.block_size;
+}
+
+static inline int check_batch(const nqb200_batch* b, bool paged) {
+  if (!b) return NQB200_ERR_NULL_POINTER;
+  if (b->batch < 0 || b->tokens < 0 || b->max_len < 0 || b->max_len > b->tokens || b->batch > 65535) return NQB200_ERR_BAD_SHAPE;
+  if (b->tokens == 0) return NQB200_OK;
+  if (b->batch == 0 || b->max_len == 0) return NQB200_ERR_BAD_SHAPE;
+  if (!b->cu || !b->pos0) return NQB200_ERR_NULL_POINTER;
+  if (paged ? (!b->table || b->table_width <= 0 || b->block_size <= 0) : !b->slot) return NQB200_ERR_NULL_POINTER;
+  return NQB200_OK;
+}
+static inline bool mixer_dtype(int dtype) { return dtype == NQB200_BF16 || dtype == NQB200_F32; }
+
+}  // namespace nqb200

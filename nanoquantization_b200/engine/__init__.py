@@ -1,1 +1,2 @@
-from .engine import BlockManager, LLMEngine, PagedKVCache, Scheduler, Sequence  # noqa: F401
+from .batch import CacheLayout, KVSpec, StepBatch  # noqa: F401
+from .engine import BlockManager, LayerStep, LLMEngine, PagedKVCache, Scheduler, Sequence, StatePool  # noqa: F401

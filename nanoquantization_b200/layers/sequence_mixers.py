@@ -1,0 +1,194 @@
+"""Sub-layers of decoders that mix tokens by other means than plain attention, over the kernels of ``mixers.py``.
+
+A mixer owns two merged weights, ``w_in [rows, width]`` (everything that reads the sub-layer's input, one product)
+and ``w_out [width, columns]`` (everything that is added to the residual stream, one product), and says what it
+keeps per sequence: ``kv_spec()`` for the paged cache, ``state_shapes()`` for the recurrent-state pool.  ``mix(proj,
+act, layer_step)`` turns the input product into the operand of the output product.  ``checkpoint(prefix)`` names
+the views of the merged weights that checkpoint tensors are copied into.
+
+Mixers that can stand side by side (``AttentionMixer``, ``RetentionMixer``) take their columns of ``proj`` and
+``act`` as offsets, so that ``ParallelMixer`` runs both on one product each; their output scale goes into the
+kernel that writes ``act``."""
+from __future__ import annotations
+
+import torch
+import torch.nn as nn
+
+from .. import _lib
+from ..engine.batch import KVSpec
+from . import mixers as ops
+
+
+def _buffer(module: nn.Module, name: str, *shape, dtype, device) -> torch.Tensor:
+    module.register_buffer(name, torch.zeros(*shape, dtype=dtype, device=device), persistent=False)
+    return getattr(module, name)
+
+
+class AttentionMixer(nn.Module):
+    """Grouped-query attention inside chunks of the sequence, partial rotary embedding, capped scores, a sink per head."""
+
+    def __init__(self, *, heads, kv_heads, dim, vdim, chunk, rot_base, rot_dims, scale, softcap, out_scale=1.0, device="cpu"):
+        super().__init__()
+        if heads % kv_heads != 0 or rot_dims % 2 != 0 or not 0 <= rot_dims <= dim:
+            raise ValueError(f"attention: {heads} heads over {kv_heads} key/value heads, {rot_dims} of {dim} dimensions rotated")
+        if chunk < 1 or softcap <= 0:
+            raise ValueError(f"attention: chunk {chunk} and softcap {softcap} must be positive")
+        self.heads, self.kv_heads, self.dim, self.vdim, self.chunk = heads, kv_heads, dim, vdim, chunk
+        self.scale, self.softcap, self.out_scale = float(scale), float(softcap), float(out_scale)
+        self.in_parts = [("q", heads * dim), ("k", kv_heads * dim), ("v", kv_heads * vdim)]
+        self.out_columns = heads * vdim
+        _buffer(self, "sink", heads, dtype=torch.float32, device=device)
+        i = torch.arange(rot_dims // 2, dtype=torch.float64)
+        self.register_buffer("inv_freq", (float(rot_base) ** (-2.0 * i / max(rot_dims, 1))).float().to(device), persistent=False)
+
+    def kv_spec(self):
+        return KVSpec(self.kv_heads, self.dim, self.vdim, self.chunk)
+
+    def state_shapes(self):
+        return {}
+
+    def checkpoint(self, prefix):
+        return {prefix + "sink": self.sink}
+
+    def desc(self) -> _lib.AttentionDesc:
+        return _lib.AttentionDesc(self.heads, self.kv_heads, self.dim, self.vdim, self.chunk, self.scale, self.softcap,
+                                  self.sink.data_ptr(), self.out_scale)
+
+    def mix(self, proj, col, act, act_col, layer_step):
+        q_off, k_off, v_off = col, col + self.heads * self.dim, col + (self.heads + self.kv_heads) * self.dim
+        ops.rope_store(proj, layer_step.k_cache, layer_step.v_cache, self.inv_freq, layer_step.batch, q_off, k_off, v_off, self.heads)
+        ops.chunk_attention(proj[:, q_off:k_off], layer_step.k_cache, layer_step.v_cache, act[:, act_col:act_col + self.out_columns],
+                            self.desc(), layer_step.batch)
+
+
+class RetentionMixer(nn.Module):
+    """Linear attention with one fixed decay per head; each head's output is RMS-normalised and gated."""
+
+    def __init__(self, *, heads, dim, vdim, decay, eps, out_scale=1.0, device="cpu"):
+        super().__init__()
+        if len(decay) != heads:
+            raise ValueError(f"retention: {len(decay)} decays for {heads} heads")
+        self.heads, self.dim, self.vdim, self.eps, self.out_scale = heads, dim, vdim, float(eps), float(out_scale)
+        self.in_parts = [("q", heads * dim), ("k", heads * dim), ("v", heads * vdim), ("g", heads * vdim)]
+        self.out_columns = heads * vdim
+        self.register_buffer("decay", torch.tensor(decay, dtype=torch.float64).float().to(device), persistent=False)
+
+    def kv_spec(self):
+        return None
+
+    def state_shapes(self):
+        return {"retention": (self.heads, self.dim, self.vdim)}
+
+    def checkpoint(self, prefix):
+        return {}
+
+    def mix(self, proj, col, act, act_col, layer_step):
+        q_off, k_off = col, col + self.heads * self.dim
+        v_off = k_off + self.heads * self.dim
+        g_off = v_off + self.heads * self.vdim
+        o = ops.retention(proj, q_off, k_off, v_off, self.decay, layer_step.state["retention"], layer_step.batch)
+        ops.head_norm_gate(o, proj[:, g_off:g_off + self.out_columns], act[:, act_col:act_col + self.out_columns], self.eps, self.out_scale)
+
+
+class ParallelMixer(nn.Module):
+    """Mixers side by side on the same input, their (scaled) outputs summed: one merged product in, one out."""
+
+    def __init__(self, width: int, parts: dict, *, dtype, device="cpu"):
+        super().__init__()
+        self.parts = nn.ModuleDict(parts)
+        self.rows = sum(n for m in parts.values() for _, n in m.in_parts)
+        self.columns = sum(m.out_columns for m in parts.values())
+        _buffer(self, "w_in", self.rows, width, dtype=dtype, device=device)
+        _buffer(self, "w_out", width, self.columns, dtype=dtype, device=device)
+
+    def kv_spec(self):
+        specs = [s for s in (m.kv_spec() for m in self.parts.values()) if s is not None]
+        if len(specs) > 1:
+            raise ValueError("one mixer of a layer keeps keys and values at most")
+        return specs[0] if specs else None
+
+    def state_shapes(self):
+        return {k: v for m in self.parts.values() for k, v in m.state_shapes().items()}
+
+    def checkpoint(self, prefix):
+        out, row, col = {}, 0, 0
+        for name, m in self.parts.items():
+            p = f"{prefix}{name}."
+            for part, n in m.in_parts:
+                out[p + part] = self.w_in[row:row + n]
+                row += n
+            out[p + "o"] = self.w_out[:, col:col + m.out_columns]
+            col += m.out_columns
+            out.update(m.checkpoint(p))
+        return out
+
+    def forward(self, x, h, layer_step):
+        """``x += mixer(h)`` on the float32 stream."""
+        proj = ops.linear(h, self.w_in)
+        act = torch.empty(h.shape[0], self.columns, dtype=h.dtype, device=h.device)
+        row = col = 0
+        for m in self.parts.values():
+            m.mix(proj, row, act, col, layer_step)
+            row += sum(n for _, n in m.in_parts)
+            col += m.out_columns
+        ops.linear_residual_(x, act, self.w_out)
+
+
+class MinGRUMixer(nn.Module):
+    """A gated element-wise recurrence whose gates read the current token only."""
+
+    def __init__(self, width: int, size: int, *, dtype, device="cpu"):
+        super().__init__()
+        self.size = size
+        _buffer(self, "w_in", 3 * size, width, dtype=dtype, device=device)
+        _buffer(self, "w_out", width, size, dtype=dtype, device=device)
+        _buffer(self, "z_bias", size, dtype=torch.float32, device=device)
+        _buffer(self, "x_bias", size, dtype=torch.float32, device=device)
+
+    def kv_spec(self):
+        return None
+
+    def state_shapes(self):
+        return {"mingru": (self.size,)}
+
+    def checkpoint(self, prefix):
+        n = self.size
+        return {prefix + "z": self.w_in[:n], prefix + "x": self.w_in[n:2 * n], prefix + "g": self.w_in[2 * n:], prefix + "o": self.w_out,
+                prefix + "z.b": self.z_bias, prefix + "x.b": self.x_bias}
+
+    def forward(self, x, h, layer_step):
+        proj = ops.linear(h, self.w_in)
+        y = ops.mingru(proj, self.size, self.z_bias, self.x_bias, layer_step.state["mingru"], layer_step.batch)
+        ops.linear_residual_(x, y, self.w_out)
+
+
+class ClampedGLU(nn.Module):
+    """Feed-forward ``down(g sigmoid(1.702 g) (u + 1))`` with g and u clamped to a limit."""
+
+    def __init__(self, width: int, ff: int, limit: float, *, dtype, device="cpu"):
+        super().__init__()
+        self.ff, self.limit = ff, float(limit)
+        _buffer(self, "w_in", 2 * ff, width, dtype=dtype, device=device)
+        _buffer(self, "w_out", width, ff, dtype=dtype, device=device)
+
+    def checkpoint(self, prefix):
+        return {prefix + "gate": self.w_in[:self.ff], prefix + "up": self.w_in[self.ff:], prefix + "down": self.w_out}
+
+    def forward(self, x, h):
+        ops.linear_residual_(x, ops.clamped_glu(ops.linear(h, self.w_in), self.limit), self.w_out)
+
+
+class ConvNorm(nn.Module):
+    """RMS norm of the residual stream, then ``h + causal_conv(h)``: what a sub-layer reads."""
+
+    def __init__(self, width: int, taps: int, eps: float, *, dtype, device="cpu"):
+        super().__init__()
+        self.eps, self.taps, self.dtype = float(eps), taps, dtype
+        _buffer(self, "weight", width, dtype=torch.float32, device=device)
+        _buffer(self, "conv", width, taps, dtype=torch.float32, device=device)
+
+    def state_shape(self):
+        return (self.taps - 1, self.weight.numel())
+
+    def forward(self, x, state, step):
+        return ops.rmsnorm_conv(x, self.weight, self.conv, state, step, self.eps, self.dtype)

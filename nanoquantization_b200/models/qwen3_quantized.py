@@ -48,6 +48,15 @@ class Qwen3Config:
     rope_theta: float = 1e6
     rms_norm_eps: float = 1e-6
 
+    @classmethod
+    def from_dict(cls, c: dict) -> "Qwen3Config":
+        """From a Hugging Face config.json with the ``quantization_config`` block the checkpoint writer adds."""
+        q = c.get("quantization_config", {})
+        return cls(c["num_hidden_layers"], c["vocab_size"], c["hidden_size"], c["num_attention_heads"], c["num_key_value_heads"],
+                   c["max_position_embeddings"], c["intermediate_size"], int(q.get("w_bits", 4)), int(q.get("group_size", 128)),
+                   c.get("head_dim"), bool(c.get("tie_word_embeddings", False)), float(c.get("rope_theta", 1e6)),
+                   float(c.get("rms_norm_eps", 1e-6)))
+
 
 # the architectures the benchmark configurations name
 QWEN3_SHAPES = {
@@ -318,6 +327,32 @@ class Qwen3QuantizedForCausalLM(nn.Module):
         return cls(cfg.num_hidden_layers, cfg.vocab_size, cfg.hidden_size, cfg.total_num_heads, cfg.total_num_kv_heads,
                    cfg.max_position_embeddings, cfg.intermediate_size, cfg.w_bits, cfg.group_size, cfg.head_dim,
                    cfg.tie_word_embeddings, cfg.rope_theta, cfg.rms_norm_eps, **kw)
+
+    delegates_attention = True  # the engine's attention over its cache, not kernels of the model's own
+
+    @property
+    def device(self) -> torch.device:
+        return self.lm_head.weight.device
+
+    @property
+    def dtype(self) -> torch.dtype:
+        return self.lm_head.weight.dtype
+
+    def cache_layout(self):
+        """Keys and values of every layer; nothing recurrent."""
+        from ..engine.batch import CacheLayout, KVSpec
+        attn = self.model.layers[0].self_attn
+        return CacheLayout([KVSpec(attn.num_kv_heads, attn.head_dim, attn.head_dim)] * len(self.model.layers))
+
+    def forward_step(self, batch, layer_step: Callable[[int], Callable], rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """An engine step: final hidden states of the given rows (all of the step's tokens if None)."""
+        h = self.model.forward_tokens(batch.tokens, batch.positions, layer_step)
+        return h if rows is None else h[rows]
+
+    def logits(self, hidden: torch.Tensor) -> torch.Tensor:
+        if self.tp_size != 1:
+            raise RuntimeError("the head is sharded over the vocabulary: only greedy_tokens() works across ranks")
+        return self.lm_head(hidden).float()
 
     def attach_peer_comm(self, comm) -> None:
         """Route the all-reduces after o_proj and down_proj through a ``PeerAllReduce``."""

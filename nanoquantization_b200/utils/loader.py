@@ -1,4 +1,7 @@
-"""Checkpoint reader and writer for the quantised Qwen3 models.
+"""Checkpoint reader and writer.
+
+A model with ``checkpoint_tensors()`` names the destination of every tensor itself (Vemedra: plain linears, merged
+when loaded) and must find all of them.  What follows is the format of the quantised Qwen3 models.
 
 On-disk format: the reference's (``nanoquantization/utils/loader.py:20-48`` reads
 it, ``scripts/qwen3_0pt6_billion.py:179-235`` writes it): ``*.safetensors``
@@ -65,7 +68,11 @@ def shard_slices(name: str, shape: tuple[int, ...], tp_size: int, tp_rank: int, 
     return full  # embeddings and norms are replicated
 
 
-def _destination(model: nn.Module, weight_name: str) -> torch.Tensor:
+def _destination(model: nn.Module, weight_name: str, named: Optional[dict] = None) -> torch.Tensor:
+    if named is not None:  # the model says where each checkpoint tensor goes (views of merged weights among them)
+        if weight_name not in named:
+            raise AttributeError(f"`{weight_name}` is not a tensor of this model")
+        return named[weight_name]
     # a parameter first, then a buffer (qweight, qscales, qzeros are buffers): loader.py:38-47
     try:
         return model.get_parameter(weight_name)
@@ -99,15 +106,20 @@ def load_model(model: nn.Module, path: str, *, tp_size: Optional[int] = None, tp
     tensor_files = sorted(glob.glob(os.path.join(path, "*.safetensors")))
     if not tensor_files:
         raise FileNotFoundError(f"no *.safetensors under {path}")
+    named = model.checkpoint_tensors() if hasattr(model, "checkpoint_tensors") else None
+    missing = set(named or ())
     for tensor_file in tensor_files:
         with safe_open(tensor_file, framework="pt", device="cpu") as f:
             for weight_name in f.keys():
-                dst = _destination(model, weight_name)
+                dst = _destination(model, weight_name, named)
+                missing.discard(weight_name)
                 src = f.get_slice(weight_name)
                 part = src[shard_slices(weight_name, tuple(src.get_shape()), tp_size, tp_rank, group_size)]
                 if tuple(part.shape) != tuple(dst.shape):
                     raise ValueError(f"`{weight_name}`: this rank's slice has shape {tuple(part.shape)}, the model expects {tuple(dst.shape)}")
                 dst.data.copy_(part)
+    if missing:
+        raise ValueError(f"the checkpoint lacks {len(missing)} tensors of the model, `{min(missing)}` among them")
 
 
 def save_model(model: nn.Module, path: str, *, config: Optional[dict] = None, w_bits: int = 4, group_size: int = 128,

@@ -8,25 +8,24 @@ from nanoquantization_b200 import _lib
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 
 
-def _declared():
-    names = []
-    inc = os.path.join(ROOT, "include")
-    for f in sorted(os.listdir(inc)):
-        if f.endswith(".h"):
-            src = open(os.path.join(inc, f)).read()
-            src = re.sub(r"/\*.*?\*/", "", src, flags=re.S)
-            names += re.findall(r"\b(nqb200_[a-z0-9_]+)\s*\(", src)
-    return sorted(set(names))
+LIBRARIES = {"nqb200.h": (_lib.load, _lib.SIGNATURES), "nqb200_mixers.h": (_lib.load_mixers, _lib.MIXER_SIGNATURES)}
+
+
+def _declared(header):
+    src = open(os.path.join(ROOT, "include", header)).read()
+    src = re.sub(r"/\*.*?\*/", "", src, flags=re.S)
+    return sorted(set(re.findall(r"\b(nqb200_[a-z0-9_]+)\s*\(", src)))
 
 
 def test_every_declared_symbol_is_exported_and_bound():
-    lib = _lib.load()
-    declared = _declared()
-    assert len(declared) >= 8
-    for name in declared:
-        assert hasattr(lib, name), f"{name} declared in include/ but not exported"
-        assert name in _lib.SIGNATURES, f"{name} has no ctypes signature"
-    assert sorted(_lib.SIGNATURES) == declared
+    assert sorted(f for f in os.listdir(os.path.join(ROOT, "include")) if f.endswith(".h")) == sorted(LIBRARIES)
+    for header, (load, signatures) in LIBRARIES.items():
+        lib, declared = load(), _declared(header)
+        assert len(declared) >= 8
+        for name in declared:
+            assert hasattr(lib, name), f"{name} declared in include/{header} but not exported"
+            assert name in signatures, f"{name} has no ctypes signature"
+        assert sorted(signatures) == declared
 
 
 def test_host_only_entry_points():
@@ -94,4 +93,5 @@ def test_prefill_dispatch_is_a_host_side_decision():
 
 def test_library_is_not_older_than_its_sources():
     from nanoquantization_b200.csrc import build
-    assert not build._stale(), "libnqb200.so is older than csrc/: rebuild with python -m nanoquantization_b200.csrc.build"
+    for path in build.LIBRARIES:
+        assert not build._stale(path), f"{path} is older than csrc/: rebuild with python -m nanoquantization_b200.csrc.build"
