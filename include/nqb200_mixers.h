@@ -39,7 +39,7 @@ int nqb200_stream_add(float* x, const int64_t* ids, const void* embed, const flo
 int nqb200_rmsnorm_rows(const float* x, const int64_t* rows, const float* weight, void* out, int64_t n_rows,
                         int64_t width, float eps, int dtype, void* stream);
 
-/* h = RMSnorm(x) * weight; out[t, c] = h[t, c] + sum_j conv[c * taps + j] h[t - taps + 1 + j, c], rounded to
+/* h = RMSnorm(x) * weight; out[t, c] = h[t, c] + sum_j conv[j * width + c] h[t - taps + 1 + j, c], rounded to
  * dtype.  state float [slots, taps - 1, width] holds each sequence's last taps - 1 rows of h and is updated. */
 int nqb200_rmsnorm_conv(const float* x, const float* weight, const float* conv, float* state, void* out,
                         const nqb200_batch* b, int64_t width, int64_t taps, float eps, int dtype, void* stream);
@@ -70,6 +70,20 @@ int nqb200_retention(const void* proj, int64_t stride, int64_t q_off, int64_t k_
                      float* state, float* o, int64_t heads, int64_t dim, int64_t vdim, const nqb200_batch* b, int dtype,
                      void* stream);
 
+typedef struct {
+  int32_t heads, dim, vdim;
+  float eps, out_scale;
+  const float* decay;     /* [heads] */
+} nqb200_retention_desc;
+
+/* Prompts (bf16): retention in chunkwise form with norm and gate.  proj holds q | k | v | gate from column off; the
+ * result goes to act from column act_col.  chunk_states: scratch, nqb200_retention_chunks(tokens, batch) * heads * dim
+ * * vdim floats. */
+int nqb200_retention_prefill(const void* proj, int64_t stride, int64_t off, void* act, int64_t act_stride, int64_t act_col,
+                             const nqb200_retention_desc* r, float* state, float* chunk_states, const nqb200_batch* b, void* stream);
+int nqb200_retention_prefill_supported(const nqb200_retention_desc* r, int64_t stride, int64_t off, int64_t act_stride, int64_t act_col);
+int64_t nqb200_retention_chunks(int64_t tokens, int64_t batch);
+
 /* out[t * out_stride + h * vdim + c] = out_scale * o / rms(o over the head) * silu(gate[t * gate_stride + h * vdim + c]). */
 int nqb200_head_norm_gate(const float* o, const void* gate, int64_t gate_stride, void* out, int64_t out_stride,
                           int64_t tokens, int64_t heads, int64_t vdim, float eps, float out_scale, int dtype, void* stream);
@@ -83,6 +97,28 @@ int nqb200_mingru(const void* proj, int64_t stride, int64_t z_off, int64_t x_off
 
 /* out[t, i] = g sigmoid(1.702 g) (u + 1), g = min(gate_up[t, i], limit), u = clamp(gate_up[t, ff + i], -limit, limit). */
 int nqb200_clamped_glu(const void* gate_up, void* out, int64_t tokens, int64_t ff, float limit, int dtype, void* stream);
+
+/* ---- decode steps: at most 16 tokens, bf16 ---------------------------------------------------------------- */
+
+enum { NQB200_DENSE_BF16 = 0, NQB200_DENSE_F32 = 1, NQB200_DENSE_RESIDUAL = 2 };
+
+/* y = x w^T, x bf16 [M, K], w bf16 [N, K], M <= 16, K % 8 == 0.  mode: y as bf16, y as float, or out float += y. */
+int nqb200_dense_decode(const void* x, const void* w, void* out, int64_t M, int64_t N, int64_t K, int mode, void* stream);
+
+/* w [2 ff, K] = gate rows, then up rows; out bf16 [M, ff] as nqb200_clamped_glu of the product (not rounded between). */
+int nqb200_dense_decode_glu(const void* x, const void* w, void* out, int64_t M, int64_t ff, int64_t K, float limit, void* stream);
+
+/* w [3 width, K] = z, x and gate rows; one token per sequence: product and nqb200_mingru update in one launch. */
+int nqb200_dense_decode_mingru(const void* x, const void* w, const float* z_bias, const float* x_bias, float* state, void* out,
+                               int64_t width, int64_t K, const nqb200_batch* b, void* stream);
+
+/* One token per sequence: rotary embedding, K/V store and attention (columns q | k | v of proj from a_off, output
+ * from column a_col of act), and retention with norm and gate (columns q | k | v | g from r_off, output from r_col),
+ * in one launch.  a or r may be NULL.  Sizes as nqb200_mixer_decode_supported says. */
+int nqb200_mixer_decode(const void* proj, int64_t stride, void* act, int64_t act_stride, const nqb200_attention* a,
+                        const float* inv_freq, int64_t rot, int64_t a_off, int64_t a_col, void* k_cache, void* v_cache,
+                        const nqb200_retention_desc* r, int64_t r_off, int64_t r_col, float* state, const nqb200_batch* b, void* stream);
+int nqb200_mixer_decode_supported(const nqb200_attention* a, const nqb200_retention_desc* r);
 
 #ifdef __cplusplus
 }

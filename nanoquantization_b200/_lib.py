@@ -79,6 +79,14 @@ class AttentionDesc(ctypes.Structure):
                 ("out_scale", ctypes.c_float)]
 
 
+class RetentionDesc(ctypes.Structure):
+    """nqb200_retention_desc of include/nqb200_mixers.h."""
+    _fields_ = [("heads", ctypes.c_int32), ("dim", ctypes.c_int32), ("vdim", ctypes.c_int32), ("eps", ctypes.c_float),
+                ("out_scale", ctypes.c_float), ("decay", _vp)]
+
+
+DENSE_BF16, DENSE_F32, DENSE_RESIDUAL = 0, 1, 2
+_ret = ctypes.POINTER(RetentionDesc)
 _step, _att, _f32 = ctypes.POINTER(StepDesc), ctypes.POINTER(AttentionDesc), ctypes.c_float
 # mirrors include/nqb200_mixers.h one to one
 MIXER_SIGNATURES = {
@@ -91,6 +99,14 @@ MIXER_SIGNATURES = {
     "nqb200_head_norm_gate": (_int, [_vp, _vp, _i64, _vp, _i64, _i64, _i64, _i64, _f32, _f32, _int, _vp]),
     "nqb200_mingru": (_int, [_vp, _i64, _i64, _i64, _i64, _vp, _vp, _vp, _vp, _i64, _step, _int, _vp]),
     "nqb200_clamped_glu": (_int, [_vp, _vp, _i64, _i64, _f32, _int, _vp]),
+    "nqb200_retention_prefill": (_int, [_vp, _i64, _i64, _vp, _i64, _i64, _ret, _vp, _vp, _step, _vp]),
+    "nqb200_retention_prefill_supported": (_int, [_ret, _i64, _i64, _i64, _i64]),
+    "nqb200_retention_chunks": (_i64, [_i64, _i64]),
+    "nqb200_dense_decode": (_int, [_vp, _vp, _vp, _i64, _i64, _i64, _int, _vp]),
+    "nqb200_dense_decode_glu": (_int, [_vp, _vp, _vp, _i64, _i64, _i64, _f32, _vp]),
+    "nqb200_dense_decode_mingru": (_int, [_vp] * 6 + [_i64, _i64, _step, _vp]),
+    "nqb200_mixer_decode_supported": (_int, [_att, _ret]),
+    "nqb200_mixer_decode": (_int, [_vp, _i64, _vp, _i64, _att, _vp, _i64, _i64, _i64, _vp, _vp, _ret, _i64, _i64, _vp, _step, _vp]),
 }
 
 _lib = None

@@ -135,6 +135,8 @@ extern "C" int nqb200_chunk_attention(const void* q, int64_t q_stride, const voi
   if (!mixer_dtype(dtype)) return NQB200_ERR_BAD_DTYPE;
   if (b->tokens == 0) return NQB200_OK;
   if (!q || !k_cache || !v_cache || !out) return NQB200_ERR_NULL_POINTER;
+  if (dtype == NQB200_BF16 && b->max_len > 1 && attention_prefill_supports(q, q_stride, k_cache, v_cache, out, out_stride, a))
+    return attention_prefill(q, q_stride, k_cache, v_cache, out, out_stride, a, b, (cudaStream_t)stream);
   const dim3 grid((unsigned)b->max_len, (unsigned)a->heads, (unsigned)b->batch), block(kSimpleKeys);
   const size_t smem = (size_t)a->dim * sizeof(float);
 #define NQB200_ATT(T)                                                                                                              \

@@ -70,7 +70,6 @@ __global__ void __launch_bounds__(256) rmsnorm_conv_kernel(const float* __restri
   const int cnt = min(tile, n - first);
   for (int c = threadIdx.x; c < width; c += blockDim.x) {
     const float w = weight[c];
-    const float* cw = conv + (size_t)c * taps;
     for (int i = 0; i < cnt; ++i) {
       const int tok = first + i;
       const float h = x[(size_t)(t0 + tok) * width + c] * inv_s[halo + i] * w;
@@ -80,9 +79,9 @@ __global__ void __launch_bounds__(256) rmsnorm_conv_kernel(const float* __restri
         float hv = 0.f;
         if (src >= 0) hv = x[(size_t)(t0 + src) * width + c] * inv_s[i + j] * w;
         else if (!fresh) hv = st[(size_t)(src + halo) * width + c];
-        acc += cw[j] * hv;
+        acc += conv[(size_t)j * width + c] * hv;
       }
-      acc += cw[halo] * h;
+      acc += conv[(size_t)halo * width + c] * h;
       out[(size_t)(t0 + tok) * width + c] = from_f<T>(h + acc);
     }
     if (head) {
@@ -95,6 +94,160 @@ __global__ void __launch_bounds__(256) rmsnorm_conv_kernel(const float* __restri
       }
     }
   }
+}
+
+template <typename T> __device__ __forceinline__ void store4(T* p, float4 v);
+template <> __device__ __forceinline__ void store4<float>(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+template <> __device__ __forceinline__ void store4<bf16>(bf16* p, float4 v) {
+  uint2 r;
+  r.x = (uint32_t)__bfloat16_as_ushort(__float2bfloat16_rn(v.x)) | ((uint32_t)__bfloat16_as_ushort(__float2bfloat16_rn(v.y)) << 16);
+  r.y = (uint32_t)__bfloat16_as_ushort(__float2bfloat16_rn(v.z)) | ((uint32_t)__bfloat16_as_ushort(__float2bfloat16_rn(v.w)) << 16);
+  *reinterpret_cast<uint2*>(p) = r;
+}
+__device__ __forceinline__ float4 ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 mul4(float4 a, float4 b) { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); }
+__device__ __forceinline__ float4 scale4(float4 a, float s) { return make_float4(a.x * s, a.y * s, a.z * s, a.w * s); }
+__device__ __forceinline__ void fma4(float4& d, float4 a, float4 b) { d.x += a.x * b.x; d.y += a.y * b.y; d.z += a.z * b.z; d.w += a.w * b.w; }
+
+// The same for widths that are multiples of 4 and short filters: float4 accesses, and the last taps - 1 rows of h
+// stay in registers while a thread walks down the tile's tokens.
+constexpr int kConvTile = 16;
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(256) rmsnorm_conv_vec_kernel(const float* __restrict__ x, const float* __restrict__ weight,
+                                                               const float* __restrict__ conv, float* state, T* __restrict__ out,
+                                                               const nqb200_batch bt, int width, float eps) {
+  constexpr int HALO = TAPS - 1;
+  __shared__ float inv_s[kConvTile + 2 * HALO];
+  grid_launch_dependents();
+  grid_dependency_wait();
+  const int b = blockIdx.y, t0 = bt.cu[b], n = bt.cu[b + 1] - t0, first = blockIdx.x * kConvTile;
+  if (first >= n) return;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const bool head = first == 0;
+  for (int r = warp; r < kConvTile + HALO + (head ? HALO : 0); r += 8) {
+    const int tok = r < kConvTile + HALO ? first - HALO + r : n - HALO + (r - HALO - kConvTile);
+    if (tok < 0 || tok >= n) continue;
+    const float* row = x + (size_t)(t0 + tok) * width;
+    float ss = 0.f;
+    for (int c = lane * 4; c < width; c += 128) {
+      const float4 v = ld4(row + c);
+      ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    }
+    ss = warp_sum(ss);
+    if (lane == 0) inv_s[r] = 1.f / sqrtf(ss / (float)width + eps);
+  }
+  __syncthreads();
+  const bool fresh = bt.pos0[b] == 0;
+  float* st = state + (size_t)bt.slot[b] * HALO * width;
+  const int cnt = min(kConvTile, n - first);
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int c = threadIdx.x * 4; c < width; c += 1024) {
+    const float4 w = ld4(weight + c);
+    float4 cw[TAPS], win[HALO];
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) cw[j] = ld4(conv + (size_t)j * width + c);
+    float4 old[HALO];   // the state as it was: read whole before it is written
+#pragma unroll
+    for (int j = 0; j < HALO; ++j) old[j] = (head && !fresh) ? ld4(st + (size_t)j * width + c) : zero;
+#pragma unroll
+    for (int j = 0; j < HALO; ++j) {
+      const int src = first - HALO + j;
+      win[j] = src >= 0 ? mul4(scale4(ld4(x + (size_t)(t0 + src) * width + c), inv_s[j]), w) : old[j];
+    }
+#pragma unroll 4
+    for (int i = 0; i < cnt; ++i) {
+      const float4 h = mul4(scale4(ld4(x + (size_t)(t0 + first + i) * width + c), inv_s[HALO + i]), w);
+      float4 acc = h;
+#pragma unroll
+      for (int j = 0; j < HALO; ++j) fma4(acc, cw[j], win[j]);
+      fma4(acc, cw[HALO], h);
+      store4<T>(out + (size_t)(t0 + first + i) * width + c, acc);
+#pragma unroll
+      for (int j = 0; j + 1 < HALO; ++j) win[j] = win[j + 1];
+      win[HALO - 1] = h;
+    }
+    if (head) {
+#pragma unroll
+      for (int r = 0; r < HALO; ++r) {
+        const int src = n - HALO + r;
+        float4 hv = zero;
+        if (src >= 0) {
+          hv = mul4(scale4(ld4(x + (size_t)(t0 + src) * width + c), inv_s[HALO + kConvTile + r]), w);
+        } else {
+#pragma unroll
+          for (int j = 0; j < HALO; ++j)
+            if (j == src + HALO) hv = old[j];
+        }
+        *reinterpret_cast<float4*>(st + (size_t)r * width + c) = hv;
+      }
+    }
+  }
+}
+
+// One token per sequence: a CTA takes the token, the row stays in shared memory between the sum of squares and the use.
+template <typename T>
+__global__ void __launch_bounds__(512) rmsnorm_conv_decode_kernel(const float* __restrict__ x, const float* __restrict__ weight,
+                                                                  const float* __restrict__ conv, float* state, T* __restrict__ out,
+                                                                  const nqb200_batch bt, int width, int taps, float eps) {
+  extern __shared__ float4 row_s[];
+  __shared__ float red[16];
+  grid_launch_dependents();
+  grid_dependency_wait();
+  const int b = blockIdx.x, t0 = bt.cu[b];
+  if (bt.cu[b + 1] == t0) return;
+  const int halo = taps - 1;
+  const float* row = x + (size_t)t0 * width;
+  float* st = state + (size_t)bt.slot[b] * halo * width;
+  const bool fresh = bt.pos0[b] == 0;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c * 4 < width; c += 512) {
+    const float4 v = ld4(row + c * 4);
+    row_s[c] = v;
+    ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+  }
+  ss = warp_sum(ss);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+  __syncthreads();
+  float tot = 0.f;
+#pragma unroll
+  for (int w = 0; w < 16; ++w) tot += red[w];
+  const float inv = 1.f / sqrtf(tot / (float)width + eps);
+  for (int c = threadIdx.x * 4; c < width; c += 2048) {
+    const float4 h = mul4(scale4(row_s[c / 4], inv), ld4(weight + c));
+    float4 acc = h;
+    fma4(acc, ld4(conv + (size_t)halo * width + c), h);
+    for (int j = 0; j < halo; ++j) {
+      const float4 s = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : ld4(st + (size_t)j * width + c);
+      fma4(acc, ld4(conv + (size_t)j * width + c), s);
+      if (j > 0) *reinterpret_cast<float4*>(st + (size_t)(j - 1) * width + c) = s;
+    }
+    if (halo > 0) *reinterpret_cast<float4*>(st + (size_t)(halo - 1) * width + c) = h;
+    store4<T>(out + (size_t)t0 * width + c, acc);
+  }
+}
+
+template <typename T>
+static int launch_rmsnorm_conv(const float* x, const float* weight, const float* conv, float* state, T* out, const nqb200_batch* b,
+                               int width, int taps, float eps, cudaStream_t st) {
+  const bool vec = width % 4 == 0 && aligned16(x) && aligned16(weight) && aligned16(conv) && aligned16(out) && (!state || aligned16(state));
+  if (vec && b->max_len == 1 && width <= 8192) {
+    return launch_overlapped(rmsnorm_conv_decode_kernel<T>, dim3((unsigned)b->batch), dim3(512), (size_t)width * 4, st, x, weight, conv, state, out,
+                             *b, width, taps, eps);
+  }
+  const dim3 block(256);
+  if (vec && taps >= 2 && taps <= 5) {
+    const dim3 grid((unsigned)((b->max_len + kConvTile - 1) / kConvTile), (unsigned)b->batch);
+#define NQB200_CONV(K) return launch_overlapped(rmsnorm_conv_vec_kernel<T, K>, grid, block, 0, st, x, weight, conv, state, out, *b, width, eps)
+    if (taps == 2) NQB200_CONV(2);
+    if (taps == 3) NQB200_CONV(3);
+    if (taps == 4) NQB200_CONV(4);
+    NQB200_CONV(5);
+#undef NQB200_CONV
+  }
+  const int halo = taps - 1, tile = halo > 8 ? halo : 8;
+  const dim3 grid((unsigned)((b->max_len + tile - 1) / tile), (unsigned)b->batch);
+  return launch_overlapped(rmsnorm_conv_kernel<T>, grid, block, (size_t)(2 * halo + tile) * sizeof(float), st, x, weight, conv, state, out, *b,
+                           width, taps, tile, eps);
 }
 
 template <typename T>
@@ -147,12 +300,9 @@ extern "C" int nqb200_rmsnorm_conv(const float* x, const float* weight, const fl
   if (!mixer_dtype(dtype)) return NQB200_ERR_BAD_DTYPE;
   if (b->tokens == 0) return NQB200_OK;
   if (!x || !weight || !conv || !out || (taps > 1 && !state)) return NQB200_ERR_NULL_POINTER;
-  const int halo = (int)taps - 1, tile = halo > 8 ? halo : 8;
-  const dim3 grid((unsigned)((b->max_len + tile - 1) / tile), (unsigned)b->batch), block(256);
-  const size_t smem = (size_t)(2 * halo + tile) * sizeof(float);
   if (dtype == NQB200_F32)
-    return launch_overlapped(rmsnorm_conv_kernel<float>, grid, block, smem, (cudaStream_t)stream, x, weight, conv, state, (float*)out, *b, (int)width, (int)taps, tile, eps);
-  return launch_overlapped(rmsnorm_conv_kernel<bf16>, grid, block, smem, (cudaStream_t)stream, x, weight, conv, state, (bf16*)out, *b, (int)width, (int)taps, tile, eps);
+    return launch_rmsnorm_conv<float>(x, weight, conv, state, (float*)out, b, (int)width, (int)taps, eps, (cudaStream_t)stream);
+  return launch_rmsnorm_conv<bf16>(x, weight, conv, state, (bf16*)out, b, (int)width, (int)taps, eps, (cudaStream_t)stream);
 }
 
 extern "C" int nqb200_clamped_glu(const void* gate_up, void* out, int64_t tokens, int64_t ff, float limit, int dtype, void* stream) {

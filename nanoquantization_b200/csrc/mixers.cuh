@@ -31,6 +31,12 @@ __device__ __forceinline__ size_t kv_row(const nqb200_batch& bt, int b, int p) {
   return (size_t)bt.table[(size_t)b * bt.table_width + p / bt.block_size] * bt.block_size + p % bt.block_size;
 }
 
+// mixer_prefill.cu: the tensor-core attention for prompts.
+bool attention_prefill_supports(const void* q, int64_t q_stride, const void* k_cache, const void* v_cache, const void* out, int64_t out_stride,
+                                const nqb200_attention* a);
+int attention_prefill(const void* q, int64_t q_stride, const void* k_cache, const void* v_cache, void* out, int64_t out_stride,
+                      const nqb200_attention* a, const nqb200_batch* b, cudaStream_t st);
+
 static inline int check_batch(const nqb200_batch* b, bool paged) {
   if (!b) return NQB200_ERR_NULL_POINTER;
   if (b->batch < 0 || b->tokens < 0 || b->max_len < 0 || b->max_len > b->tokens || b->batch > 65535) return NQB200_ERR_BAD_SHAPE;

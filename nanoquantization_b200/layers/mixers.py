@@ -41,11 +41,12 @@ def rmsnorm_rows(x: torch.Tensor, rows: Optional[torch.Tensor], weight: torch.Te
 
 def rmsnorm_conv(x: torch.Tensor, weight: torch.Tensor, conv: torch.Tensor, state: torch.Tensor, step, eps: float,
                  dtype: torch.dtype) -> torch.Tensor:
-    """``h + causal_conv(h)`` with ``h`` the RMS norm of ``x``; ``state [slots, taps - 1, width]`` carries the last h."""
+    """``h + causal_conv(h)`` with ``h`` the RMS norm of ``x``; ``conv [taps, width]``; ``state [slots, taps - 1, width]``
+    carries the last h."""
     _lib.require_cuda(x, weight, conv)
     out = torch.empty(x.shape, dtype=dtype, device=x.device)
     _call("nqb200_rmsnorm_conv", x.data_ptr(), weight.data_ptr(), conv.data_ptr(), _ptr(state), out.data_ptr(), ctypes.byref(step.desc),
-          x.shape[1], conv.shape[1], eps, _lib.mixer_dtype_code(dtype))
+          x.shape[1], conv.shape[0], eps, _lib.mixer_dtype_code(dtype))
     return out
 
 
@@ -79,6 +80,28 @@ def head_norm_gate(o: torch.Tensor, gate: torch.Tensor, out: torch.Tensor, eps: 
           out_scale, _lib.mixer_dtype_code(out.dtype))
 
 
+RETENTION_PREFILL_TOKENS = 17   # shorter portions take the token-by-token kernel
+
+
+def retention_gated(proj: torch.Tensor, off: int, desc: _lib.RetentionDesc, decay: torch.Tensor, state: torch.Tensor, act: torch.Tensor,
+                    act_col: int, step) -> None:
+    """Retention with norm and gate: ``proj`` holds q | k | v | gate from column ``off``, the result goes to ``act``
+    from column ``act_col``.  Prompts in bfloat16 run chunkwise on the tensor cores, the rest token by token."""
+    lib = _lib.load_mixers()
+    _, heads, dim, vdim = state.shape
+    if (proj.dtype == torch.bfloat16 and step.max_len >= RETENTION_PREFILL_TOKENS
+            and lib.nqb200_retention_prefill_supported(ctypes.byref(desc), proj.stride(0), off, act.stride(0), act_col)):
+        chunks = lib.nqb200_retention_chunks(step.num_tokens, step.batch)
+        scratch = torch.empty(chunks, heads, dim, vdim, dtype=torch.float32, device=proj.device)
+        _call("nqb200_retention_prefill", proj.data_ptr(), proj.stride(0), off, act.data_ptr(), act.stride(0), act_col, ctypes.byref(desc),
+              state.data_ptr(), scratch.data_ptr(), ctypes.byref(step.desc))
+        return
+    k_off, v_off = off + heads * dim, off + 2 * heads * dim
+    g_off = v_off + heads * vdim
+    o = retention(proj, off, k_off, v_off, decay, state, step)
+    head_norm_gate(o, proj[:, g_off:g_off + heads * vdim], act[:, act_col:act_col + heads * vdim], desc.eps, desc.out_scale)
+
+
 def mingru(proj: torch.Tensor, width: int, z_bias: torch.Tensor, x_bias: torch.Tensor, state: torch.Tensor, step) -> torch.Tensor:
     """``proj [tokens, z | x | g]`` -> gated states ``[tokens, width]``; ``state [slots, width]`` is carried."""
     out = torch.empty(proj.shape[0], width, dtype=proj.dtype, device=proj.device)
@@ -94,15 +117,64 @@ def clamped_glu(gate_up: torch.Tensor, limit: float) -> torch.Tensor:
     return out
 
 
+DECODE_TOKENS = 16   # up to here the linears run as kernels that stream the weights once
+
+
+def decode_sized(x: torch.Tensor, weight: torch.Tensor) -> bool:
+    return x.dtype == torch.bfloat16 and 0 < x.shape[0] <= DECODE_TOKENS and weight.shape[1] % 8 == 0
+
+
+def _dense(x, weight, out, mode):
+    _call("nqb200_dense_decode", x.data_ptr(), weight.data_ptr(), out.data_ptr(), x.shape[0], weight.shape[0], weight.shape[1], mode)
+    return out
+
+
 def linear(x: torch.Tensor, weight: torch.Tensor, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
-    """``x @ weight.T`` with 32-bit accumulation."""
-    if x.dtype == torch.float32 or out_dtype in (None, x.dtype):
+    """``x @ weight.T`` with 32-bit accumulation: the streaming kernel for decode sizes, a library product otherwise."""
+    dtype = out_dtype or x.dtype
+    if decode_sized(x, weight):
+        out = torch.empty(x.shape[0], weight.shape[0], dtype=dtype, device=x.device)
+        return _dense(x, weight, out, _lib.DENSE_F32 if dtype == torch.float32 else _lib.DENSE_BF16)
+    if x.dtype == dtype:
         return torch.mm(x, weight.t())
-    return torch.mm(x, weight.t(), out_dtype=out_dtype)
+    return torch.mm(x, weight.t(), out_dtype=dtype)
 
 
 def linear_residual_(stream: torch.Tensor, y: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
     """``stream += y @ weight.T``: the product is added to the float32 stream before any rounding."""
+    if decode_sized(y, weight):
+        return _dense(y, weight, stream, _lib.DENSE_RESIDUAL)
     if y.dtype == torch.float32:
         return stream.addmm_(y, weight.t())
     return torch.addmm(stream, y, weight.t(), out_dtype=torch.float32, out=stream)
+
+
+def dense_glu(x: torch.Tensor, weight: torch.Tensor, limit: float) -> torch.Tensor:
+    """Decode sizes: the merged gate | up product with the clamped GLU inside."""
+    out = torch.empty(x.shape[0], weight.shape[0] // 2, dtype=x.dtype, device=x.device)
+    _call("nqb200_dense_decode_glu", x.data_ptr(), weight.data_ptr(), out.data_ptr(), x.shape[0], out.shape[1], weight.shape[1], limit)
+    return out
+
+
+def dense_mingru(x: torch.Tensor, weight: torch.Tensor, z_bias: torch.Tensor, x_bias: torch.Tensor, state: torch.Tensor, step) -> torch.Tensor:
+    """Decode sizes, one token per sequence: the merged z | x | g product with the minGRU update inside."""
+    width = weight.shape[0] // 3
+    out = torch.empty(x.shape[0], width, dtype=x.dtype, device=x.device)
+    _call("nqb200_dense_decode_mingru", x.data_ptr(), weight.data_ptr(), z_bias.data_ptr(), x_bias.data_ptr(), state.data_ptr(), out.data_ptr(),
+          width, weight.shape[1], ctypes.byref(step.desc))
+    return out
+
+
+def mixer_decode_supported(att: Optional[_lib.AttentionDesc], ret: Optional[_lib.RetentionDesc]) -> bool:
+    lib = _lib.load_mixers()
+    return bool(lib.nqb200_mixer_decode_supported(None if att is None else ctypes.byref(att), None if ret is None else ctypes.byref(ret)))
+
+
+def mixer_decode(proj: torch.Tensor, act: torch.Tensor, att, ret, step) -> None:
+    """One token per sequence, attention and retention in one launch.  ``att = (desc, inv_freq, first projection
+    column, first output column, k_cache, v_cache)``, ``ret = (desc, first projection column, first output column,
+    state)``; either may be None."""
+    a = (None, None, 0, 0, 0, None, None) if att is None else (
+        ctypes.byref(att[0]), _ptr(att[1]), 2 * att[1].numel(), att[2], att[3], att[4].data_ptr(), att[5].data_ptr())
+    r = (None, 0, 0, None) if ret is None else (ctypes.byref(ret[0]), ret[1], ret[2], ret[3].data_ptr())
+    _call("nqb200_mixer_decode", proj.data_ptr(), proj.stride(0), act.data_ptr(), act.stride(0), *a, *r, ctypes.byref(step.desc))

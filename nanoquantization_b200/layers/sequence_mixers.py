@@ -82,12 +82,11 @@ class RetentionMixer(nn.Module):
     def checkpoint(self, prefix):
         return {}
 
+    def desc(self) -> _lib.RetentionDesc:
+        return _lib.RetentionDesc(self.heads, self.dim, self.vdim, self.eps, self.out_scale, self.decay.data_ptr())
+
     def mix(self, proj, col, act, act_col, layer_step):
-        q_off, k_off = col, col + self.heads * self.dim
-        v_off = k_off + self.heads * self.dim
-        g_off = v_off + self.heads * self.vdim
-        o = ops.retention(proj, q_off, k_off, v_off, self.decay, layer_step.state["retention"], layer_step.batch)
-        ops.head_norm_gate(o, proj[:, g_off:g_off + self.out_columns], act[:, act_col:act_col + self.out_columns], self.eps, self.out_scale)
+        ops.retention_gated(proj, col, self.desc(), self.decay, layer_step.state["retention"], act, act_col, layer_step.batch)
 
 
 class ParallelMixer(nn.Module):
@@ -100,6 +99,26 @@ class ParallelMixer(nn.Module):
         self.columns = sum(m.out_columns for m in parts.values())
         _buffer(self, "w_in", self.rows, width, dtype=dtype, device=device)
         _buffer(self, "w_out", width, self.columns, dtype=dtype, device=device)
+        # (mixer, first row of its projections, first column of its output), for the one-launch decode step
+        self._attention = self._retention = None
+        self._at_once = None
+        row = col = 0
+        for m in parts.values():
+            if isinstance(m, AttentionMixer):
+                self._attention = (m, row, col)
+            elif isinstance(m, RetentionMixer):
+                self._retention = (m, row, col)
+            row += sum(n for _, n in m.in_parts)
+            col += m.out_columns
+
+    def _decodes_at_once(self, h, batch) -> bool:
+        if batch.max_len != 1 or h.dtype != torch.bfloat16:
+            return False
+        if self._at_once is None:
+            self._at_once = (len(self.parts) == (self._attention is not None) + (self._retention is not None)
+                             and ops.mixer_decode_supported(self._attention and self._attention[0].desc(),
+                                                            self._retention and self._retention[0].desc()))
+        return self._at_once
 
     def kv_spec(self):
         specs = [s for s in (m.kv_spec() for m in self.parts.values()) if s is not None]
@@ -126,6 +145,12 @@ class ParallelMixer(nn.Module):
         """``x += mixer(h)`` on the float32 stream."""
         proj = ops.linear(h, self.w_in)
         act = torch.empty(h.shape[0], self.columns, dtype=h.dtype, device=h.device)
+        if self._decodes_at_once(h, layer_step.batch):
+            att, ret = self._attention, self._retention
+            ops.mixer_decode(proj, act, att and (att[0].desc(), att[0].inv_freq, att[1], att[2], layer_step.k_cache, layer_step.v_cache),
+                             ret and (ret[0].desc(), ret[1], ret[2], layer_step.state["retention"]), layer_step.batch)
+            ops.linear_residual_(x, act, self.w_out)
+            return
         row = col = 0
         for m in self.parts.values():
             m.mix(proj, row, act, col, layer_step)
@@ -157,6 +182,10 @@ class MinGRUMixer(nn.Module):
                 prefix + "z.b": self.z_bias, prefix + "x.b": self.x_bias}
 
     def forward(self, x, h, layer_step):
+        if layer_step.batch.max_len == 1 and ops.decode_sized(h, self.w_in):
+            y = ops.dense_mingru(h, self.w_in, self.z_bias, self.x_bias, layer_step.state["mingru"], layer_step.batch)
+            ops.linear_residual_(x, y, self.w_out)
+            return
         proj = ops.linear(h, self.w_in)
         y = ops.mingru(proj, self.size, self.z_bias, self.x_bias, layer_step.state["mingru"], layer_step.batch)
         ops.linear_residual_(x, y, self.w_out)
@@ -175,6 +204,9 @@ class ClampedGLU(nn.Module):
         return {prefix + "gate": self.w_in[:self.ff], prefix + "up": self.w_in[self.ff:], prefix + "down": self.w_out}
 
     def forward(self, x, h):
+        if ops.decode_sized(h, self.w_in):
+            ops.linear_residual_(x, ops.dense_glu(h, self.w_in, self.limit), self.w_out)
+            return
         ops.linear_residual_(x, ops.clamped_glu(ops.linear(h, self.w_in), self.limit), self.w_out)
 
 
@@ -185,7 +217,10 @@ class ConvNorm(nn.Module):
         super().__init__()
         self.eps, self.taps, self.dtype = float(eps), taps, dtype
         _buffer(self, "weight", width, dtype=torch.float32, device=device)
-        _buffer(self, "conv", width, taps, dtype=torch.float32, device=device)
+        _buffer(self, "conv", taps, width, dtype=torch.float32, device=device)   # the checkpoint's [width, taps], transposed
+
+    def checkpoint(self, norm, conv):
+        return {norm: self.weight, conv: self.conv.t()}
 
     def state_shape(self):
         return (self.taps - 1, self.weight.numel())

@@ -78,10 +78,10 @@ class VemedraLayer(nn.Module):
 
     def checkpoint(self, prefix: str) -> dict:
         out = self.mixer.checkpoint(prefix + "mix.")
-        out.update({prefix + "norm1": self.norm1.weight, prefix + "canon1": self.norm1.conv})
+        out.update(self.norm1.checkpoint(prefix + "norm1", prefix + "canon1"))
         if self.mlp is not None:
             out.update(self.mlp.checkpoint(prefix + "mlp."))
-            out.update({prefix + "norm2": self.norm2.weight, prefix + "canon2": self.norm2.conv})
+            out.update(self.norm2.checkpoint(prefix + "norm2", prefix + "canon2"))
         return out
 
     def forward(self, x: torch.Tensor, layer_step) -> None:

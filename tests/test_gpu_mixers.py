@@ -105,7 +105,7 @@ def test_norm_with_input_convolution(schedule, taps, width, dtype):
     w, cw = 1 + 0.3 * rand(width, seed=9), rand(width, taps, seed=10)
     r = Replay(LENGTHS, schedule)
     state = torch.full((r.num_slots, taps - 1, width), 1e4, device=DEV)     # what an earlier owner left
-    got = r.run(x, lambda b, rows: ops.rmsnorm_conv(rows, w.to(DEV), cw.to(DEV), state, b, 1e-3, dtype))
+    got = r.run(x, lambda b, rows: ops.rmsnorm_conv(rows, w.to(DEV), cw.t().contiguous().to(DEV), state, b, 1e-3, dtype))
     for i in range(len(LENGTHS)):
         h = O.rms_norm(x[i].double(), 1e-3, w.double())
         close(got[i], h + O.causal_conv(h, cw.double()), dtype)
@@ -284,6 +284,161 @@ def test_clamped_glu(dtype):
     gu = (rand(13, 2 * 75, seed=1) * 3).to(dtype)
     gu[0, :4] = torch.tensor([1.5, 1.50001, -9.0, 0.0])
     close(ops.clamped_glu(gu.to(DEV), 1.5), O.clamped_glu(gu[:, :75].double(), gu[:, 75:].double(), 1.5), dtype)
+
+
+# ------------------------------------------------------------------ retention with norm and gate, prompts in bf16
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("sizes", [(2, 64, 64), (3, 32, 128), (1, 128, 256), (2, 256, 48), (2, 24, 200), (1, 20, 28)], ids=str)
+@pytest.mark.parametrize("lengths", [(300, 70), (530, 1, 256)], ids=str)
+def test_retention_of_prompts(lengths, sizes, dtype):
+    """Chunk borders of the chunkwise form fall elsewhere in every schedule; a slow decay carries far."""
+    H, D, V = sizes
+    decay = [1 - 2.0 ** -(3 + 3 * h) for h in range(H)]
+    off, col, eps, scale = 8, 4, 1e-4, 1.3
+    parts = [[rand(n, H, d, seed=10 * i + j).to(dtype) for j, d in enumerate((D, D, V, V))] for i, n in enumerate(lengths)]
+    for q, k, v, g in parts:
+        q += 0.5                       # outputs of ordinary size: the norm would blow up rounding where they vanish
+        k += 0.5
+    want = [scale * O.rms_norm(O.retention(q.double(), k.double() * D ** -0.5, v.double(), decay), eps).flatten(1) * O.silu(g.double().flatten(1))
+            for q, k, v, g in parts]
+    proj = [torch.cat([torch.zeros(len(p[0]), off, dtype=dtype)] + [t.flatten(1) for t in p], 1) for p in parts]
+    dec = torch.tensor(decay, dtype=torch.float64).float().to(DEV)
+    desc = _lib.RetentionDesc(H, D, V, eps, scale, dec.data_ptr())
+    total = sum(lengths)
+    whole = [[(s, n) for s, n in enumerate(lengths)]]
+    cuts = [[(s, k)] for s, n in enumerate(lengths) for k in cut(n, [100, 2, 40, 1, 259])]
+    halves = [[(s, n // 2) for s, n in enumerate(lengths) if n // 2], [(s, n - n // 2) for s, n in enumerate(lengths)]]
+    for schedule in (whole, cuts, halves):
+        r = Replay(lengths, schedule)
+        state = torch.full((r.num_slots, H, D, V), 1e4, device=DEV)
+
+        def fn(b, rows):
+            act = torch.full((rows.shape[0], H * V + 10), 7.0, dtype=dtype, device=DEV)
+            ops.retention_gated(rows, off, desc, dec, state, act, col, b)
+            assert (act[:, :col] == 7).all() and (act[:, col + H * V:] == 7).all()
+            return act[:, col:col + H * V]
+        got = r.run(proj, fn)
+        for i, (q, k, v, g) in enumerate(parts):
+            close(got[i], want[i], dtype, f32=1e-3, bf16=3e-2)
+            S = torch.zeros(H, D, V, dtype=torch.float64)
+            dd = torch.tensor(decay, dtype=torch.float64)[:, None, None]
+            for t in range(lengths[i]):
+                S = dd * S + k[t].double()[:, :, None] * D ** -0.5 * v[t].double()[:, None, :]
+            close(state[r.slots[i]], S, torch.float32, f32=2e-4)
+    assert total > 300
+
+
+# ------------------------------------------------------------------ decode steps
+def dense_case(M, N, K, seed=0):
+    return rand(M, K, seed=seed).bfloat16(), (rand(N, K, seed=seed + 1) * K ** -0.5).bfloat16()
+
+
+@pytest.mark.parametrize("M,N,K", [(1, 16, 8), (1, 40, 40), (3, 33, 104), (8, 512, 256), (9, 100, 1000), (16, 300, 4096), (5, 1, 2056)])
+def test_dense_decode(M, N, K):
+    x, w = dense_case(M, N, K)
+    want = x.double() @ w.double().t()
+    xd, wd = x.to(DEV), w.to(DEV)
+    assert ops.decode_sized(xd, wd)
+    close(ops.linear(xd, wd), want, torch.bfloat16)
+    close(ops.linear(xd, wd, torch.float32), want, torch.float32)
+    stream = rand(M, N, seed=5)
+    close(ops.linear_residual_(stream.to(DEV), xd, wd), stream.double() + want, torch.float32)
+
+
+def test_linears_of_other_sizes_take_the_library():
+    for M, N, K in ((17, 24, 64), (2, 24, 36)):
+        x, w = dense_case(M, N, K)
+        want = x.double() @ w.double().t()
+        assert not ops.decode_sized(x.to(DEV), w.to(DEV))
+        close(ops.linear(x.to(DEV), w.to(DEV), torch.float32), want, torch.float32)
+        stream = rand(M, N, seed=5)
+        got = stream.to(DEV)
+        assert ops.linear_residual_(got, x.to(DEV), w.to(DEV)) is got
+        close(got, stream.double() + want, torch.float32)
+        close(ops.linear_residual_(stream.to(DEV), x.float().to(DEV), w.float().to(DEV)), stream.double() + want, torch.float32)
+
+
+@pytest.mark.parametrize("M,ff,K", [(1, 24, 64), (7, 130, 256), (16, 72, 1000)])
+def test_dense_with_clamped_glu(M, ff, K):
+    x, w = dense_case(M, 2 * ff, K)
+    x *= 3
+    y = x.double() @ w.double().t()
+    close(ops.dense_glu(x.to(DEV), w.to(DEV), 1.7), O.clamped_glu(y[:, :ff], y[:, ff:], 1.7), torch.bfloat16)
+
+
+@pytest.mark.parametrize("B,width,K", [(1, 40, 64), (5, 33, 256), (16, 128, 1000)])
+def test_dense_with_mingru(B, width, K):
+    """Three tokens of every sequence, the first from a slot that another sequence has left."""
+    w = (rand(3 * width, K, seed=1) * K ** -0.5).bfloat16()
+    zb, xb = rand(width, seed=2), rand(width, seed=3)
+    xs = [rand(3, K, seed=10 + i).bfloat16() for i in range(B)]
+    r = Replay((3,) * B, [[(s, 1) for s in range(B)]] * 3)
+    state = torch.full((r.num_slots, width), 1e4, device=DEV)
+    got = r.run(xs, lambda b, rows: ops.dense_mingru(rows, w.to(DEV), zb.to(DEV), xb.to(DEV), state, b))
+    for i in range(B):
+        z, u, g = (xs[i].double() @ w.double().t()).split(width, 1)
+        S = O.min_gru(z + zb.double(), u + xb.double())
+        close(got[i], S * O.silu(g), torch.bfloat16)
+        close(state[r.slots[i]], S[-1], torch.float32)
+
+
+@pytest.mark.parametrize("att", [(4, 2, 24, 40, 13, 16), (2, 2, 64, 64, 1000, 64), (12, 1, 128, 128, 40, 64), (6, 2, 256, 256, 300, 0), (5, 1, 8, 8, 1, 8), None], ids=str)
+@pytest.mark.parametrize("ret", [(3, 20, 28), (2, 64, 64), (2, 128, 256), (1, 9, 33), (1, 300, 600), None], ids=str)
+def test_one_launch_decode_step(att, ret):
+    """Attention and retention of a decode step, side by side in one launch: after a prompt that the other kernels
+    read, and from the first token on."""
+    if att is None and ret is None:
+        return
+    dtype, lengths, decoded = torch.bfloat16, (330, 1, 45), 9
+    H, G, D, V, chunk, rot = att or (0, 0, 0, 0, 1, 0)
+    RH, RD, RV = ret or (0, 0, 0)
+    na, a_off, a_col = H * D + G * (D + V), 3, 6
+    r_off, r_col = a_off + na + 2, a_col + H * V + 3
+    decay = [1 - 2.0 ** -(2 + 3 * h) for h in range(RH)]
+    dec = torch.tensor(decay or [0.0]).float().to(DEV)
+    sink = rand(max(H, 1), seed=3)
+    m = AttentionMixer(heads=H, kv_heads=G, dim=D, vdim=V, chunk=chunk, rot_base=70.0, rot_dims=rot, scale=0.3, softcap=4.0, out_scale=1.7, device=DEV) if att else None
+    if att:
+        m.sink.copy_(sink)
+    rdesc = _lib.RetentionDesc(RH, RD, RV, 1e-4, 0.8, dec.data_ptr()) if ret else None
+    assert ops.mixer_decode_supported(m and m.desc(), rdesc)
+    width = r_off + 2 * RH * (RD + RV) + 1
+    proj = [rand(n, width, seed=i).to(dtype) for i, n in enumerate(lengths)]
+    for p in proj:
+        p[:, r_off:r_off + 2 * RH * RD] += 0.5
+    schedule = [[(s, n - decoded) for s, n in enumerate(lengths) if n > decoded]] + [[(s, 1) for s, n in enumerate(lengths) if k < n and (n > decoded or k == 0)] for k in range(decoded)]
+    r = Replay(lengths, schedule, block_size=16)
+    kc = torch.full((r.num_blocks, 16, max(G, 1), max(D, 1)), 300.0, dtype=dtype, device=DEV)
+    vc = torch.full((r.num_blocks, 16, max(G, 1), max(V, 1)), 300.0, dtype=dtype, device=DEV)
+    state = torch.full((r.num_slots, max(RH, 1), max(RD, 1), max(RV, 1)), 1e4, device=DEV)
+
+    class Step:
+        k_cache, v_cache, batch = kc, vc, None
+
+    def fn(b, rows):
+        act = torch.full((rows.shape[0], r_col + RH * RV + 2), 7.0, dtype=dtype, device=DEV)
+        rows = rows.contiguous()
+        if b.max_len == 1:
+            ops.mixer_decode(rows, act, att and (m.desc(), m.inv_freq, a_off, a_col, kc, vc), ret and (rdesc, r_off, r_col, state), b)
+            assert (act[:, :a_col] == 7).all() and (act[:, a_col + H * V:r_col] == 7).all() and (act[:, -2:] == 7).all()
+            return act
+        Step.batch = b
+        if att:
+            m.mix(rows, a_off, act, a_col, Step)
+        if ret:
+            ops.retention_gated(rows, r_off, rdesc, dec, state, act, r_col, b)
+        return act
+    got = r.run(proj, fn)
+    for i, n in enumerate(lengths):
+        if att:
+            q, k, v = proj[i][:, a_off:a_off + na].float().split([H * D, G * D, G * V], 1)
+            want = oracle_attend(m, q.reshape(n, H, D), k.reshape(n, G, D), v.reshape(n, G, V), 70.0, rot, sink)
+            close(got[i][-decoded:, a_col:a_col + H * V], want.flatten(1)[-decoded:], dtype, bf16=2e-2)
+        if ret:
+            q, k, v, g = proj[i][:, r_off:-1].double().split([RH * RD, RH * RD, RH * RV, RH * RV], 1)
+            o = O.retention(q.reshape(n, RH, RD), k.reshape(n, RH, RD) * RD ** -0.5, v.reshape(n, RH, RV), decay)
+            want = 0.8 * O.rms_norm(o, 1e-4).flatten(1) * O.silu(g)
+            close(got[i][-decoded:, r_col:r_col + RH * RV], want[-decoded:], dtype, bf16=3e-2)
 
 
 def test_bad_arguments_are_errors():
