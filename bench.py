@@ -705,6 +705,268 @@ def decode_bench(world, rank, dev, dtype, batches=(1, 16, 64), context=2048, ste
 
 
 # --------------------------------------------------------------------------
+# Vemedra: layers of a real model's size beside the Qwen3 layers of the same size (--vemedra)
+# --------------------------------------------------------------------------
+VEMEDRA_LAYERS = 8
+
+
+def vemedra_config(layers=VEMEDRA_LAYERS, chunk=4096):
+    """Widths of the Qwen3-8B architecture: 4096 wide, 32 query heads over 8, head size 128, feed-forward 12288; every
+    fourth layer a minGRU, the others attention in chunks beside 16 retention heads."""
+    ff = {"kind": "dense", "ff": 12288, "limit": 7.0}
+    gru = {"type": "mingru", "mixer": {"width": 4096}, "mlp": ff}
+    par = {"type": "parallel", "mlp": ff, "mixer": {
+        "left": {"heads": 32, "kv_heads": 8, "dim": 128, "vdim": 128, "mask": {"size": chunk}, "rot": {"base": 1e6, "dims": 128},
+                 "scale": 128 ** -0.5, "softcap": 50.0},
+        "right": {"heads": 16, "dim": 128, "vdim": 256, "decay": [1 - 2.0 ** -(5 + 0.5 * h) for h in range(16)]}, "left_scale": 1.0, "right_scale": 0.5}}
+    return {"architecture": "Vemedra", "vocab": 151936, "width": 4096, "canon": {"taps": 4}, "norm": {"eps": 1e-6},
+            "layers": [gru if i % 4 == 0 else par for i in range(layers)]}
+
+
+def _device_us(fn, reps):
+    """Microseconds per call of ``fn(i)``, i = 0 .. reps - 1, replayed as one CUDA graph."""
+    fn(0)
+    torch.cuda.synchronize()
+    side = torch.cuda.Stream()
+    side.wait_stream(torch.cuda.current_stream())
+    with torch.cuda.stream(side):
+        for i in range(reps):
+            fn(i)
+    torch.cuda.current_stream().wait_stream(side)
+    torch.cuda.synchronize()
+    graph = torch.cuda.CUDAGraph()
+    with torch.cuda.graph(graph):
+        for i in range(reps):
+            fn(i)
+    for _ in range(3):
+        graph.replay()
+    torch.cuda.synchronize()
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    e0.record()
+    for _ in range(3):
+        graph.replay()
+    e1.record()
+    torch.cuda.synchronize()
+    return e0.elapsed_time(e1) * 1e3 / (3 * reps)
+
+
+def _engine_throughput(eng, vocab, batches, context, prefill, steps=16):
+    """Decode steps per batch size over a given context, and one prompt, as in the Qwen3-8B section."""
+    from nanoquantization_b200.engine import Sequence
+    g = torch.Generator().manual_seed(1)
+    out = {"decode": [], "context": context}
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    for B in batches:
+        eng._graphs.clear()
+        seqs = []
+        for i in range(B):
+            s = Sequence(i, torch.randint(0, vocab, (context,), generator=g).tolist(), 10 ** 9)
+            eng._hold(s, context + 8)
+            s.output.append(1)
+            seqs.append(s)
+        for _ in range(3):
+            eng._decode(seqs)
+        torch.cuda.synchronize()
+        e0.record()
+        for _ in range(steps):
+            eng._decode(seqs)
+        e1.record()
+        torch.cuda.synchronize()
+        ms = e0.elapsed_time(e1) / steps
+        graph = next(iter(eng._graphs.values()))[0]
+        e0.record()
+        for _ in range(steps):
+            graph.replay()
+        e1.record()
+        torch.cuda.synchronize()
+        out["decode"].append({"batch": B, "ms_per_step": round(ms, 3), "tok_per_s": round(B / ms * 1e3, 1),
+                              "graph_ms": round(e0.elapsed_time(e1) / steps, 3)})
+        for s in seqs:
+            eng.drop(s)
+    eng._graphs.clear()
+    seq = Sequence(10 ** 6, torch.randint(0, vocab, (prefill,), generator=g).tolist(), 1)
+    times = []
+    for k in range(5):
+        eng._hold(seq, prefill + 1)
+        torch.cuda.synchronize()
+        e0.record()
+        eng._prefill([seq])
+        e1.record()
+        torch.cuda.synchronize()
+        times.append(e0.elapsed_time(e1))
+        eng.drop(seq)
+    ms = sorted(times[2:])[1]
+    out["prefill"] = {"tokens": prefill, "ms": round(ms, 3), "tok_per_s": round(prefill / ms * 1e3, 1)}
+    return out
+
+
+def vemedra_kernels(dev, peaks, T=8192, context=2048):
+    """Each kernel of a layer on its own, on inputs larger than L2 (rotating copies), against its roofline, and the
+    kernels of a Qwen3 layer that do the like."""
+    import torch.nn.functional as F
+    from nanoquantization_b200.engine import StepBatch
+    from nanoquantization_b200.layers import fused, mixers as ops
+    from nanoquantization_b200.layers.sequence_mixers import AttentionMixer
+    from nanoquantization_b200 import _lib
+    hbm, bf16 = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    W, H, G, D, RH, RD, RV, FF, chunk, bs = 4096, 32, 8, 128, 16, 128, 256, 12288, 4096, 256
+    rows = []
+    dt = torch.bfloat16
+
+    def rnd(*shape, dtype=dt):
+        return torch.randn(*shape, device=dev, dtype=torch.float32).to(dtype)
+
+    def add(phase, name, us, nbytes=0, flops=0):
+        tb, tf = nbytes / hbm * 1e6, flops / bf16 * 1e6
+        rows.append({"phase": phase, "kernel": name, "us": round(us, 2), "bound": "hbm" if tb >= tf else "tensor",
+                     "of_roofline": round(max(tb, tf) / us, 3)})
+
+    def step(n, B, start):
+        blocks = -(-(start + n) // bs)
+        return StepBatch.host([[0] * n] * B, [start] * B, [[b * blocks + i for i in range(blocks)] for b in range(B)], list(range(B)), blocks, bs).to(dev)
+    one = step(T, 1, 0)
+    nin = H * D + 2 * G * D + 2 * RH * RD + 2 * RH * RV
+    att = AttentionMixer(heads=H, kv_heads=G, dim=D, vdim=D, chunk=chunk, rot_base=1e6, rot_dims=D, scale=D ** -0.5, softcap=50.0, device=dev)
+    decay = torch.tensor([1 - 2.0 ** -(5 + 0.5 * h) for h in range(RH)], device=dev)
+    ret = _lib.RetentionDesc(RH, RD, RV, 1e-6, 0.5, decay.data_ptr())
+    # prefill
+    x, nw, cw = [rnd(T, W, dtype=torch.float32) for _ in range(2)], rnd(W, dtype=torch.float32), rnd(4, W, dtype=torch.float32)
+    cst = torch.zeros(65, 3, W, device=dev)
+    add("prefill", "rmsnorm + convolution", _device_us(lambda i: ops.rmsnorm_conv(x[i % 2], nw, cw, cst, one, 1e-6, dt), 8), T * W * 6)
+    x16, r16, n16 = [rnd(T, W) for _ in range(2)], [rnd(T, W) for _ in range(2)], rnd(W)
+    add("prefill", "Qwen3: residual add + rmsnorm", _device_us(lambda i: fused.add_rmsnorm(x16[i % 2], r16[i % 2], n16, 1e-6), 8), T * W * 8)
+    del r16
+    proj = [rnd(T, nin) for _ in range(2)]
+    kc, vc = torch.zeros(T // bs + 1, bs, G, D, dtype=dt, device=dev), torch.zeros(T // bs + 1, bs, G, D, dtype=dt, device=dev)
+    add("prefill", "rotary + K/V store", _device_us(lambda i: ops.rope_store(proj[i % 2], kc, vc, att.inv_freq, one, 0, H * D, (H + G) * D, H), 8),
+        T * (2 * H * D + 4 * G * D) * 2)
+    qkv, qn, cs = [rnd(T, (H + 2 * G) * D) for _ in range(3)], rnd(D), rnd(T, 1, D, dtype=torch.float32)
+    add("prefill", "Qwen3: QK-norm + rotary + K/V store",
+        _device_us(lambda i: fused.qknorm_rope_(qkv[i % 3], qn, qn, cs, one.positions, H, G, D, 1e-6, (kc, vc, one.rows)), 9), T * (2 * H * D + 4 * G * D) * 2)
+    act = rnd(T, H * D + RH * RV)
+    for name, c in ((f"attention, chunks of {chunk}", chunk), ("attention, one chunk of all", T)):
+        att.chunk = c
+        d = att.desc()
+        us = _device_us(lambda i: ops.chunk_attention(proj[i % 2][:, :H * D], kc, vc, act[:, :H * D], d, one), 4)
+        add("prefill", name, us, flops=T // c * (c * c / 2) * 4 * D * H)
+    q, k, v = (qkv[0][:, o:o + n * D].reshape(1, T, n, D).transpose(1, 2).contiguous() for o, n in ((0, H), (H * D, G), ((H + G) * D, G)))
+    us = _device_us(lambda i: F.scaled_dot_product_attention(q, k, v, is_causal=True, enable_gqa=True), 4)
+    add("prefill", "Qwen3: scaled_dot_product_attention, all", us, flops=T * T / 2 * 4 * D * H)
+    del q, k, v, qkv
+    st, off = torch.zeros(65, RH, RD, RV, device=dev), (H + 2 * G) * D
+    us = _device_us(lambda i: ops.retention_gated(proj[i % 2], off, ret, decay, st, act, H * D, one), 4)
+    add("prefill", "retention + norm + gate (3 launches)", us, T * (2 * RH * RD + 3 * RH * RV) * 2, 4 * T * RH * RD * RV)
+    zb, gst, p3 = rnd(W, dtype=torch.float32), torch.zeros(65, W, device=dev), [rnd(T, 3 * W) for _ in range(2)]
+    add("prefill", "minGRU scan", _device_us(lambda i: ops.mingru(p3[i % 2], W, zb, zb, gst, one), 8), T * W * 8)
+    del p3
+    gu = [rnd(T, 2 * FF) for _ in range(2)]
+    add("prefill", "clamped GLU", _device_us(lambda i: ops.clamped_glu(gu[i % 2], 7.0), 8), T * FF * 6)
+    add("prefill", "Qwen3: silu(gate) * up", _device_us(lambda i: fused.silu_mul(gu[i % 2]), 8), T * FF * 6)
+    del gu
+    w = rnd(nin, W)
+    add("prefill", "merged input product (library)", _device_us(lambda i: ops.linear(x16[i % 2], w), 4), flops=2 * T * W * nin)
+    w2 = rnd(W, FF)
+    y = rnd(T, FF)
+    add("prefill", "down product + residual (library)", _device_us(lambda i: ops.linear_residual_(x[i % 2], y, w2), 4), flops=2 * T * W * FF)
+    lin = make_layer(W, 2 * FF, 11, dev, dt)
+    add("prefill", "Qwen3: gate | up product, 4-bit weights", _device_us(lambda i: lin(x16[i % 2]), 4), flops=2 * T * W * 2 * FF)
+    del proj, act, x, x16, y, w, w2, lin
+    torch.cuda.empty_cache()
+    # decode: the weights rotate over copies larger than L2
+    for B in (1, 16):
+        ph, h = f"decode, batch {B}", rnd(B, W)
+        s = step(1, B, context - 1)
+        stream, f12 = rnd(B, W, dtype=torch.float32), rnd(B, FF)
+        ws = [rnd(nin, W) for _ in range(3)]
+        add(ph, "merged input product", _device_us(lambda i: ops.linear(h, ws[i % 3]), 12), nin * W * 2)
+        ws = [rnd(2 * FF, W) for _ in range(2)]
+        add(ph, "gate | up product + clamped GLU", _device_us(lambda i: ops.dense_glu(h, ws[i % 2], 7.0), 8), 2 * FF * W * 2)
+        ws = [rnd(W, FF) for _ in range(3)]
+        add(ph, "down product + residual", _device_us(lambda i: ops.linear_residual_(stream, f12, ws[i % 3]), 12), FF * W * 2)
+        ws = [rnd(W, H * D + RH * RV) for _ in range(4)]
+        a8 = rnd(B, H * D + RH * RV)
+        add(ph, "output product + residual", _device_us(lambda i: ops.linear_residual_(stream, a8, ws[i % 4]), 12), W * (H * D + RH * RV) * 2)
+        ws = [rnd(3 * W, W) for _ in range(3)]
+        add(ph, "z | x | g product + minGRU", _device_us(lambda i: ops.dense_mingru(h, ws[i % 3], zb, zb, gst, s), 12), 3 * W * W * 2)
+        del ws
+        for (K, N) in ((W, 2 * FF), (FF, W), (W, (H + 2 * G) * D)):
+            n = max(2, -(-int(1.5 * L2_BYTES) // weight_bytes(K, N)))
+            lins = [make_layer(K, N, 7 + c, dev, dt) for c in range(n)]
+            xk = rnd(B, K)
+            add(ph, f"Qwen3: 4-bit linear {K} -> {N}", _device_us(lambda i: lins[i % n](xk), 2 * n), weight_bytes(K, N))
+            del lins
+        n = 8 if B == 1 else 2   # copies of cache and state
+        copies = []
+        for _ in range(n):
+            nb = B * (context // bs)
+            copies.append((rnd(nb, bs, G, D), rnd(nb, bs, G, D), torch.zeros(B, RH, RD, RV, device=dev)))
+        pr, ac = rnd(B, nin), rnd(B, H * D + RH * RV)
+        att.chunk = chunk
+        d = att.desc()
+        kv_bytes, st_bytes = B * context * 2 * G * D * 2, 2 * B * RH * RD * RV * 4
+        both = lambda i: ops.mixer_decode(pr, ac, (d, att.inv_freq, 0, 0, copies[i % n][0], copies[i % n][1]), (ret, off, H * D, copies[i % n][2]), s)  # noqa: E731
+        add(ph, "attention + retention", _device_us(both, 2 * n), kv_bytes + st_bytes)
+        add(ph, "  attention alone", _device_us(lambda i: ops.mixer_decode(pr, ac, (d, att.inv_freq, 0, 0, copies[i % n][0], copies[i % n][1]), None, s), 2 * n), kv_bytes)
+        add(ph, "  retention alone", _device_us(lambda i: ops.mixer_decode(pr, ac, None, (ret, off, H * D, copies[i % n][2]), s), 2 * n), st_bytes)
+        try:
+            from flash_attn import flash_attn_with_kvcache
+            q1 = rnd(B, 1, H, D)
+            add(ph, "Qwen3: flash_attn_with_kvcache", _device_us(lambda i: flash_attn_with_kvcache(
+                q1, copies[i % n][0], copies[i % n][1], cache_seqlens=s.ctx, block_table=s.table, causal=True), 2 * n), kv_bytes)
+        except ImportError:
+            pass
+        add(ph, "rmsnorm + convolution", _device_us(lambda i: ops.rmsnorm_conv(stream, nw, cw, cst, s, 1e-6, dt), 16), B * W * (6 + 24) + W * 20)
+        add(ph, "Qwen3: residual add + rmsnorm", _device_us(lambda i: fused.add_rmsnorm(h, h, n16, 1e-6), 16), B * W * 8)
+        del copies
+    return rows
+
+
+def run_vemedra(args):
+    """--vemedra: random-init layers of real sizes through the engine, beside Qwen3 layers (4-bit weights) of the same
+    width, heads and feed-forward, and every kernel against its roofline."""
+    from nanoquantization_b200 import WQLinear_GEMM
+    from nanoquantization_b200.engine import LLMEngine
+    from nanoquantization_b200.models import QWEN3_SHAPES, Qwen3QuantizedForCausalLM, VemedraConfig, VemedraForCausalLM
+    torch.cuda.set_device(0)
+    dev, dt = torch.device("cuda", 0), torch.bfloat16
+    torch.manual_seed(0)
+    with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as fh:
+        peaks = json.load(fh)
+    line = {"what": "Vemedra beside Qwen3 (4-bit weights), random init, one GPU, bf16", "layers": VEMEDRA_LAYERS,
+            "note": "weights and caches larger than L2; rooflines are the measured copy bandwidth and bf16 peak"}
+    sampler = ClockSampler(0)
+    sampler.start()
+    if not args.vemedra_kernels_only:
+        batches, context, prefill = (1, 16, 64), 2047, 8192
+        model = VemedraForCausalLM(VemedraConfig.from_dict(vemedra_config()), device=dev, dtype=dt)
+        for name, t in model.checkpoint_tensors().items():
+            if "norm" in name:
+                t.fill_(1.0)
+            else:
+                t.copy_(torch.randn(t.shape, device=dev) * (t.shape[-1] ** -0.5 if t.dim() > 1 else 0.1))
+        eng = LLMEngine(model, num_blocks=64 * 9 + 40, max_batch=64)
+        line["vemedra"] = _engine_throughput(eng, 151936, batches, context, prefill)
+        line["vemedra"]["weights_gb"] = round(sum(t.numel() * t.element_size() for t in model.buffers()) / 1e9, 2)
+        del eng, model
+        torch.cuda.empty_cache()
+        shp = QWEN3_SHAPES["qwen3-8b"]
+        model = Qwen3QuantizedForCausalLM(VEMEDRA_LAYERS, 151936, shp["hidden_size"], shp["total_num_heads"], shp["total_num_kv_heads"], 8400,
+                                          shp["intermediate_size"], 4, GROUP, 128, False, 1e6, 1e-6, device=dev, dtype=dt)
+        for n, mod in enumerate(m for m in model.modules() if isinstance(m, WQLinear_GEMM)):
+            fill_layer(mod, 5000 + n, dev, dt)
+        torch.nn.init.normal_(model.model.embed_tokens.weight, std=0.02)
+        torch.nn.init.normal_(model.lm_head.weight, std=0.02)
+        model.fuse_projections()
+        eng = LLMEngine(model, num_blocks=64 * 9 + 40, max_batch=64)
+        line["qwen3"] = _engine_throughput(eng, 151936, batches, context, prefill)
+        del eng, model
+        torch.cuda.empty_cache()
+    line["kernels"] = vemedra_kernels(dev, peaks)
+    line["clocks"] = sampler.stop()
+    emit(json.dumps(line))
+
+
+# --------------------------------------------------------------------------
 # checker legs of our arm (after the timed regions)
 # --------------------------------------------------------------------------
 def reference_gpu_leg(layers, xs_dev, points, per_point, dev):
@@ -1029,6 +1291,9 @@ def main():
     ap.add_argument("--dtype", default="f16", choices=["f16", "bf16"])
     ap.add_argument("--serve", nargs="?", const="qwen3-32b", default=None,
                     help="instead of the sweep: the continuous-batching workload on this architecture (tensor-parallel under torchrun)")
+    ap.add_argument("--vemedra", action="store_true",
+                    help="instead of the sweep: Vemedra layers of real sizes beside Qwen3 layers of the same size, and every kernel against its roofline")
+    ap.add_argument("--vemedra-kernels-only", action="store_true", help="with --vemedra: the kernels alone")
     ap.add_argument("--requests", type=int, default=256)
     ap.add_argument("--decode-only", type=int, default=0, metavar="BATCH",
                     help="only the Qwen3-8B decode point of this batch size, 1 GPU (the case a launch list is taken of)")
@@ -1038,6 +1303,8 @@ def main():
         torch.cuda.set_device(0)
         dtype = torch.bfloat16 if args.dtype == "bf16" else torch.float16
         emit(json.dumps(decode_bench(1, 0, torch.device("cuda", 0), dtype, batches=(args.decode_only,), steps=4, prefill=False)))
+    elif args.vemedra:
+        run_vemedra(args)
     elif args.serve:
         run_serve(args)
     elif args.point:

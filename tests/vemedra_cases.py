@@ -71,6 +71,11 @@ def weights(c, seed=0):
         elif name != "embed":
             w = 1.5 * w * shape[-1] ** -0.5
         out[name] = w.to(torch.bfloat16)
+    # Keys of the retention lean towards its queries: where q.k is about zero at the first tokens, a head's output
+    # almost vanishes, and its norm would blow up plain rounding to the size of the logits.
+    for name in out:
+        if name.endswith("right.k"):
+            out[name] = (0.8 * out[name[:-1] + "q"].float() + 0.6 * out[name].float()).to(torch.bfloat16)
     return out
 
 
