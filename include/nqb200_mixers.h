@@ -90,10 +90,12 @@ int nqb200_head_norm_gate(const float* o, const void* gate, int64_t gate_stride,
 
 /* minGRU over proj [tokens, stride]: z, x and gate pre-activations at columns z_off, x_off, g_off.
  * z = sigmoid(zp + z_bias), u = xp + x_bias, candidate = u >= 0 ? u + 1/2 : sigmoid(u),
- * S <- (1 - z) S + z candidate, out = S silu(g).  state float [slots, width]. */
+ * S <- (1 - z) S + z candidate, out = S silu(g).  state float [slots, width].
+ * scratch: nqb200_mingru_scratch() floats (may be NULL where no sequence brings more than 128 tokens). */
 int nqb200_mingru(const void* proj, int64_t stride, int64_t z_off, int64_t x_off, int64_t g_off, const float* z_bias,
-                  const float* x_bias, float* state, void* out, int64_t width, const nqb200_batch* b, int dtype,
-                  void* stream);
+                  const float* x_bias, float* state, void* out, int64_t width, float* scratch, const nqb200_batch* b,
+                  int dtype, void* stream);
+int64_t nqb200_mingru_scratch(int64_t tokens, int64_t batch, int64_t width);
 
 /* out[t, i] = g sigmoid(1.702 g) (u + 1), g = min(gate_up[t, i], limit), u = clamp(gate_up[t, ff + i], -limit, limit). */
 int nqb200_clamped_glu(const void* gate_up, void* out, int64_t tokens, int64_t ff, float limit, int dtype, void* stream);

@@ -97,7 +97,8 @@ MIXER_SIGNATURES = {
     "nqb200_chunk_attention": (_int, [_vp, _i64, _vp, _vp, _vp, _i64, _att, _step, _int, _vp]),
     "nqb200_retention": (_int, [_vp, _i64, _i64, _i64, _i64, _vp, _vp, _vp, _i64, _i64, _i64, _step, _int, _vp]),
     "nqb200_head_norm_gate": (_int, [_vp, _vp, _i64, _vp, _i64, _i64, _i64, _i64, _f32, _f32, _int, _vp]),
-    "nqb200_mingru": (_int, [_vp, _i64, _i64, _i64, _i64, _vp, _vp, _vp, _vp, _i64, _step, _int, _vp]),
+    "nqb200_mingru": (_int, [_vp, _i64, _i64, _i64, _i64, _vp, _vp, _vp, _vp, _i64, _vp, _step, _int, _vp]),
+    "nqb200_mingru_scratch": (_i64, [_i64, _i64, _i64]),
     "nqb200_clamped_glu": (_int, [_vp, _vp, _i64, _i64, _f32, _int, _vp]),
     "nqb200_retention_prefill": (_int, [_vp, _i64, _i64, _vp, _i64, _i64, _ret, _vp, _vp, _step, _vp]),
     "nqb200_retention_prefill_supported": (_int, [_ret, _i64, _i64, _i64, _i64]),

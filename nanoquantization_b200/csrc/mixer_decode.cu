@@ -12,9 +12,11 @@ namespace cg = cooperative_groups;
 namespace nqb200 {
 
 constexpr int kDecThreads = 128;
-constexpr int kDecTile = 128;      // keys per pass of a CTA
+constexpr int kDecTile = 64;       // keys per pass of a CTA: 16 per warp
+constexpr int kDecStages = 3;      // passes whose keys and values are under way
 constexpr int kDecHeads = 8;       // query heads per cluster at most (columns of one mma)
 constexpr int kDecMaxDim = 256;
+constexpr int kDecPS = kDecTile + 8;
 
 struct DecodeArgs {
   const bf16* proj; int64_t stride;
@@ -31,15 +33,15 @@ struct DecodeArgs {
   float eps, r_scale;
 };
 
+// Fixed part of the attention's shared memory; the key / value ring follows it.
 struct AttSmem {
   alignas(16) bf16 q[kDecHeads][kDecMaxDim + 8];
+  alignas(16) bf16 p[16][kDecPS];             // weights, rows 8 .. 15 stay zero
   alignas(16) bf16 knew[kDecMaxDim];
-  float p[kDecHeads][kDecTile + 4];
+  float s[kDecHeads][kDecTile + 4];
   float cs[kDecMaxDim];
   float m[kDecHeads], l[kDecHeads], corr[kDecHeads];
-  int rows[kDecTile];
   float out[kDecHeads][kDecMaxDim];           // this CTA's share, read by the cluster
-  float red[kDecThreads * kDecHeads * 8];     // partial sums of the key groups
 };
 
 struct RetSmem {
@@ -49,33 +51,75 @@ struct RetSmem {
   float ss, wsum[4];
 };
 
-__device__ __forceinline__ void mma_bf16(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
+__device__ __forceinline__ uint32_t dec_smem(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void dec_cp16(uint32_t dst, const void* src, bool ok) {
+  const int n = ok ? 16 : 0;
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(n));
+}
+__device__ __forceinline__ void dec_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void dec_ldsm4(uint32_t (&r)[4], uint32_t a) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
+}
+__device__ __forceinline__ void dec_ldsm4t(uint32_t (&r)[4], uint32_t a) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
+}
+__device__ __forceinline__ void dec_ldsm2(uint32_t (&r)[2], uint32_t a) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(a));
 }
 
-// R: query heads of this cluster (compile-time bound RM).
-template <int RM>
-__device__ void attention_decode(const DecodeArgs& a, AttSmem& sm, int b, int unit, cg::cluster_group& cl) {
+__host__ __device__ constexpr int att_ks(int dim) { return (dim + 15) / 16 * 16 + 8; }   // row strides of the ring, in elements
+__host__ __device__ constexpr int att_stage(int dim, int vp) { return kDecTile * (att_ks(dim) + vp + 8); }
+
+// VP: value columns padded to 64, 128 or 256; a warp owns a quarter of them.
+template <int VP>
+__device__ void attention_decode(const DecodeArgs& a, uint8_t* smem, int b, int unit, cg::cluster_group& cl) {
+  AttSmem& sm = *reinterpret_cast<AttSmem*>(smem);
+  bf16* ring = reinterpret_cast<bf16*>(smem + sizeof(AttSmem));
   const nqb200_attention& at = a.at;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, rank = (int)cl.block_rank(), csize = (int)cl.num_blocks();
   const int per_kv = at.heads / at.kv_heads, kvh = unit / a.head_groups, hg = unit % a.head_groups;
-  const int h0 = kvh * per_kv + hg * RM, R = min(RM, per_kv - hg * RM);   // query heads h0 .. h0 + R - 1
+  const int h0 = kvh * per_kv + hg * kDecHeads, R = min(kDecHeads, per_kv - hg * kDecHeads);   // query heads h0 .. h0 + R - 1
   const int D = at.dim, V = at.vdim, pos = a.bt.pos0[b];
   const int lo = at.chunk > 0 ? pos / at.chunk * at.chunk : 0, nk = pos - lo + 1;
   const int per = (nk + csize - 1) / csize, k0 = lo + rank * per, k1 = min(lo + nk, k0 + per);   // this CTA's keys
+  const int tiles = k1 > k0 ? (k1 - k0 + kDecTile - 1) / kDecTile : 0;
+  const int KS = att_ks(D), D8 = D / 8, V8 = V / 8, half = a.rot / 2;
+  constexpr int VS = VP + 8, NT = VP / 32;       // n-tiles of 8 columns per warp
   const bf16* row = a.proj + (size_t)b * a.stride;
-  const int half = a.rot / 2, dpad = (D + 31) / 32 * 32;
+  const bool newest = k0 <= pos && pos < k1;
 
+  auto load_tile = [&](int i) {
+    if (i < tiles) {
+      bf16* kd = ring + (size_t)(i % kDecStages) * att_stage(D, VP) + (tid >> 1) * KS;
+      bf16* vd = ring + (size_t)(i % kDecStages) * att_stage(D, VP) + kDecTile * KS + (tid >> 1) * VS;
+      const int j = k0 + i * kDecTile + (tid >> 1);            // two threads per key
+      const bool ok = j < k1 && j != pos;
+      const size_t r = kv_row(a.bt, b, ok ? j : k0) * at.kv_heads + kvh;
+      for (int c = tid & 1; c < D8; c += 2) dec_cp16(dec_smem(kd + c * 8), a.k_cache + r * D + c * 8, ok);
+      for (int c = tid & 1; c < V8; c += 2) dec_cp16(dec_smem(vd + c * 8), a.v_cache + r * V + c * 8, ok);
+    }
+    asm volatile("cp.async.commit_group;");
+  };
+#pragma unroll
+  for (int i = 0; i < kDecStages - 1; ++i) load_tile(i);
+
+  // while those are under way: padding columns, the rotated queries and (in the CTA that holds the newest key) key
+  for (int e = tid; e < kDecStages * kDecTile * (KS - 8 - D); e += kDecThreads) {
+    const int r = e / (KS - 8 - D), c = e % (KS - 8 - D);
+    ring[(size_t)(r / kDecTile) * att_stage(D, VP) + (r % kDecTile) * KS + D + c] = __float2bfloat16_rn(0.f);
+  }
+  for (int e = tid; e < kDecStages * kDecTile * (VP - V); e += kDecThreads) {
+    const int r = e / (VP - V), c = e % (VP - V);
+    ring[(size_t)(r / kDecTile) * att_stage(D, VP) + kDecTile * KS + (r % kDecTile) * VS + V + c] = __float2bfloat16_rn(0.f);
+  }
+  for (int e = tid; e < kDecHeads * (KS - 8); e += kDecThreads) sm.q[e / (KS - 8)][e % (KS - 8)] = __float2bfloat16_rn(0.f);
+  for (int e = tid; e < 16 * kDecPS; e += kDecThreads) sm.p[e / kDecPS][e % kDecPS] = __float2bfloat16_rn(0.f);
   for (int f = tid; f < half; f += kDecThreads) sincosf((float)pos * a.inv_freq[f], &sm.cs[half + f], &sm.cs[f]);
-  for (int e = tid; e < kDecHeads * dpad; e += kDecThreads) sm.q[e / dpad][e % dpad] = __float2bfloat16_rn(0.f);
   if (tid < kDecHeads) { sm.m[tid] = -INFINITY; sm.l[tid] = 0.f; }
   __syncthreads();
-  // rotate q (R heads) and, in the CTA that holds the newest key, k; that CTA also stores k and v
-  const bool newest = k0 <= pos && pos < k1;
-  const size_t nrow = newest ? kv_row(a.bt, b, pos) : 0;
-  bf16* kdst = a.k_cache + (nrow * at.kv_heads + kvh) * D;
-  bf16* vdst = a.v_cache + (nrow * at.kv_heads + kvh) * V;
   const int pairs = half + (D - a.rot), nvec = R + (newest ? 1 : 0);
   for (int e = tid; e < nvec * pairs; e += kDecThreads) {
     const int r = e / pairs, j = e % pairs;
@@ -89,120 +133,93 @@ __device__ void attention_decode(const DecodeArgs& a, AttSmem& sm, int b, int un
       dst[j + half] = src[j + half];
     }
   }
-  __syncthreads();
-  if (newest && hg == 0) {   // every head group of the key/value head would write the same
-    for (int d = tid; d < D; d += kDecThreads) kdst[d] = sm.knew[d];
-    for (int d = tid; d < V; d += kDecThreads) vdst[d] = row[a.v_off + (size_t)kvh * V + d];
-  }
-
-  const int CG = V / 8, KG = kDecThreads / CG, cgi = tid % CG, kgi = tid / CG;   // 8 value columns x a key group per thread
-  const bool pv = kgi < KG;
-  float acc[RM][8];
-#pragma unroll
-  for (int r = 0; r < RM; ++r)
-#pragma unroll
-    for (int c = 0; c < 8; ++c) acc[r][c] = 0.f;
+  const uint32_t k_lane = (uint32_t)((warp * 16 + (lane & 15)) * KS + (lane >> 4) * 8) * 2;
+  const uint32_t v_lane = (uint32_t)(((lane & 7) + (((lane >> 3) & 1) << 3)) * VS + warp * (VP / 4) + (lane >> 4) * 8) * 2;
+  const uint32_t q_addr = dec_smem(&sm.q[lane & 7][((lane >> 3) & 1) * 8]);
+  const uint32_t p_addr = dec_smem(&sm.p[lane & 15][(lane >> 4) * 8]);
   const int g = lane >> 2, t = lane & 3;
-  for (int j0 = k0; j0 < k1; j0 += kDecTile) {
-    const int cnt = min(kDecTile, k1 - j0);
-    __syncthreads();
-    if (tid < cnt) sm.rows[tid] = (int)kv_row(a.bt, b, j0 + tid);
-    __syncthreads();
-    // scores: 16 keys per warp and turn, keys as rows of the mma, query heads as its columns
-    for (int kk = warp * 16; kk < cnt; kk += 64) {
-      const bf16* kp[2];
+  float O[NT][4];
 #pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        const int key = kk + g + 8 * i;
-        kp[i] = (key < cnt && j0 + key != pos) ? a.k_cache + ((size_t)sm.rows[key] * at.kv_heads + kvh) * D : sm.knew;
-        if (key >= cnt) kp[i] = nullptr;
-      }
-      float c[4] = {0.f, 0.f, 0.f, 0.f};
-      for (int d0 = 0; d0 < dpad; d0 += 32) {
-        const int d = d0 + t * 8;
-        uint4 ka = make_uint4(0, 0, 0, 0), kb = ka;
-        if (d < D && kp[0]) ka = *reinterpret_cast<const uint4*>(kp[0] + d);
-        if (d < D && kp[1]) kb = *reinterpret_cast<const uint4*>(kp[1] + d);
-        const uint4 qv = *reinterpret_cast<const uint4*>(&sm.q[g][d]);
-        mma_bf16(c, ka.x, kb.x, ka.y, kb.y, qv.x, qv.y);
-        mma_bf16(c, ka.z, kb.z, ka.w, kb.w, qv.z, qv.w);
-      }
+  for (int i = 0; i < NT; ++i)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int key = kk + g + 8 * (e >> 1), r = t * 2 + (e & 1);
-        float s = c[e] * at.scale;
-        if (at.softcap > 0.f) s = at.softcap * tanhf(s / at.softcap);
-        sm.p[r][key] = key < cnt ? s : -INFINITY;
+    for (int e = 0; e < 4; ++e) O[i][e] = 0.f;
+
+  for (int i = 0; i < tiles; ++i) {
+    asm volatile("cp.async.wait_group %0;" ::"n"(kDecStages - 2));
+    __syncthreads();               // tile i has landed for every thread; tile i - 1 is no longer read
+    load_tile(i + kDecStages - 1);
+    const int j0 = k0 + i * kDecTile, cnt = min(kDecTile, k1 - j0);
+    bf16* kt = ring + (size_t)(i % kDecStages) * att_stage(D, VP);
+    bf16* vt = kt + kDecTile * KS;
+    if (pos >= j0 && pos < j0 + cnt) {   // the newest key and value: into the tile, and into the cache
+      const size_t nrow = kv_row(a.bt, b, pos) * at.kv_heads + kvh;
+      for (int d = tid; d < D; d += kDecThreads) {
+        kt[(pos - j0) * KS + d] = sm.knew[d];
+        if (hg == 0) a.k_cache[nrow * D + d] = sm.knew[d];
       }
+      for (int d = tid; d < V; d += kDecThreads) {
+        const bf16 v = row[a.v_off + (size_t)kvh * V + d];
+        vt[(pos - j0) * VS + d] = v;
+        if (hg == 0) a.v_cache[nrow * V + d] = v;
+      }
+      __syncthreads();
+    }
+    // scores: keys as rows of the mma, query heads as its columns
+    float c[4] = {0.f, 0.f, 0.f, 0.f};
+    const uint32_t ka = dec_smem(kt) + k_lane;
+#pragma unroll 4
+    for (int d = 0; d < KS - 8; d += 16) {
+      uint32_t kf[4], qf[2];
+      dec_ldsm4(kf, ka + d * 2);
+      dec_ldsm2(qf, q_addr + d * 2);
+      dec_mma(c, kf, qf[0], qf[1]);
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int key = warp * 16 + g + 8 * (e >> 1), r = t * 2 + (e & 1);
+      float s = c[e] * at.scale;
+      if (at.softcap > 0.f) s = at.softcap * tanhf(s / at.softcap);
+      sm.s[r][key] = key < cnt ? s : -INFINITY;
     }
     __syncthreads();
-    // softmax of the tile: a warp per head
-    for (int r = warp; r < R; r += 4) {
-      float mx = -INFINITY;
-      for (int i = lane; i < cnt; i += 32) mx = fmaxf(mx, sm.p[r][i]);
-      const float m_old = sm.m[r], m_new = fmaxf(m_old, warp_max(mx));
-      float s = 0.f;
-      for (int i = lane; i < cnt; i += 32) {
-        const float e = expf(sm.p[r][i] - m_new);
-        sm.p[r][i] = e;
-        s += e;
-      }
-      s = warp_sum(s);
+    // softmax of the tile: two heads per warp, two keys per lane
+#pragma unroll
+    for (int q = 0; q < 2; ++q) {
+      const int r = warp * 2 + q;
+      if (r >= R) break;
+      const float s0 = sm.s[r][lane], s1 = sm.s[r][lane + 32], m_old = sm.m[r], m_new = fmaxf(m_old, warp_max(fmaxf(s0, s1)));
+      const float e0 = expf(s0 - m_new), e1 = expf(s1 - m_new), sum = warp_sum(e0 + e1);
+      sm.p[r][lane] = __float2bfloat16_rn(e0);
+      sm.p[r][lane + 32] = __float2bfloat16_rn(e1);
       __syncwarp();
       if (lane == 0) {
         const float corr = expf(m_old - m_new);
         sm.corr[r] = corr;
         sm.m[r] = m_new;
-        sm.l[r] = sm.l[r] * corr + s;
+        sm.l[r] = sm.l[r] * corr + sum;
       }
     }
     __syncthreads();
-    if (pv) {
+    const float corr = g < R ? sm.corr[g] : 0.f;
 #pragma unroll
-      for (int r = 0; r < RM; ++r) {
-        const float corr = r < R ? sm.corr[r] : 0.f;
+    for (int n = 0; n < NT; ++n) { O[n][0] *= corr; O[n][1] *= corr; }
+    const uint32_t va = dec_smem(vt) + v_lane;
 #pragma unroll
-        for (int c = 0; c < 8; ++c) acc[r][c] *= corr;
-      }
-#pragma unroll 4
-      for (int i = kgi; i < cnt; i += KG) {
-        const bf16* vp = (j0 + i != pos) ? a.v_cache + ((size_t)sm.rows[i] * at.kv_heads + kvh) * V : row + a.v_off + (size_t)kvh * V;
-        float vf[8];
-        if (j0 + i != pos) {
-          const uint4 v = *reinterpret_cast<const uint4*>(vp + cgi * 8);
-          const uint32_t w[4] = {v.x, v.y, v.z, v.w};
+    for (int kk = 0; kk < kDecTile / 16; ++kk) {
+      uint32_t pf[4];
+      dec_ldsm4(pf, p_addr + kk * 32);
 #pragma unroll
-          for (int c = 0; c < 4; ++c) { vf[2 * c] = __uint_as_float(w[c] << 16); vf[2 * c + 1] = __uint_as_float(w[c] & 0xFFFF0000u); }
-        } else {   // the new token's v stands in the projection, at any alignment
-#pragma unroll
-          for (int c = 0; c < 8; ++c) vf[c] = to_f(vp[cgi * 8 + c]);
-        }
-#pragma unroll
-        for (int r = 0; r < RM; ++r) {
-          if (r >= R) break;
-          const float w = sm.p[r][i];
-#pragma unroll
-          for (int c = 0; c < 8; ++c) acc[r][c] += w * vf[c];
-        }
+      for (int n = 0; n < NT / 2; ++n) {
+        uint32_t vf[4];
+        dec_ldsm4t(vf, va + (kk * 16 * VS + n * 16) * 2);
+        dec_mma(O[2 * n], pf, vf[0], vf[1]);
+        dec_mma(O[2 * n + 1], pf, vf[2], vf[3]);
       }
     }
   }
-  __syncthreads();
-  // sum over the key groups, then over the cluster's CTAs
-  if (pv) {
+  asm volatile("cp.async.wait_group 0;");
 #pragma unroll
-    for (int r = 0; r < RM; ++r)
-#pragma unroll
-      for (int c = 0; c < 8; ++c)
-        if (r < R) sm.red[(kgi * RM + r) * V + cgi * 8 + c] = acc[r][c];
-  }
-  __syncthreads();
-  for (int e = tid; e < R * V; e += kDecThreads) {
-    const int r = e / V, c = e % V;
-    float s = 0.f;
-    for (int k = 0; k < KG; ++k) s += sm.red[(k * RM + r) * V + c];
-    sm.out[r][c] = s;
-  }
+  for (int n = 0; n < NT; ++n) *reinterpret_cast<float2*>(&sm.out[g][warp * (VP / 4) + n * 8 + 2 * t]) = make_float2(O[n][0], O[n][1]);
   cl.sync();
   for (int e = rank * kDecThreads + tid; e < R * V; e += csize * kDecThreads) {
     const int r = e / V, c = e % V;
@@ -247,21 +264,31 @@ __device__ void retention_decode(const DecodeArgs& a, RetSmem& sm, int b, int h,
     if (rgi < RG) {
 #pragma unroll
       for (int i = 0; i < VEC; ++i) v[i] = to_f(row[a.rv_off + (size_t)h * V + col + i]);
-#pragma unroll 4
-      for (int r = rgi; r < D; r += RG) {
-        float* sp = st + (size_t)r * V + col;
-        float s[VEC];
-        if (VEC == 4) {
-          float4 f = fresh ? make_float4(0, 0, 0, 0) : *reinterpret_cast<const float4*>(sp);
-          s[0] = f.x; s[1 % VEC] = f.y; s[2 % VEC] = f.z; s[3 % VEC] = f.w;
-        } else {
-          s[0] = fresh ? 0.f : *sp;
-        }
-        const float kr = sm.k[r], qr = sm.q[r];
+      constexpr int U = 16;   // rows under way per thread
+      for (int r0 = rgi; r0 < D; r0 += U * RG) {
+        float S[U][VEC];
 #pragma unroll
-        for (int i = 0; i < VEC; ++i) { s[i] = d * s[i] + kr * v[i]; acc[i] += s[i] * qr; }
-        if (VEC == 4) *reinterpret_cast<float4*>(sp) = make_float4(s[0], s[1 % VEC], s[2 % VEC], s[3 % VEC]);
-        else *sp = s[0];
+        for (int u = 0; u < U; ++u) {
+          const int r = r0 + u * RG;
+          const float* sp = st + (size_t)r * V + col;
+          if (VEC == 4) {
+            const float4 f = (fresh || r >= D) ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(sp);
+            S[u][0] = f.x; S[u][1 % VEC] = f.y; S[u][2 % VEC] = f.z; S[u][3 % VEC] = f.w;
+          } else {
+            S[u][0] = (fresh || r >= D) ? 0.f : *sp;
+          }
+        }
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+          const int r = r0 + u * RG;
+          if (r >= D) break;
+          const float kr = sm.k[r], qr = sm.q[r];
+#pragma unroll
+          for (int i = 0; i < VEC; ++i) { S[u][i] = d * S[u][i] + kr * v[i]; acc[i] += S[u][i] * qr; }
+          float* sp = st + (size_t)r * V + col;
+          if (VEC == 4) *reinterpret_cast<float4*>(sp) = make_float4(S[u][0], S[u][1 % VEC], S[u][2 % VEC], S[u][3 % VEC]);
+          else *sp = S[u][0];
+        }
       }
 #pragma unroll
       for (int i = 0; i < VEC; ++i) sm.red[(rgi * width + cgi) * VEC + i] = acc[i];
@@ -291,21 +318,23 @@ __device__ void retention_decode(const DecodeArgs& a, RetSmem& sm, int b, int h,
   cl.sync();
 }
 
-template <int RM, int VEC>
+template <int VP, int VEC>
 __global__ void __launch_bounds__(kDecThreads) mixer_decode_kernel(const DecodeArgs a) {
   extern __shared__ __align__(16) uint8_t smem[];
   grid_launch_dependents();
   grid_dependency_wait();
   cg::cluster_group cl = cg::this_cluster();
   const int unit = blockIdx.y, b = blockIdx.z;
-  if (unit < a.att_clusters) attention_decode<RM>(a, *reinterpret_cast<AttSmem*>(smem), b, unit, cl);
+  if (unit < a.att_clusters) attention_decode<VP>(a, smem, b, unit, cl);
   else retention_decode<VEC>(a, *reinterpret_cast<RetSmem*>(smem), b, unit - a.att_clusters, cl);
 }
 
-template <int RM, int VEC>
+template <int VP, int VEC>
 static int launch_decode(const DecodeArgs& a, int csize, cudaStream_t st) {
-  const size_t smem = sizeof(AttSmem) > sizeof(RetSmem) ? sizeof(AttSmem) : sizeof(RetSmem);
-  if (cudaFuncSetAttribute(mixer_decode_kernel<RM, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+  size_t smem = a.ret_heads > 0 ? sizeof(RetSmem) : 0;
+  const size_t att = a.att_clusters > 0 ? sizeof(AttSmem) + (size_t)kDecStages * att_stage(a.at.dim, VP) * sizeof(bf16) : 0;
+  if (att > smem) smem = att;
+  if (cudaFuncSetAttribute(mixer_decode_kernel<VP, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
     cudaGetLastError();
     return NQB200_ERR_LAUNCH;
   }
@@ -323,7 +352,7 @@ static int launch_decode(const DecodeArgs& a, int csize, cudaStream_t st) {
   attr[1].val.clusterDim.z = 1;
   cfg.attrs = attr;
   cfg.numAttrs = 2;
-  if (cudaLaunchKernelEx(&cfg, mixer_decode_kernel<RM, VEC>, a) != cudaSuccess) {
+  if (cudaLaunchKernelEx(&cfg, mixer_decode_kernel<VP, VEC>, a) != cudaSuccess) {
     cudaGetLastError();
     return NQB200_ERR_LAUNCH;
   }
@@ -358,21 +387,20 @@ extern "C" int nqb200_mixer_decode(const void* proj, int64_t stride, void* act, 
   if (r && !aligned16(state)) return NQB200_ERR_MISALIGNED;
   DecodeArgs p = {};
   p.proj = (const bf16*)proj; p.stride = stride; p.act = (bf16*)act; p.act_stride = act_stride; p.bt = *b;
-  int csize = 1, rm = 1;
+  int csize = 1, want = 1;
   int64_t units = 0;
   if (a) {
     const int per_kv = a->heads / a->kv_heads;
-    rm = per_kv >= 5 ? 8 : per_kv >= 3 ? 4 : per_kv;
     p.at = *a;
     p.inv_freq = inv_freq; p.rot = (int)rot;
     p.q_off = (int)a_off; p.k_off = (int)(a_off + (int64_t)a->heads * a->dim); p.v_off = p.k_off + a->kv_heads * a->dim;
     p.a_col = (int)a_col; p.k_cache = (bf16*)k_cache; p.v_cache = (bf16*)v_cache;
-    p.head_groups = (per_kv + rm - 1) / rm;
+    p.head_groups = (per_kv + kDecHeads - 1) / kDecHeads;
     p.att_clusters = a->kv_heads * p.head_groups;
     units += p.att_clusters;
     int64_t keys = (int64_t)b->table_width * b->block_size;
     if (a->chunk > 0 && a->chunk < keys) keys = a->chunk;
-    while (csize < 8 && keys > (int64_t)csize * kDecTile) csize *= 2;
+    while (want < 8 && keys > (int64_t)want * kDecTile) want *= 2;
   }
   if (r) {
     p.ret_heads = r->heads; p.rdim = r->dim; p.rvdim = r->vdim;
@@ -380,16 +408,15 @@ extern "C" int nqb200_mixer_decode(const void* proj, int64_t stride, void* act, 
     p.rg_off = p.rv_off + r->heads * r->vdim; p.r_col = (int)r_col;
     p.decay = r->decay; p.rstate = state; p.eps = r->eps; p.r_scale = r->out_scale;
     units += r->heads;
-    int64_t bytes = (int64_t)r->dim * r->vdim * 4;    // a CTA moves about 16 KB of state each way
-    while (csize < 8 && bytes > (int64_t)csize * 16384 && csize * 8 <= r->vdim) csize *= 2;
+    while (want < 8 && (int64_t)r->dim * r->vdim * 4 > (int64_t)want * 16384 && want * 8 <= r->vdim) want *= 2;
   }
-  while (csize > 1 && units * b->batch * csize > kNumSMs * 8) csize /= 2;
+  // enough CTAs for two per SM, and no more than there is work for
+  while (csize < want && units * b->batch * csize < 2 * kNumSMs) csize *= 2;
   cudaStream_t st = (cudaStream_t)stream;
   const bool v4 = !r || r->vdim % 4 == 0;
-#define NQB200_DEC(RM) return v4 ? launch_decode<RM, 4>(p, csize, st) : launch_decode<RM, 1>(p, csize, st)
-  if (rm == 1) NQB200_DEC(1);
-  if (rm == 2) NQB200_DEC(2);
-  if (rm == 4) NQB200_DEC(4);
-  NQB200_DEC(8);
+#define NQB200_DEC(VP) return v4 ? launch_decode<VP, 4>(p, csize, st) : launch_decode<VP, 1>(p, csize, st)
+  if (!a || a->vdim <= 64) NQB200_DEC(64);
+  if (a->vdim <= 128) NQB200_DEC(128);
+  NQB200_DEC(256);
 #undef NQB200_DEC
 }

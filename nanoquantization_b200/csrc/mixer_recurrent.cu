@@ -167,9 +167,121 @@ __global__ void __launch_bounds__(kGruSegs* kGruCols) mingru_kernel(const T* __r
   if (seg == 0 && live) st[c] = carry[col];
 }
 
+// Two channels per thread (even widths): a CTA takes 64 channels x 128 tokens, a warp 16 of the tokens, so that the
+// chunks of a prompt run side by side.  A first launch folds each chunk into S -> A S + B; the second combines the
+// chunks ahead of its own, scans its 8 warps' folds and replays the tokens.  The sequence's state at the step's start is
+// copied aside by the first launch, because the last chunk's CTA overwrites it while others still need it.
+constexpr int kGruChunk = 128, kGruWarpTokens = 16;
+
+__device__ __forceinline__ float2 ld_pair(const float* p) { return *reinterpret_cast<const float2*>(p); }
+__device__ __forceinline__ float2 ld_pair(const bf16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); }
+__device__ __forceinline__ void st_pair(float* p, float2 v) { *reinterpret_cast<float2*>(p) = v; }
+__device__ __forceinline__ void st_pair(bf16* p, float2 v) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(v.x, v.y); }
+__device__ __forceinline__ float sigmoid_fast(float v) { return __fdividef(1.f, 1.f + __expf(-v)); }
+template <typename T> __device__ __forceinline__ float gate_sigmoid(float v) { return sigmoid_f(v); }
+template <> __device__ __forceinline__ float gate_sigmoid<bf16>(float v) { return sigmoid_fast(v); }
+
+struct GruArgs {
+  int64_t stride;
+  int z_off, x_off, g_off, width;
+  const float* z_bias; const float* x_bias;
+  float* state; float2* folds; float* start;   // folds [chunk id][width], start [batch][width]
+  nqb200_batch bt;
+};
+__device__ __forceinline__ size_t gru_chunk_id(const nqb200_batch& bt, int b, int c) { return (size_t)(bt.cu[b] / kGruChunk + b + c); }
+
+template <typename T, bool FOLD>
+__global__ void __launch_bounds__(256) mingru_chunk_kernel(const T* __restrict__ proj, T* __restrict__ out, const GruArgs p) {
+  __shared__ float2 As[8][32], Bs[8][32];
+  grid_launch_dependents();
+  grid_dependency_wait();
+  const int b = blockIdx.z, chunk = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int t0 = p.bt.cu[b], n = p.bt.cu[b + 1] - t0, first = chunk * kGruChunk, c = blockIdx.x * 64 + lane * 2;
+  if (first >= n) return;
+  const bool live = c < p.width, fresh = p.bt.pos0[b] == 0;
+  const int tok0 = first + warp * kGruWarpTokens, cnt = max(0, min(kGruWarpTokens, n - tok0));
+  float* own = p.state + (size_t)p.bt.slot[b] * p.width + c;
+  float2 a[kGruWarpTokens], v[kGruWarpTokens], A = make_float2(1.f, 1.f), B = make_float2(0.f, 0.f);
+  const float2 zb = live ? ld_pair(p.z_bias + c) : B, xb = live ? ld_pair(p.x_bias + c) : B;
+  const T* row = proj + (size_t)(t0 + tok0) * p.stride + c;
+#pragma unroll
+  for (int i = 0; i < kGruWarpTokens; ++i) {
+    const bool ok = live && i < cnt;
+    a[i] = ok ? ld_pair(row + (size_t)i * p.stride + p.z_off) : B;
+    v[i] = ok ? ld_pair(row + (size_t)i * p.stride + p.x_off) : B;
+  }
+#pragma unroll
+  for (int i = 0; i < kGruWarpTokens; ++i) {
+    const float zx = gate_sigmoid<T>(a[i].x + zb.x), zy = gate_sigmoid<T>(a[i].y + zb.y), ux = v[i].x + xb.x, uy = v[i].y + xb.y;
+    const bool ok = i < cnt;
+    a[i] = ok ? make_float2(1.f - zx, 1.f - zy) : make_float2(1.f, 1.f);
+    v[i] = ok ? make_float2(zx * (ux >= 0.f ? ux + 0.5f : gate_sigmoid<T>(ux)), zy * (uy >= 0.f ? uy + 0.5f : gate_sigmoid<T>(uy))) : make_float2(0.f, 0.f);
+    A.x *= a[i].x; A.y *= a[i].y;
+    B.x = a[i].x * B.x + v[i].x; B.y = a[i].y * B.y + v[i].y;
+  }
+  As[warp][lane] = A;
+  Bs[warp][lane] = B;
+  float2 S = make_float2(0.f, 0.f);   // FOLD: the fold's own B; else the state at the chunk's start
+  if (!FOLD && live) {
+    if (n <= kGruChunk) {
+      if (!fresh) S = ld_pair(own);
+    } else {   // several CTAs need the state and the last one's replaces it: from the copy
+      S = ld_pair(p.start + (size_t)b * p.width + c);
+      const float2* f = p.folds + 2 * (gru_chunk_id(p.bt, b, 0) * (p.width / 2) + c / 2);
+#pragma unroll 8
+      for (int k = 0; k < chunk; ++k) {
+        const float4 ab = *reinterpret_cast<const float4*>(f + (size_t)k * p.width);   // A of both channels, B of both
+        S.x = ab.x * S.x + ab.z;
+        S.y = ab.y * S.y + ab.w;
+      }
+    }
+  }
+  __syncthreads();
+  if (FOLD) {
+    if (warp == 0 && live) {
+      float2 FA = make_float2(1.f, 1.f), FB = make_float2(0.f, 0.f);
+#pragma unroll
+      for (int w = 0; w < 8; ++w) {
+        const float2 wa = As[w][lane], wb = Bs[w][lane];
+        FA.x *= wa.x; FA.y *= wa.y;
+        FB.x = wa.x * FB.x + wb.x; FB.y = wa.y * FB.y + wb.y;
+      }
+      *reinterpret_cast<float4*>(p.folds + 2 * (gru_chunk_id(p.bt, b, chunk) * (p.width / 2) + c / 2)) = make_float4(FA.x, FA.y, FB.x, FB.y);
+      if (chunk == 0) st_pair(p.start + (size_t)b * p.width + c, fresh ? make_float2(0.f, 0.f) : ld_pair(own));
+    }
+    return;
+  }
+  for (int w = 0; w < warp; ++w) {
+    const float2 wa = As[w][lane], wb = Bs[w][lane];
+    S.x = wa.x * S.x + wb.x; S.y = wa.y * S.y + wb.y;
+  }
+  T* orow = out + (size_t)(t0 + tok0) * p.width + c;
+#pragma unroll
+  for (int i = 0; i < kGruWarpTokens; ++i) {
+    S.x = a[i].x * S.x + v[i].x; S.y = a[i].y * S.y + v[i].y;
+    if (live && i < cnt) {
+      const float2 g = ld_pair(row + (size_t)i * p.stride + p.g_off);
+      st_pair(orow + (size_t)i * p.width, make_float2(S.x * (g.x * gate_sigmoid<T>(g.x)), S.y * (g.y * gate_sigmoid<T>(g.y))));
+    }
+  }
+  // every warp has read the state (of a sequence with one chunk) before the last one replaces it
+  __syncthreads();
+  if (live && warp == 7 && first + kGruChunk >= n) st_pair(own, S);
+}
+
 }  // namespace nqb200
 
 using namespace nqb200;
+
+template <typename T>
+static int mingru_chunked(const void* proj, void* out, const GruArgs& p, cudaStream_t st) {
+  const dim3 grid((unsigned)((p.width + 63) / 64), (unsigned)((p.bt.max_len + kGruChunk - 1) / kGruChunk), (unsigned)p.bt.batch), block(256);
+  if (grid.y > 1) {
+    const int rc = launch_overlapped(mingru_chunk_kernel<T, true>, grid, block, 0, st, (const T*)proj, (T*)nullptr, p);
+    if (rc != NQB200_OK) return rc;
+  }
+  return launch_overlapped(mingru_chunk_kernel<T, false>, grid, block, 0, st, (const T*)proj, (T*)out, p);
+}
 
 template <typename T, int DPT>
 static int retention_simple(const void* proj, int64_t stride, int64_t q_off, int64_t k_off, int64_t v_off, const float* decay, float* state,
@@ -225,18 +337,35 @@ extern "C" int nqb200_head_norm_gate(const float* o, const void* gate, int64_t g
                            out_stride, pairs, (int)heads, (int)vdim, eps, out_scale);
 }
 
+extern "C" int64_t nqb200_mingru_scratch(int64_t tokens, int64_t batch, int64_t width) {
+  return (tokens / kGruChunk + batch) * width * 2 + batch * width;
+}
+
 extern "C" int nqb200_mingru(const void* proj, int64_t stride, int64_t z_off, int64_t x_off, int64_t g_off, const float* z_bias,
-                             const float* x_bias, float* state, void* out, int64_t width, const nqb200_batch* b, int dtype, void* stream) {
+                             const float* x_bias, float* state, void* out, int64_t width, float* scratch, const nqb200_batch* b, int dtype,
+                             void* stream) {
   const int s = check_batch(b, false);
   if (s != NQB200_OK) return s;
   if (width <= 0 || width > INT32_MAX || stride <= 0) return NQB200_ERR_BAD_SHAPE;
   if (!mixer_dtype(dtype)) return NQB200_ERR_BAD_DTYPE;
   if (b->tokens == 0) return NQB200_OK;
   if (!proj || !z_bias || !x_bias || !state || !out) return NQB200_ERR_NULL_POINTER;
+  cudaStream_t st = (cudaStream_t)stream;
+  const bool pairs = width % 2 == 0 && stride % 2 == 0 && z_off % 2 == 0 && x_off % 2 == 0 && g_off % 2 == 0 && aligned16(proj) && aligned16(out) &&
+                     aligned16(z_bias) && aligned16(x_bias) && aligned16(state);
+  if (pairs && b->max_len > 1 && (b->max_len + kGruChunk - 1) / kGruChunk <= 65535) {
+    if (b->max_len > kGruChunk && (!scratch || !aligned16(scratch))) return NQB200_ERR_WORKSPACE;
+    GruArgs p = {};
+    p.stride = stride; p.z_off = (int)z_off; p.x_off = (int)x_off; p.g_off = (int)g_off; p.width = (int)width;
+    p.z_bias = z_bias; p.x_bias = x_bias; p.state = state; p.bt = *b;
+    p.folds = reinterpret_cast<float2*>(scratch);
+    p.start = scratch ? scratch + (b->tokens / kGruChunk + b->batch) * width * 2 : nullptr;
+    return dtype == NQB200_F32 ? mingru_chunked<float>(proj, out, p, st) : mingru_chunked<bf16>(proj, out, p, st);
+  }
   const dim3 grid((unsigned)((width + kGruCols - 1) / kGruCols), (unsigned)b->batch), block(kGruSegs * kGruCols);
   if (dtype == NQB200_F32)
-    return launch_overlapped(mingru_kernel<float>, grid, block, 0, (cudaStream_t)stream, (const float*)proj, stride, (int)z_off, (int)x_off,
-                             (int)g_off, z_bias, x_bias, state, (float*)out, (int)width, *b);
-  return launch_overlapped(mingru_kernel<bf16>, grid, block, 0, (cudaStream_t)stream, (const bf16*)proj, stride, (int)z_off, (int)x_off,
-                           (int)g_off, z_bias, x_bias, state, (bf16*)out, (int)width, *b);
+    return launch_overlapped(mingru_kernel<float>, grid, block, 0, st, (const float*)proj, stride, (int)z_off, (int)x_off, (int)g_off, z_bias,
+                             x_bias, state, (float*)out, (int)width, *b);
+  return launch_overlapped(mingru_kernel<bf16>, grid, block, 0, st, (const bf16*)proj, stride, (int)z_off, (int)x_off, (int)g_off, z_bias, x_bias,
+                           state, (bf16*)out, (int)width, *b);
 }

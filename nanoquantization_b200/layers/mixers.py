@@ -105,8 +105,11 @@ def retention_gated(proj: torch.Tensor, off: int, desc: _lib.RetentionDesc, deca
 def mingru(proj: torch.Tensor, width: int, z_bias: torch.Tensor, x_bias: torch.Tensor, state: torch.Tensor, step) -> torch.Tensor:
     """``proj [tokens, z | x | g]`` -> gated states ``[tokens, width]``; ``state [slots, width]`` is carried."""
     out = torch.empty(proj.shape[0], width, dtype=proj.dtype, device=proj.device)
+    scratch = None
+    if step.max_len > 128:
+        scratch = torch.empty(_lib.load_mixers().nqb200_mingru_scratch(step.num_tokens, step.batch, width), dtype=torch.float32, device=proj.device)
     _call("nqb200_mingru", proj.data_ptr(), proj.stride(0), 0, width, 2 * width, z_bias.data_ptr(), x_bias.data_ptr(), state.data_ptr(),
-          out.data_ptr(), width, ctypes.byref(step.desc), _lib.mixer_dtype_code(proj.dtype))
+          out.data_ptr(), width, _ptr(scratch), ctypes.byref(step.desc), _lib.mixer_dtype_code(proj.dtype))
     return out
 
 

@@ -449,4 +449,4 @@ def test_bad_arguments_are_errors():
     with pytest.raises(RuntimeError, match="bad shape"):
         _lib.check_mixers(_lib.load_mixers().nqb200_clamped_glu(x.data_ptr(), x.data_ptr(), 1, 0, 1.0, _lib.F32, None))
     with pytest.raises(RuntimeError, match="null pointer"):
-        _lib.check_mixers(_lib.load_mixers().nqb200_mingru(None, 8, 0, 1, 2, None, None, None, None, 4, b.desc, _lib.F32, None))
+        _lib.check_mixers(_lib.load_mixers().nqb200_mingru(None, 8, 0, 1, 2, None, None, None, None, 4, None, b.desc, _lib.F32, None))
