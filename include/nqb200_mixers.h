@@ -59,10 +59,12 @@ typedef struct {
   float out_scale;
 } nqb200_attention;
 
-/* Attention of rotated q (rows of `q`, row stride q_stride, head h at column h * dim) over the paged caches.
- * out[t * out_stride + h * vdim + c] = out_scale * o, rounded to dtype. */
+/* Attention of rotated q (rows of `q`, row stride q_stride, head h at column h * dim) over the paged caches of
+ * cache_rows rows.  out[t * out_stride + h * vdim + c] = out_scale * o, rounded to dtype.  status (may be NULL): an int
+ * on the device that takes NQB200_ERR_WAIT_TIMEOUT if a bounded wait gives up. */
 int nqb200_chunk_attention(const void* q, int64_t q_stride, const void* k_cache, const void* v_cache, void* out,
-                           int64_t out_stride, const nqb200_attention* a, const nqb200_batch* b, int dtype, void* stream);
+                           int64_t out_stride, int64_t cache_rows, const nqb200_attention* a, const nqb200_batch* b, int* status, int dtype,
+                           void* stream);
 
 /* Retention.  proj holds q and k (heads x dim at q_off, k_off) and v (heads x vdim at v_off).
  * S <- decay[h] S + (dim^-1/2 k) v^T, o = S^T q, state float [slots, heads, dim, vdim].  o float [tokens, heads * vdim]. */

@@ -94,7 +94,7 @@ MIXER_SIGNATURES = {
     "nqb200_rmsnorm_rows": (_int, [_vp, _vp, _vp, _vp, _i64, _i64, _f32, _int, _vp]),
     "nqb200_rmsnorm_conv": (_int, [_vp, _vp, _vp, _vp, _vp, _step, _i64, _i64, _f32, _int, _vp]),
     "nqb200_rope_store": (_int, [_vp, _vp, _vp, _vp, _step] + [_i64] * 9 + [_int, _vp]),
-    "nqb200_chunk_attention": (_int, [_vp, _i64, _vp, _vp, _vp, _i64, _att, _step, _int, _vp]),
+    "nqb200_chunk_attention": (_int, [_vp, _i64, _vp, _vp, _vp, _i64, _i64, _att, _step, _vp, _int, _vp]),
     "nqb200_retention": (_int, [_vp, _i64, _i64, _i64, _i64, _vp, _vp, _vp, _i64, _i64, _i64, _step, _int, _vp]),
     "nqb200_head_norm_gate": (_int, [_vp, _vp, _i64, _vp, _i64, _i64, _i64, _i64, _f32, _f32, _int, _vp]),
     "nqb200_mingru": (_int, [_vp, _i64, _i64, _i64, _i64, _vp, _vp, _vp, _vp, _i64, _vp, _step, _int, _vp]),
@@ -160,6 +160,26 @@ _STATUS = ("ok", "bad shape", "bad dtype", "misaligned pointer", "null pointer",
 def check_mixers(status: int) -> None:
     if status != 0:
         raise RuntimeError(f"nqb200_mixers: {_STATUS[status] if status < len(_STATUS) else 'unknown status'} (status {status})")
+
+
+_mixer_status: dict[int, torch.Tensor] = {}
+
+
+def mixer_status(dev: torch.device) -> torch.Tensor:
+    """The device's status word for bounded waits of the mixer kernels (0: none gave up)."""
+    idx = dev.index if dev.index is not None else torch.cuda.current_device()
+    if idx not in _mixer_status:
+        _mixer_status[idx] = torch.zeros(1, dtype=torch.int32, device=dev)
+    return _mixer_status[idx]
+
+
+def check_mixer_status() -> None:
+    """Synchronise and raise if a bounded wait of a mixer kernel gave up; the word is cleared."""
+    for word in _mixer_status.values():
+        status = int(word.item())
+        if status != 0:
+            word.zero_()
+            check_mixers(status)
 
 
 def mixer_dtype_code(dtype: torch.dtype) -> int:

@@ -18,8 +18,8 @@ LIB_PATH = os.path.join(LIB_DIR, "libnqb200.so")
 MIXERS_PATH = os.path.join(LIB_DIR, "libnqb200_mixers.so")
 SOURCES = ["api.cu", "unpack_dequant.cu", "gemm_decode.cu", "gemm_stream.cu", "gemm_umma_prefill.cu", "gemm_umma_pair.cu", "quantize_pack.cu", "fused_elementwise.cu", "peer_allreduce.cu"]
 HEADERS = ["common.cuh", "tma_utils.cuh", "umma_utils.cuh", os.path.join(ROOT, "include", "nqb200.h")]
-MIXER_SOURCES = ["mixer_norm.cu", "mixer_attention.cu", "mixer_recurrent.cu", "mixer_dense.cu", "mixer_decode.cu", "mixer_prefill.cu"]
-MIXER_HEADERS = ["common.cuh", "mixers.cuh", os.path.join(ROOT, "include", "nqb200.h"), os.path.join(ROOT, "include", "nqb200_mixers.h")]
+MIXER_SOURCES = ["mixer_norm.cu", "mixer_attention.cu", "mixer_recurrent.cu", "mixer_dense.cu", "mixer_decode.cu", "mixer_prefill.cu", "mixer_attention_umma.cu"]
+MIXER_HEADERS = ["common.cuh", "mixers.cuh", "tma_utils.cuh", "umma_utils.cuh", os.path.join(ROOT, "include", "nqb200.h"), os.path.join(ROOT, "include", "nqb200_mixers.h")]
 LIBRARIES = {LIB_PATH: (SOURCES, HEADERS), MIXERS_PATH: (MIXER_SOURCES, MIXER_HEADERS)}
 
 

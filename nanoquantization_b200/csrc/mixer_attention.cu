@@ -125,7 +125,8 @@ extern "C" int nqb200_rope_store(void* proj, void* k_cache, void* v_cache, const
 }
 
 extern "C" int nqb200_chunk_attention(const void* q, int64_t q_stride, const void* k_cache, const void* v_cache, void* out,
-                                      int64_t out_stride, const nqb200_attention* a, const nqb200_batch* b, int dtype, void* stream) {
+                                      int64_t out_stride, int64_t cache_rows, const nqb200_attention* a, const nqb200_batch* b, int* status,
+                                      int dtype, void* stream) {
   const int st = check_batch(b, true);
   if (st != NQB200_OK) return st;
   if (!a) return NQB200_ERR_NULL_POINTER;
@@ -135,6 +136,8 @@ extern "C" int nqb200_chunk_attention(const void* q, int64_t q_stride, const voi
   if (!mixer_dtype(dtype)) return NQB200_ERR_BAD_DTYPE;
   if (b->tokens == 0) return NQB200_OK;
   if (!q || !k_cache || !v_cache || !out) return NQB200_ERR_NULL_POINTER;
+  if (dtype == NQB200_BF16 && attention_umma_supports(q, q_stride, k_cache, v_cache, out, out_stride, cache_rows, a, b))
+    return attention_umma(q, q_stride, k_cache, v_cache, out, out_stride, cache_rows, a, b, status, (cudaStream_t)stream);
   if (dtype == NQB200_BF16 && b->max_len > 1 && attention_prefill_supports(q, q_stride, k_cache, v_cache, out, out_stride, a))
     return attention_prefill(q, q_stride, k_cache, v_cache, out, out_stride, a, b, (cudaStream_t)stream);
   const dim3 grid((unsigned)b->max_len, (unsigned)a->heads, (unsigned)b->batch), block(kSimpleKeys);

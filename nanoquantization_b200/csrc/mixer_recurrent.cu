@@ -251,7 +251,7 @@ __global__ void __launch_bounds__(256) mingru_chunk_kernel(const T* __restrict__
     }
     return;
   }
-  for (int w = 0; w < warp; ++w) {
+  for (int w = 0; w < (FOLD ? 0 : warp); ++w) {
     const float2 wa = As[w][lane], wb = Bs[w][lane];
     S.x = wa.x * S.x + wb.x; S.y = wa.y * S.y + wb.y;
   }

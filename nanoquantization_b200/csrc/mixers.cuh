@@ -31,7 +31,12 @@ __device__ __forceinline__ size_t kv_row(const nqb200_batch& bt, int b, int p) {
   return (size_t)bt.table[(size_t)b * bt.table_width + p / bt.block_size] * bt.block_size + p % bt.block_size;
 }
 
-// mixer_prefill.cu: the tensor-core attention for prompts.
+// mixer_attention_umma.cu: attention of prompts with tcgen05.
+bool attention_umma_supports(const void* q, int64_t q_stride, const void* k_cache, const void* v_cache, const void* out, int64_t out_stride,
+                             int64_t cache_rows, const nqb200_attention* a, const nqb200_batch* b);
+int attention_umma(const void* q, int64_t q_stride, const void* k_cache, const void* v_cache, void* out, int64_t out_stride, int64_t cache_rows,
+                   const nqb200_attention* a, const nqb200_batch* b, int* status, cudaStream_t st);
+// mixer_prefill.cu: the same for the sizes and pages that kernel does not take, and for short portions.
 bool attention_prefill_supports(const void* q, int64_t q_stride, const void* k_cache, const void* v_cache, const void* out, int64_t out_stride,
                                 const nqb200_attention* a);
 int attention_prefill(const void* q, int64_t q_stride, const void* k_cache, const void* v_cache, void* out, int64_t out_stride,

@@ -458,6 +458,7 @@ class LLMEngine:
             comm.check()
         if self.device.type == "cuda":
             _lib.check_workspaces()
+            _lib.check_mixer_status()
 
     def generate(self, prompts: Seq[Seq[int]], max_new_tokens) -> list[list[int]]:
         if isinstance(max_new_tokens, int):

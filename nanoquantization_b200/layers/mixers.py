@@ -61,7 +61,7 @@ def rope_store(proj: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
 def chunk_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, out: torch.Tensor, desc: _lib.AttentionDesc, step) -> None:
     """Attention over the paged cache; ``q`` and ``out`` are column ranges of row-major buffers."""
     _call("nqb200_chunk_attention", q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), out.stride(0),
-          ctypes.byref(desc), ctypes.byref(step.desc), _lib.mixer_dtype_code(q.dtype))
+          k_cache.shape[0] * k_cache.shape[1], ctypes.byref(desc), ctypes.byref(step.desc), _lib.mixer_status(q.device).data_ptr(), _lib.mixer_dtype_code(q.dtype))
 
 
 def retention(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, decay: torch.Tensor, state: torch.Tensor, step) -> torch.Tensor:

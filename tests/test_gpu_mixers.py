@@ -128,12 +128,12 @@ def test_final_norm_takes_rows_and_stream_add_adds():
         assert torch.allclose(y.cpu(), 2 * e.float()[ids] + 2 * step, atol=1e-6)
 
 
-def attend(r, mixer, q, k, v, dtype):
+def attend(r, mixer, q, k, v, dtype, pad=3, col=4):
     """Rotate, store, attend: the mixer's own call on a projection [q | k | v]; returns o [T, heads, vdim] per sequence."""
     H, G, D, V = mixer.heads, mixer.kv_heads, mixer.dim, mixer.vdim
     kc = torch.full((r.num_blocks, r.bs, G, D), 300.0, dtype=dtype, device=DEV)
     vc = torch.full((r.num_blocks, r.bs, G, V), 300.0, dtype=dtype, device=DEV)
-    pad = 3   # the projection's columns start inside a wider buffer
+    # the projection's columns start inside a wider buffer, and the output's in another
     proj = [torch.cat([torch.zeros(len(a), pad), a.flatten(1), b.flatten(1), c.flatten(1)], 1).to(dtype) for a, b, c in zip(q, k, v)]
 
     class Step:
@@ -141,16 +141,42 @@ def attend(r, mixer, q, k, v, dtype):
 
     def fn(b, rows):
         Step.batch = b
-        act = torch.full((rows.shape[0], H * V + 5), 7.0, dtype=dtype, device=DEV)
-        mixer.mix(rows.contiguous(), pad, act, 4, Step)
-        assert (act[:, :4] == 7).all() and (act[:, -1] == 7).all()
-        return act[:, 4:-1].reshape(-1, H, V)
+        act = torch.full((rows.shape[0], H * V + 2 * col), 7.0, dtype=dtype, device=DEV)
+        mixer.mix(rows.contiguous(), pad, act, col, Step)
+        assert (act[:, :col] == 7).all() and (act[:, -col:] == 7).all()
+        return act[:, col:-col].reshape(-1, H, V)
     return r.run(proj, fn)
 
 
 def oracle_attend(m, q, k, v, base, rot, sink):
     q, k = O.rotate(q.double(), base, rot), O.rotate(k.double(), base, rot)
     return O.chunk_attention(q, k, v.double(), m.scale, m.softcap, m.chunk, sink.double()) * m.out_scale
+
+
+def fast_attend(m, q, k, v, base, rot, sink):
+    """The oracle's attention for long sequences: the same definition on whole score matrices."""
+    T, H, G = q.shape[0], m.heads, m.kv_heads
+    p = torch.arange(T, dtype=torch.float64)
+
+    def turn(x):
+        x = x.double().clone()
+        a = p[:, None, None] * base ** (-2.0 * torch.arange(rot // 2, dtype=torch.float64) / rot)
+        u, w = x[..., :rot // 2].clone(), x[..., rot // 2:rot].clone()
+        x[..., :rot // 2], x[..., rot // 2:rot] = u * a.cos() - w * a.sin(), w * a.cos() + u * a.sin()
+        return x
+    q, k = turn(q), turn(k).repeat_interleave(H // G, 1)
+    s = torch.einsum("ihd,jhd->hij", q, k) * m.scale
+    s = m.softcap * torch.tanh(s / m.softcap)
+    i, j = p.long()[:, None], p.long()[None, :]
+    s = s.masked_fill((j > i) | (i // m.chunk != j // m.chunk), float("-inf"))
+    s = torch.cat([s, sink.double()[:, None, None].expand(H, T, 1)], -1).softmax(-1)[..., :-1]
+    return torch.einsum("hij,jhd->ihd", s, v.double().repeat_interleave(H // G, 1)) * m.out_scale
+
+
+def test_the_two_forms_of_the_attention_oracle_agree():
+    m = AttentionMixer(heads=2, kv_heads=1, dim=8, vdim=4, chunk=7, rot_base=50.0, rot_dims=6, scale=0.5, softcap=2.0, out_scale=1.5)
+    q, k, v, sink = rand(20, 2, 8, seed=1), rand(20, 1, 8, seed=2), rand(20, 1, 4, seed=3), rand(2, seed=4)
+    assert torch.allclose(fast_attend(m, q, k, v, 50.0, 6, sink), oracle_attend(m, q, k, v, 50.0, 6, sink))
 
 
 ATTENTION_SIZES = [  # heads, kv_heads, dim, vdim, chunk, rot
@@ -214,6 +240,35 @@ def test_attention_over_many_keys(dtype):
     for steps in ([T], [T - 5, 1, 1, 1, 1, 1], [599, 2, 50, 49], [301, 297, 1, 1, 1, 99]):
         r = Replay((T,), [[(0, n)] for n in steps], block_size=64)
         close(attend(r, m, [q], [k], [v], dtype)[0], want, dtype, bf16=2e-2)
+
+
+@pytest.mark.parametrize("D,V", [(128, 128), (64, 64), (128, 64), (64, 128)])
+@pytest.mark.parametrize("chunk,softcap", [(100000, 4.0), (512, 60.0), (700, 3.0), (1000, 0.5)])
+def test_attention_of_long_prompts(chunk, softcap, D, V):
+    """The sizes and pages of the tcgen05 kernel: chunk borders inside its tiles, portions that start anywhere, caps that
+    are far away and caps that bind, rows whose maximum moves late (loud keys near the end), two requests at once."""
+    lengths, H, G, dtype = (1300, 389), 4, 2, torch.bfloat16
+    m = AttentionMixer(heads=H, kv_heads=G, dim=D, vdim=V, chunk=chunk, rot_base=1e4, rot_dims=32, scale=0.25, softcap=softcap, out_scale=0.7, device=DEV)
+    sink = rand(H, seed=5)
+    m.sink.copy_(sink)
+    qkv = []
+    for i, n in enumerate(lengths):
+        q, k, v = rand(n, H, D, seed=6 + i), rand(n, G, D, seed=17 + i), rand(n, G, V, seed=28 + i)
+        k[n // 3, :, 40] = 9.0
+        k[n - 100:, :, 41] = 6.0
+        q[n // 2:, :, 40] = 4.0
+        q[n - 60:, :, 41] = 5.0
+        qkv.append([t.to(dtype).float() for t in (q, k, v)])
+    q, k, v = zip(*qkv)
+    want = [fast_attend(m, *t, 1e4, 32, sink) for t in qkv]
+    whole = [[(s, n) for s, n in enumerate(lengths)]]
+    cuts = [[(0, 300), (1, 130)], [(0, 511), (1, 200)], [(0, 2)], [(0, 487), (1, 59)]]
+    for schedule, bs in ((whole, 256), (whole, 128), (cuts, 128)):
+        r = Replay(lengths, schedule, block_size=bs)
+        got = attend(r, m, q, k, v, dtype, pad=8, col=8)
+        for a, b in zip(got, want):
+            close(a, b, dtype, bf16=2e-2)
+    assert int(_lib.mixer_status(torch.device(DEV)).item()) == 0
 
 
 RETENTION_SIZES = [(3, 20, 28), (1, 9, 33), (2, 64, 64), (2, 32, 128), (4, 128, 64), (1, 80, 48)]
