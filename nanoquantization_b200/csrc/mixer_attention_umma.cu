@@ -51,11 +51,11 @@ __device__ __forceinline__ bool wait_bar(uint64_t* bar, uint32_t parity, volatil
   }
 }
 
-// D[tmem] (+)= A[smem descriptor] * B[smem descriptor]
-__device__ __forceinline__ void umma_ss(uint32_t d_tmem, uint64_t a_desc, uint64_t b_desc, uint32_t idesc, uint32_t accumulate) {
-  asm volatile("{\n .reg .pred p;\n setp.ne.b32 p, %4, 0;\n"
-               " tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n}"
-               ::"r"(d_tmem), "l"(a_desc), "l"(b_desc), "r"(idesc), "r"(accumulate) : "memory");
+// D[tmem] (+)= A[smem descriptor] * B[smem descriptor]; the descriptors' high halves are the same.
+__device__ __forceinline__ void umma_ss_lohi(uint32_t d_tmem, uint32_t a_lo, uint32_t b_lo, uint32_t hi, uint32_t idesc, uint32_t accumulate) {
+  asm volatile("{\n .reg .pred p;\n .reg .b64 a, b;\n setp.ne.b32 p, %5, 0;\n mov.b64 a, {%1, %3};\n mov.b64 b, {%2, %3};\n"
+               " tcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %4, p;\n}"
+               ::"r"(d_tmem), "r"(a_lo), "r"(b_lo), "r"(hi), "r"(idesc), "r"(accumulate) : "memory");
 }
 // Operand whose rows in shared memory run along k (the contraction), 64 columns = 128 swizzled bytes a row: 8-row groups
 // 1024 bytes apart along k, further blocks of 64 columns `block_bytes` apart.
@@ -180,48 +180,74 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
     }
   } else if (warp == 1) {
     // ------------------------------------------------------------------ MMA
+    // One thread runs both tiles as two little state machines and never blocks on one of them: it polls for a tile's
+    // weights (then issues O += P V) and for that product's end (P has been read: then S of the next key tile may
+    // overwrite it).  A ring stage is handed back by whichever tile uses it second.
     if (lane == 0) {
       const uint32_t idesc_s = umma_idesc(1, 128, kTile);
       const uint32_t idesc_o = umma_idesc(1, 128, V) | (1u << 16);   // B's rows run along k
+      const uint64_t dq = umma_smem_desc_sw128(smem), dk = umma_smem_desc_sw128(smem + kOffK), dv = smem_desc_mn(smem + kOffV, kBox);
+      const uint32_t k_hi = (uint32_t)(dq >> 32), v_hi = (uint32_t)(dv >> 32), q_lo = (uint32_t)dq, k_lo = (uint32_t)dk, v_lo = (uint32_t)dv;
       auto scores = [&](int q, int s) {
+        const uint32_t a = q_lo + q * (kQBytes >> 4), bk = k_lo + s * (kKBytes >> 4), d = tmem + kColS + q * 128;
 #pragma unroll
         for (int ks = 0; ks < D / 16; ++ks)
-          umma_ss(tmem + kColS + q * 128, umma_smem_desc_sw128(smem + q * kQBytes + (ks >> 2) * kBox + (ks & 3) * 32),
-                  umma_smem_desc_sw128(smem + kOffK + s * kKBytes + (ks >> 2) * kBox + (ks & 3) * 32), idesc_s, ks > 0 ? 1u : 0u);
+          umma_ss_lohi(d, a + (ks >> 2) * (kBox >> 4) + (ks & 3) * 2, bk + (ks >> 2) * (kBox >> 4) + (ks & 3) * 2, k_hi, idesc_s, ks > 0 ? 1u : 0u);
         umma_commit(smem_u32(&bar_s[q]));
       };
       bool ok = wait_bar(&bar_q, 0, s_abort, p.status) && wait_bar(&bar_kfull[0], 0, s_abort, p.status);
+      const int users = nq[1] > 0 ? 2 : 1;
+      // tile of the next product, whether it is under way, users that have still to issue on K / V tile j (by j & 1)
+      int jq[2] = {0, 0};
+      bool busy[2] = {false, false};
+      auto users_of = [&](int j) { return users == 2 ? (j < nq[0]) + (j < nq[1]) : 1; };
+      int kleft[2] = {0, users_of(1)}, vleft[2] = {users_of(0), users_of(1)};
       if (ok) {
         tc_fence_after();
-        for (int q = 0; q < 2; ++q) if (nq[q] > 0) scores(q, 0);
+        for (int q = 0; q < users; ++q) scores(q, 0);
         umma_commit(smem_u32(&bar_kfree[0]));
+        kleft[0] = users_of(2);
       }
-      for (int j = 0; ok && j < nmax; ++j) {
-        const int s = j & 1, sn = s ^ 1;
-        bool v_here = false, k_here = false;
-        for (int q = 0; ok && q < 2; ++q) {
-          if (j >= nq[q]) continue;
-          ok = wait_bar(&bar_p[q], j & 1, s_abort, p.status);
-          if (ok && !v_here) { ok = wait_bar(&bar_vfull[s], (j >> 1) & 1, s_abort, p.status); v_here = true; }
-          if (!ok) break;
-          tc_fence_after();
+      unsigned long long t_last = global_timer_ns();
+      uint32_t polls = 0;
+      while (ok && (jq[0] < nq[0] || jq[1] < nq[1])) {
+        bool moved = false;
 #pragma unroll
-          for (int ks = 0; ks < kTile / 16; ++ks)
-            umma_ts(tmem + kColO + q * 128, tmem + kColS + q * 128 + ks * 8, smem_desc_mn(smem + kOffV + s * kVBytes + ks * 2048, kBox), idesc_o,
-                    (j > 0 || ks > 0) ? 1u : 0u);
-          umma_commit(smem_u32(&bar_pv[q]));
-          if (j == nq[q] - 1) umma_commit(smem_u32(&bar_o[q]));
-          if (j + 1 < nq[q]) {
-            if (!k_here) { ok = wait_bar(&bar_kfull[sn], ((j + 1) >> 1) & 1, s_abort, p.status); k_here = true; }
-            ok = ok && wait_bar(&bar_pv[q], j & 1, s_abort, p.status);   // P has been read: S may overwrite it
-            if (!ok) break;
+        for (int q = 0; q < 2; ++q) {
+          const int j = jq[q], s = j & 1, sn = s ^ 1;
+          if (j >= nq[q]) continue;
+          if (!busy[q]) {
+            if (!mbar_test_wait(smem_u32(&bar_p[q]), s) || !mbar_test_wait(smem_u32(&bar_vfull[s]), (j >> 1) & 1)) continue;
+            tc_fence_after();
+            const uint32_t d = tmem + kColO + q * 128, pa = tmem + kColS + q * 128, bv = v_lo + s * (kVBytes >> 4);
+#pragma unroll
+            for (int ks = 0; ks < kTile / 16; ++ks) umma_ts_lohi(d, pa + ks * 8, bv + ks * (2048 >> 4), v_hi, idesc_o, (j > 0 || ks > 0) ? 1u : 0u);
+            umma_commit(smem_u32(&bar_pv[q]));
+            if (--vleft[s] == 0) { umma_commit(smem_u32(&bar_vfree[s])); vleft[s] = users_of(j + 2); }
+            if (j == nq[q] - 1) { umma_commit(smem_u32(&bar_o[q])); jq[q] = j + 1; }
+            else busy[q] = true;
+          } else {
+            if (!mbar_test_wait(smem_u32(&bar_pv[q]), s) || !mbar_test_wait(smem_u32(&bar_kfull[sn]), ((j + 1) >> 1) & 1)) continue;
             tc_fence_after();
             scores(q, sn);
+            if (--kleft[sn] == 0) { umma_commit(smem_u32(&bar_kfree[sn])); kleft[sn] = users_of(j + 3); }
+            jq[q] = j + 1;
+            busy[q] = false;
+          }
+          moved = true;
+        }
+        if (moved) {
+          polls = 0;
+        } else if ((++polls & 63u) == 0) {
+          const unsigned long long now = global_timer_ns();
+          if (polls == 64) t_last = now;
+          if (*s_abort) ok = false;
+          else if (now - t_last > kWaitLimitNs) {
+            *s_abort = 1;
+            if (p.status) atomicExch(p.status, NQB200_ERR_WAIT_TIMEOUT);
+            ok = false;
           }
         }
-        if (!ok) break;
-        umma_commit(smem_u32(&bar_vfree[s]));
-        if (k_here) umma_commit(smem_u32(&bar_kfree[sn]));
       }
       // everything issued has completed before tensor memory may be released
       umma_commit(smem_u32(&bar_drain));
@@ -244,7 +270,7 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
     const float sink = p.sink ? p.sink[h] * kLog2e : -INFINITY;
     float m = sink, l = 0.f;
     uint64_t lsum = pair2(0.f, 0.f);
-    uint32_t r[32];
+    uint32_t buf[2][32];   // a chunk of 32 columns is read while the one before it is worked on
     bool ok = true;
     for (int j = 0; j < nq[q]; ++j) {
       ok = wait_bar(&bar_s[q], j & 1, s_abort, p.status);
@@ -253,10 +279,12 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
       const int key0 = kstart + j * kTile;
       const bool masked = key0 + kTile - 1 > wfirst || key0 < lo_last;     // for any row of the warp
       float mx = -INFINITY, ab = 0.f;
+      tmem_ld32(tS, buf[0]);
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
-        tmem_ld32(tS + c * 32, r);
         tc_wait_ld();
+        uint32_t (&r)[32] = buf[c & 1];
+        tmem_ld32(tS + (c < 3 ? c + 1 : 0) * 32, buf[(c + 1) & 1]);   // after the last chunk: the first one again, for the second pass
         if (masked) {
 #pragma unroll
           for (int e = 0; e < 32; ++e) {
@@ -286,6 +314,7 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
           lsum = pair2(a * f, c2 * f);
 #pragma unroll
           for (int c = 0; c < V / 32; ++c) {
+            uint32_t (&r)[32] = buf[1];
             tmem_ld32(tO + c * 32, r);
             tc_wait_ld();
 #pragma unroll
@@ -300,8 +329,9 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
       const uint64_t nm2 = pair2(-mu, -mu);
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
-        tmem_ld32(tS + c * 32, r);
         tc_wait_ld();
+        uint32_t (&r)[32] = buf[c & 1];
+        if (c < 3) tmem_ld32(tS + (c + 1) * 32, buf[(c + 1) & 1]);
         uint32_t w[16];
         if (series) {
 #pragma unroll
@@ -351,6 +381,7 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
         bf16* dst = p.out + (size_t)(t0 + i) * p.out_stride + (size_t)h * V;
 #pragma unroll
         for (int c = 0; c < V / 32; ++c) {
+          uint32_t (&r)[32] = buf[0];
           tmem_ld32(tO + c * 32, r);
           tc_wait_ld();
           if (i < n) {

@@ -40,6 +40,7 @@ struct AttSmem {
   alignas(16) bf16 knew[kDecMaxDim];
   float s[kDecHeads][kDecTile + 4];
   float cs[kDecMaxDim];
+  int rows[4][kDecTile];                      // cache rows of the keys of four successive tiles
   float m[kDecHeads], l[kDecHeads], corr[kDecHeads];
   float out[kDecHeads][kDecMaxDim];           // this CTA's share, read by the cluster
 };
@@ -93,16 +94,28 @@ __device__ void attention_decode(const DecodeArgs& a, uint8_t* smem, int b, int 
 
   auto load_tile = [&](int i) {
     if (i < tiles) {
-      bf16* kd = ring + (size_t)(i % kDecStages) * att_stage(D, VP) + (tid >> 1) * KS;
-      bf16* vd = ring + (size_t)(i % kDecStages) * att_stage(D, VP) + kDecTile * KS + (tid >> 1) * VS;
-      const int j = k0 + i * kDecTile + (tid >> 1);            // two threads per key
-      const bool ok = j < k1 && j != pos;
-      const size_t r = kv_row(a.bt, b, ok ? j : k0) * at.kv_heads + kvh;
-      for (int c = tid & 1; c < D8; c += 2) dec_cp16(dec_smem(kd + c * 8), a.k_cache + r * D + c * 8, ok);
-      for (int c = tid & 1; c < V8; c += 2) dec_cp16(dec_smem(vd + c * 8), a.v_cache + r * V + c * 8, ok);
+      bf16* kd = ring + (size_t)(i % kDecStages) * att_stage(D, VP);
+      bf16* vd = kd + kDecTile * KS;
+      // neighbouring threads copy neighbouring 16-byte pieces of a row
+      for (int e = tid; e < kDecTile * D8; e += kDecThreads) {
+        const int key = e / D8, c = e - key * D8, j = k0 + i * kDecTile + key;
+        dec_cp16(dec_smem(kd + key * KS + c * 8), a.k_cache + ((size_t)sm.rows[i & 3][key] * at.kv_heads + kvh) * D + c * 8, j < k1 && j != pos);
+      }
+      for (int e = tid; e < kDecTile * V8; e += kDecThreads) {
+        const int key = e / V8, c = e - key * V8, j = k0 + i * kDecTile + key;
+        dec_cp16(dec_smem(vd + key * VS + c * 8), a.v_cache + ((size_t)sm.rows[i & 3][key] * at.kv_heads + kvh) * V + c * 8, j < k1 && j != pos);
+      }
     }
     asm volatile("cp.async.commit_group;");
   };
+  auto find_rows = [&](int first, int count) {   // of tiles first .. first + count - 1
+    for (int e = tid; e < count * kDecTile; e += kDecThreads) {
+      const int i = first + e / kDecTile, key = e % kDecTile;
+      if (i < tiles) sm.rows[i & 3][key] = (int)kv_row(a.bt, b, min(k0 + i * kDecTile + key, k1 - 1));
+    }
+  };
+  find_rows(0, 4);
+  __syncthreads();
 #pragma unroll
   for (int i = 0; i < kDecStages - 1; ++i) load_tile(i);
 
@@ -148,6 +161,7 @@ __device__ void attention_decode(const DecodeArgs& a, uint8_t* smem, int b, int 
     asm volatile("cp.async.wait_group %0;" ::"n"(kDecStages - 2));
     __syncthreads();               // tile i has landed for every thread; tile i - 1 is no longer read
     load_tile(i + kDecStages - 1);
+    find_rows(i + 4, 1);           // over tile i's, whose loads are done; read after the next barrier at the earliest
     const int j0 = k0 + i * kDecTile, cnt = min(kDecTile, k1 - j0);
     bf16* kt = ring + (size_t)(i % kDecStages) * att_stage(D, VP);
     bf16* vt = kt + kDecTile * KS;
@@ -224,14 +238,22 @@ __device__ void attention_decode(const DecodeArgs& a, uint8_t* smem, int b, int 
   for (int e = rank * kDecThreads + tid; e < R * V; e += csize * kDecThreads) {
     const int r = e / V, c = e % V;
     const float sink = at.sink ? at.sink[h0 + r] : -INFINITY;
-    float m = sink;
-    for (int k = 0; k < csize; ++k) m = fmaxf(m, cl.map_shared_rank(&sm, k)->m[r]);
+    float pm[8], pl[8], po[8], m = sink;   // all of the cluster's shares at once
+#pragma unroll
+    for (int k = 0; k < 8; ++k) {
+      const AttSmem* s = cl.map_shared_rank(&sm, k < csize ? k : 0);
+      pm[k] = k < csize ? s->m[r] : -INFINITY;
+      pl[k] = s->l[r];
+      po[k] = s->out[r][c];
+    }
+#pragma unroll
+    for (int k = 0; k < 8; ++k) m = fmaxf(m, pm[k]);
     float l = at.sink ? expf(sink - m) : 0.f, o = 0.f;
-    for (int k = 0; k < csize; ++k) {
-      const AttSmem* s = cl.map_shared_rank(&sm, k);
-      const float f = expf(s->m[r] - m);      // 0 for a CTA without keys
-      l += s->l[r] * f;
-      o += s->out[r][c] * f;
+#pragma unroll
+    for (int k = 0; k < 8; ++k) {
+      const float f = expf(pm[k] - m);      // 0 for a CTA without keys, and beyond the cluster
+      l += pl[k] * f;
+      o += po[k] * f;
     }
     a.act[(size_t)b * a.act_stride + a.a_col + (size_t)(h0 + r) * V + c] = __float2bfloat16_rn(o / l * at.out_scale);
   }
@@ -410,8 +432,8 @@ extern "C" int nqb200_mixer_decode(const void* proj, int64_t stride, void* act, 
     units += r->heads;
     while (want < 8 && (int64_t)r->dim * r->vdim * 4 > (int64_t)want * 16384 && want * 8 <= r->vdim) want *= 2;
   }
-  // enough CTAs for two per SM, and no more than there is work for
-  while (csize < want && units * b->batch * csize < 2 * kNumSMs) csize *= 2;
+  // CTAs for one wave at two per SM, and no more than there is work for
+  while (csize < want && units * b->batch * csize * 2 <= 2 * kNumSMs) csize *= 2;
   cudaStream_t st = (cudaStream_t)stream;
   const bool v4 = !r || r->vdim % 4 == 0;
 #define NQB200_DEC(VP) return v4 ? launch_decode<VP, 4>(p, csize, st) : launch_decode<VP, 1>(p, csize, st)

@@ -323,29 +323,40 @@ __global__ void __launch_bounds__(128) retention_chunk_kernel(const ChunkStateAr
   const uint32_t a_addr = smem_addr(ks + ((lane & 7) + ((lane >> 4) << 3)) * kTS + warp * 16 + ((lane >> 3) & 1) * 8);
   const uint32_t b_lane = (((lane & 7) + (((lane >> 3) & 1) << 3)) * kTS + (lane >> 4) * 8) * 2;
   const uint4 zero = make_uint4(0, 0, 0, 0);
+  // a thread's 16-byte pieces: rows tid / 8 + 16 i of the tile, loaded a tile ahead (from places that exist) into registers
+  const int r0 = tid >> 3, cc = (tid & 7) * 8, kcol = min(d0 + cc, a.dim - 8), vcol = min(v0 + cc, a.vdim - 8);
+  uint4 kreg[4], vreg[4];
+  auto fetch = [&](int j0) {
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const size_t row = (size_t)(t0 + first + min(j0 + r0 + 16 * i, len - 1)) * a.stride;
+      kreg[i] = *reinterpret_cast<const uint4*>(a.k + row + (size_t)h * a.dim + kcol);
+      vreg[i] = *reinterpret_cast<const uint4*>(a.v + row + (size_t)h * a.vdim + vcol);
+    }
+  };
+  fetch(0);
   for (int j0 = 0; j0 < len; j0 += 64) {
     __syncthreads();
-    for (int e = tid; e < 64 * 8; e += 128) {
-      const int r = e / 8, cc = e % 8 * 8, j = j0 + r;
-      const size_t row = (size_t)(t0 + first + min(j, len - 1)) * a.stride;
-      uint4 kv = zero, vv = zero;
-      if (j < len && d0 + cc < a.dim) kv = *reinterpret_cast<const uint4*>(a.k + row + (size_t)h * a.dim + d0 + cc);
-      if (j < len && v0 + cc < a.vdim) vv = *reinterpret_cast<const uint4*>(a.v + row + (size_t)h * a.vdim + v0 + cc);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int r = r0 + 16 * i, j = j0 + r;
+      const uint4 kv = d0 + cc < a.dim ? kreg[i] : zero, vv = v0 + cc < a.vdim ? vreg[i] : zero;
       *reinterpret_cast<uint4*>(ks + r * kTS + cc) = kv;
       const float w = j < len ? kscale * decay_pow(log2d, len - 1 - j) : 0.f;
       const uint32_t in[4] = {vv.x, vv.y, vv.z, vv.w};
       uint32_t hi[4], lo[4];
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const float x = __uint_as_float(in[i] << 16) * w, y = __uint_as_float(in[i] & 0xFFFF0000u) * w;
+      for (int k = 0; k < 4; ++k) {
+        const float x = __uint_as_float(in[k] << 16) * w, y = __uint_as_float(in[k] & 0xFFFF0000u) * w;
         const float hx = __bfloat162float(__float2bfloat16_rn(x)), hy = __bfloat162float(__float2bfloat16_rn(y));
-        hi[i] = pack2(hx, hy);
-        lo[i] = pack2(x - hx, y - hy);
+        hi[k] = pack2(hx, hy);
+        lo[k] = pack2(x - hx, y - hy);
       }
       *reinterpret_cast<uint4*>(vh + r * kTS + cc) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
       *reinterpret_cast<uint4*>(vl + r * kTS + cc) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
     }
     __syncthreads();
+    if (j0 + 64 < len) fetch(j0 + 64);
 #pragma unroll
     for (int kt = 0; kt < 4; ++kt) {
       uint32_t ka[4];

@@ -203,12 +203,13 @@ __global__ void __launch_bounds__(256) mingru_chunk_kernel(const T* __restrict__
   float* own = p.state + (size_t)p.bt.slot[b] * p.width + c;
   float2 a[kGruWarpTokens], v[kGruWarpTokens], A = make_float2(1.f, 1.f), B = make_float2(0.f, 0.f);
   const float2 zb = live ? ld_pair(p.z_bias + c) : B, xb = live ? ld_pair(p.x_bias + c) : B;
-  const T* row = proj + (size_t)(t0 + tok0) * p.stride + c;
+  // every load is made, from a place that exists (what does not count is masked below), so that all are under way at once
+  const T* base = proj + (live ? c : 0);
 #pragma unroll
   for (int i = 0; i < kGruWarpTokens; ++i) {
-    const bool ok = live && i < cnt;
-    a[i] = ok ? ld_pair(row + (size_t)i * p.stride + p.z_off) : B;
-    v[i] = ok ? ld_pair(row + (size_t)i * p.stride + p.x_off) : B;
+    const T* row = base + (size_t)(t0 + min(tok0 + i, n - 1)) * p.stride;
+    a[i] = ld_pair(row + p.z_off);
+    v[i] = ld_pair(row + p.x_off);
   }
 #pragma unroll
   for (int i = 0; i < kGruWarpTokens; ++i) {
@@ -256,11 +257,14 @@ __global__ void __launch_bounds__(256) mingru_chunk_kernel(const T* __restrict__
     S.x = wa.x * S.x + wb.x; S.y = wa.y * S.y + wb.y;
   }
   T* orow = out + (size_t)(t0 + tok0) * p.width + c;
+  float2 gate[kGruWarpTokens];
+#pragma unroll
+  for (int i = 0; i < kGruWarpTokens; ++i) gate[i] = ld_pair(base + (size_t)(t0 + min(tok0 + i, n - 1)) * p.stride + p.g_off);
 #pragma unroll
   for (int i = 0; i < kGruWarpTokens; ++i) {
     S.x = a[i].x * S.x + v[i].x; S.y = a[i].y * S.y + v[i].y;
     if (live && i < cnt) {
-      const float2 g = ld_pair(row + (size_t)i * p.stride + p.g_off);
+      const float2 g = gate[i];
       st_pair(orow + (size_t)i * p.width, make_float2(S.x * (g.x * gate_sigmoid<T>(g.x)), S.y * (g.y * gate_sigmoid<T>(g.y))));
     }
   }
