@@ -79,8 +79,8 @@ typedef struct {
 } nqb200_retention_desc;
 
 /* Prompts (bf16): retention in chunkwise form with norm and gate.  proj holds q | k | v | gate from column off; the
- * result goes to act from column act_col.  chunk_states: scratch, nqb200_retention_chunks(tokens, batch) * heads * dim
- * * vdim floats. */
+ * result goes to act from column act_col.  chunk_states: scratch, 2 * nqb200_retention_chunks(tokens, batch) * heads *
+ * dim * vdim floats. */
 int nqb200_retention_prefill(const void* proj, int64_t stride, int64_t off, void* act, int64_t act_stride, int64_t act_col,
                              const nqb200_retention_desc* r, float* state, float* chunk_states, const nqb200_batch* b, void* stream);
 int nqb200_retention_prefill_supported(const nqb200_retention_desc* r, int64_t stride, int64_t off, int64_t act_stride, int64_t act_col);

@@ -77,13 +77,9 @@ __device__ __forceinline__ void tmem_ld32(uint32_t taddr, uint32_t (&r)[32]) {
                  "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
                : "r"(taddr) : "memory");
 }
-__device__ __forceinline__ void tmem_st32(uint32_t taddr, const uint32_t (&r)[32]) {
-  asm volatile("tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,"
-               "%24,%25,%26,%27,%28,%29,%30,%31,%32};"
-               ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]),
-                 "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]), "r"(r[16]), "r"(r[17]), "r"(r[18]), "r"(r[19]),
-                 "r"(r[20]), "r"(r[21]), "r"(r[22]), "r"(r[23]), "r"(r[24]), "r"(r[25]), "r"(r[26]), "r"(r[27]), "r"(r[28]), "r"(r[29]),
-                 "r"(r[30]), "r"(r[31]) : "memory");
+__device__ __forceinline__ void tmem_st8(uint32_t taddr, const uint32_t (&r)[8]) {
+  asm volatile("tcgen05.st.sync.aligned.32x32b.x8.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8};"
+               ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]) : "memory");
 }
 __device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t (&r)[16]) {
   asm volatile("tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16};"
@@ -263,14 +259,13 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
     const float ysc = capped ? p.scale / p.softcap : p.scale, top = capped ? p.softcap * kLog2e : kLog2e;
     auto score = [&](float s) {   // in log2 units
       const float y = s * ysc;
-      return top * (capped ? 1.f - __fdividef(2.f, 1.f + ex2(y * (2.f * kLog2e))) : y);
+      return top * (capped ? tanh_fast(y) : y);
     };
     const uint64_t ysc2 = pair2(ysc, ysc), k1 = pair2(top, top), k3 = pair2(-top / 3.f, -top / 3.f), k5 = pair2(top * (2.f / 15.f), top * (2.f / 15.f)),
                    k7 = pair2(-top * (17.f / 315.f), -top * (17.f / 315.f)), k9 = pair2(top * (62.f / 2835.f), top * (62.f / 2835.f));
     const float sink = p.sink ? p.sink[h] * kLog2e : -INFINITY;
     float m = sink, l = 0.f;
     uint64_t lsum = pair2(0.f, 0.f);
-    uint32_t buf[2][32];   // a chunk of 32 columns is read while the one before it is worked on
     bool ok = true;
     for (int j = 0; j < nq[q]; ++j) {
       ok = wait_bar(&bar_s[q], j & 1, s_abort, p.status);
@@ -278,26 +273,30 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
       tc_fence_after();
       const int key0 = kstart + j * kTile;
       const bool masked = key0 + kTile - 1 > wfirst || key0 < lo_last;     // for any row of the warp
-      float mx = -INFINITY, ab = 0.f;
-      tmem_ld32(tS, buf[0]);
+      uint32_t r[4][32];     // the row's scores, all of them
 #pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        tc_wait_ld();
-        uint32_t (&r)[32] = buf[c & 1];
-        tmem_ld32(tS + (c < 3 ? c + 1 : 0) * 32, buf[(c + 1) & 1]);   // after the last chunk: the first one again, for the second pass
-        if (masked) {
+      for (int c = 0; c < 4; ++c) tmem_ld32(tS + c * 32, r[c]);
+      tc_wait_ld();
+      float mx = -INFINITY, ab = 0.f;
+      if (!masked) {
+        float mv[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY}, av[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+        for (int c = 0; c < 4; ++c)
+#pragma unroll
+          for (int e = 0; e < 32; ++e) {
+            mv[e & 3] = fmaxf(mv[e & 3], __uint_as_float(r[c][e]));
+            av[e & 3] = fmaxf(av[e & 3], fabsf(__uint_as_float(r[c][e])));
+          }
+        mx = fmaxf(fmaxf(mv[0], mv[1]), fmaxf(mv[2], mv[3]));
+        ab = fmaxf(fmaxf(av[0], av[1]), fmaxf(av[2], av[3]));
+      } else {
+#pragma unroll
+        for (int c = 0; c < 4; ++c)
 #pragma unroll
           for (int e = 0; e < 32; ++e) {
             const int key = key0 + c * 32 + e;
-            if (key <= pos && key >= lo) mx = fmaxf(mx, __uint_as_float(r[e]));
+            mx = (key <= pos && key >= lo) ? fmaxf(mx, __uint_as_float(r[c][e])) : mx;
           }
-        } else {
-#pragma unroll
-          for (int e = 0; e < 32; ++e) {
-            mx = fmaxf(mx, __uint_as_float(r[e]));
-            ab = fmaxf(ab, fabsf(__uint_as_float(r[e])));
-          }
-        }
       }
       const float mt = mx == -INFINITY ? mx : score(mx), mn = fmaxf(m, mt);
       if (j == 0) {
@@ -312,31 +311,27 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
           float a, c2;
           unpair2(lsum, a, c2);
           lsum = pair2(a * f, c2 * f);
-#pragma unroll
-          for (int c = 0; c < V / 32; ++c) {
-            uint32_t (&r)[32] = buf[1];
-            tmem_ld32(tO + c * 32, r);
+#pragma unroll 1
+          for (int c = 0; c < V / 8; ++c) {   // rare: small pieces, few registers
+            uint32_t o[8];
+            tmem_ld_32x32b_x8(tO + c * 8, o);
             tc_wait_ld();
 #pragma unroll
-            for (int e = 0; e < 32; ++e) r[e] = __float_as_uint(__uint_as_float(r[e]) * f);
-            tmem_st32(tO + c * 32, r);
+            for (int e = 0; e < 8; ++e) o[e] = __float_as_uint(__uint_as_float(o[e]) * f);
+            tmem_st8(tO + c * 8, o);
           }
           tc_wait_st();
         }
       }
       const float mu = m == -INFINITY ? 0.f : m;
-      const bool series = !masked && (!capped || __all_sync(0xFFFFFFFFu, ab * ysc <= kSeriesRange));
-      const uint64_t nm2 = pair2(-mu, -mu);
+      if (!masked && (!capped || __all_sync(0xFFFFFFFFu, ab * ysc <= kSeriesRange))) {
+        const uint64_t nm2 = pair2(-mu, -mu);
 #pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        tc_wait_ld();
-        uint32_t (&r)[32] = buf[c & 1];
-        if (c < 3) tmem_ld32(tS + (c + 1) * 32, buf[(c + 1) & 1]);
-        uint32_t w[16];
-        if (series) {
+        for (int c = 0; c < 4; ++c) {
+          uint32_t w[16];
 #pragma unroll
           for (int e = 0; e < 16; ++e) {
-            const uint64_t y = mul2(pair2(__uint_as_float(r[2 * e]), __uint_as_float(r[2 * e + 1])), ysc2);
+            const uint64_t y = mul2(pair2(__uint_as_float(r[c][2 * e]), __uint_as_float(r[c][2 * e + 1])), ysc2);
             uint64_t arg;
             if (capped) {
               const uint64_t y2 = mul2(y, y);
@@ -351,20 +346,28 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
             lsum = add2(lsum, pair2(x0, x1));
             w[e] = pack_bf16(x0, x1);
           }
-        } else {
+          tmem_st16(tS + c * 16, w);
+        }
+      } else {
+        // from tensor memory again, a piece at a time: compact code for the few tiles at the edges
+#pragma unroll 1
+        for (int c = 0; c < 8; ++c) {
+          uint32_t v[16], w[8];
+          tmem_ld_32x32b_x16(tS + c * 16, v);
+          tc_wait_ld();
 #pragma unroll
-          for (int e = 0; e < 16; ++e) {
+          for (int e = 0; e < 8; ++e) {
             float x[2];
 #pragma unroll
             for (int u = 0; u < 2; ++u) {
-              const int key = key0 + c * 32 + 2 * e + u;
-              x[u] = (key <= pos && key >= lo) ? ex2(score(__uint_as_float(r[2 * e + u])) - mu) : 0.f;
+              const int key = key0 + c * 16 + 2 * e + u;
+              x[u] = (key <= pos && key >= lo) ? ex2(score(__uint_as_float(v[2 * e + u])) - mu) : 0.f;
             }
             lsum = add2(lsum, pair2(x[0], x[1]));
             w[e] = pack_bf16(x[0], x[1]);
           }
+          tmem_st8(tS + c * 8, w);      // lies behind what has been read of S
         }
-        tmem_st16(tS + c * 16, w);      // lies behind what has been read of S
       }
       tc_wait_st();
       tc_fence_before();
@@ -381,7 +384,7 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
         bf16* dst = p.out + (size_t)(t0 + i) * p.out_stride + (size_t)h * V;
 #pragma unroll
         for (int c = 0; c < V / 32; ++c) {
-          uint32_t (&r)[32] = buf[0];
+          uint32_t r[32];
           tmem_ld32(tO + c * 32, r);
           tc_wait_ld();
           if (i < n) {

@@ -11,12 +11,12 @@ namespace cg = cooperative_groups;
 
 namespace nqb200 {
 
-constexpr int kDecThreads = 128;
-constexpr int kDecTile = 64;       // keys per pass of a CTA: 16 per warp
-constexpr int kDecStages = 3;      // passes whose keys and values are under way
+constexpr int kDecThreads = 256;
+constexpr int kDecMaxTile = 128;   // keys per pass of a CTA at most: 16 per warp
+constexpr int kDecStages = 2;      // passes in the ring
 constexpr int kDecHeads = 8;       // query heads per cluster at most (columns of one mma)
 constexpr int kDecMaxDim = 256;
-constexpr int kDecPS = kDecTile + 8;
+constexpr int kDecPS = kDecMaxTile + 8;
 
 struct DecodeArgs {
   const bf16* proj; int64_t stride;
@@ -38,9 +38,9 @@ struct AttSmem {
   alignas(16) bf16 q[kDecHeads][kDecMaxDim + 8];
   alignas(16) bf16 p[16][kDecPS];             // weights, rows 8 .. 15 stay zero
   alignas(16) bf16 knew[kDecMaxDim];
-  float s[kDecHeads][kDecTile + 4];
+  float s[kDecHeads][kDecMaxTile + 4];
   float cs[kDecMaxDim];
-  int rows[4][kDecTile];                      // cache rows of the keys of four successive tiles
+  int rows[4][kDecMaxTile];                   // cache rows of the keys of four successive tiles
   float m[kDecHeads], l[kDecHeads], corr[kDecHeads];
   float out[kDecHeads][kDecMaxDim];           // this CTA's share, read by the cluster
 };
@@ -49,7 +49,7 @@ struct RetSmem {
   float q[1024], k[1024];
   float red[kDecThreads * 4];
   float o[1024];
-  float ss, wsum[4];
+  float ss, wsum[kDecThreads / 32];
 };
 
 __device__ __forceinline__ uint32_t dec_smem(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -72,10 +72,10 @@ __device__ __forceinline__ void dec_ldsm2(uint32_t (&r)[2], uint32_t a) {
 }
 
 __host__ __device__ constexpr int att_ks(int dim) { return (dim + 15) / 16 * 16 + 8; }   // row strides of the ring, in elements
-__host__ __device__ constexpr int att_stage(int dim, int vp) { return kDecTile * (att_ks(dim) + vp + 8); }
+__host__ __device__ constexpr int att_stage(int dim, int vp, int tile) { return tile * (att_ks(dim) + vp + 8); }
 
-// VP: value columns padded to 64, 128 or 256; a warp owns a quarter of them.
-template <int VP>
+// VP: value columns padded to 64, 128 or 256; a warp owns a quarter of them and half of a tile's keys.
+template <int VP, int TILE>
 __device__ void attention_decode(const DecodeArgs& a, uint8_t* smem, int b, int unit, cg::cluster_group& cl) {
   AttSmem& sm = *reinterpret_cast<AttSmem*>(smem);
   bf16* ring = reinterpret_cast<bf16*>(smem + sizeof(AttSmem));
@@ -86,7 +86,7 @@ __device__ void attention_decode(const DecodeArgs& a, uint8_t* smem, int b, int 
   const int D = at.dim, V = at.vdim, pos = a.bt.pos0[b];
   const int lo = at.chunk > 0 ? pos / at.chunk * at.chunk : 0, nk = pos - lo + 1;
   const int per = (nk + csize - 1) / csize, k0 = lo + rank * per, k1 = min(lo + nk, k0 + per);   // this CTA's keys
-  const int tiles = k1 > k0 ? (k1 - k0 + kDecTile - 1) / kDecTile : 0;
+  const int tiles = k1 > k0 ? (k1 - k0 + TILE - 1) / TILE : 0;
   const int KS = att_ks(D), D8 = D / 8, V8 = V / 8, half = a.rot / 2;
   constexpr int VS = VP + 8, NT = VP / 32;       // n-tiles of 8 columns per warp
   const bf16* row = a.proj + (size_t)b * a.stride;
@@ -94,24 +94,29 @@ __device__ void attention_decode(const DecodeArgs& a, uint8_t* smem, int b, int 
 
   auto load_tile = [&](int i) {
     if (i < tiles) {
-      bf16* kd = ring + (size_t)(i % kDecStages) * att_stage(D, VP);
-      bf16* vd = kd + kDecTile * KS;
+      bf16* kd = ring + (size_t)(i % kDecStages) * att_stage(D, VP, TILE);
+      bf16* vd = kd + TILE * KS;
       // neighbouring threads copy neighbouring 16-byte pieces of a row
-      for (int e = tid; e < kDecTile * D8; e += kDecThreads) {
-        const int key = e / D8, c = e - key * D8, j = k0 + i * kDecTile + key;
-        dec_cp16(dec_smem(kd + key * KS + c * 8), a.k_cache + ((size_t)sm.rows[i & 3][key] * at.kv_heads + kvh) * D + c * 8, j < k1 && j != pos);
-      }
-      for (int e = tid; e < kDecTile * V8; e += kDecThreads) {
-        const int key = e / V8, c = e - key * V8, j = k0 + i * kDecTile + key;
-        dec_cp16(dec_smem(vd + key * VS + c * 8), a.v_cache + ((size_t)sm.rows[i & 3][key] * at.kv_heads + kvh) * V + c * 8, j < k1 && j != pos);
-      }
+      const int j0 = k0 + i * TILE;
+      auto copy = [&](bf16* dst, int dstride, const bf16* cache, int n8, int size) {
+        const int dk = kDecThreads / n8, dc = kDecThreads % n8;
+        for (int key = tid / n8, c = tid % n8; key < TILE;) {
+          dec_cp16(dec_smem(dst + key * dstride + c * 8), cache + ((size_t)sm.rows[i & 3][key] * at.kv_heads + kvh) * size + c * 8,
+                   j0 + key < k1 && j0 + key != pos);
+          key += dk;
+          c += dc;
+          if (c >= n8) { c -= n8; ++key; }
+        }
+      };
+      copy(kd, KS, a.k_cache, D8, D);
+      copy(vd, VS, a.v_cache, V8, V);
     }
     asm volatile("cp.async.commit_group;");
   };
   auto find_rows = [&](int first, int count) {   // of tiles first .. first + count - 1
-    for (int e = tid; e < count * kDecTile; e += kDecThreads) {
-      const int i = first + e / kDecTile, key = e % kDecTile;
-      if (i < tiles) sm.rows[i & 3][key] = (int)kv_row(a.bt, b, min(k0 + i * kDecTile + key, k1 - 1));
+    for (int e = tid; e < count * TILE; e += kDecThreads) {
+      const int i = first + e / TILE, key = e % TILE;
+      if (i < tiles) sm.rows[i & 3][key] = (int)kv_row(a.bt, b, min(k0 + i * TILE + key, k1 - 1));
     }
   };
   find_rows(0, 4);
@@ -120,13 +125,13 @@ __device__ void attention_decode(const DecodeArgs& a, uint8_t* smem, int b, int 
   for (int i = 0; i < kDecStages - 1; ++i) load_tile(i);
 
   // while those are under way: padding columns, the rotated queries and (in the CTA that holds the newest key) key
-  for (int e = tid; e < kDecStages * kDecTile * (KS - 8 - D); e += kDecThreads) {
+  for (int e = tid; e < kDecStages * TILE * (KS - 8 - D); e += kDecThreads) {
     const int r = e / (KS - 8 - D), c = e % (KS - 8 - D);
-    ring[(size_t)(r / kDecTile) * att_stage(D, VP) + (r % kDecTile) * KS + D + c] = __float2bfloat16_rn(0.f);
+    ring[(size_t)(r / TILE) * att_stage(D, VP, TILE) + (r % TILE) * KS + D + c] = __float2bfloat16_rn(0.f);
   }
-  for (int e = tid; e < kDecStages * kDecTile * (VP - V); e += kDecThreads) {
+  for (int e = tid; e < kDecStages * TILE * (VP - V); e += kDecThreads) {
     const int r = e / (VP - V), c = e % (VP - V);
-    ring[(size_t)(r / kDecTile) * att_stage(D, VP) + kDecTile * KS + (r % kDecTile) * VS + V + c] = __float2bfloat16_rn(0.f);
+    ring[(size_t)(r / TILE) * att_stage(D, VP, TILE) + TILE * KS + (r % TILE) * VS + V + c] = __float2bfloat16_rn(0.f);
   }
   for (int e = tid; e < kDecHeads * (KS - 8); e += kDecThreads) sm.q[e / (KS - 8)][e % (KS - 8)] = __float2bfloat16_rn(0.f);
   for (int e = tid; e < 16 * kDecPS; e += kDecThreads) sm.p[e / kDecPS][e % kDecPS] = __float2bfloat16_rn(0.f);
@@ -146,10 +151,12 @@ __device__ void attention_decode(const DecodeArgs& a, uint8_t* smem, int b, int 
       dst[j + half] = src[j + half];
     }
   }
+  const float inv_cap = at.softcap > 0.f ? 1.f / at.softcap : 0.f;
   const uint32_t k_lane = (uint32_t)((warp * 16 + (lane & 15)) * KS + (lane >> 4) * 8) * 2;
-  const uint32_t v_lane = (uint32_t)(((lane & 7) + (((lane >> 3) & 1) << 3)) * VS + warp * (VP / 4) + (lane >> 4) * 8) * 2;
+  const int quarter = warp & 3, half_keys = (warp >> 2) * (TILE / 2);
+  const uint32_t v_lane = (uint32_t)((half_keys + (lane & 7) + (((lane >> 3) & 1) << 3)) * VS + quarter * (VP / 4) + (lane >> 4) * 8) * 2;
   const uint32_t q_addr = dec_smem(&sm.q[lane & 7][((lane >> 3) & 1) * 8]);
-  const uint32_t p_addr = dec_smem(&sm.p[lane & 15][(lane >> 4) * 8]);
+  const uint32_t p_addr = dec_smem(&sm.p[lane & 15][half_keys + (lane >> 4) * 8]);
   const int g = lane >> 2, t = lane & 3;
   float O[NT][4];
 #pragma unroll
@@ -162,9 +169,9 @@ __device__ void attention_decode(const DecodeArgs& a, uint8_t* smem, int b, int 
     __syncthreads();               // tile i has landed for every thread; tile i - 1 is no longer read
     load_tile(i + kDecStages - 1);
     find_rows(i + 4, 1);           // over tile i's, whose loads are done; read after the next barrier at the earliest
-    const int j0 = k0 + i * kDecTile, cnt = min(kDecTile, k1 - j0);
-    bf16* kt = ring + (size_t)(i % kDecStages) * att_stage(D, VP);
-    bf16* vt = kt + kDecTile * KS;
+    const int j0 = k0 + i * TILE, cnt = min(TILE, k1 - j0);
+    bf16* kt = ring + (size_t)(i % kDecStages) * att_stage(D, VP, TILE);
+    bf16* vt = kt + TILE * KS;
     if (pos >= j0 && pos < j0 + cnt) {   // the newest key and value: into the tile, and into the cache
       const size_t nrow = kv_row(a.bt, b, pos) * at.kv_heads + kvh;
       for (int d = tid; d < D; d += kDecThreads) {
@@ -178,39 +185,44 @@ __device__ void attention_decode(const DecodeArgs& a, uint8_t* smem, int b, int 
       }
       __syncthreads();
     }
-    // scores: keys as rows of the mma, query heads as its columns
-    float c[4] = {0.f, 0.f, 0.f, 0.f};
-    const uint32_t ka = dec_smem(kt) + k_lane;
+    // scores: keys as rows of the mma, query heads as its columns; 16 keys per warp
+    if (warp * 16 < TILE) {
+      float c[4] = {0.f, 0.f, 0.f, 0.f};
+      const uint32_t ka = dec_smem(kt) + k_lane;
 #pragma unroll 4
-    for (int d = 0; d < KS - 8; d += 16) {
-      uint32_t kf[4], qf[2];
-      dec_ldsm4(kf, ka + d * 2);
-      dec_ldsm2(qf, q_addr + d * 2);
-      dec_mma(c, kf, qf[0], qf[1]);
-    }
+      for (int d = 0; d < KS - 8; d += 16) {
+        uint32_t kf[4], qf[2];
+        dec_ldsm4(kf, ka + d * 2);
+        dec_ldsm2(qf, q_addr + d * 2);
+        dec_mma(c, kf, qf[0], qf[1]);
+      }
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int key = warp * 16 + g + 8 * (e >> 1), r = t * 2 + (e & 1);
-      float s = c[e] * at.scale;
-      if (at.softcap > 0.f) s = at.softcap * tanhf(s / at.softcap);
-      sm.s[r][key] = key < cnt ? s : -INFINITY;
+      for (int e = 0; e < 4; ++e) {
+        const int key = warp * 16 + g + 8 * (e >> 1), r = t * 2 + (e & 1);
+        float s = c[e] * at.scale;
+        if (at.softcap > 0.f) s = at.softcap * tanh_fast(s * inv_cap);
+        sm.s[r][key] = key < cnt ? s : -INFINITY;
+      }
     }
     __syncthreads();
-    // softmax of the tile: two heads per warp, two keys per lane
+    // softmax of the tile: a head per warp, TILE / 32 keys per lane
+    if (warp < R) {
+      float x[TILE / 32], mx = -INFINITY, sum = 0.f;
 #pragma unroll
-    for (int q = 0; q < 2; ++q) {
-      const int r = warp * 2 + q;
-      if (r >= R) break;
-      const float s0 = sm.s[r][lane], s1 = sm.s[r][lane + 32], m_old = sm.m[r], m_new = fmaxf(m_old, warp_max(fmaxf(s0, s1)));
-      const float e0 = expf(s0 - m_new), e1 = expf(s1 - m_new), sum = warp_sum(e0 + e1);
-      sm.p[r][lane] = __float2bfloat16_rn(e0);
-      sm.p[r][lane + 32] = __float2bfloat16_rn(e1);
-      __syncwarp();
+      for (int k = 0; k < TILE / 32; ++k) { x[k] = sm.s[warp][lane + 32 * k]; mx = fmaxf(mx, x[k]); }
+      const float m_old = sm.m[warp], m_new = fmaxf(m_old, warp_max(mx));
+#pragma unroll
+      for (int k = 0; k < TILE / 32; ++k) {
+        x[k] = exp_fast(x[k] - m_new);
+        sum += x[k];
+        sm.p[warp][lane + 32 * k] = __float2bfloat16_rn(x[k]);
+      }
+      sum = warp_sum(sum);
       if (lane == 0) {
-        const float corr = expf(m_old - m_new);
-        sm.corr[r] = corr;
-        sm.m[r] = m_new;
-        sm.l[r] = sm.l[r] * corr + sum;
+        const float corr = exp_fast(m_old - m_new);
+        sm.corr[warp] = corr;
+        sm.m[warp] = m_new;
+        sm.l[warp] = sm.l[warp] * corr + sum;
       }
     }
     __syncthreads();
@@ -219,7 +231,7 @@ __device__ void attention_decode(const DecodeArgs& a, uint8_t* smem, int b, int 
     for (int n = 0; n < NT; ++n) { O[n][0] *= corr; O[n][1] *= corr; }
     const uint32_t va = dec_smem(vt) + v_lane;
 #pragma unroll
-    for (int kk = 0; kk < kDecTile / 16; ++kk) {
+    for (int kk = 0; kk < TILE / 32; ++kk) {
       uint32_t pf[4];
       dec_ldsm4(pf, p_addr + kk * 32);
 #pragma unroll
@@ -232,8 +244,17 @@ __device__ void attention_decode(const DecodeArgs& a, uint8_t* smem, int b, int 
     }
   }
   asm volatile("cp.async.wait_group 0;");
+  // the two halves of the keys, one after the other
+  for (int half_no = 0; half_no < 2; ++half_no) {
+    if ((warp >> 2) == half_no) {
 #pragma unroll
-  for (int n = 0; n < NT; ++n) *reinterpret_cast<float2*>(&sm.out[g][warp * (VP / 4) + n * 8 + 2 * t]) = make_float2(O[n][0], O[n][1]);
+      for (int n = 0; n < NT; ++n) {
+        float2* o = reinterpret_cast<float2*>(&sm.out[g][quarter * (VP / 4) + n * 8 + 2 * t]);
+        *o = half_no ? make_float2(o->x + O[n][0], o->y + O[n][1]) : make_float2(O[n][0], O[n][1]);
+      }
+    }
+    __syncthreads();
+  }
   cl.sync();
   for (int e = rank * kDecThreads + tid; e < R * V; e += csize * kDecThreads) {
     const int r = e / V, c = e % V;
@@ -327,7 +348,12 @@ __device__ void retention_decode(const DecodeArgs& a, RetSmem& sm, int b, int h,
   ss = warp_sum(ss);
   if ((tid & 31) == 0) sm.wsum[tid >> 5] = ss;
   __syncthreads();
-  if (tid == 0) sm.ss = sm.wsum[0] + sm.wsum[1] + sm.wsum[2] + sm.wsum[3];
+  if (tid == 0) {
+    float s = 0.f;
+#pragma unroll
+    for (int w = 0; w < kDecThreads / 32; ++w) s += sm.wsum[w];
+    sm.ss = s;
+  }
   cl.sync();
   float tot = 0.f;
   for (int k = 0; k < csize; ++k) tot += cl.map_shared_rank(&sm, k)->ss;
@@ -340,23 +366,23 @@ __device__ void retention_decode(const DecodeArgs& a, RetSmem& sm, int b, int h,
   cl.sync();
 }
 
-template <int VP, int VEC>
-__global__ void __launch_bounds__(kDecThreads) mixer_decode_kernel(const DecodeArgs a) {
+template <int VP, int VEC, int TILE>
+__global__ void __launch_bounds__(kDecThreads, 1) mixer_decode_kernel(const DecodeArgs a) {
   extern __shared__ __align__(16) uint8_t smem[];
   grid_launch_dependents();
   grid_dependency_wait();
   cg::cluster_group cl = cg::this_cluster();
   const int unit = blockIdx.y, b = blockIdx.z;
-  if (unit < a.att_clusters) attention_decode<VP>(a, smem, b, unit, cl);
+  if (unit < a.att_clusters) attention_decode<VP, TILE>(a, smem, b, unit, cl);
   else retention_decode<VEC>(a, *reinterpret_cast<RetSmem*>(smem), b, unit - a.att_clusters, cl);
 }
 
-template <int VP, int VEC>
+template <int VP, int VEC, int TILE>
 static int launch_decode(const DecodeArgs& a, int csize, cudaStream_t st) {
   size_t smem = a.ret_heads > 0 ? sizeof(RetSmem) : 0;
-  const size_t att = a.att_clusters > 0 ? sizeof(AttSmem) + (size_t)kDecStages * att_stage(a.at.dim, VP) * sizeof(bf16) : 0;
+  const size_t att = a.att_clusters > 0 ? sizeof(AttSmem) + (size_t)kDecStages * att_stage(a.at.dim, VP, TILE) * sizeof(bf16) : 0;
   if (att > smem) smem = att;
-  if (cudaFuncSetAttribute(mixer_decode_kernel<VP, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+  if (cudaFuncSetAttribute(mixer_decode_kernel<VP, VEC, TILE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
     cudaGetLastError();
     return NQB200_ERR_LAUNCH;
   }
@@ -374,7 +400,7 @@ static int launch_decode(const DecodeArgs& a, int csize, cudaStream_t st) {
   attr[1].val.clusterDim.z = 1;
   cfg.attrs = attr;
   cfg.numAttrs = 2;
-  if (cudaLaunchKernelEx(&cfg, mixer_decode_kernel<VP, VEC>, a) != cudaSuccess) {
+  if (cudaLaunchKernelEx(&cfg, mixer_decode_kernel<VP, VEC, TILE>, a) != cudaSuccess) {
     cudaGetLastError();
     return NQB200_ERR_LAUNCH;
   }
@@ -422,7 +448,7 @@ extern "C" int nqb200_mixer_decode(const void* proj, int64_t stride, void* act, 
     units += p.att_clusters;
     int64_t keys = (int64_t)b->table_width * b->block_size;
     if (a->chunk > 0 && a->chunk < keys) keys = a->chunk;
-    while (want < 8 && keys > (int64_t)want * kDecTile) want *= 2;
+    while (want < 8 && keys > (int64_t)want * 64) want *= 2;
   }
   if (r) {
     p.ret_heads = r->heads; p.rdim = r->dim; p.rvdim = r->vdim;
@@ -432,13 +458,16 @@ extern "C" int nqb200_mixer_decode(const void* proj, int64_t stride, void* act, 
     units += r->heads;
     while (want < 8 && (int64_t)r->dim * r->vdim * 4 > (int64_t)want * 16384 && want * 8 <= r->vdim) want *= 2;
   }
-  // CTAs for one wave at two per SM, and no more than there is work for
-  while (csize < want && units * b->batch * csize * 2 <= 2 * kNumSMs) csize *= 2;
+  // about one CTA of attention per SM (its ring takes most of the shared memory), and no more than there is work for
+  while (csize < want && units * b->batch * csize * 2 <= (a ? kNumSMs * 3 / 2 : kNumSMs * 4)) csize *= 2;
   cudaStream_t st = (cudaStream_t)stream;
   const bool v4 = !r || r->vdim % 4 == 0;
-#define NQB200_DEC(VP) return v4 ? launch_decode<VP, 4>(p, csize, st) : launch_decode<VP, 1>(p, csize, st)
-  if (!a || a->vdim <= 64) NQB200_DEC(64);
-  if (a->vdim <= 128) NQB200_DEC(128);
-  NQB200_DEC(256);
+  // 128 keys a pass where two stages of them fit
+#define NQB200_DEC(VP, TILE) return v4 ? launch_decode<VP, 4, TILE>(p, csize, st) : launch_decode<VP, 1, TILE>(p, csize, st)
+  const bool big = a && a->dim + a->vdim > 256;
+  if (!a || (a->vdim <= 64 && !big)) NQB200_DEC(64, 128);
+  if (a->vdim <= 128 && !big) NQB200_DEC(128, 128);
+  if (a->vdim <= 128) NQB200_DEC(128, 64);
+  NQB200_DEC(256, 64);
 #undef NQB200_DEC
 }

@@ -281,7 +281,7 @@ __global__ void __launch_bounds__(256) clamped_glu_vec_kernel(const bf16* __rest
       for (int e = 0; e < 2; ++e) {
         const float g = fminf(__uint_as_float(e ? gw[k] & 0xFFFF0000u : gw[k] << 16), limit);
         const float u = fminf(fmaxf(__uint_as_float(e ? uw[k] & 0xFFFF0000u : uw[k] << 16), -limit), limit);
-        y[e] = g * __fdividef(1.f, 1.f + __expf(-1.702f * g)) * (u + 1.f);
+        y[e] = g * sigmoid_fast(1.702f * g) * (u + 1.f);
       }
       ow[k] = (uint32_t)__bfloat16_as_ushort(__float2bfloat16_rn(y[0])) | ((uint32_t)__bfloat16_as_ushort(__float2bfloat16_rn(y[1])) << 16);
     }

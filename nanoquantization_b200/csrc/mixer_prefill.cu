@@ -64,7 +64,7 @@ struct PrefillArgs {
   const float* sink;
   // retention: k, v, gate in the same buffer as q
   const bf16* k; const bf16* v; const bf16* gate;
-  const float* decay; const float* states;   // states [chunk id][heads][dim][vdim]
+  const float* decay; const bf16* states;    // states [chunk id][heads][high part, rest][dim][vdim]
   float eps;
 };
 
@@ -144,16 +144,18 @@ __global__ void __launch_bounds__(kThreads, 1) prefill_kernel(const PrefillArgs 
     cp_wait<0>();
     __syncthreads();
     // the part from before this chunk: q S, then rows times decay^(i + 1)
-    const float* S = a.states + (chunk_id(a.bt, b, kstart / kRetChunk) * a.heads + h) * (size_t)a.dim * a.vdim;
+    const bf16* S = a.states + (chunk_id(a.bt, b, kstart / kRetChunk) * a.heads + h) * (size_t)(2 * a.dim * a.vdim);
     for (int d0 = 0; d0 < DP; d0 += kKeys) {
       __syncthreads();
-      for (int e = tid; e < kKeys * (a.vdim / 2); e += kThreads) {
-        const int r = e / (a.vdim / 2), c = e % (a.vdim / 2) * 2;
-        const float2 f = d0 + r < a.dim ? *reinterpret_cast<const float2*>(S + (size_t)(d0 + r) * a.vdim + c) : make_float2(0.f, 0.f);
-        const float hx = __bfloat162float(__float2bfloat16_rn(f.x)), hy = __bfloat162float(__float2bfloat16_rn(f.y));
-        *reinterpret_cast<uint32_t*>(vs + r * VS + c) = pack2(hx, hy);
-        *reinterpret_cast<uint32_t*>(vs + (kKeys + r) * VS + c) = pack2(f.x - hx, f.y - hy);
+      const int r = tid >> 2;             // four threads per row, both parts
+      const bool ok = d0 + r < a.dim;
+      const bf16* src = S + (size_t)(ok ? d0 + r : 0) * a.vdim;
+      for (int c = tid & 3; c < V8; c += 4) {
+        cp16(smem_addr(vs + r * VS + c * 8), src + c * 8, ok);
+        cp16(smem_addr(vs + (kKeys + r) * VS + c * 8), src + (size_t)a.dim * a.vdim + c * 8, ok);
       }
+      cp_commit();
+      cp_wait<0>();
       __syncthreads();
 #pragma unroll
       for (int kt = 0; kt < kKeys / 16; ++kt) {
@@ -292,9 +294,10 @@ __global__ void __launch_bounds__(kThreads, 1) prefill_kernel(const PrefillArgs 
       if (c >= a.vdim) break;
       float x = O[i][2 * r] * f, y = O[i][2 * r + 1] * f;
       if (RET) {
-        const float gx = to_f(gp[c]), gy = to_f(gp[c + 1]);
-        x *= gx * sigmoid_f(gx);
-        y *= gy * sigmoid_f(gy);
+        const uint32_t gw = *reinterpret_cast<const uint32_t*>(gp + c);
+        const float gx = __uint_as_float(gw << 16), gy = __uint_as_float(gw & 0xFFFF0000u);
+        x *= gx * sigmoid_fast(gx);
+        y *= gy * sigmoid_fast(gy);
       }
       *reinterpret_cast<uint32_t*>(dst + c) = pack2(x, y);
     }
@@ -384,9 +387,9 @@ __global__ void __launch_bounds__(128) retention_chunk_kernel(const ChunkStateAr
     }
 }
 
-// states[c] <- the state ahead of chunk c; the sequence's own state moves to the end of the step.
-__global__ void __launch_bounds__(256) retention_scan_kernel(float* states, float* state, const float* __restrict__ decay, int heads,
-                                                             int per_head, const nqb200_batch bt) {
+// starts[c] <- the state ahead of chunk c, split into two bf16 numbers; the sequence's own state moves to the end of the step.
+__global__ void __launch_bounds__(256) retention_scan_kernel(const float* __restrict__ states, bf16* __restrict__ starts, float* state,
+                                                             const float* __restrict__ decay, int heads, int per_head, const nqb200_batch bt) {
   grid_launch_dependents();
   grid_dependency_wait();
   const int b = blockIdx.z, h = blockIdx.y, e = (blockIdx.x * 256 + threadIdx.x) * 4, n = bt.cu[b + 1] - bt.cu[b];
@@ -395,13 +398,17 @@ __global__ void __launch_bounds__(256) retention_scan_kernel(float* states, floa
   float* own = state + ((size_t)bt.slot[b] * heads + h) * per_head + e;
   float4 S = bt.pos0[b] == 0 ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(own);
   const int chunks = (n + kRetChunk - 1) / kRetChunk;
-  float* p = states + (chunk_id(bt, b, 0) * heads + h) * (size_t)per_head + e;
+  const float* p = states + (chunk_id(bt, b, 0) * heads + h) * (size_t)per_head + e;
+  bf16* o = starts + (chunk_id(bt, b, 0) * heads + h) * (size_t)(2 * per_head) + e;
   const size_t step = (size_t)heads * per_head;
   float4 next = *reinterpret_cast<const float4*>(p);
-  for (int c = 0; c < chunks; ++c, p += step) {
+  for (int c = 0; c < chunks; ++c, p += step, o += 2 * step) {
     const float4 dl = next;
     if (c + 1 < chunks) next = *reinterpret_cast<const float4*>(p + step);
-    *reinterpret_cast<float4*>(p) = S;
+    const float hx = __bfloat162float(__float2bfloat16_rn(S.x)), hy = __bfloat162float(__float2bfloat16_rn(S.y));
+    const float hz = __bfloat162float(__float2bfloat16_rn(S.z)), hw = __bfloat162float(__float2bfloat16_rn(S.w));
+    *reinterpret_cast<uint2*>(o) = make_uint2(pack2(hx, hy), pack2(hz, hw));
+    *reinterpret_cast<uint2*>(o + per_head) = make_uint2(pack2(S.x - hx, S.y - hy), pack2(S.z - hz, S.w - hw));
     const float f = decay_pow(log2d, min(kRetChunk, n - c * kRetChunk));
     S.x = f * S.x + dl.x; S.y = f * S.y + dl.y; S.z = f * S.z + dl.z; S.w = f * S.w + dl.w;
   }
@@ -486,13 +493,14 @@ extern "C" int nqb200_retention_prefill(const void* proj, int64_t stride, int64_
   int rc = launch_overlapped(retention_chunk_kernel, dim3(chunks, (unsigned)(r->heads * ((r->dim + 63) / 64) * c.vtiles), (unsigned)b->batch), dim3(128), 0, st, c);
   if (rc != NQB200_OK) return rc;
   const int per_head = r->dim * r->vdim;
+  bf16* starts = reinterpret_cast<bf16*>(chunk_states + nqb200_retention_chunks(b->tokens, b->batch) * r->heads * per_head);
   rc = launch_overlapped(retention_scan_kernel, dim3((unsigned)((per_head / 4 + 255) / 256), (unsigned)r->heads, (unsigned)b->batch), dim3(256), 0, st,
-                         chunk_states, state, r->decay, r->heads, per_head, *b);
+                         (const float*)chunk_states, starts, state, r->decay, r->heads, per_head, *b);
   if (rc != NQB200_OK) return rc;
   PrefillArgs p = {};
   p.q = q; p.q_stride = stride; p.out = (bf16*)act + act_col; p.out_stride = act_stride; p.bt = *b;
   p.heads = r->heads; p.dim = r->dim; p.vdim = r->vdim; p.out_scale = r->out_scale; p.kv_heads = r->heads;
   p.k = q + qk; p.v = q + 2 * qk; p.gate = q + 2 * qk + vv;
-  p.decay = r->decay; p.states = chunk_states; p.eps = r->eps; p.scale = 1.f / sqrtf((float)r->dim);
+  p.decay = r->decay; p.states = starts; p.eps = r->eps; p.scale = 1.f / sqrtf((float)r->dim);
   return dispatch_prefill<true>(p, st);
 }

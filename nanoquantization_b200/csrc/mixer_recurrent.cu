@@ -168,16 +168,15 @@ __global__ void __launch_bounds__(kGruSegs* kGruCols) mingru_kernel(const T* __r
 }
 
 // Two channels per thread (even widths): a CTA takes 64 channels x 128 tokens, a warp 16 of the tokens, so that the
-// chunks of a prompt run side by side.  A first launch folds each chunk into S -> A S + B; the second combines the
-// chunks ahead of its own, scans its 8 warps' folds and replays the tokens.  The sequence's state at the step's start is
-// copied aside by the first launch, because the last chunk's CTA overwrites it while others still need it.
+// chunks of a prompt run side by side.  A first launch folds each chunk into S -> A S + B, a second walks over the folds
+// and leaves every chunk's starting state in its fold's place, and the third scans its 8 warps' folds and replays the
+// tokens.
 constexpr int kGruChunk = 128, kGruWarpTokens = 16;
 
 __device__ __forceinline__ float2 ld_pair(const float* p) { return *reinterpret_cast<const float2*>(p); }
 __device__ __forceinline__ float2 ld_pair(const bf16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); }
 __device__ __forceinline__ void st_pair(float* p, float2 v) { *reinterpret_cast<float2*>(p) = v; }
 __device__ __forceinline__ void st_pair(bf16* p, float2 v) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(v.x, v.y); }
-__device__ __forceinline__ float sigmoid_fast(float v) { return __fdividef(1.f, 1.f + __expf(-v)); }
 template <typename T> __device__ __forceinline__ float gate_sigmoid(float v) { return sigmoid_f(v); }
 template <> __device__ __forceinline__ float gate_sigmoid<bf16>(float v) { return sigmoid_fast(v); }
 
@@ -185,7 +184,7 @@ struct GruArgs {
   int64_t stride;
   int z_off, x_off, g_off, width;
   const float* z_bias; const float* x_bias;
-  float* state; float2* folds; float* start;   // folds [chunk id][width], start [batch][width]
+  float* state; float2* folds;   // folds [chunk id][width / 2]: A of both channels, then B of both
   nqb200_batch bt;
 };
 __device__ __forceinline__ size_t gru_chunk_id(const nqb200_batch& bt, int b, int c) { return (size_t)(bt.cu[b] / kGruChunk + b + c); }
@@ -224,21 +223,11 @@ __global__ void __launch_bounds__(256) mingru_chunk_kernel(const T* __restrict__
   Bs[warp][lane] = B;
   float2 S = make_float2(0.f, 0.f);   // FOLD: the fold's own B; else the state at the chunk's start
   if (!FOLD && live) {
-    if (n <= kGruChunk) {
-      if (!fresh) S = ld_pair(own);
-    } else {   // several CTAs need the state and the last one's replaces it: from the copy
-      S = ld_pair(p.start + (size_t)b * p.width + c);
-      const float2* f = p.folds + 2 * (gru_chunk_id(p.bt, b, 0) * (p.width / 2) + c / 2);
-#pragma unroll 8
-      for (int k = 0; k < chunk; ++k) {
-        const float4 ab = *reinterpret_cast<const float4*>(f + (size_t)k * p.width);   // A of both channels, B of both
-        S.x = ab.x * S.x + ab.z;
-        S.y = ab.y * S.y + ab.w;
-      }
-    }
+    if (n > kGruChunk) S = p.folds[2 * (gru_chunk_id(p.bt, b, chunk) * (p.width / 2) + c / 2)];   // where the scan left it
+    else if (!fresh) S = ld_pair(own);
   }
   __syncthreads();
-  if (FOLD) {
+  if constexpr (FOLD) {
     if (warp == 0 && live) {
       float2 FA = make_float2(1.f, 1.f), FB = make_float2(0.f, 0.f);
 #pragma unroll
@@ -248,11 +237,9 @@ __global__ void __launch_bounds__(256) mingru_chunk_kernel(const T* __restrict__
         FB.x = wa.x * FB.x + wb.x; FB.y = wa.y * FB.y + wb.y;
       }
       *reinterpret_cast<float4*>(p.folds + 2 * (gru_chunk_id(p.bt, b, chunk) * (p.width / 2) + c / 2)) = make_float4(FA.x, FA.y, FB.x, FB.y);
-      if (chunk == 0) st_pair(p.start + (size_t)b * p.width + c, fresh ? make_float2(0.f, 0.f) : ld_pair(own));
     }
-    return;
-  }
-  for (int w = 0; w < (FOLD ? 0 : warp); ++w) {
+  } else {
+  for (int w = 0; w < warp; ++w) {
     const float2 wa = As[w][lane], wb = Bs[w][lane];
     S.x = wa.x * S.x + wb.x; S.y = wa.y * S.y + wb.y;
   }
@@ -271,6 +258,29 @@ __global__ void __launch_bounds__(256) mingru_chunk_kernel(const T* __restrict__
   // every warp has read the state (of a sequence with one chunk) before the last one replaces it
   __syncthreads();
   if (live && warp == 7 && first + kGruChunk >= n) st_pair(own, S);
+  }
+}
+
+__global__ void __launch_bounds__(64) mingru_scan_kernel(const GruArgs p) {
+  grid_launch_dependents();
+  grid_dependency_wait();
+  const int b = blockIdx.y, pair = blockIdx.x * 64 + threadIdx.x, n = p.bt.cu[b + 1] - p.bt.cu[b];
+  if (pair * 2 >= p.width || n <= kGruChunk) return;
+  const int chunks = (n + kGruChunk - 1) / kGruChunk;
+  float2 S = p.bt.pos0[b] == 0 ? make_float2(0.f, 0.f) : ld_pair(p.state + (size_t)p.bt.slot[b] * p.width + pair * 2);
+  float2* f = p.folds + 2 * (gru_chunk_id(p.bt, b, 0) * (p.width / 2) + pair);
+  for (int c0 = 0; c0 < chunks; c0 += 16) {
+    float4 ab[16];
+#pragma unroll
+    for (int k = 0; k < 16; ++k) ab[k] = *reinterpret_cast<const float4*>(f + (size_t)min(c0 + k, chunks - 1) * p.width);
+#pragma unroll
+    for (int k = 0; k < 16; ++k) {
+      if (c0 + k >= chunks) break;
+      f[(size_t)(c0 + k) * p.width] = S;
+      S.x = ab[k].x * S.x + ab[k].z;
+      S.y = ab[k].y * S.y + ab[k].w;
+    }
+  }
 }
 
 }  // namespace nqb200
@@ -281,7 +291,8 @@ template <typename T>
 static int mingru_chunked(const void* proj, void* out, const GruArgs& p, cudaStream_t st) {
   const dim3 grid((unsigned)((p.width + 63) / 64), (unsigned)((p.bt.max_len + kGruChunk - 1) / kGruChunk), (unsigned)p.bt.batch), block(256);
   if (grid.y > 1) {
-    const int rc = launch_overlapped(mingru_chunk_kernel<T, true>, grid, block, 0, st, (const T*)proj, (T*)nullptr, p);
+    int rc = launch_overlapped(mingru_chunk_kernel<T, true>, grid, block, 0, st, (const T*)proj, (T*)nullptr, p);
+    if (rc == NQB200_OK) rc = launch_overlapped(mingru_scan_kernel, dim3((unsigned)((p.width / 2 + 63) / 64), (unsigned)p.bt.batch), dim3(64), 0, st, p);
     if (rc != NQB200_OK) return rc;
   }
   return launch_overlapped(mingru_chunk_kernel<T, false>, grid, block, 0, st, (const T*)proj, (T*)out, p);
@@ -342,7 +353,7 @@ extern "C" int nqb200_head_norm_gate(const float* o, const void* gate, int64_t g
 }
 
 extern "C" int64_t nqb200_mingru_scratch(int64_t tokens, int64_t batch, int64_t width) {
-  return (tokens / kGruChunk + batch) * width * 2 + batch * width;
+  return (tokens / kGruChunk + batch) * width * 2;
 }
 
 extern "C" int nqb200_mingru(const void* proj, int64_t stride, int64_t z_off, int64_t x_off, int64_t g_off, const float* z_bias,
@@ -363,7 +374,6 @@ extern "C" int nqb200_mingru(const void* proj, int64_t stride, int64_t z_off, in
     p.stride = stride; p.z_off = (int)z_off; p.x_off = (int)x_off; p.g_off = (int)g_off; p.width = (int)width;
     p.z_bias = z_bias; p.x_bias = x_bias; p.state = state; p.bt = *b;
     p.folds = reinterpret_cast<float2*>(scratch);
-    p.start = scratch ? scratch + (b->tokens / kGruChunk + b->batch) * width * 2 : nullptr;
     return dtype == NQB200_F32 ? mingru_chunked<float>(proj, out, p, st) : mingru_chunked<bf16>(proj, out, p, st);
   }
   const dim3 grid((unsigned)((width + kGruCols - 1) / kGruCols), (unsigned)b->batch), block(kGruSegs * kGruCols);

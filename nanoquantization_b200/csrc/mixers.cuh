@@ -15,6 +15,14 @@ template <> __device__ __forceinline__ bf16 from_f<bf16>(float v) { return __flo
 
 __device__ __forceinline__ float sigmoid_f(float v) { return 1.f / (1.f + expf(-v)); }
 
+// For bf16 results: a few float ulps, out of the hardware's exponential and reciprocal.
+__device__ __forceinline__ float ex2_fast(float x) { float r; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x)); return r; }
+__device__ __forceinline__ float rcp_fast(float x) { float r; asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x)); return r; }
+__device__ __forceinline__ float sigmoid_fast(float v) { return rcp_fast(1.f + ex2_fast(v * -1.4426950408889634f)); }
+__device__ __forceinline__ float exp_fast(float v) { return ex2_fast(v * 1.4426950408889634f); }
+// tanh as 1 - 2 / (1 + e^2y): absolute error of a few 1e-7, right at both ends
+__device__ __forceinline__ float tanh_fast(float y) { return 1.f - 2.f * rcp_fast(1.f + ex2_fast(y * 2.8853900817779268f)); }
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xFFFFFFFFu, v, o);

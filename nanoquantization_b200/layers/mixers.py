@@ -92,7 +92,7 @@ def retention_gated(proj: torch.Tensor, off: int, desc: _lib.RetentionDesc, deca
     if (proj.dtype == torch.bfloat16 and step.max_len >= RETENTION_PREFILL_TOKENS
             and lib.nqb200_retention_prefill_supported(ctypes.byref(desc), proj.stride(0), off, act.stride(0), act_col)):
         chunks = lib.nqb200_retention_chunks(step.num_tokens, step.batch)
-        scratch = torch.empty(chunks, heads, dim, vdim, dtype=torch.float32, device=proj.device)
+        scratch = torch.empty(2, chunks, heads, dim, vdim, dtype=torch.float32, device=proj.device)
         _call("nqb200_retention_prefill", proj.data_ptr(), proj.stride(0), off, act.data_ptr(), act.stride(0), act_col, ctypes.byref(desc),
               state.data_ptr(), scratch.data_ptr(), ctypes.byref(step.desc))
         return
