@@ -94,6 +94,8 @@ __device__ __forceinline__ uint64_t add2(uint64_t a, uint64_t b) { uint64_t r; a
 __device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
   uint64_t r; asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c)); return r;
 }
+__device__ __forceinline__ float max3(float a, float b, float c) { float r; asm("max.f32 %0, %1, %2, %3;" : "=f"(r) : "f"(a), "f"(b), "f"(c)); return r; }
+__device__ __forceinline__ float min3(float a, float b, float c) { float r; asm("min.f32 %0, %1, %2, %3;" : "=f"(r) : "f"(a), "f"(b), "f"(c)); return r; }
 __device__ __forceinline__ float ex2(float x) { float r; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x)); return r; }
 __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
   const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
@@ -107,7 +109,7 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
   constexpr uint32_t kQBytes = kTile * D * 2, kKBytes = kTile * D * 2, kVBytes = kTile * V * 2, kBox = kTile * 128;
   constexpr uint32_t kOffK = 2 * kQBytes, kOffV = kOffK + 2 * kKBytes;
   extern __shared__ uint8_t smem_raw[];
-  __shared__ __align__(8) uint64_t bar_q, bar_kfull[2], bar_kfree[2], bar_vfull[2], bar_vfree[2], bar_s[2], bar_p[2], bar_pv[2], bar_o[2], bar_drain;
+  __shared__ __align__(8) uint64_t bar_q, bar_kfull[2], bar_kfree[2], bar_vfull[2], bar_vfree[2], bar_s[2], bar_p[2][2], bar_pv[2], bar_o[2], bar_drain;
   __shared__ uint32_t s_tmem;
   __shared__ int s_abort_i;
   volatile int* s_abort = &s_abort_i;
@@ -132,7 +134,7 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
     for (int s = 0; s < 2; ++s) {
       mbar_init(smem_u32(&bar_kfull[s]), 1); mbar_init(smem_u32(&bar_kfree[s]), 1);
       mbar_init(smem_u32(&bar_vfull[s]), 1); mbar_init(smem_u32(&bar_vfree[s]), 1);
-      mbar_init(smem_u32(&bar_s[s]), 1); mbar_init(smem_u32(&bar_p[s]), 4);
+      mbar_init(smem_u32(&bar_s[s]), 1); mbar_init(smem_u32(&bar_p[s][0]), 4); mbar_init(smem_u32(&bar_p[s][1]), 4);
       mbar_init(smem_u32(&bar_pv[s]), 1); mbar_init(smem_u32(&bar_o[s]), 1);
     }
     mbar_init(smem_u32(&bar_drain), 1);
@@ -176,9 +178,9 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
     }
   } else if (warp == 1) {
     // ------------------------------------------------------------------ MMA
-    // One thread runs both tiles as two little state machines and never blocks on one of them: it polls for a tile's
-    // weights (then issues O += P V) and for that product's end (P has been read: then S of the next key tile may
-    // overwrite it).  A ring stage is handed back by whichever tile uses it second.
+    // One thread runs both tiles as two little state machines and never blocks on one of them: it polls for the first
+    // and the second half of a tile's weights (then issues that half of O += P V) and for that product's end (P has been
+    // read: then S of the next key tile may overwrite it).  A ring stage is handed back by whichever tile uses it second.
     if (lane == 0) {
       const uint32_t idesc_s = umma_idesc(1, 128, kTile);
       const uint32_t idesc_o = umma_idesc(1, 128, V) | (1u << 16);   // B's rows run along k
@@ -193,9 +195,10 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
       };
       bool ok = wait_bar(&bar_q, 0, s_abort, p.status) && wait_bar(&bar_kfull[0], 0, s_abort, p.status);
       const int users = nq[1] > 0 ? 2 : 1;
-      // tile of the next product, whether it is under way, users that have still to issue on K / V tile j (by j & 1)
+      // tile of the next product; 0, 1: waits for that half of the weights, 2: for the product; users that have still to
+      // issue on K / V tile j (by j & 1)
       int jq[2] = {0, 0};
-      bool busy[2] = {false, false};
+      int phase[2] = {0, 0};
       auto users_of = [&](int j) { return users == 2 ? (j < nq[0]) + (j < nq[1]) : 1; };
       int kleft[2] = {0, users_of(1)}, vleft[2] = {users_of(0), users_of(1)};
       if (ok) {
@@ -212,23 +215,27 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
         for (int q = 0; q < 2; ++q) {
           const int j = jq[q], s = j & 1, sn = s ^ 1;
           if (j >= nq[q]) continue;
-          if (!busy[q]) {
-            if (!mbar_test_wait(smem_u32(&bar_p[q]), s) || !mbar_test_wait(smem_u32(&bar_vfull[s]), (j >> 1) & 1)) continue;
+          if (phase[q] < 2) {
+            const int half = phase[q];
+            if (!mbar_test_wait(smem_u32(&bar_p[q][half]), s) || !mbar_test_wait(smem_u32(&bar_vfull[s]), (j >> 1) & 1)) continue;
             tc_fence_after();
-            const uint32_t d = tmem + kColO + q * 128, pa = tmem + kColS + q * 128, bv = v_lo + s * (kVBytes >> 4);
+            const uint32_t d = tmem + kColO + q * 128, pa = tmem + kColS + q * 128 + half * 32, bv = v_lo + s * (kVBytes >> 4) + half * (8192 >> 4);
 #pragma unroll
-            for (int ks = 0; ks < kTile / 16; ++ks) umma_ts_lohi(d, pa + ks * 8, bv + ks * (2048 >> 4), v_hi, idesc_o, (j > 0 || ks > 0) ? 1u : 0u);
-            umma_commit(smem_u32(&bar_pv[q]));
-            if (--vleft[s] == 0) { umma_commit(smem_u32(&bar_vfree[s])); vleft[s] = users_of(j + 2); }
-            if (j == nq[q] - 1) { umma_commit(smem_u32(&bar_o[q])); jq[q] = j + 1; }
-            else busy[q] = true;
+            for (int ks = 0; ks < kTile / 32; ++ks)
+              umma_ts_lohi(d, pa + ks * 8, bv + ks * (2048 >> 4), v_hi, idesc_o, (j > 0 || half > 0 || ks > 0) ? 1u : 0u);
+            phase[q] = half + 1;
+            if (half == 1) {
+              umma_commit(smem_u32(&bar_pv[q]));
+              if (--vleft[s] == 0) { umma_commit(smem_u32(&bar_vfree[s])); vleft[s] = users_of(j + 2); }
+              if (j == nq[q] - 1) { umma_commit(smem_u32(&bar_o[q])); jq[q] = j + 1; }
+            }
           } else {
             if (!mbar_test_wait(smem_u32(&bar_pv[q]), s) || !mbar_test_wait(smem_u32(&bar_kfull[sn]), ((j + 1) >> 1) & 1)) continue;
             tc_fence_after();
             scores(q, sn);
             if (--kleft[sn] == 0) { umma_commit(smem_u32(&bar_kfree[sn])); kleft[sn] = users_of(j + 3); }
             jq[q] = j + 1;
-            busy[q] = false;
+            phase[q] = 0;
           }
           moved = true;
         }
@@ -263,6 +270,12 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
     };
     const uint64_t ysc2 = pair2(ysc, ysc), k1 = pair2(top, top), k3 = pair2(-top / 3.f, -top / 3.f), k5 = pair2(top * (2.f / 15.f), top * (2.f / 15.f)),
                    k7 = pair2(-top * (17.f / 315.f), -top * (17.f / 315.f)), k9 = pair2(top * (62.f / 2835.f), top * (62.f / 2835.f));
+    auto half_done = [&](int half) {   // that half of the weights is in tensor memory
+      tc_wait_st();
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(smem_u32(&bar_p[q][half]));
+    };
     const float sink = p.sink ? p.sink[h] * kLog2e : -INFINITY;
     float m = sink, l = 0.f;
     uint64_t lsum = pair2(0.f, 0.f);
@@ -279,16 +292,17 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
       tc_wait_ld();
       float mx = -INFINITY, ab = 0.f;
       if (!masked) {
-        float mv[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY}, av[4] = {0.f, 0.f, 0.f, 0.f};
+        float hi[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY}, lw[4] = {INFINITY, INFINITY, INFINITY, INFINITY};
 #pragma unroll
         for (int c = 0; c < 4; ++c)
 #pragma unroll
-          for (int e = 0; e < 32; ++e) {
-            mv[e & 3] = fmaxf(mv[e & 3], __uint_as_float(r[c][e]));
-            av[e & 3] = fmaxf(av[e & 3], fabsf(__uint_as_float(r[c][e])));
+          for (int e = 0; e < 32; e += 2) {
+            const int k = (e >> 1) & 3;
+            hi[k] = max3(hi[k], __uint_as_float(r[c][e]), __uint_as_float(r[c][e + 1]));
+            lw[k] = min3(lw[k], __uint_as_float(r[c][e]), __uint_as_float(r[c][e + 1]));
           }
-        mx = fmaxf(fmaxf(mv[0], mv[1]), fmaxf(mv[2], mv[3]));
-        ab = fmaxf(fmaxf(av[0], av[1]), fmaxf(av[2], av[3]));
+        mx = fmaxf(fmaxf(hi[0], hi[1]), fmaxf(hi[2], hi[3]));
+        ab = fmaxf(mx, -fminf(fminf(lw[0], lw[1]), fminf(lw[2], lw[3])));
       } else {
 #pragma unroll
         for (int c = 0; c < 4; ++c)
@@ -326,6 +340,7 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
       const float mu = m == -INFINITY ? 0.f : m;
       if (!masked && (!capped || __all_sync(0xFFFFFFFFu, ab * ysc <= kSeriesRange))) {
         const uint64_t nm2 = pair2(-mu, -mu);
+        uint64_t ls[4] = {lsum, 0, 0, 0};
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
           uint32_t w[16];
@@ -343,11 +358,13 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
             unpair2(arg, x0, x1);
             x0 = ex2(x0);
             x1 = ex2(x1);
-            lsum = add2(lsum, pair2(x0, x1));
+            ls[e & 3] = add2(ls[e & 3], pair2(x0, x1));
             w[e] = pack_bf16(x0, x1);
           }
           tmem_st16(tS + c * 16, w);
+          if (c == 1) half_done(0);
         }
+        lsum = add2(add2(ls[0], ls[1]), add2(ls[2], ls[3]));
       } else {
         // from tensor memory again, a piece at a time: compact code for the few tiles at the edges
 #pragma unroll 1
@@ -367,12 +384,10 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
             w[e] = pack_bf16(x[0], x[1]);
           }
           tmem_st8(tS + c * 8, w);      // lies behind what has been read of S
+          if (c == 3) half_done(0);
         }
       }
-      tc_wait_st();
-      tc_fence_before();
-      __syncwarp();
-      if (lane == 0) mbar_arrive(smem_u32(&bar_p[q]));
+      half_done(1);
     }
     if (ok && nq[q] > 0) {
       ok = wait_bar(&bar_o[q], 0, s_abort, p.status);

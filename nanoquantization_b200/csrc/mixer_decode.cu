@@ -433,6 +433,12 @@ extern "C" int nqb200_mixer_decode(const void* proj, int64_t stride, void* act, 
   if (a && (rot < 0 || rot % 2 != 0 || rot > a->dim)) return NQB200_ERR_BAD_SHAPE;
   if (a && (!aligned16(k_cache) || !aligned16(v_cache))) return NQB200_ERR_MISALIGNED;
   if (r && !aligned16(state)) return NQB200_ERR_MISALIGNED;
+  if (a && r && (int64_t)(a->kv_heads + r->heads) * b->batch > kNumSMs) {
+    // more than one wave: each with the shared memory and the cluster size that suit it
+    const int rc = nqb200_mixer_decode(proj, stride, act, act_stride, a, inv_freq, rot, a_off, a_col, k_cache, v_cache, nullptr, 0, 0, nullptr, b, stream);
+    return rc != NQB200_OK ? rc
+                           : nqb200_mixer_decode(proj, stride, act, act_stride, nullptr, nullptr, 0, 0, 0, nullptr, nullptr, r, r_off, r_col, state, b, stream);
+  }
   DecodeArgs p = {};
   p.proj = (const bf16*)proj; p.stride = stride; p.act = (bf16*)act; p.act_stride = act_stride; p.bt = *b;
   int csize = 1, want = 1;
