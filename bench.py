@@ -841,14 +841,16 @@ def vemedra_kernels(dev, peaks, T=8192, context=2048):
     add("prefill", "rotary + K/V store", _device_us(lambda i: ops.rope_store(proj[i % 2], kc, vc, att.inv_freq, one, 0, H * D, (H + G) * D, H), 8),
         T * (2 * H * D + 4 * G * D) * 2)
     qkv, qn, cs = [rnd(T, (H + 2 * G) * D) for _ in range(3)], rnd(D), rnd(T, 1, D, dtype=torch.float32)
+    kq, vq = torch.zeros_like(kc), torch.zeros_like(vc)
     add("prefill", "Qwen3: QK-norm + rotary + K/V store",
-        _device_us(lambda i: fused.qknorm_rope_(qkv[i % 3], qn, qn, cs, one.positions, H, G, D, 1e-6, (kc, vc, one.rows)), 9), T * (2 * H * D + 4 * G * D) * 2)
+        _device_us(lambda i: fused.qknorm_rope_(qkv[i % 3], qn, qn, cs, one.positions, H, G, D, 1e-6, (kq, vq, one.rows)), 9), T * (2 * H * D + 4 * G * D) * 2)
     act = rnd(T, H * D + RH * RV)
-    for name, c in ((f"attention, chunks of {chunk}", chunk), ("attention, one chunk of all", T)):
-        att.chunk = c
+    for name, c, cap in ((f"attention, chunks of {chunk}", chunk, 50.0), ("attention, one chunk of all", T, 50.0), ("attention, the same with scores beyond the cap", T, 3.0)):
+        att.chunk, att.softcap = c, cap
         d = att.desc()
         us = _device_us(lambda i: ops.chunk_attention(proj[i % 2][:, :H * D], kc, vc, act[:, :H * D], d, one), 4)
         add("prefill", name, us, flops=T // c * (c * c / 2) * 4 * D * H)
+    att.softcap = 50.0
     q, k, v = (qkv[0][:, o:o + n * D].reshape(1, T, n, D).transpose(1, 2).contiguous() for o, n in ((0, H), (H * D, G), ((H + G) * D, G)))
     us = _device_us(lambda i: F.scaled_dot_product_attention(q, k, v, is_causal=True, enable_gqa=True), 4)
     add("prefill", "Qwen3: scaled_dot_product_attention, all", us, flops=T * T / 2 * 4 * D * H)

@@ -10,8 +10,9 @@
 // tiles take turns on the tensor pipe while the other one's softmax runs.  The running maximum is only moved (and O
 // rescaled) when it falls behind by more than 8 in log2 units: the weights stay below 2^8 and the sums exact enough,
 // and after a row's first tiles it hardly ever happens.  The cap is monotonic, so the maximum is taken over raw scores.
-// For scores well inside the cap tanh is its Taylor series, which costs fused multiply-adds on register pairs only; a
-// warp whose tile has a larger score, or needs a mask, takes the general path.
+// For scores well inside the cap tanh is its Taylor series, which costs fused multiply-adds on register pairs only; up to
+// twice the cap it is the seventh convergent of Lambert's continued fraction (one reciprocal more per score); a warp
+// whose tile has a larger score, or needs a mask, takes the general path.
 //
 // Every wait is bounded; on expiry NQB200_ERR_WAIT_TIMEOUT goes to the status word, all roles drain and tensor memory is
 // released.
@@ -24,7 +25,7 @@ namespace att {
 
 constexpr int kTile = 128, kThreads = 384;
 constexpr uint32_t kColS = 0, kColO = 256, kTmemCols = 512;
-constexpr float kLog2e = 1.4426950408889634f, kLag = 8.f, kSeriesRange = 0.4f;
+constexpr float kLog2e = 1.4426950408889634f, kLag = 8.f, kSeriesRange = 0.4f, kFractionRange = 2.f;
 
 struct Params {
   nqb200_batch bt;
@@ -338,7 +339,32 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
         }
       }
       const float mu = m == -INFINITY ? 0.f : m;
-      if (!masked && (!capped || __all_sync(0xFFFFFFFFu, ab * ysc <= kSeriesRange))) {
+      const int range = masked ? 2 : !capped || __all_sync(0xFFFFFFFFu, ab * ysc <= kSeriesRange) ? 0 : __all_sync(0xFFFFFFFFu, ab * ysc <= kFractionRange) ? 1 : 2;
+      if (range == 1) {
+        // tanh y = y (10395 + 1260 y^2 + 21 y^4) / (10395 + 4725 y^2 + 210 y^4 + y^6)
+        const uint64_t n0 = pair2(10395.f, 10395.f), n1 = pair2(1260.f, 1260.f), n2 = pair2(21.f, 21.f), d1 = pair2(4725.f, 4725.f), d2 = pair2(210.f, 210.f),
+                       nm2 = pair2(-mu, -mu);
+        uint64_t ls[2] = {lsum, 0};
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          uint32_t w[16];
+#pragma unroll
+          for (int e = 0; e < 16; ++e) {
+            const uint64_t y = mul2(pair2(__uint_as_float(r[c][2 * e]), __uint_as_float(r[c][2 * e + 1])), ysc2), y2 = mul2(y, y);
+            const uint64_t num = mul2(mul2(y, k1), fma2(fma2(n2, y2, n1), y2, n0)), den = fma2(fma2(add2(y2, d2), y2, d1), y2, n0);
+            float a, c2, x0, x1;
+            unpair2(den, a, c2);
+            unpair2(fma2(num, pair2(rcp_fast(a), rcp_fast(c2)), nm2), x0, x1);
+            x0 = ex2(x0);
+            x1 = ex2(x1);
+            ls[e & 1] = add2(ls[e & 1], pair2(x0, x1));
+            w[e] = pack_bf16(x0, x1);
+          }
+          tmem_st16(tS + c * 16, w);
+          if (c == 1) half_done(0);
+        }
+        lsum = add2(ls[0], ls[1]);
+      } else if (range == 0) {
         const uint64_t nm2 = pair2(-mu, -mu);
         uint64_t ls[4] = {lsum, 0, 0, 0};
 #pragma unroll
