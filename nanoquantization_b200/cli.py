@@ -21,7 +21,7 @@ import sys
 
 DTYPES = ("bfloat16", "float16", "float32")
 TRACE_REQUESTS = 16      # requests that can be live at once when replaying
-TRACE_BLOCK = 64
+TRACE_BLOCK = 256        # the engine's own block size: the kernels are those of serving
 
 
 def _model(args):
