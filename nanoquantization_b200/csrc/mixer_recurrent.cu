@@ -239,25 +239,25 @@ __global__ void __launch_bounds__(256) mingru_chunk_kernel(const T* __restrict__
       *reinterpret_cast<float4*>(p.folds + 2 * (gru_chunk_id(p.bt, b, chunk) * (p.width / 2) + c / 2)) = make_float4(FA.x, FA.y, FB.x, FB.y);
     }
   } else {
-  for (int w = 0; w < warp; ++w) {
-    const float2 wa = As[w][lane], wb = Bs[w][lane];
-    S.x = wa.x * S.x + wb.x; S.y = wa.y * S.y + wb.y;
-  }
-  T* orow = out + (size_t)(t0 + tok0) * p.width + c;
-  float2 gate[kGruWarpTokens];
-#pragma unroll
-  for (int i = 0; i < kGruWarpTokens; ++i) gate[i] = ld_pair(base + (size_t)(t0 + min(tok0 + i, n - 1)) * p.stride + p.g_off);
-#pragma unroll
-  for (int i = 0; i < kGruWarpTokens; ++i) {
-    S.x = a[i].x * S.x + v[i].x; S.y = a[i].y * S.y + v[i].y;
-    if (live && i < cnt) {
-      const float2 g = gate[i];
-      st_pair(orow + (size_t)i * p.width, make_float2(S.x * (g.x * gate_sigmoid<T>(g.x)), S.y * (g.y * gate_sigmoid<T>(g.y))));
+    for (int w = 0; w < warp; ++w) {
+      const float2 wa = As[w][lane], wb = Bs[w][lane];
+      S.x = wa.x * S.x + wb.x; S.y = wa.y * S.y + wb.y;
     }
-  }
-  // every warp has read the state (of a sequence with one chunk) before the last one replaces it
-  __syncthreads();
-  if (live && warp == 7 && first + kGruChunk >= n) st_pair(own, S);
+    T* orow = out + (size_t)(t0 + tok0) * p.width + c;
+    float2 gate[kGruWarpTokens];
+#pragma unroll
+    for (int i = 0; i < kGruWarpTokens; ++i) gate[i] = ld_pair(base + (size_t)(t0 + min(tok0 + i, n - 1)) * p.stride + p.g_off);
+#pragma unroll
+    for (int i = 0; i < kGruWarpTokens; ++i) {
+      S.x = a[i].x * S.x + v[i].x; S.y = a[i].y * S.y + v[i].y;
+      if (live && i < cnt) {
+        const float2 g = gate[i];
+        st_pair(orow + (size_t)i * p.width, make_float2(S.x * (g.x * gate_sigmoid<T>(g.x)), S.y * (g.y * gate_sigmoid<T>(g.y))));
+      }
+    }
+    // every warp has read the state (of a sequence with one chunk) before the last one replaces it
+    __syncthreads();
+    if (live && warp == 7 && first + kGruChunk >= n) st_pair(own, S);
   }
 }
 

@@ -223,3 +223,32 @@ def test_fused_decode_block_vs_oracle(dtype, M):
     gu = O.w4a16_ref(xn, b["qweight"], b["qscales"], b["qzeros"]).to(dtype)
     want = (torch.nn.functional.silu(gu[:, :I]).to(dtype) * gu[:, I:]).float()
     assert O.rel_err(y, want) <= 2 * tol   # three 16-bit roundings (y, silu, product) on top of the GEMM's
+
+
+@torch.no_grad()
+def test_prompt_in_portions_gives_the_same_logits():
+    """Later portions read the earlier ones' keys from the pages; single tokens take the decode path."""
+    from nanoquantization_b200.engine import Sequence
+    m = _tiny(seed=4)
+    m.fuse_projections()
+    toks = torch.randint(0, 512, (45,), generator=torch.Generator().manual_seed(5)).tolist()
+    eng = LLMEngine(m, num_blocks=16, block_size=16, max_batch=2)
+
+    def run(sizes):
+        seq, out, i = Sequence(0, [], 1), [], 0
+        for n in sizes:
+            out += eng.extend([(seq, toks[i:i + n], list(range(n)))])
+            i += n
+        eng.drop(seq)
+        return torch.cat(out)
+    whole = run([45])
+    for sizes in ([20, 2, 23], [17, 27, 1], [40, 1, 1, 1, 1, 1]):
+        assert float((run(sizes) - whole).abs().max()) <= 3e-2 * float(whole.abs().max())
+    assert len(eng.blocks.free) == 16
+
+
+def test_scheduler_portions_through_generate():
+    m = _tiny(seed=2)
+    eng = LLMEngine(m, num_blocks=24, block_size=16, max_batch=3, prefill_portion=7)
+    outs = eng.generate([[1 + i] * (4 + 9 * i) for i in range(4)], [2, 5, 3, 4])
+    assert [len(o) for o in outs] == [2, 5, 3, 4] and len(eng.blocks.free) == 24

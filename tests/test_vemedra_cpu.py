@@ -149,7 +149,6 @@ def test_scheduler_frees_half_read_prompts_when_nothing_else_can_move():
 
 
 def test_step_batch_bookkeeping():
-
     b = StepBatch.host([[5, 6], [9]], [6, 0], [[-1, 3], [2]], [4, 1], 3, 4)
     assert b.tokens.tolist() == [5, 6, 9] and b.positions.tolist() == [6, 7, 0] and b.rows.tolist() == [14, 15, 8]
     assert b.cu.tolist() == [0, 2, 3] and b.pos0.tolist() == [6, 0] and b.ctx.tolist() == [8, 1] and b.slot.tolist() == [4, 1]
