@@ -1,6 +1,7 @@
-/* nqb200_mixers -- C ABI of the sequence-mixing kernels (sm_100a): input convolution fused with RMS norm,
- * partial rotary embedding with a paged K/V store, chunk-masked attention with a score cap and a sink,
- * retention, minGRU, clamped GLU, and the skinny dense linears of decode steps with these steps inside.
+/* nqb200_mixers -- C ABI of the sequence-mixing kernels (sm_100a): input convolution fused with RMS norm, norms after
+ * the residual sum, partial rotary embedding with a paged K/V store, chunk-masked attention with a score cap and a
+ * sink or with sigmoid weights, retention, gated linear attention, minGRU, clamped GLU, per-layer token inputs, and
+ * the skinny dense linears of decode steps with these steps inside.
  *
  * Conventions as in nqb200.h: plain device pointers, asynchronous on `stream`, status codes, nothing here
  * allocates.  `dtype` is the type of activations, weights and K/V caches: NQB200_BF16, or NQB200_F32 where
@@ -39,6 +40,23 @@ int nqb200_stream_add(float* x, const int64_t* ids, const void* embed, const flo
 int nqb200_rmsnorm_rows(const float* x, const int64_t* rows, const float* weight, void* out, int64_t n_rows,
                         int64_t width, float eps, int dtype, void* stream);
 
+/* RMS norm in groups: the row is split into `groups` equal consecutive parts, each divided by its own root mean square,
+ * and the whole multiplied by weight [width].
+ * nqb200_group_norm_rows: out[r] = norm(x[rows ? rows[r] : r]), rounded to dtype.
+ * nqb200_post_norm: x[t] = norm(alpha * x[t] + sum_{j < terms} y[t * terms + j]) in place; h[t] = x[t] rounded to dtype.
+ * y [tokens * terms, width] is of y_dtype (NQB200_BF16 or NQB200_F32); terms = 0: nothing is added, y may be NULL. */
+int nqb200_group_norm_rows(const float* x, const int64_t* rows, const float* weight, void* out, int64_t n_rows,
+                           int64_t width, int64_t groups, float eps, int dtype, void* stream);
+int nqb200_post_norm(float* x, const void* y, int y_dtype, int64_t terms, float alpha, const float* weight, void* h,
+                     int64_t tokens, int64_t width, int64_t groups, float eps, int dtype, void* stream);
+
+/* What a layer adds per token: out[t, i] = gelu_tanh(gate[t, i]) * table[ids[t] * table_stride + column + i], i < dim, and
+ * x[t] += y[t] / rms(y[t]) * weight with h[t] = the sum rounded to dtype (y float [tokens, width]). */
+int nqb200_gelu_table(const void* gate, const int64_t* ids, const void* table, int64_t table_stride, int64_t column,
+                      void* out, int64_t tokens, int64_t dim, int dtype, void* stream);
+int nqb200_add_normed(float* x, const float* y, const float* weight, void* h, int64_t tokens, int64_t width, float eps,
+                      int dtype, void* stream);
+
 /* h = RMSnorm(x) * weight; out[t, c] = h[t, c] + sum_j conv[j * width + c] h[t - taps + 1 + j, c], rounded to
  * dtype.  state float [slots, taps - 1, width] holds each sequence's last taps - 1 rows of h and is updated. */
 int nqb200_rmsnorm_conv(const float* x, const float* weight, const float* conv, float* state, void* out,
@@ -53,10 +71,28 @@ int nqb200_rope_store(void* proj, void* k_cache, void* v_cache, const float* inv
 
 typedef struct {
   int32_t heads, kv_heads, dim, vdim;
+  int32_t rot;             /* the first rot dimensions turn */
+  int32_t interleaved;     /* pairs (2i, 2i + 1); else (i, i + rot/2) */
+  const float* inv_freq;   /* [rot / 2] */
+  const float* q_norm;     /* [dim] RMS norm over each head ahead of the rotation, or NULL */
+  const float* k_norm;
+  float eps;
+} nqb200_rope;
+
+/* nqb200_rope_store with both pair layouts and a norm ahead of the rotation.  v_off may be k_off: the values are then the
+ * keys as projected.  k_cache NULL: k is turned in place and nothing is stored. */
+int nqb200_norm_rope(void* proj, void* k_cache, void* v_cache, const nqb200_rope* r, const nqb200_batch* b, int64_t stride,
+                     int64_t q_off, int64_t k_off, int64_t v_off, int dtype, void* stream);
+
+typedef struct {
+  int32_t heads, kv_heads, dim, vdim;
   int32_t chunk;          /* a query sees keys j <= i with j / chunk == i / chunk; <= 0: no chunks */
   float scale, softcap;   /* softcap <= 0: none */
   const float* sink;      /* [heads] or NULL */
   float out_scale;
+  const float* temp;      /* [heads] factor of the scores, or NULL; sigmoid only */
+  const float* bias;      /* [heads] added to the scores, or NULL; sigmoid only */
+  int32_t sigmoid;        /* a key's weight is sigmoid(scale temp q.k + bias), not normalised: no softcap, no sink */
 } nqb200_attention;
 
 /* Attention of rotated q (rows of `q`, row stride q_stride, head h at column h * dim) over the paged caches of
@@ -67,9 +103,10 @@ int nqb200_chunk_attention(const void* q, int64_t q_stride, const void* k_cache,
                            void* stream);
 
 /* Retention.  proj holds q and k (heads x dim at q_off, k_off) and v (heads x vdim at v_off).
- * S <- decay[h] S + (dim^-1/2 k) v^T, o = S^T q, state float [slots, heads, dim, vdim].  o float [tokens, heads * vdim]. */
+ * S <- decay[h] S + (dim^-1/2 k) v^T, o = S^T q, state float [slots, heads, dim, vdim].  o float [tokens, heads * vdim].
+ * log_decay [tokens, heads * dim] (then decay is not read): gated linear attention, S <- diag(exp(log_decay)) S + ... */
 int nqb200_retention(const void* proj, int64_t stride, int64_t q_off, int64_t k_off, int64_t v_off, const float* decay,
-                     float* state, float* o, int64_t heads, int64_t dim, int64_t vdim, const nqb200_batch* b, int dtype,
+                     const float* log_decay, float* state, float* o, int64_t heads, int64_t dim, int64_t vdim, const nqb200_batch* b, int dtype,
                      void* stream);
 
 typedef struct {
@@ -86,8 +123,14 @@ int nqb200_retention_prefill(const void* proj, int64_t stride, int64_t off, void
 int nqb200_retention_prefill_supported(const nqb200_retention_desc* r, int64_t stride, int64_t off, int64_t act_stride, int64_t act_col);
 int64_t nqb200_retention_chunks(int64_t tokens, int64_t batch);
 
-/* out[t * out_stride + h * vdim + c] = out_scale * o / rms(o over the head) * silu(gate[t * gate_stride + h * vdim + c]). */
-int nqb200_head_norm_gate(const float* o, const void* gate, int64_t gate_stride, void* out, int64_t out_stride,
+/* log_decay[t, c] = log(sigmoid(a2[c] . low[t] + bias[c])) / tau for c < channels; low [tokens, rank] with row stride
+ * low_stride and a2 [channels, rank] of dtype. */
+int nqb200_gla_log_decay(const void* low, int64_t low_stride, const void* a2, const float* bias, float* log_decay,
+                         int64_t tokens, int64_t channels, int64_t rank, float tau, int dtype, void* stream);
+
+/* out[t * out_stride + h * vdim + c] = out_scale * o / rms(o over the head) * weight[c] * silu(gate[t * gate_stride + h *
+ * vdim + c]); weight [vdim] or NULL. */
+int nqb200_head_norm_gate(const float* o, const void* gate, int64_t gate_stride, const float* weight, void* out, int64_t out_stride,
                           int64_t tokens, int64_t heads, int64_t vdim, float eps, float out_scale, int dtype, void* stream);
 
 /* minGRU over proj [tokens, stride]: z, x and gate pre-activations at columns z_off, x_off, g_off.
@@ -106,8 +149,12 @@ int nqb200_clamped_glu(const void* gate_up, void* out, int64_t tokens, int64_t f
 
 enum { NQB200_DENSE_BF16 = 0, NQB200_DENSE_F32 = 1, NQB200_DENSE_RESIDUAL = 2 };
 
-/* y = x w^T, x bf16 [M, K], w bf16 [N, K], M <= 16, K % 8 == 0.  mode: y as bf16, y as float, or out float += y. */
-int nqb200_dense_decode(const void* x, const void* w, void* out, int64_t M, int64_t N, int64_t K, int mode, void* stream);
+/* y = x w^T, x bf16 [M, K], w bf16 [N, K], M <= 16, K % 8 == 0.  mode: y as bf16, y as float, or float out = beta out + y. */
+int nqb200_dense_decode(const void* x, const void* w, void* out, int64_t M, int64_t N, int64_t K, int mode, float beta, void* stream);
+
+/* nqb200_gelu_table of the product (not rounded between): w [dim, K], out bf16 [M, dim]. */
+int nqb200_dense_decode_gelu_table(const void* x, const void* w, const int64_t* ids, const void* table, int64_t table_stride,
+                                   int64_t column, void* out, int64_t M, int64_t dim, int64_t K, void* stream);
 
 /* w [2 ff, K] = gate rows, then up rows; out bf16 [M, ff] as nqb200_clamped_glu of the product (not rounded between). */
 int nqb200_dense_decode_glu(const void* x, const void* w, void* out, int64_t M, int64_t ff, int64_t K, float limit, void* stream);

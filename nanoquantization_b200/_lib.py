@@ -14,6 +14,7 @@ import torch
 _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(_HERE, "lib", "libnqb200.so")
 MIXERS_PATH = os.path.join(_HERE, "lib", "libnqb200_mixers.so")
+MOE_PATH = os.path.join(_HERE, "lib", "libnqb200_moe.so")
 
 F16, BF16, F32 = 0, 1, 2
 _vp, _i64, _int, _sz = ctypes.c_void_p, ctypes.c_int64, ctypes.c_int, ctypes.c_size_t
@@ -76,7 +77,14 @@ class AttentionDesc(ctypes.Structure):
     """nqb200_attention of include/nqb200_mixers.h."""
     _fields_ = [("heads", ctypes.c_int32), ("kv_heads", ctypes.c_int32), ("dim", ctypes.c_int32), ("vdim", ctypes.c_int32),
                 ("chunk", ctypes.c_int32), ("scale", ctypes.c_float), ("softcap", ctypes.c_float), ("sink", _vp),
-                ("out_scale", ctypes.c_float)]
+                ("out_scale", ctypes.c_float), ("temp", _vp), ("bias", _vp), ("sigmoid", ctypes.c_int32)]
+
+
+class RopeDesc(ctypes.Structure):
+    """nqb200_rope of include/nqb200_mixers.h."""
+    _fields_ = [("heads", ctypes.c_int32), ("kv_heads", ctypes.c_int32), ("dim", ctypes.c_int32), ("vdim", ctypes.c_int32),
+                ("rot", ctypes.c_int32), ("interleaved", ctypes.c_int32), ("inv_freq", _vp), ("q_norm", _vp), ("k_norm", _vp),
+                ("eps", ctypes.c_float)]
 
 
 class RetentionDesc(ctypes.Structure):
@@ -85,33 +93,60 @@ class RetentionDesc(ctypes.Structure):
                 ("out_scale", ctypes.c_float), ("decay", _vp)]
 
 
+class RouterDesc(ctypes.Structure):
+    """nqb200_router of include/nqb200_moe.h."""
+    _fields_ = [("experts", ctypes.c_int32), ("top", ctypes.c_int32), ("groups", ctypes.c_int32), ("keep", ctypes.c_int32),
+                ("scale", ctypes.c_float), ("correction", _vp)]
+
+
+class MoePlan(ctypes.Structure):
+    """nqb200_moe_plan of include/nqb200_moe.h."""
+    _fields_ = [("expert", _vp), ("weight", _vp), ("offsets", _vp), ("order", _vp), ("active", _vp), ("counters", _vp)]
+
+
+MOE_UP, MOE_DOWN = 0, 1
 DENSE_BF16, DENSE_F32, DENSE_RESIDUAL = 0, 1, 2
 _ret = ctypes.POINTER(RetentionDesc)
 _step, _att, _f32 = ctypes.POINTER(StepDesc), ctypes.POINTER(AttentionDesc), ctypes.c_float
+_rope, _router, _plan = ctypes.POINTER(RopeDesc), ctypes.POINTER(RouterDesc), ctypes.POINTER(MoePlan)
 # mirrors include/nqb200_mixers.h one to one
 MIXER_SIGNATURES = {
     "nqb200_stream_add": (_int, [_vp, _vp, _vp, _vp, _int, _i64, _i64, _int, _vp]),
     "nqb200_rmsnorm_rows": (_int, [_vp, _vp, _vp, _vp, _i64, _i64, _f32, _int, _vp]),
+    "nqb200_group_norm_rows": (_int, [_vp, _vp, _vp, _vp, _i64, _i64, _i64, _f32, _int, _vp]),
+    "nqb200_post_norm": (_int, [_vp, _vp, _int, _i64, _f32, _vp, _vp, _i64, _i64, _i64, _f32, _int, _vp]),
+    "nqb200_gelu_table": (_int, [_vp, _vp, _vp, _i64, _i64, _vp, _i64, _i64, _int, _vp]),
+    "nqb200_add_normed": (_int, [_vp, _vp, _vp, _vp, _i64, _i64, _f32, _int, _vp]),
     "nqb200_rmsnorm_conv": (_int, [_vp, _vp, _vp, _vp, _vp, _step, _i64, _i64, _f32, _int, _vp]),
     "nqb200_rope_store": (_int, [_vp, _vp, _vp, _vp, _step] + [_i64] * 9 + [_int, _vp]),
+    "nqb200_norm_rope": (_int, [_vp, _vp, _vp, _rope, _step, _i64, _i64, _i64, _i64, _int, _vp]),
     "nqb200_chunk_attention": (_int, [_vp, _i64, _vp, _vp, _vp, _i64, _i64, _att, _step, _vp, _int, _vp]),
-    "nqb200_retention": (_int, [_vp, _i64, _i64, _i64, _i64, _vp, _vp, _vp, _i64, _i64, _i64, _step, _int, _vp]),
-    "nqb200_head_norm_gate": (_int, [_vp, _vp, _i64, _vp, _i64, _i64, _i64, _i64, _f32, _f32, _int, _vp]),
+    "nqb200_retention": (_int, [_vp, _i64, _i64, _i64, _i64, _vp, _vp, _vp, _vp, _i64, _i64, _i64, _step, _int, _vp]),
+    "nqb200_gla_log_decay": (_int, [_vp, _i64, _vp, _vp, _vp, _i64, _i64, _i64, _f32, _int, _vp]),
+    "nqb200_head_norm_gate": (_int, [_vp, _vp, _i64, _vp, _vp, _i64, _i64, _i64, _i64, _f32, _f32, _int, _vp]),
     "nqb200_mingru": (_int, [_vp, _i64, _i64, _i64, _i64, _vp, _vp, _vp, _vp, _i64, _vp, _step, _int, _vp]),
     "nqb200_mingru_scratch": (_i64, [_i64, _i64, _i64]),
     "nqb200_clamped_glu": (_int, [_vp, _vp, _i64, _i64, _f32, _int, _vp]),
     "nqb200_retention_prefill": (_int, [_vp, _i64, _i64, _vp, _i64, _i64, _ret, _vp, _vp, _step, _vp]),
     "nqb200_retention_prefill_supported": (_int, [_ret, _i64, _i64, _i64, _i64]),
     "nqb200_retention_chunks": (_i64, [_i64, _i64]),
-    "nqb200_dense_decode": (_int, [_vp, _vp, _vp, _i64, _i64, _i64, _int, _vp]),
+    "nqb200_dense_decode": (_int, [_vp, _vp, _vp, _i64, _i64, _i64, _int, _f32, _vp]),
+    "nqb200_dense_decode_gelu_table": (_int, [_vp, _vp, _vp, _vp, _i64, _i64, _vp, _i64, _i64, _i64, _vp]),
     "nqb200_dense_decode_glu": (_int, [_vp, _vp, _vp, _i64, _i64, _i64, _f32, _vp]),
     "nqb200_dense_decode_mingru": (_int, [_vp] * 6 + [_i64, _i64, _step, _vp]),
     "nqb200_mixer_decode_supported": (_int, [_att, _ret]),
     "nqb200_mixer_decode": (_int, [_vp, _i64, _vp, _i64, _att, _vp, _i64, _i64, _i64, _vp, _vp, _ret, _i64, _i64, _vp, _step, _vp]),
 }
 
+# mirrors include/nqb200_moe.h one to one
+MOE_SIGNATURES = {
+    "nqb200_moe_route": (_int, [_vp, _router, _plan, _i64, _vp]),
+    "nqb200_moe_linear": (_int, [_vp, _vp, _vp, _int, _i64, _i64, _i64, _router, _plan, _int, _int, _vp, _vp]),
+    "nqb200_moe_linear_kernel": (ctypes.c_char_p, [_i64, _i64, _i64, _i64, _int]),
+}
+
 _lib = None
-_mixers = None
+_more: dict[str, ctypes.CDLL] = {}
 _lock = threading.Lock()
 
 
@@ -136,21 +171,31 @@ def load() -> ctypes.CDLL:
     return _lib
 
 
-def load_mixers() -> ctypes.CDLL:
-    """Load the library of sequence-mixing kernels once; raise if it has not been built."""
-    global _mixers
-    if _mixers is None:
+def _load_once(path: str, signatures: dict) -> ctypes.CDLL:
+    lib = _more.get(path)
+    if lib is None:
         with _lock:
-            if _mixers is None:
-                if not os.path.exists(MIXERS_PATH):
-                    raise RuntimeError(f"{MIXERS_PATH} is missing: build it with `python -m nanoquantization_b200.csrc.build` "
+            if path not in _more:
+                if not os.path.exists(path):
+                    raise RuntimeError(f"{path} is missing: build it with `python -m nanoquantization_b200.csrc.build` "
                                        "(needs nvcc). There is no CPU or PyTorch fallback for these kernels.")
-                lib = ctypes.CDLL(MIXERS_PATH)
-                for name, (res, args) in MIXER_SIGNATURES.items():
+                lib = ctypes.CDLL(path)
+                for name, (res, args) in signatures.items():
                     fn = getattr(lib, name)
                     fn.restype, fn.argtypes = res, args
-                _mixers = lib
-    return _mixers
+                _more[path] = lib
+            lib = _more[path]
+    return lib
+
+
+def load_mixers() -> ctypes.CDLL:
+    """Load the library of sequence-mixing kernels once; raise if it has not been built."""
+    return _load_once(MIXERS_PATH, MIXER_SIGNATURES)
+
+
+def load_moe() -> ctypes.CDLL:
+    """Load the library of mixture-of-experts kernels once; raise if it has not been built."""
+    return _load_once(MOE_PATH, MOE_SIGNATURES)
 
 
 _STATUS = ("ok", "bad shape", "bad dtype", "misaligned pointer", "null pointer", "workspace missing or too small",

@@ -1,7 +1,7 @@
 """Build the libraries (sm_100a) in-tree with nvcc.  Cross-compiles without a GPU.
 
-Two shared objects: ``libnqb200.so`` (the W4A16 linears, their elementwise neighbours and the peer all-reduce) and
-``libnqb200_mixers.so`` (the sequence-mixing kernels).  They are built separately so that a model compiles only what
+Three shared objects: ``libnqb200.so`` (the W4A16 linears, their elementwise neighbours and the peer all-reduce),
+``libnqb200_mixers.so`` (the sequence-mixing kernels) and ``libnqb200_moe.so`` (mixtures of experts).  They are built separately so that a model compiles only what
 it uses; the sources of a library are compiled side by side."""
 from __future__ import annotations
 
@@ -16,11 +16,14 @@ ROOT = os.path.dirname(os.path.dirname(HERE))
 LIB_DIR = os.path.join(os.path.dirname(HERE), "lib")
 LIB_PATH = os.path.join(LIB_DIR, "libnqb200.so")
 MIXERS_PATH = os.path.join(LIB_DIR, "libnqb200_mixers.so")
+MOE_PATH = os.path.join(LIB_DIR, "libnqb200_moe.so")
 SOURCES = ["api.cu", "unpack_dequant.cu", "gemm_decode.cu", "gemm_stream.cu", "gemm_umma_prefill.cu", "gemm_umma_pair.cu", "quantize_pack.cu", "fused_elementwise.cu", "peer_allreduce.cu"]
 HEADERS = ["common.cuh", "tma_utils.cuh", "umma_utils.cuh", os.path.join(ROOT, "include", "nqb200.h")]
 MIXER_SOURCES = ["mixer_norm.cu", "mixer_attention.cu", "mixer_recurrent.cu", "mixer_dense.cu", "mixer_decode.cu", "mixer_prefill.cu", "mixer_attention_umma.cu"]
 MIXER_HEADERS = ["common.cuh", "mixers.cuh", "tma_utils.cuh", "umma_utils.cuh", os.path.join(ROOT, "include", "nqb200.h"), os.path.join(ROOT, "include", "nqb200_mixers.h")]
-LIBRARIES = {LIB_PATH: (SOURCES, HEADERS), MIXERS_PATH: (MIXER_SOURCES, MIXER_HEADERS)}
+MOE_SOURCES = ["moe_route.cu", "moe_experts.cu", "moe_umma.cu"]
+MOE_HEADERS = MIXER_HEADERS + ["moe.cuh", os.path.join(ROOT, "include", "nqb200_moe.h")]
+LIBRARIES = {LIB_PATH: (SOURCES, HEADERS), MIXERS_PATH: (MIXER_SOURCES, MIXER_HEADERS), MOE_PATH: (MOE_SOURCES, MOE_HEADERS)}
 
 
 def _stale(path: str = LIB_PATH) -> bool:

@@ -38,6 +38,47 @@ __global__ void __launch_bounds__(256) rope_store_kernel(T* __restrict__ proj, T
   for (int e = threadIdx.x; e < kv_heads * vdim; e += blockDim.x) vd[e] = row[v_off + e];
 }
 
+// One CTA per token and a warp per head: optional RMS norm of the head, rotation in either pair layout, store.
+template <typename T>
+__global__ void __launch_bounds__(256) norm_rope_kernel(T* __restrict__ proj, T* __restrict__ k_cache, T* __restrict__ v_cache, const nqb200_rope r,
+                                                        const nqb200_batch bt, int64_t stride, int q_off, int k_off, int v_off) {
+  extern __shared__ float cs[];  // [rot/2] cos, [rot/2] sin
+  grid_launch_dependents();
+  grid_dependency_wait();
+  const int b = blockIdx.y, i = blockIdx.x, t0 = bt.cu[b], half = r.rot / 2, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (i >= bt.cu[b + 1] - t0) return;
+  const int p = bt.pos0[b] + i;
+  for (int f = threadIdx.x; f < half; f += blockDim.x) sincosf((float)p * r.inv_freq[f], &cs[half + f], &cs[f]);
+  __syncthreads();
+  T* row = proj + (size_t)(t0 + i) * stride;
+  const size_t slot = k_cache ? kv_row(bt, b, p) : 0;
+  const int first = r.interleaved ? 1 : half, step = r.interleaved ? 2 : 1;   // distance inside a pair, and between pairs
+  for (int hd = warp; hd < r.heads + r.kv_heads; hd += 8) {
+    const bool isq = hd < r.heads;
+    const T* src = row + (isq ? q_off + hd * r.dim : k_off + (hd - r.heads) * r.dim);
+    T* dst = isq || !k_cache ? const_cast<T*>(src) : k_cache + slot * r.kv_heads * r.dim + (hd - r.heads) * r.dim;
+    const float* w = isq ? r.q_norm : r.k_norm;
+    float inv = 1.f;
+    if (w) {
+      float ss = 0.f;
+      for (int d = lane; d < r.dim; d += 32) { const float x = to_f(src[d]); ss += x * x; }
+      inv = 1.f / sqrtf(warp_sum(ss) / (float)r.dim + r.eps);
+    }
+    for (int j = lane; j < half; j += 32) {
+      const int a = j * step, c = a + first;
+      float u = to_f(src[a]), v = to_f(src[c]);
+      if (w) { u = u * inv * w[a]; v = v * inv * w[c]; }
+      dst[a] = from_f<T>(u * cs[j] - v * cs[half + j]);
+      dst[c] = from_f<T>(v * cs[j] + u * cs[half + j]);
+    }
+    for (int d = r.rot + lane; d < r.dim; d += 32) dst[d] = w ? from_f<T>(to_f(src[d]) * inv * w[d]) : src[d];
+  }
+  if (k_cache) {
+    T* vd = v_cache + slot * r.kv_heads * r.vdim;
+    for (int e = threadIdx.x; e < r.kv_heads * r.vdim; e += blockDim.x) vd[e] = row[v_off + e];
+  }
+}
+
 constexpr int kSimpleKeys = 128;   // keys per pass = threads
 constexpr int kSimpleVCols = 8;    // value columns per thread at most: vdim <= 1024
 
@@ -58,6 +99,7 @@ __global__ void __launch_bounds__(kSimpleKeys) attention_simple_kernel(const T* 
   const T* qr = q + (size_t)(t0 + i) * q_stride + (size_t)h * at.dim;
   for (int d = tid; d < at.dim; d += kSimpleKeys) qs[d] = to_f(qr[d]);
   float m = at.sink ? at.sink[h] : -INFINITY, l = at.sink ? 1.f : 0.f;
+  const float factor = at.scale * (at.temp ? at.temp[h] : 1.f), shift = at.bias ? at.bias[h] : 0.f;
   float acc[kSimpleVCols] = {};
   for (int j0 = lo; j0 <= p; j0 += kSimpleKeys) {
     const int j = j0 + tid;
@@ -69,21 +111,28 @@ __global__ void __launch_bounds__(kSimpleKeys) attention_simple_kernel(const T* 
       const T* kr = k_cache + (r * at.kv_heads + g) * at.dim;
       float d = 0.f;
       for (int c = 0; c < at.dim; ++c) d += qs[c] * to_f(kr[c]);
-      s = d * at.scale;
+      s = d * factor + shift;
       if (at.softcap > 0.f) s = at.softcap * tanhf(s / at.softcap);
     }
-    const float wm = warp_max(s);
-    if ((tid & 31) == 0) red[tid >> 5] = wm;
-    __syncthreads();
-    const float m_new = fmaxf(m, fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3])));
-    const float corr = expf(m - m_new), e = expf(s - m_new);
-    sc[tid] = e;
-    const float ws = warp_sum(e);
-    __syncthreads();
-    if ((tid & 31) == 0) red[tid >> 5] = ws;
-    __syncthreads();
-    l = l * corr + (red[0] + red[1] + red[2] + red[3]);
-    m = m_new;
+    float corr = 1.f;
+    if (at.sigmoid) {
+      sc[tid] = sigmoid_f(s);
+      __syncthreads();
+    } else {
+      const float wm = warp_max(s);
+      if ((tid & 31) == 0) red[tid >> 5] = wm;
+      __syncthreads();
+      const float m_new = fmaxf(m, fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3])));
+      const float e = expf(s - m_new);
+      corr = expf(m - m_new);
+      sc[tid] = e;
+      const float ws = warp_sum(e);
+      __syncthreads();
+      if ((tid & 31) == 0) red[tid >> 5] = ws;
+      __syncthreads();
+      l = l * corr + (red[0] + red[1] + red[2] + red[3]);
+      m = m_new;
+    }
     const int cnt = min(kSimpleKeys, p - j0 + 1);
 #pragma unroll
     for (int c = 0; c < kSimpleVCols; ++c) {
@@ -94,7 +143,7 @@ __global__ void __launch_bounds__(kSimpleKeys) attention_simple_kernel(const T* 
       acc[c] = a;
     }
   }
-  const float f = at.out_scale / l;
+  const float f = at.sigmoid ? at.out_scale : at.out_scale / l;
 #pragma unroll
   for (int c = 0; c < kSimpleVCols; ++c) {
     const int col = tid + c * kSimpleKeys;
@@ -124,6 +173,27 @@ extern "C" int nqb200_rope_store(void* proj, void* k_cache, void* v_cache, const
 #undef NQB200_ROPE
 }
 
+extern "C" int nqb200_norm_rope(void* proj, void* k_cache, void* v_cache, const nqb200_rope* r, const nqb200_batch* b, int64_t stride,
+                                int64_t q_off, int64_t k_off, int64_t v_off, int dtype, void* stream) {
+  const int st = check_batch(b, k_cache != nullptr);
+  if (st != NQB200_OK) return st;
+  if (!r) return NQB200_ERR_NULL_POINTER;
+  if (r->heads <= 0 || r->kv_heads <= 0 || r->dim <= 0 || r->rot < 0 || r->rot > r->dim || r->rot % 2 != 0 || stride <= 0 || r->rot > 8192 ||
+      (k_cache && r->vdim <= 0))
+    return NQB200_ERR_BAD_SHAPE;
+  if (!mixer_dtype(dtype)) return NQB200_ERR_BAD_DTYPE;
+  if (b->tokens == 0) return NQB200_OK;
+  if (!proj || (k_cache && !v_cache) || (r->rot > 0 && !r->inv_freq)) return NQB200_ERR_NULL_POINTER;
+  const dim3 grid((unsigned)b->max_len, (unsigned)b->batch), block(256);
+  const size_t smem = (size_t)r->rot * sizeof(float);
+  cudaStream_t s = (cudaStream_t)stream;
+  if (dtype == NQB200_F32)
+    return launch_overlapped(norm_rope_kernel<float>, grid, block, smem, s, (float*)proj, (float*)k_cache, (float*)v_cache, *r, *b, stride,
+                             (int)q_off, (int)k_off, (int)v_off);
+  return launch_overlapped(norm_rope_kernel<bf16>, grid, block, smem, s, (bf16*)proj, (bf16*)k_cache, (bf16*)v_cache, *r, *b, stride, (int)q_off,
+                           (int)k_off, (int)v_off);
+}
+
 extern "C" int nqb200_chunk_attention(const void* q, int64_t q_stride, const void* k_cache, const void* v_cache, void* out,
                                       int64_t out_stride, int64_t cache_rows, const nqb200_attention* a, const nqb200_batch* b, int* status,
                                       int dtype, void* stream) {
@@ -131,14 +201,15 @@ extern "C" int nqb200_chunk_attention(const void* q, int64_t q_stride, const voi
   if (st != NQB200_OK) return st;
   if (!a) return NQB200_ERR_NULL_POINTER;
   if (a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads != 0 || a->dim <= 0 || a->dim > 4096 || a->vdim <= 0 ||
-      a->vdim > kSimpleKeys * kSimpleVCols || a->heads > 65535)
+      a->vdim > kSimpleKeys * kSimpleVCols || a->heads > 65535 || (a->sigmoid && (a->softcap > 0.f || a->sink)) ||
+      (!a->sigmoid && (a->temp || a->bias)))
     return NQB200_ERR_BAD_SHAPE;
   if (!mixer_dtype(dtype)) return NQB200_ERR_BAD_DTYPE;
   if (b->tokens == 0) return NQB200_OK;
   if (!q || !k_cache || !v_cache || !out) return NQB200_ERR_NULL_POINTER;
-  if (dtype == NQB200_BF16 && attention_umma_supports(q, q_stride, k_cache, v_cache, out, out_stride, cache_rows, a, b))
+  if (dtype == NQB200_BF16 && !a->sigmoid && attention_umma_supports(q, q_stride, k_cache, v_cache, out, out_stride, cache_rows, a, b))
     return attention_umma(q, q_stride, k_cache, v_cache, out, out_stride, cache_rows, a, b, status, (cudaStream_t)stream);
-  if (dtype == NQB200_BF16 && b->max_len > 1 && attention_prefill_supports(q, q_stride, k_cache, v_cache, out, out_stride, a))
+  if (dtype == NQB200_BF16 && !a->sigmoid && b->max_len > 1 && attention_prefill_supports(q, q_stride, k_cache, v_cache, out, out_stride, a))
     return attention_prefill(q, q_stride, k_cache, v_cache, out, out_stride, a, b, (cudaStream_t)stream);
   const dim3 grid((unsigned)b->max_len, (unsigned)a->heads, (unsigned)b->batch), block(kSimpleKeys);
   const size_t smem = (size_t)a->dim * sizeof(float);

@@ -9,13 +9,15 @@
 
 namespace nqb200 {
 
-enum DenseMode { kPlain = 0, kFloat = 1, kResidual = 2, kGlu = 3, kMinGru = 4 };
+enum DenseMode { kPlain = 0, kFloat = 1, kResidual = 2, kGlu = 3, kMinGru = 4, kTable = 5 };
 
 struct DenseArgs {
   const bf16* x; const bf16* w; void* out;
   int M, N, K;            // N: rows of one group (outputs)
+  float beta;             // residual
   float limit;            // GLU
   const float* z_bias; const float* x_bias; float* state; const int32_t* slot; const int32_t* pos0;  // minGRU
+  const int64_t* ids; const bf16* table; int64_t table_stride;   // token table (its first column added)
 };
 
 __device__ __forceinline__ uint4 ld_weight(const bf16* p) {
@@ -101,7 +103,10 @@ __global__ void __launch_bounds__(256) dense_decode_kernel(const DenseArgs p) {
   } else if (MODE == kFloat) {
     reinterpret_cast<float*>(p.out)[at] = v[0];
   } else if (MODE == kResidual) {
-    reinterpret_cast<float*>(p.out)[at] += v[0];
+    float* o = reinterpret_cast<float*>(p.out) + at;
+    *o = p.beta * *o + v[0];
+  } else if (MODE == kTable) {
+    reinterpret_cast<bf16*>(p.out)[at] = __float2bfloat16_rn(gelu_tanh_f(v[0]) * to_f(p.table[(size_t)p.ids[tok] * p.table_stride + n]));
   } else if (MODE == kGlu) {
     const float gt = fminf(v[0], p.limit), up = fminf(fmaxf(v[NG - 1], -p.limit), p.limit);
     reinterpret_cast<bf16*>(p.out)[at] = __float2bfloat16_rn(gt * sigmoid_f(1.702f * gt) * (up + 1.f));
@@ -131,15 +136,25 @@ using namespace nqb200;
 
 static bool dense_sizes(int64_t M, int64_t N, int64_t K) { return M >= 0 && M <= 16 && N > 0 && K > 0 && N <= (1 << 28) && K <= (1 << 28); }
 
-extern "C" int nqb200_dense_decode(const void* x, const void* w, void* out, int64_t M, int64_t N, int64_t K, int mode, void* stream) {
+extern "C" int nqb200_dense_decode(const void* x, const void* w, void* out, int64_t M, int64_t N, int64_t K, int mode, float beta, void* stream) {
   if (!dense_sizes(M, N, K)) return NQB200_ERR_BAD_SHAPE;
   DenseArgs p = {};
-  p.x = (const bf16*)x; p.w = (const bf16*)w; p.out = out; p.M = (int)M; p.N = (int)N; p.K = (int)K;
+  p.x = (const bf16*)x; p.w = (const bf16*)w; p.out = out; p.M = (int)M; p.N = (int)N; p.K = (int)K; p.beta = beta;
   cudaStream_t st = (cudaStream_t)stream;
   if (mode == NQB200_DENSE_BF16) return launch_dense<kPlain>(p, st);
   if (mode == NQB200_DENSE_F32) return launch_dense<kFloat>(p, st);
   if (mode == NQB200_DENSE_RESIDUAL) return launch_dense<kResidual>(p, st);
   return NQB200_ERR_BAD_DTYPE;
+}
+
+extern "C" int nqb200_dense_decode_gelu_table(const void* x, const void* w, const int64_t* ids, const void* table, int64_t table_stride,
+                                              int64_t column, void* out, int64_t M, int64_t dim, int64_t K, void* stream) {
+  if (!dense_sizes(M, dim, K) || column < 0 || table_stride < column + dim) return NQB200_ERR_BAD_SHAPE;
+  if (M > 0 && (!ids || !table)) return NQB200_ERR_NULL_POINTER;
+  DenseArgs p = {};
+  p.x = (const bf16*)x; p.w = (const bf16*)w; p.out = out; p.M = (int)M; p.N = (int)dim; p.K = (int)K;
+  p.ids = ids; p.table = (const bf16*)table + column; p.table_stride = table_stride;
+  return launch_dense<kTable>(p, (cudaStream_t)stream);
 }
 
 extern "C" int nqb200_dense_decode_glu(const void* x, const void* w, void* out, int64_t M, int64_t ff, int64_t K, float limit, void* stream) {

@@ -1,6 +1,6 @@
-// The residual stream's own steps: embedding / loop entry, RMS norm, RMS norm + input convolution, and the
-// clamped GLU between the feed-forward's linears.  The stream is float; a norm reads it once and leaves the
-// 16-bit operand of the next linear.
+// The residual stream's own steps: embedding / loop entry, RMS norm, RMS norm + input convolution, norms after the
+// residual sum, per-layer token inputs, and the clamped GLU between the feed-forward's linears.  The stream is float; a
+// norm reads it once and leaves the 16-bit operand of the next linear.
 #include "mixers.cuh"
 
 namespace nqb200 {
@@ -105,6 +105,11 @@ template <> __device__ __forceinline__ void store4<bf16>(bf16* p, float4 v) {
   *reinterpret_cast<uint2*>(p) = r;
 }
 __device__ __forceinline__ float4 ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4(const float* p) { return ld4(p); }
+__device__ __forceinline__ float4 load4(const bf16* p) {
+  const uint2 r = *reinterpret_cast<const uint2*>(p);
+  return make_float4(__uint_as_float(r.x << 16), __uint_as_float(r.x & 0xFFFF0000u), __uint_as_float(r.y << 16), __uint_as_float(r.y & 0xFFFF0000u));
+}
 __device__ __forceinline__ float4 mul4(float4 a, float4 b) { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); }
 __device__ __forceinline__ float4 scale4(float4 a, float s) { return make_float4(a.x * s, a.y * s, a.z * s, a.w * s); }
 __device__ __forceinline__ void fma4(float4& d, float4 a, float4 b) { d.x += a.x * b.x; d.y += a.y * b.y; d.z += a.z * b.z; d.w += a.w * b.w; }
@@ -250,6 +255,141 @@ static int launch_rmsnorm_conv(const float* x, const float* weight, const float*
                            width, taps, tile, eps);
 }
 
+// Norms after the sum.  A CTA takes a token; the row (alpha x + the terms of y) stays in shared memory between the sums of
+// squares and the use.  The groups of the row are split into about as many pieces as there are warps, a warp sums whole
+// pieces, and the group's scale is taken from its pieces.  out: the row rounded to T; x (if written): the row itself.
+constexpr int kNormThreads = 256, kNormWarps = kNormThreads / 32;
+template <typename T, typename Y>
+__global__ void __launch_bounds__(kNormThreads) group_norm_kernel(float* x, const int64_t* __restrict__ rows, const Y* __restrict__ y, int terms, float alpha,
+                                                                  const float* __restrict__ weight, T* __restrict__ out, int width, int groups, int pieces,
+                                                                  float eps, int write_x) {
+  extern __shared__ float4 norm_smem[];
+  float* row_s = reinterpret_cast<float*>(norm_smem);        // [width]
+  float* part = row_s + (width + 3) / 4 * 4;                 // [groups * pieces]
+  grid_launch_dependents();
+  grid_dependency_wait();
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int64_t at = rows ? rows[blockIdx.x] : blockIdx.x;
+  float* xr = x + (size_t)at * width;
+  const Y* yr = y + (size_t)blockIdx.x * terms * width;
+  const int size = width / groups;
+  const bool vec = size % 4 == 0;
+  if (vec) {
+    for (int c = tid * 4; c < width; c += kNormThreads * 4) {
+      float4 v = scale4(ld4(xr + c), alpha);
+      for (int j = 0; j < terms; ++j) {
+        const float4 a = load4(yr + (size_t)j * width + c);
+        v.x += a.x; v.y += a.y; v.z += a.z; v.w += a.w;
+      }
+      *reinterpret_cast<float4*>(row_s + c) = v;
+    }
+  } else {
+    for (int c = tid; c < width; c += kNormThreads) {
+      float v = alpha * xr[c];
+      for (int j = 0; j < terms; ++j) v += to_f(yr[(size_t)j * width + c]);
+      row_s[c] = v;
+    }
+  }
+  __syncthreads();
+  const int len = (size + pieces - 1) / pieces;
+  for (int q = warp; q < groups * pieces; q += kNormWarps) {
+    const int g = q / pieces, lo = (q - g * pieces) * len, hi = min(lo + len, size);
+    const float* s = row_s + g * size;
+    float ss = 0.f;
+    for (int c = lo + lane; c < hi; c += 32) ss += s[c] * s[c];
+    ss = warp_sum(ss);
+    if (lane == 0) part[q] = ss;
+  }
+  __syncthreads();
+  for (int g = tid; g < groups; g += kNormThreads) {   // a thread per group; its pieces' places become free for the scale
+    float ss = 0.f;
+    for (int k = 0; k < pieces; ++k) ss += part[g * pieces + k];
+    part[g * pieces] = 1.f / sqrtf(ss / (float)size + eps);
+  }
+  __syncthreads();
+  T* o = out + (size_t)blockIdx.x * width;
+  if (vec) {
+    for (int c = tid * 4; c < width; c += kNormThreads * 4) {
+      const float4 v = mul4(scale4(*reinterpret_cast<const float4*>(row_s + c), part[c / size * pieces]), ld4(weight + c));
+      if (write_x) *reinterpret_cast<float4*>(xr + c) = v;
+      store4<T>(o + c, v);
+    }
+  } else {
+    for (int c = tid; c < width; c += kNormThreads) {
+      const float v = row_s[c] * part[c / size * pieces] * weight[c];
+      if (write_x) xr[c] = v;
+      o[c] = from_f<T>(v);
+    }
+  }
+}
+
+// x += y / rms(y) * weight, and the sum rounded to T.
+template <typename T>
+__global__ void __launch_bounds__(kNormThreads) add_normed_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ weight,
+                                                                  T* __restrict__ out, int width, float eps) {
+  __shared__ float red[kNormWarps];
+  grid_launch_dependents();
+  grid_dependency_wait();
+  float* xr = x + (size_t)blockIdx.x * width;
+  const float* yr = y + (size_t)blockIdx.x * width;
+  T* o = out + (size_t)blockIdx.x * width;
+  const int tid = threadIdx.x;
+  const bool vec = width % 4 == 0;
+  float ss = 0.f;
+  if (vec) {
+    for (int c = tid * 4; c < width; c += kNormThreads * 4) { const float4 v = ld4(yr + c); ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
+  } else {
+    for (int c = tid; c < width; c += kNormThreads) ss += yr[c] * yr[c];
+  }
+  ss = warp_sum(ss);
+  if ((tid & 31) == 0) red[tid >> 5] = ss;
+  __syncthreads();
+  float tot = 0.f;
+#pragma unroll
+  for (int w = 0; w < kNormWarps; ++w) tot += red[w];
+  const float inv = 1.f / sqrtf(tot / (float)width + eps);
+  if (vec) {
+    for (int c = tid * 4; c < width; c += kNormThreads * 4) {
+      float4 v = ld4(xr + c);
+      fma4(v, scale4(ld4(yr + c), inv), ld4(weight + c));
+      *reinterpret_cast<float4*>(xr + c) = v;
+      store4<T>(o + c, v);
+    }
+  } else {
+    for (int c = tid; c < width; c += kNormThreads) {
+      const float v = xr[c] + yr[c] * inv * weight[c];
+      xr[c] = v;
+      o[c] = from_f<T>(v);
+    }
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) gelu_table_kernel(const T* __restrict__ gate, const int64_t* __restrict__ ids, const T* __restrict__ table,
+                                                         int64_t table_stride, T* __restrict__ out, int64_t tokens, int dim) {
+  grid_launch_dependents();
+  grid_dependency_wait();
+  const int64_t total = tokens * (int64_t)dim;
+  for (int64_t e = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; e < total; e += (int64_t)gridDim.x * blockDim.x) {
+    const int64_t t = e / dim, i = e - t * dim;
+    out[e] = from_f<T>(gelu_tanh_f(to_f(gate[e])) * to_f(table[ids[t] * table_stride + i]));
+  }
+}
+
+template <typename T, typename Y>
+static int launch_group_norm(float* x, const int64_t* rows, const void* y, int64_t terms, float alpha, const float* weight, void* out, int64_t n,
+                             int64_t width, int64_t groups, float eps, int write_x, cudaStream_t st) {
+  const int pieces = groups >= kNormWarps ? 1 : (int)((kNormWarps + groups - 1) / groups);
+  const size_t smem = ((size_t)(width + 3) / 4 * 4 + (size_t)groups * pieces) * sizeof(float);
+  if (smem > 200 * 1024) return NQB200_ERR_TOO_LARGE;
+  if (smem > 48 * 1024 && cudaFuncSetAttribute(group_norm_kernel<T, Y>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+    cudaGetLastError();
+    return NQB200_ERR_LAUNCH;
+  }
+  return launch_overlapped(group_norm_kernel<T, Y>, dim3((unsigned)n), dim3(kNormThreads), smem, st, x, rows, (const Y*)y, (int)terms, alpha, weight,
+                           (T*)out, (int)width, (int)groups, pieces, eps, write_x);
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256) clamped_glu_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int64_t tokens, int ff,
                                                           float limit) {
@@ -315,6 +455,67 @@ extern "C" int nqb200_rmsnorm_rows(const float* x, const int64_t* rows, const fl
   if (dtype == NQB200_F32)
     return launch_overlapped(rmsnorm_rows_kernel<float>, grid, block, 0, (cudaStream_t)stream, x, rows, weight, (float*)out, (int)width, eps);
   return launch_overlapped(rmsnorm_rows_kernel<bf16>, grid, block, 0, (cudaStream_t)stream, x, rows, weight, (bf16*)out, (int)width, eps);
+}
+
+static int group_norm_shape(int64_t n, int64_t width, int64_t groups, int dtype) {
+  if (n < 0 || width <= 0 || n > INT32_MAX || width > INT32_MAX || groups <= 0 || width % groups != 0) return NQB200_ERR_BAD_SHAPE;
+  return mixer_dtype(dtype) ? NQB200_OK : NQB200_ERR_BAD_DTYPE;
+}
+
+extern "C" int nqb200_group_norm_rows(const float* x, const int64_t* rows, const float* weight, void* out, int64_t n_rows, int64_t width, int64_t groups,
+                                      float eps, int dtype, void* stream) {
+  const int s = group_norm_shape(n_rows, width, groups, dtype);
+  if (s != NQB200_OK || n_rows == 0) return s;
+  if (!x || !weight || !out) return NQB200_ERR_NULL_POINTER;
+  if (!aligned16(x) || !aligned16(weight) || !aligned16(out)) return NQB200_ERR_MISALIGNED;
+  cudaStream_t st = (cudaStream_t)stream;
+  float* xs = const_cast<float*>(x);   // not written
+  if (dtype == NQB200_F32) return launch_group_norm<float, float>(xs, rows, nullptr, 0, 1.f, weight, out, n_rows, width, groups, eps, 0, st);
+  return launch_group_norm<bf16, float>(xs, rows, nullptr, 0, 1.f, weight, out, n_rows, width, groups, eps, 0, st);
+}
+
+extern "C" int nqb200_post_norm(float* x, const void* y, int y_dtype, int64_t terms, float alpha, const float* weight, void* h, int64_t tokens,
+                                int64_t width, int64_t groups, float eps, int dtype, void* stream) {
+  const int s = group_norm_shape(tokens, width, groups, dtype);
+  if (s != NQB200_OK) return s;
+  if (terms < 0 || terms > INT32_MAX) return NQB200_ERR_BAD_SHAPE;
+  if (!mixer_dtype(y_dtype)) return NQB200_ERR_BAD_DTYPE;
+  if (tokens == 0) return NQB200_OK;
+  if (!x || !weight || !h || (terms > 0 && !y)) return NQB200_ERR_NULL_POINTER;
+  if (!aligned16(x) || !aligned16(weight) || !aligned16(h) || !aligned16(y)) return NQB200_ERR_MISALIGNED;
+  cudaStream_t st = (cudaStream_t)stream;
+  if (dtype == NQB200_F32)
+    return y_dtype == NQB200_F32 ? launch_group_norm<float, float>(x, nullptr, y, terms, alpha, weight, h, tokens, width, groups, eps, 1, st)
+                                 : launch_group_norm<float, bf16>(x, nullptr, y, terms, alpha, weight, h, tokens, width, groups, eps, 1, st);
+  return y_dtype == NQB200_F32 ? launch_group_norm<bf16, float>(x, nullptr, y, terms, alpha, weight, h, tokens, width, groups, eps, 1, st)
+                               : launch_group_norm<bf16, bf16>(x, nullptr, y, terms, alpha, weight, h, tokens, width, groups, eps, 1, st);
+}
+
+extern "C" int nqb200_gelu_table(const void* gate, const int64_t* ids, const void* table, int64_t table_stride, int64_t column, void* out, int64_t tokens,
+                                 int64_t dim, int dtype, void* stream) {
+  if (tokens < 0 || dim <= 0 || dim > INT32_MAX || column < 0 || table_stride < column + dim) return NQB200_ERR_BAD_SHAPE;
+  if (!mixer_dtype(dtype)) return NQB200_ERR_BAD_DTYPE;
+  if (tokens == 0) return NQB200_OK;
+  if (!gate || !ids || !table || !out) return NQB200_ERR_NULL_POINTER;
+  const int64_t want = (tokens * dim + 255) / 256;
+  const dim3 grid((unsigned)(want < (int64_t)kNumSMs * 16 ? want : (int64_t)kNumSMs * 16)), block(256);
+  if (dtype == NQB200_F32)
+    return launch_overlapped(gelu_table_kernel<float>, grid, block, 0, (cudaStream_t)stream, (const float*)gate, ids, (const float*)table + column,
+                             table_stride, (float*)out, tokens, (int)dim);
+  return launch_overlapped(gelu_table_kernel<bf16>, grid, block, 0, (cudaStream_t)stream, (const bf16*)gate, ids, (const bf16*)table + column, table_stride,
+                           (bf16*)out, tokens, (int)dim);
+}
+
+extern "C" int nqb200_add_normed(float* x, const float* y, const float* weight, void* h, int64_t tokens, int64_t width, float eps, int dtype,
+                                 void* stream) {
+  const int s = group_norm_shape(tokens, width, 1, dtype);
+  if (s != NQB200_OK || tokens == 0) return s;
+  if (!x || !y || !weight || !h) return NQB200_ERR_NULL_POINTER;
+  if (!aligned16(x) || !aligned16(y) || !aligned16(weight) || !aligned16(h)) return NQB200_ERR_MISALIGNED;
+  const dim3 grid((unsigned)tokens), block(kNormThreads);
+  if (dtype == NQB200_F32)
+    return launch_overlapped(add_normed_kernel<float>, grid, block, 0, (cudaStream_t)stream, x, y, weight, (float*)h, (int)width, eps);
+  return launch_overlapped(add_normed_kernel<bf16>, grid, block, 0, (cudaStream_t)stream, x, y, weight, (bf16*)h, (int)width, eps);
 }
 
 extern "C" int nqb200_rmsnorm_conv(const float* x, const float* weight, const float* conv, float* state, void* out,

@@ -10,7 +10,8 @@ constexpr int kRetCols = 32, kRetGroups = 8, kRetTokens = 16;
 // group, group + 8, ... of its column of S in registers.
 template <typename T, int DPT>
 __global__ void __launch_bounds__(kRetCols* kRetGroups) retention_simple_kernel(const T* __restrict__ proj, int64_t stride, int q_off, int k_off,
-                                                                                int v_off, const float* __restrict__ decay, float* state,
+                                                                                int v_off, const float* __restrict__ decay,
+                                                                                const float* __restrict__ log_decay, float* state,
                                                                                 float* __restrict__ o, int heads, int dim, int vdim,
                                                                                 const nqb200_batch bt) {
   extern __shared__ float sm[];
@@ -18,6 +19,7 @@ __global__ void __launch_bounds__(kRetCols* kRetGroups) retention_simple_kernel(
   float* ks = qs + kRetTokens * dim;            // [tokens][dim], scaled
   float* vs = ks + kRetTokens * dim;            // [tokens][cols]
   float* part = vs + kRetTokens * kRetCols;     // [tokens][groups][cols]
+  float* ds = part + kRetTokens * kRetGroups * kRetCols;   // [tokens][dim] decays, where every channel has its own
   grid_launch_dependents();
   grid_dependency_wait();
   const int b = blockIdx.z, h = blockIdx.y, col = threadIdx.x % kRetCols, grp = threadIdx.x / kRetCols, tid = threadIdx.x;
@@ -25,7 +27,7 @@ __global__ void __launch_bounds__(kRetCols* kRetGroups) retention_simple_kernel(
   if (n <= 0) return;
   float* st = state + ((size_t)bt.slot[b] * heads + h) * dim * vdim;
   const bool live = c < vdim, fresh = bt.pos0[b] == 0;
-  const float d = decay[h], kscale = 1.f / sqrtf((float)dim);
+  const float d = log_decay ? 0.f : decay[h], kscale = 1.f / sqrtf((float)dim);
   float S[DPT];
 #pragma unroll
   for (int r = 0; r < DPT; ++r) {
@@ -40,6 +42,7 @@ __global__ void __launch_bounds__(kRetCols* kRetGroups) retention_simple_kernel(
       const T* row = proj + (size_t)(t0 + base + i) * stride + (size_t)h * dim + r;
       qs[e] = to_f(row[q_off]);
       ks[e] = to_f(row[k_off]) * kscale;
+      if (log_decay) ds[e] = expf(log_decay[((size_t)(t0 + base + i) * heads + h) * dim + r]);
     }
     for (int e = tid; e < cnt * kRetCols; e += blockDim.x) {
       const int i = e / kRetCols, cc = blockIdx.x * kRetCols + e % kRetCols;
@@ -53,7 +56,7 @@ __global__ void __launch_bounds__(kRetCols* kRetGroups) retention_simple_kernel(
       for (int r = 0; r < DPT; ++r) {
         const int row = r * kRetGroups + grp;
         if (row < dim) {
-          S[r] = d * S[r] + ks[i * dim + row] * v;
+          S[r] = (log_decay ? ds[i * dim + row] : d) * S[r] + ks[i * dim + row] * v;
           acc += S[r] * qs[i * dim + row];
         }
       }
@@ -81,7 +84,7 @@ __global__ void __launch_bounds__(kRetCols* kRetGroups) retention_simple_kernel(
 // One warp per (token, head).
 template <typename T>
 __global__ void __launch_bounds__(256) head_norm_gate_kernel(const float* __restrict__ o, const T* __restrict__ gate, int64_t gate_stride,
-                                                             T* __restrict__ out, int64_t out_stride, int64_t pairs, int heads, int vdim,
+                                                             const float* __restrict__ weight, T* __restrict__ out, int64_t out_stride, int64_t pairs, int heads, int vdim,
                                                              float eps, float out_scale) {
   grid_launch_dependents();
   grid_dependency_wait();
@@ -95,8 +98,37 @@ __global__ void __launch_bounds__(256) head_norm_gate_kernel(const float* __rest
   const float inv = out_scale / sqrtf(warp_sum(ss) / (float)vdim + eps);
   for (int c = lane; c < vdim; c += 32) {
     const float g = to_f(gate[t * gate_stride + (int64_t)h * vdim + c]);
-    out[t * out_stride + (int64_t)h * vdim + c] = from_f<T>(row[c] * inv * (g * sigmoid_f(g)));
+    out[t * out_stride + (int64_t)h * vdim + c] = from_f<T>(row[c] * inv * (weight ? weight[c] : 1.f) * (g * sigmoid_f(g)));
   }
+}
+
+// A thread per channel and 16 tokens: log of the decays, from the gate's low-rank projection.
+constexpr int kDecayTokens = 16;
+template <typename T>
+__global__ void __launch_bounds__(256) gla_log_decay_kernel(const T* __restrict__ low, int64_t low_stride, const T* __restrict__ a2,
+                                                            const float* __restrict__ bias, float* __restrict__ out, int64_t tokens, int channels,
+                                                            int rank, float inv_tau) {
+  extern __shared__ float low_s[];   // [kDecayTokens][rank]
+  grid_launch_dependents();
+  grid_dependency_wait();
+  const int64_t t0 = (int64_t)blockIdx.y * kDecayTokens;
+  const int cnt = (int)min((int64_t)kDecayTokens, tokens - t0);
+  for (int e = threadIdx.x; e < cnt * rank; e += 256) low_s[e] = to_f(low[(t0 + e / rank) * low_stride + e % rank]);
+  __syncthreads();
+  const int c = blockIdx.x * 256 + threadIdx.x;
+  if (c >= channels) return;
+  float z[kDecayTokens];
+  const float b = bias[c];
+#pragma unroll
+  for (int i = 0; i < kDecayTokens; ++i) z[i] = 0.f;
+  for (int r = 0; r < rank; ++r) {
+    const float w = to_f(a2[(size_t)c * rank + r]);
+#pragma unroll
+    for (int i = 0; i < kDecayTokens; ++i) z[i] += w * (i < cnt ? low_s[i * rank + r] : 0.f);
+  }
+#pragma unroll
+  for (int i = 0; i < kDecayTokens; ++i)
+    if (i < cnt) out[(t0 + i) * channels + c] = log_sigmoid_f(z[i] + b) * inv_tau;
 }
 
 constexpr int kGruSegs = 32, kGruCols = 32, kGruLen = 4;  // 128 tokens per pass
@@ -299,30 +331,30 @@ static int mingru_chunked(const void* proj, void* out, const GruArgs& p, cudaStr
 }
 
 template <typename T, int DPT>
-static int retention_simple(const void* proj, int64_t stride, int64_t q_off, int64_t k_off, int64_t v_off, const float* decay, float* state,
-                            float* o, int64_t heads, int64_t dim, int64_t vdim, const nqb200_batch* b, cudaStream_t st) {
+static int retention_simple(const void* proj, int64_t stride, int64_t q_off, int64_t k_off, int64_t v_off, const float* decay,
+                            const float* log_decay, float* state, float* o, int64_t heads, int64_t dim, int64_t vdim, const nqb200_batch* b, cudaStream_t st) {
   const dim3 grid((unsigned)((vdim + kRetCols - 1) / kRetCols), (unsigned)heads, (unsigned)b->batch), block(kRetCols * kRetGroups);
-  const size_t smem = (size_t)kRetTokens * (2 * dim + kRetCols + kRetGroups * kRetCols) * sizeof(float);
+  const size_t smem = (size_t)kRetTokens * ((log_decay ? 3 : 2) * dim + kRetCols + kRetGroups * kRetCols) * sizeof(float);
   if (smem > 48 * 1024 &&
       cudaFuncSetAttribute(retention_simple_kernel<T, DPT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
     cudaGetLastError();
     return NQB200_ERR_LAUNCH;
   }
   return launch_overlapped(retention_simple_kernel<T, DPT>, grid, block, smem, st, (const T*)proj, stride, (int)q_off, (int)k_off, (int)v_off,
-                           decay, state, o, (int)heads, (int)dim, (int)vdim, *b);
+                           decay, log_decay, state, o, (int)heads, (int)dim, (int)vdim, *b);
 }
 
 extern "C" int nqb200_retention(const void* proj, int64_t stride, int64_t q_off, int64_t k_off, int64_t v_off, const float* decay,
-                                float* state, float* o, int64_t heads, int64_t dim, int64_t vdim, const nqb200_batch* b, int dtype,
+                                const float* log_decay, float* state, float* o, int64_t heads, int64_t dim, int64_t vdim, const nqb200_batch* b, int dtype,
                                 void* stream) {
   const int s = check_batch(b, false);
   if (s != NQB200_OK) return s;
   if (heads <= 0 || heads > 65535 || dim <= 0 || dim > 1024 || vdim <= 0 || stride <= 0) return NQB200_ERR_BAD_SHAPE;
   if (!mixer_dtype(dtype)) return NQB200_ERR_BAD_DTYPE;
   if (b->tokens == 0) return NQB200_OK;
-  if (!proj || !decay || !state || !o) return NQB200_ERR_NULL_POINTER;
+  if (!proj || (!decay && !log_decay) || !state || !o) return NQB200_ERR_NULL_POINTER;
   cudaStream_t st = (cudaStream_t)stream;
-#define NQB200_RET(T, D) return retention_simple<T, D>(proj, stride, q_off, k_off, v_off, decay, state, o, heads, dim, vdim, b, st)
+#define NQB200_RET(T, D) return retention_simple<T, D>(proj, stride, q_off, k_off, v_off, decay, log_decay, state, o, heads, dim, vdim, b, st)
 #define NQB200_RET_T(T)                                                                                       \
   do {                                                                                                        \
     if (dim <= 64) NQB200_RET(T, 8);                                                                          \
@@ -337,7 +369,24 @@ extern "C" int nqb200_retention(const void* proj, int64_t stride, int64_t q_off,
 #undef NQB200_RET
 }
 
-extern "C" int nqb200_head_norm_gate(const float* o, const void* gate, int64_t gate_stride, void* out, int64_t out_stride, int64_t tokens,
+extern "C" int nqb200_gla_log_decay(const void* low, int64_t low_stride, const void* a2, const float* bias, float* log_decay, int64_t tokens,
+                                    int64_t channels, int64_t rank, float tau, int dtype, void* stream) {
+  if (tokens < 0 || channels <= 0 || channels > INT32_MAX || rank <= 0 || rank > 512 || low_stride < rank || !(tau > 0.f)) return NQB200_ERR_BAD_SHAPE;
+  if (!mixer_dtype(dtype)) return NQB200_ERR_BAD_DTYPE;
+  if (tokens == 0) return NQB200_OK;
+  if (!low || !a2 || !bias || !log_decay) return NQB200_ERR_NULL_POINTER;
+  const int64_t ty = (tokens + kDecayTokens - 1) / kDecayTokens;
+  if (ty > 65535) return NQB200_ERR_TOO_LARGE;
+  const dim3 grid((unsigned)((channels + 255) / 256), (unsigned)ty), block(256);
+  const size_t smem = (size_t)kDecayTokens * rank * sizeof(float);
+  if (dtype == NQB200_F32)
+    return launch_overlapped(gla_log_decay_kernel<float>, grid, block, smem, (cudaStream_t)stream, (const float*)low, low_stride, (const float*)a2, bias,
+                             log_decay, tokens, (int)channels, (int)rank, 1.f / tau);
+  return launch_overlapped(gla_log_decay_kernel<bf16>, grid, block, smem, (cudaStream_t)stream, (const bf16*)low, low_stride, (const bf16*)a2, bias,
+                           log_decay, tokens, (int)channels, (int)rank, 1.f / tau);
+}
+
+extern "C" int nqb200_head_norm_gate(const float* o, const void* gate, int64_t gate_stride, const float* weight, void* out, int64_t out_stride, int64_t tokens,
                                      int64_t heads, int64_t vdim, float eps, float out_scale, int dtype, void* stream) {
   if (tokens < 0 || heads <= 0 || vdim <= 0) return NQB200_ERR_BAD_SHAPE;
   if (!mixer_dtype(dtype)) return NQB200_ERR_BAD_DTYPE;
@@ -346,9 +395,9 @@ extern "C" int nqb200_head_norm_gate(const float* o, const void* gate, int64_t g
   const int64_t pairs = tokens * heads;
   const dim3 grid((unsigned)((pairs + 7) / 8)), block(256);
   if (dtype == NQB200_F32)
-    return launch_overlapped(head_norm_gate_kernel<float>, grid, block, 0, (cudaStream_t)stream, o, (const float*)gate, gate_stride, (float*)out,
+    return launch_overlapped(head_norm_gate_kernel<float>, grid, block, 0, (cudaStream_t)stream, o, (const float*)gate, gate_stride, weight, (float*)out,
                              out_stride, pairs, (int)heads, (int)vdim, eps, out_scale);
-  return launch_overlapped(head_norm_gate_kernel<bf16>, grid, block, 0, (cudaStream_t)stream, o, (const bf16*)gate, gate_stride, (bf16*)out,
+  return launch_overlapped(head_norm_gate_kernel<bf16>, grid, block, 0, (cudaStream_t)stream, o, (const bf16*)gate, gate_stride, weight, (bf16*)out,
                            out_stride, pairs, (int)heads, (int)vdim, eps, out_scale);
 }
 

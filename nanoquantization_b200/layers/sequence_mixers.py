@@ -17,11 +17,17 @@ import torch.nn as nn
 from .. import _lib
 from ..engine.batch import KVSpec
 from . import mixers as ops
+from . import moe
 
 
 def _buffer(module: nn.Module, name: str, *shape, dtype, device) -> torch.Tensor:
     module.register_buffer(name, torch.zeros(*shape, dtype=dtype, device=device), persistent=False)
     return getattr(module, name)
+
+
+def _inverse_frequencies(base, dims, device):
+    i = torch.arange(dims // 2, dtype=torch.float64)
+    return (float(base) ** (-2.0 * i / max(dims, 1))).float().to(device)
 
 
 class AttentionMixer(nn.Module):
@@ -38,8 +44,7 @@ class AttentionMixer(nn.Module):
         self.in_parts = [("q", heads * dim), ("k", kv_heads * dim), ("v", kv_heads * vdim)]
         self.out_columns = heads * vdim
         _buffer(self, "sink", heads, dtype=torch.float32, device=device)
-        i = torch.arange(rot_dims // 2, dtype=torch.float64)
-        self.register_buffer("inv_freq", (float(rot_base) ** (-2.0 * i / max(rot_dims, 1))).float().to(device), persistent=False)
+        self.register_buffer("inv_freq", _inverse_frequencies(rot_base, rot_dims, device), persistent=False)
 
     def kv_spec(self):
         return KVSpec(self.kv_heads, self.dim, self.vdim, self.chunk)
@@ -52,7 +57,7 @@ class AttentionMixer(nn.Module):
 
     def desc(self) -> _lib.AttentionDesc:
         return _lib.AttentionDesc(self.heads, self.kv_heads, self.dim, self.vdim, self.chunk, self.scale, self.softcap,
-                                  self.sink.data_ptr(), self.out_scale)
+                                  self.sink.data_ptr(), self.out_scale, None, None, 0)
 
     def mix(self, proj, col, act, act_col, layer_step):
         q_off, k_off, v_off = col, col + self.heads * self.dim, col + (self.heads + self.kv_heads) * self.dim
@@ -61,17 +66,62 @@ class AttentionMixer(nn.Module):
                             self.desc(), layer_step.batch)
 
 
-class RetentionMixer(nn.Module):
-    """Linear attention with one fixed decay per head; each head's output is RMS-normalised and gated."""
+class SigmoidAttentionMixer(nn.Module):
+    """Grouped-query attention whose weights are sigmoids of the scores (plus a number per head), not normalised over the
+    keys.  Queries and keys are RMS-normed per head and partially rotated; the values are the keys as projected."""
 
-    def __init__(self, *, heads, dim, vdim, decay, eps, out_scale=1.0, device="cpu"):
+    def __init__(self, *, heads, kv_heads, dim, rot_base, rot_dims, interleaved, scale, eps, out_scale=1.0, device="cpu"):
         super().__init__()
+        if heads % kv_heads != 0 or rot_dims % 2 != 0 or not 0 <= rot_dims <= dim:
+            raise ValueError(f"attention: {heads} heads over {kv_heads} key/value heads, {rot_dims} of {dim} dimensions rotated")
+        self.heads, self.kv_heads, self.dim, self.vdim, self.rot = heads, kv_heads, dim, dim, rot_dims
+        self.scale, self.eps, self.out_scale, self.interleaved = float(scale), float(eps), float(out_scale), bool(interleaved)
+        self.in_parts = [("q", heads * dim), ("k", kv_heads * dim)]
+        self.out_columns = heads * dim
+        for name, n in (("q_norm", dim), ("k_norm", dim), ("temp", heads), ("bias", heads)):
+            _buffer(self, name, n, dtype=torch.float32, device=device)
+        self.register_buffer("inv_freq", _inverse_frequencies(rot_base, rot_dims, device), persistent=False)
+
+    def kv_spec(self):
+        return KVSpec(self.kv_heads, self.dim, self.vdim)
+
+    def state_shapes(self):
+        return {}
+
+    def checkpoint(self, prefix):
+        return {prefix + "q.norm": self.q_norm, prefix + "k.norm": self.k_norm, prefix + "temp": self.temp, prefix + "pb": self.bias}
+
+    def desc(self) -> _lib.AttentionDesc:
+        return _lib.AttentionDesc(self.heads, self.kv_heads, self.dim, self.vdim, 0, self.scale, 0.0, None, self.out_scale, self.temp.data_ptr(),
+                                  self.bias.data_ptr(), 1)
+
+    def rope_desc(self) -> _lib.RopeDesc:
+        return _lib.RopeDesc(self.heads, self.kv_heads, self.dim, self.vdim, self.rot, int(self.interleaved), self.inv_freq.data_ptr(),
+                             self.q_norm.data_ptr(), self.k_norm.data_ptr(), self.eps)
+
+    def mix(self, proj, col, act, act_col, layer_step):
+        q_off, k_off = col, col + self.heads * self.dim
+        ops.norm_rope(proj, layer_step.k_cache, layer_step.v_cache, self.rope_desc(), layer_step.batch, q_off, k_off, k_off)
+        ops.chunk_attention(proj[:, q_off:k_off], layer_step.k_cache, layer_step.v_cache, act[:, act_col:act_col + self.out_columns],
+                            self.desc(), layer_step.batch)
+
+
+class RetentionMixer(nn.Module):
+    """Linear attention with one fixed decay per head, queries and keys rotated where ``rot_dims`` says so (pairs i, i +
+    rot_dims / 2); each head's output is RMS-normalised and gated."""
+
+    def __init__(self, *, heads, dim, vdim, decay, eps, out_scale=1.0, rot_base=1.0, rot_dims=0, device="cpu"):
+        super().__init__()
+        if rot_dims % 2 != 0 or not 0 <= rot_dims <= dim:
+            raise ValueError(f"retention: {rot_dims} of {dim} dimensions rotated")
         if len(decay) != heads:
             raise ValueError(f"retention: {len(decay)} decays for {heads} heads")
         self.heads, self.dim, self.vdim, self.eps, self.out_scale = heads, dim, vdim, float(eps), float(out_scale)
         self.in_parts = [("q", heads * dim), ("k", heads * dim), ("v", heads * vdim), ("g", heads * vdim)]
         self.out_columns = heads * vdim
+        self.rot = rot_dims
         self.register_buffer("decay", torch.tensor(decay, dtype=torch.float64).float().to(device), persistent=False)
+        self.register_buffer("inv_freq", _inverse_frequencies(rot_base, rot_dims, device), persistent=False)
 
     def kv_spec(self):
         return None
@@ -85,16 +135,51 @@ class RetentionMixer(nn.Module):
     def desc(self) -> _lib.RetentionDesc:
         return _lib.RetentionDesc(self.heads, self.dim, self.vdim, self.eps, self.out_scale, self.decay.data_ptr())
 
+    def rope_desc(self) -> _lib.RopeDesc:
+        return _lib.RopeDesc(self.heads, self.heads, self.dim, self.vdim, self.rot, 0, self.inv_freq.data_ptr(), None, None, 0.0)
+
     def mix(self, proj, col, act, act_col, layer_step):
+        if self.rot > 0:
+            ops.norm_rope(proj, None, None, self.rope_desc(), layer_step.batch, col, col + self.heads * self.dim, 0)
         ops.retention_gated(proj, col, self.desc(), self.decay, layer_step.state["retention"], act, act_col, layer_step.batch)
 
 
-class ParallelMixer(nn.Module):
-    """Mixers side by side on the same input, their (scaled) outputs summed: one merged product in, one out."""
+class GatedLinearMixer(nn.Module):
+    """Gated linear attention: a decay per key channel and token, sigmoid(z)^(1 / tau) with z a low-rank projection of the
+    input; each head's output is RMS-normalised with a weight and gated."""
 
-    def __init__(self, width: int, parts: dict, *, dtype, device="cpu"):
+    def __init__(self, *, heads, dim, vdim, rank, tau, eps, out_scale=1.0, dtype=torch.bfloat16, device="cpu"):
         super().__init__()
-        self.parts = nn.ModuleDict(parts)
+        if tau <= 0:
+            raise ValueError(f"gated linear attention: tau {tau} must be positive")
+        self.heads, self.dim, self.vdim, self.rank = heads, dim, vdim, rank
+        self.tau, self.eps, self.out_scale = float(tau), float(eps), float(out_scale)
+        self.in_parts = [("q", heads * dim), ("k", heads * dim), ("v", heads * vdim), ("g", heads * vdim), ("a1", rank)]
+        self.out_columns = heads * vdim
+        _buffer(self, "a2", heads * dim, rank, dtype=dtype, device=device)
+        _buffer(self, "a2_bias", heads * dim, dtype=torch.float32, device=device)
+        _buffer(self, "norm", vdim, dtype=torch.float32, device=device)
+
+    def kv_spec(self):
+        return None
+
+    def state_shapes(self):
+        return {"gla": (self.heads, self.dim, self.vdim)}
+
+    def checkpoint(self, prefix):
+        return {prefix + "a2": self.a2, prefix + "a2.b": self.a2_bias, prefix + "norm": self.norm}
+
+    def mix(self, proj, col, act, act_col, layer_step):
+        ops.gla_gated(proj, col, self, layer_step.state["gla"], act, act_col, layer_step.batch)
+
+
+class ParallelMixer(nn.Module):
+    """Mixers side by side on the same input, their (scaled) outputs summed: one merged product in, one out.  ``beta``
+    scales the stream that the sum is added to; ``prefixes`` names a part's tensors where they do not start with its name."""
+
+    def __init__(self, width: int, parts: dict, *, dtype, device="cpu", beta=1.0, prefixes=None):
+        super().__init__()
+        self.parts, self.beta, self.prefixes = nn.ModuleDict(parts), float(beta), prefixes or {k: k + "." for k in parts}
         self.rows = sum(n for m in parts.values() for _, n in m.in_parts)
         self.columns = sum(m.out_columns for m in parts.values())
         _buffer(self, "w_in", self.rows, width, dtype=dtype, device=device)
@@ -116,6 +201,7 @@ class ParallelMixer(nn.Module):
             return False
         if self._at_once is None:
             self._at_once = (len(self.parts) == (self._attention is not None) + (self._retention is not None)
+                             and not (self._retention and self._retention[0].rot)
                              and ops.mixer_decode_supported(self._attention and self._attention[0].desc(),
                                                             self._retention and self._retention[0].desc()))
         return self._at_once
@@ -132,7 +218,7 @@ class ParallelMixer(nn.Module):
     def checkpoint(self, prefix):
         out, row, col = {}, 0, 0
         for name, m in self.parts.items():
-            p = f"{prefix}{name}."
+            p = prefix + self.prefixes[name]
             for part, n in m.in_parts:
                 out[p + part] = self.w_in[row:row + n]
                 row += n
@@ -142,21 +228,21 @@ class ParallelMixer(nn.Module):
         return out
 
     def forward(self, x, h, layer_step):
-        """``x += mixer(h)`` on the float32 stream."""
+        """``x = beta * x + mixer(h)`` on the float32 stream."""
         proj = ops.linear(h, self.w_in)
         act = torch.empty(h.shape[0], self.columns, dtype=h.dtype, device=h.device)
         if self._decodes_at_once(h, layer_step.batch):
             att, ret = self._attention, self._retention
             ops.mixer_decode(proj, act, att and (att[0].desc(), att[0].inv_freq, att[1], att[2], layer_step.k_cache, layer_step.v_cache),
                              ret and (ret[0].desc(), ret[1], ret[2], layer_step.state["retention"]), layer_step.batch)
-            ops.linear_residual_(x, act, self.w_out)
+            ops.linear_residual_(x, act, self.w_out, self.beta)
             return
         row = col = 0
         for m in self.parts.values():
             m.mix(proj, row, act, col, layer_step)
             row += sum(n for _, n in m.in_parts)
             col += m.out_columns
-        ops.linear_residual_(x, act, self.w_out)
+        ops.linear_residual_(x, act, self.w_out, self.beta)
 
 
 class MinGRUMixer(nn.Module):
@@ -208,6 +294,71 @@ class ClampedGLU(nn.Module):
             ops.linear_residual_(x, ops.dense_glu(h, self.w_in, self.limit), self.w_out)
             return
         ops.linear_residual_(x, ops.clamped_glu(ops.linear(h, self.w_in), self.limit), self.w_out)
+
+
+class RoutedExperts(nn.Module):
+    """Feed-forward of many small experts ``down(gelu(up h))``, of which each token uses ``top``, chosen by sigmoid scores
+    plus a correction among the best groups of neighbouring experts."""
+
+    def __init__(self, width: int, ff: int, *, experts, top, groups, keep, scale, dtype, device="cpu"):
+        super().__init__()
+        if groups < 1 or experts % groups != 0 or not 1 <= keep <= groups or not 1 <= top <= keep * (experts // groups):
+            raise ValueError(f"experts: {top} of {experts} from {keep} of {groups} groups")
+        self.experts, self.top, self.groups, self.keep, self.scale = experts, top, groups, keep, float(scale)
+        _buffer(self, "router", experts, width, dtype=dtype, device=device)
+        _buffer(self, "correction", experts, dtype=torch.float32, device=device)
+        _buffer(self, "up", experts, ff, width, dtype=dtype, device=device)
+        _buffer(self, "down", experts, width, ff, dtype=dtype, device=device)
+
+    def checkpoint(self, prefix):
+        out = {prefix + "router": self.router, prefix + "correction": self.correction}
+        for e in range(self.experts):
+            out.update({f"{prefix}e{e}.up": self.up[e], f"{prefix}e{e}.down": self.down[e]})
+        return out
+
+    def router_desc(self) -> _lib.RouterDesc:
+        return _lib.RouterDesc(self.experts, self.top, self.groups, self.keep, self.scale, self.correction.data_ptr())
+
+    def forward(self, h):
+        """The weighted outputs of every token's experts, ``[tokens, top, width]``; the caller adds them up."""
+        plan = moe.route(ops.linear(h, self.router, torch.float32), self.router_desc())
+        return moe.experts_down(moe.experts_up(h, self.up, plan), self.down, plan)
+
+
+class GroupNorm(nn.Module):
+    """RMS norm in groups after the residual sum: ``x = norm(alpha x + y)`` on the stream, and its rounding for what reads it."""
+
+    def __init__(self, width: int, groups: int, eps: float, *, dtype, device="cpu"):
+        super().__init__()
+        if groups < 1 or width % groups != 0:
+            raise ValueError(f"norm: {width} in {groups} groups")
+        self.groups, self.eps, self.dtype = groups, float(eps), dtype
+        _buffer(self, "weight", width, dtype=torch.float32, device=device)
+
+    def rows(self, x, rows):
+        return ops.group_norm_rows(x, rows, self.weight, self.groups, self.eps, self.dtype)
+
+    def forward(self, x, y=None, alpha=1.0):
+        return ops.post_norm_(x, y, alpha, self.weight, self.groups, self.eps, self.dtype)
+
+
+class TokenSideInput(nn.Module):
+    """What a layer adds per token: ``x += rmsnorm(proj(gelu_tanh(gate x) * e))``, e a slice of the token's row in a table
+    that all layers share."""
+
+    def __init__(self, width: int, dim: int, column: int, eps: float, *, dtype, device="cpu"):
+        super().__init__()
+        self.dim, self.column, self.eps = dim, column, float(eps)
+        _buffer(self, "gate", dim, width, dtype=dtype, device=device)
+        _buffer(self, "proj", width, dim, dtype=dtype, device=device)
+        _buffer(self, "norm", width, dtype=torch.float32, device=device)
+
+    def checkpoint(self, prefix):
+        return {prefix + "gate": self.gate, prefix + "proj": self.proj, prefix + "norm": self.norm}
+
+    def forward(self, x, h, tokens, table):
+        g = ops.linear_gelu_table(h, self.gate, tokens, table, self.column)
+        return ops.add_normed_(x, ops.linear(g, self.proj, torch.float32), self.norm, self.eps, h.dtype)
 
 
 class ConvNorm(nn.Module):

@@ -4,13 +4,14 @@ from __future__ import annotations
 import json
 import os
 from dataclasses import dataclass
-from typing import Callable
+from typing import Callable, Optional
 
 import torch
 
-from ..utils.loader import load_model
+from ..utils.loader import load_model, tensor_shapes
 from .qwen3_quantized import Qwen3Config, Qwen3QuantizedForCausalLM
 from .vemedra import VemedraConfig, VemedraForCausalLM
+from .verozen import VerozenConfig, VerozenForCausalLM
 
 
 @dataclass(frozen=True)
@@ -20,11 +21,15 @@ class ModelEntry:
     dtypes: tuple                           # what the model's kernels run in
     libraries: tuple                        # kernel libraries it needs (names in csrc.build)
     prepare: Callable[[torch.nn.Module], None] = lambda model: None   # after loading
+    # config.json and {tensor name: shape} -> config.json with the sizes that only the tensors give
+    complete: Optional[Callable[[dict, dict], dict]] = None
 
 
 MODELS: dict[str, ModelEntry] = {
     "Qwen3ForCausalLM": ModelEntry(Qwen3Config.from_dict, Qwen3QuantizedForCausalLM.from_config, (torch.bfloat16, torch.float16),
                                    ("LIB_PATH",), lambda model: model.fuse_projections()),
+    "Verozen": ModelEntry(VerozenConfig.from_dict, VerozenForCausalLM, (torch.bfloat16, torch.float32), ("MIXERS_PATH", "MOE_PATH"),
+                          complete=VerozenConfig.complete),
     "Vemedra": ModelEntry(VemedraConfig.from_dict, VemedraForCausalLM, (torch.bfloat16, torch.float32), ("MIXERS_PATH",)),
 }
 
@@ -48,6 +53,8 @@ def build_model(path: str, *, device="cuda:0", dtype=torch.bfloat16) -> torch.nn
     entry = model_class(config)
     if dtype not in entry.dtypes:
         raise TypeError(f"this model runs in {', '.join(str(d) for d in entry.dtypes)}, not {dtype}")
+    if entry.complete is not None:
+        config = entry.complete(config, tensor_shapes(path))
     model = entry.build(entry.config(config), device=device, dtype=dtype)
     load_model(model, path)
     entry.prepare(model)

@@ -1,7 +1,7 @@
 """Checkpoint reader and writer.
 
-A model with ``checkpoint_tensors()`` names the destination of every tensor itself (Vemedra: plain linears, merged
-when loaded) and must find all of them.  What follows is the format of the quantised Qwen3 models.
+A model with ``checkpoint_tensors()`` names the destination of every tensor itself (Vemedra, Verozen: plain linears,
+merged when loaded) and must find all of them.  What follows is the format of the quantised Qwen3 models.
 
 On-disk format: the reference's (``nanoquantization/utils/loader.py:20-48`` reads
 it, ``scripts/qwen3_0pt6_billion.py:179-235`` writes it): ``*.safetensors``
@@ -66,6 +66,16 @@ def shard_slices(name: str, shape: tuple[int, ...], tp_size: int, tp_rank: int, 
     if _VOCAB.search(name):
         return (slice(*_bounds(shape[0], tp_size, tp_rank, 1, name)),) + full[1:]
     return full  # embeddings and norms are replicated
+
+
+def tensor_shapes(path: str) -> dict[str, tuple[int, ...]]:
+    """Name -> shape of every tensor of the checkpoint directory, from the files' headers."""
+    from safetensors import safe_open
+    out = {}
+    for tensor_file in sorted(glob.glob(os.path.join(path, "*.safetensors"))):
+        with safe_open(tensor_file, framework="pt", device="cpu") as f:
+            out.update({name: tuple(f.get_slice(name).get_shape()) for name in f.keys()})
+    return out
 
 
 def _destination(model: nn.Module, weight_name: str, named: Optional[dict] = None) -> torch.Tensor:
