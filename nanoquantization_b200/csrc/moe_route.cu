@@ -31,7 +31,8 @@ __device__ void route_token(const float* __restrict__ z, const nqb200_router& r,
   for (int e = lane; e < r.experts; e += 32) {
     const float v = sigmoid_f(z[e]);
     s[e] = v;
-    choice[e] = v + (r.correction ? r.correction[e] : 0.f);
+    const float c = v + (r.correction ? r.correction[e] : 0.f);
+    choice[e] = c == c ? c : -INFINITY;    // so that any two compare, and every lane ends with the same expert
   }
   __syncwarp();
   const int size = r.experts / r.groups;
@@ -44,7 +45,8 @@ __device__ void route_token(const float* __restrict__ z, const nqb200_router& r,
         const float v = choice[g * size + k];
         if (v > a) { b = a; a = v; } else if (v > b) { b = v; }
       }
-      gs[g] = size > 1 ? a + b : a;
+      const float sum = size > 1 ? a + b : a;
+      gs[g] = sum == sum ? sum : -INFINITY;
       gopen |= 1u << i;
     }
     __syncwarp();

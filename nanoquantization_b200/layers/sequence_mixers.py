@@ -227,21 +227,24 @@ class ParallelMixer(nn.Module):
             out.update(m.checkpoint(p))
         return out
 
-    def forward(self, x, h, layer_step):
-        """``x = beta * x + mixer(h)`` on the float32 stream."""
-        proj = ops.linear(h, self.w_in)
-        act = torch.empty(h.shape[0], self.columns, dtype=h.dtype, device=h.device)
-        if self._decodes_at_once(h, layer_step.batch):
+    def mix(self, proj, act, layer_step):
+        """The input product -> the operand of the output product; a decode step in one launch where its kernel takes the sizes."""
+        if self._decodes_at_once(proj, layer_step.batch):
             att, ret = self._attention, self._retention
             ops.mixer_decode(proj, act, att and (att[0].desc(), att[0].inv_freq, att[1], att[2], layer_step.k_cache, layer_step.v_cache),
                              ret and (ret[0].desc(), ret[1], ret[2], layer_step.state["retention"]), layer_step.batch)
-            ops.linear_residual_(x, act, self.w_out, self.beta)
             return
         row = col = 0
         for m in self.parts.values():
             m.mix(proj, row, act, col, layer_step)
             row += sum(n for _, n in m.in_parts)
             col += m.out_columns
+
+    def forward(self, x, h, layer_step):
+        """``x = beta * x + mixer(h)`` on the float32 stream."""
+        proj = ops.linear(h, self.w_in)
+        act = torch.empty(h.shape[0], self.columns, dtype=h.dtype, device=h.device)
+        self.mix(proj, act, layer_step)
         ops.linear_residual_(x, act, self.w_out, self.beta)
 
 

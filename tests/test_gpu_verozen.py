@@ -1,0 +1,248 @@
+"""The Verozen model through the engine on a GPU, against the plain whole-sequence oracle."""
+import json
+import os
+import subprocess
+import sys
+
+import pytest
+import torch
+
+import verozen_cases as C
+from nanoquantization_b200.engine import LLMEngine, Sequence
+from oracle.verozen_oracle import VerozenOracle
+
+pytestmark = pytest.mark.gpu
+DEV = "cuda:0"
+ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+DTYPES = [torch.float32, torch.bfloat16]
+
+CONFIGS = {
+    "small": C.config(),
+    "side-only": C.config([C.gla(2, 16, 16, 1.0, 3), C.attention(2, 1, 24, 0)], width=32, vocab=50, norm_groups=1, alpha=1.0, side_dim=16),
+    "attention-first": C.config([C.attention(8, 4, 32, 32, 1e4, 0.2, C.experts(32, 8, 2, 2, 1)), C.retention(2, 32, 32, 32, mlp=C.experts(24, 6, 3, 1, 1))],
+                                width=64, norm_groups=16, alpha=2.5),
+    "retention-only": C.config([C.retention(4, 64, 64, 64), C.retention(2, 16, 128, 4, mlp=C.experts(56, 4, 4, 2, 2, 1.0))], width=96, vocab=130, norm_groups=2, eps=1e-5),
+    "gla-only": C.config([C.gla(4, 32, 32, 16.0, 16, C.experts(48, 16, 3, 2, 1)), C.gla(2, 64, 128, 4.0, 8, C.experts(64, 5, 1, 5, 2))], width=128, norm_groups=4, side_dim=24),
+    "wide": C.config([C.gla(4, 64, 64, 16.0, 16, C.experts(128, 16, 4, 4, 2)), C.attention(4, 2, 128, 64, 1e4, 0.09, C.experts(96, 8, 2, 2, 1, 2.5)),
+                      C.retention(2, 64, 128, 64, 1e4, C.experts(128, 8, 2, 1, 1))], width=256, norm_groups=4, side_dim=32, alpha=3.0),
+}
+
+
+def prompt(n, vocab, seed=0):
+    return torch.randint(0, vocab, (n,), generator=torch.Generator().manual_seed(seed)).tolist()
+
+
+class Oracle(VerozenOracle):
+    """Also notes how close each token's choice of experts was (the smallest gap over its layers, in units of the scores)."""
+
+    def feed_forward(self, p, f, h):
+        r, size = f["router"], f["router"]["experts"] // f["router"]["groups"]["count"]
+        choice = torch.sigmoid(h @ self.w[p + "router"].T) + self.w[p + "correction"]
+        score = choice.view(len(h), -1, size).topk(min(2, size)).values.sum(-1)
+        keep, top = r["groups"]["keep"], r["top"]
+        order = score.sort(descending=True)
+        gaps = [order.values[:, keep - 1] - order.values[:, keep]] if keep < score.shape[1] else []
+        allowed = torch.zeros_like(score, dtype=torch.bool).scatter(1, order.indices[:, :keep], True).repeat_interleave(size, 1)
+        best = choice.masked_fill(~allowed, float("-inf")).sort(descending=True).values
+        if top < choice.shape[1]:
+            gaps.append(best[:, top - 1] - best[:, top])
+        for g in gaps:
+            self.gap = torch.minimum(self.gap, g)
+        return super().feed_forward(p, f, h)
+
+    def forward(self, tokens, layers_out=None):
+        self.gap = torch.full((len(tokens),), 9.0, dtype=torch.float64)
+        return super().forward(tokens, layers_out)
+
+
+_made = {}
+
+
+def made(name, dtype):
+    """(configuration, model, oracle); the oracle computes in float64."""
+    c = CONFIGS[name]
+    if name not in _made:
+        _made[name] = Oracle(c, C.weights(c, 7)), {}
+    oracle, models = _made[name]
+    if dtype not in models:
+        models[dtype] = C.build(c, C.weights(c, 7), DEV, dtype)
+    return c, models[dtype], oracle
+
+
+_logits = {}
+
+
+def expected(name, tokens):
+    key = (name, tuple(tokens))
+    if key not in _logits:
+        y = _made[name][0].forward(tokens)
+        y.gap = _made[name][0].gap
+        _logits[key] = y
+    return _logits[key]
+
+
+def engine(model, **kw):
+    return LLMEngine(model, **dict(dict(num_blocks=40, block_size=8, max_batch=4), **kw))
+
+
+def check(got, want, dtype, over=0.06, worst=1.0):
+    """Root mean square error per position, in units of the logits' spread; a few positions may be badly conditioned.  In
+    bfloat16 positions where the choice of an expert is a close call are left out: rounding decides them."""
+    d = got.double().cpu() - want
+    d = d - d.mean(-1, keepdim=True)
+    err = d.pow(2).mean(-1).sqrt() / want.std()
+    limit = 3e-5 if dtype == torch.float32 else 0.08
+    if dtype == torch.bfloat16 and hasattr(want, "gap"):
+        clear = want.gap > 0.04
+        assert float(clear.double().mean()) > 0.3
+        err = err[clear]
+    assert int((err > limit).sum()) <= over * len(err) + 1, err.sort().values[-8:]
+    assert float(err.max()) <= (5e-4 if dtype == torch.float32 else worst), float(err.max())
+
+
+def feed(eng, seq, tokens, sizes):
+    """All logits of a sequence that is given in portions."""
+    out, i, j = [], 0, 0
+    while i < len(tokens):
+        n = min(sizes[j % len(sizes)], len(tokens) - i)
+        out += eng.extend([(seq, tokens[i:i + n], list(range(n)))])
+        i += n
+        j += 1
+    return torch.cat(out)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", CONFIGS)
+def test_prompt_portions_and_decoding_give_the_same_logits(name, dtype):
+    c, model, _ = made(name, dtype)
+    toks = prompt(75, c["vocab"], 1)
+    want = expected(name, toks)
+    eng = engine(model)
+    for sizes in ([75], [2], [31, 2, 7, 3], [20, 17, 18], [40] + [1] * 35, [1]):
+        seq = Sequence(0, [], 1)
+        check(feed(eng, seq, toks, sizes), want, dtype)
+        eng.drop(seq)
+    assert len(eng.blocks.free) == 40 and len(eng.states.free) == 4
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", ["small", "wide"])
+def test_unequal_requests_together_and_reused_slots(name, dtype):
+    """Requests of different lengths in one step, some in prompts and some decoding; when one ends, the next takes
+    over its pages and its slot."""
+    c, model, _ = made(name, dtype)
+    toks = [prompt(n, c["vocab"], 10 + n) for n in (41, 9, 64, 23, 30)]
+    want = [expected(name, t) for t in toks]
+    eng = engine(model, max_batch=3, num_blocks=22)
+    live, waiting, got = {}, [0, 1, 2, 3, 4], [[] for _ in toks]
+    at, k = [0] * 5, 0
+    while live or waiting:
+        while waiting and len(live) < 3:
+            i = waiting.pop(0)
+            live[i] = Sequence(i, [], 1)
+        entries, who = [], []
+        for i, seq in live.items():
+            n = min(len(toks[i]) - at[i], 1 if k % 2 else 2 + (3 * i + k) % 6)
+            entries.append((seq, toks[i][at[i]:at[i] + n], list(range(n))))
+            who.append(i)
+            at[i] += n
+        for i, y in zip(who, eng.extend(entries)):
+            got[i].append(y)
+        for i in who:
+            if at[i] == len(toks[i]):
+                eng.drop(live.pop(i))
+        k += 1
+    for i in range(5):
+        check(torch.cat(got[i]), want[i], dtype)
+    assert len(eng.blocks.free) == 22 and len(eng.states.free) == 3
+
+
+def test_generation_is_the_oracles_greedy_choice():
+    """Through add_request / the scheduler: whole prompts and portions, graphs and plain launches, room for all and
+    so little that requests are preempted."""
+    c, model, oracle = made("small", torch.float32)
+    prompts = [prompt(n, c["vocab"], 30 + n) for n in (12, 33, 5)]
+    steps = 14
+    want = []
+    for p in prompts:
+        ids = list(p)
+        y = oracle.forward(ids)[-1]
+        top = y.topk(2).values
+        for _ in range(steps):
+            assert float(top[0] - top[1]) > 5e-4          # a clear choice, so that equality is a fair demand
+            ids.append(int(y.argmax()))
+            y = oracle.forward(ids)[-1]
+            top = y.topk(2).values
+        want.append(ids[len(p):])
+    for kw in ({}, {"use_cuda_graph": False}, {"prefill_portion": 6}, {"prefill_portion": 9, "max_batch": 2}, {"num_blocks": 7}):
+        eng = engine(model, **kw)
+        assert eng.generate(prompts, steps) == want, kw
+        assert len(eng.blocks.free) == kw.get("num_blocks", 40) and len(eng.states.free) == kw.get("max_batch", 4)
+
+
+def test_graph_and_plain_decoding_agree_in_bf16():
+    c, model, _ = made("wide", torch.bfloat16)
+    prompts = [prompt(n, c["vocab"], n) for n in (50, 3, 97)]
+    assert engine(model, num_blocks=60).generate(prompts, 20) == engine(model, num_blocks=60, use_cuda_graph=False).generate(prompts, 20)
+
+
+def test_long_decoding_keeps_to_the_prompt_path():
+    """500 decoded tokens, against the same tokens as one prompt (float32)."""
+    c, model, _ = made("gla-only", torch.float32)
+    toks = prompt(520, c["vocab"], 8)
+    eng = engine(model, num_blocks=80)
+    a, b = Sequence(0, [], 1), Sequence(1, [], 1)
+    whole = feed(eng, a, toks, [520])
+    single = feed(eng, b, toks, [20] + [1] * 500)
+    d = (whole - single).double()
+    assert float(d.abs().max()) <= 3e-4 * float(whole.abs().max())
+
+
+def test_larger_decode_batches_and_long_prompts_in_bf16():
+    """More sequences than a decode-sized linear takes, and a prompt of several hundred tokens: the logits of the
+    float32 model within bf16 rounding."""
+    c, m32, _ = made("wide", torch.float32)
+    _, m16, _ = made("wide", torch.bfloat16)
+    toks = [prompt(30 + 9 * i, c["vocab"], 50 + i) for i in range(20)] + [prompt(450, c["vocab"], 99)]
+    outs = []
+    for m in (m32, m16):
+        eng = engine(m, num_blocks=400, max_batch=32)
+        seqs = [Sequence(i, [], 1) for i in range(21)]
+        ys = eng.extend([(s, t[:-2], list(range(len(t) - 2))) for s, t in zip(seqs, toks)])
+        ys += eng.extend([(s, t[-2:-1], [0]) for s, t in zip(seqs, toks)])
+        ys += eng.extend([(s, t[-1:], [0]) for s, t in zip(seqs, toks)])
+        outs.append(torch.cat(ys))
+    check(outs[1], outs[0].double().cpu(), torch.bfloat16, over=0.2, worst=1.5)     # close calls of the routers among them
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_command_line_replays_and_generates(tmp_path, dtype):
+    from safetensors.torch import save_file
+    c, _, oracle = made("small" if dtype == "float32" else "side-only", torch.float32)
+    (tmp_path / "m").mkdir()
+    (tmp_path / "m" / "config.json").write_text(json.dumps(c))
+    save_file(C.weights(c, 7), str(tmp_path / "m" / "model.safetensors"))
+    a, b = prompt(20, c["vocab"], 1), prompt(6, c["vocab"], 2)
+    steps = [{"step": 0, "entries": [{"id": "a", "tokens": a[:15], "want": [3, 14]}], "end": []},
+             {"step": 1, "entries": [{"id": "a", "tokens": a[15:16], "want": []}], "end": []},
+             {"step": 2, "entries": [{"id": "a", "tokens": a[16:17], "want": [0]}], "end": ["a"]},
+             {"step": 3, "entries": [{"id": "b", "tokens": b, "want": [5]}], "end": ["b"]}]
+    out = subprocess.run([os.path.join(ROOT, "bin", "trace_run"), "--model", str(tmp_path / "m"), "--dtype", dtype, "--out", str(tmp_path),
+                          "--max-tokens", "64"], input="".join(json.dumps(s) + "\n" for s in steps), capture_output=True, text=True, check=True)
+    assert [x for x in out.stdout.splitlines() if x.startswith("done")] == [f"done {i}" for i in range(4)]
+    assert not (tmp_path / "1.f32").exists()
+    import numpy as np
+
+    def read(i):
+        return torch.from_numpy(np.fromfile(tmp_path / f"{i}.f32", "<f4").reshape(-1, c["vocab"]))
+    ya, yb = oracle.forward(a[:17]), oracle.forward(b)
+    check(read(0), ya[[3, 14]], getattr(torch, dtype))
+    check(read(2), ya[[16]], getattr(torch, dtype))
+    check(read(3), yb[[5]], getattr(torch, dtype))
+    if dtype == "float32":
+        bad = subprocess.run([os.path.join(ROOT, "bin", "trace_run"), "--model", str(tmp_path / "m"), "--dtype", "float16", "--out", str(tmp_path)],
+                             input="", capture_output=True, text=True)
+        assert bad.returncode == 3
+        gen = subprocess.run([sys.executable, "-m", "nanoquantization_b200.cli", "generate", "--model", str(tmp_path / "m"), "--dtype", dtype,
+                              "--max-new-tokens", "1"], input=" ".join(map(str, b)) + "\n", capture_output=True, text=True, check=True, cwd=ROOT)
+        assert gen.stdout.split() == [str(int(yb[-1].argmax()))]
