@@ -906,9 +906,9 @@ def vemedra_kernels(dev, peaks, T=8192, context=2048):
         att.chunk = chunk
         d = att.desc()
         kv_bytes, st_bytes = B * context * 2 * G * D * 2, 2 * B * RH * RD * RV * 4
-        both = lambda i: ops.mixer_decode(pr, ac, (d, att.inv_freq, 0, 0, copies[i % n][0], copies[i % n][1]), (ret, off, H * D, copies[i % n][2]), s)  # noqa: E731
+        both = lambda i: ops.mixer_decode(pr, ac, (d, att.rope_desc(), 0, att.value_column(0), 0, copies[i % n][0], copies[i % n][1]), (ret, off, H * D, copies[i % n][2]), s)  # noqa: E731
         add(ph, "attention + retention", _device_us(both, 2 * n), kv_bytes + st_bytes)
-        add(ph, "  attention alone", _device_us(lambda i: ops.mixer_decode(pr, ac, (d, att.inv_freq, 0, 0, copies[i % n][0], copies[i % n][1]), None, s), 2 * n), kv_bytes)
+        add(ph, "  attention alone", _device_us(lambda i: ops.mixer_decode(pr, ac, (d, att.rope_desc(), 0, att.value_column(0), 0, copies[i % n][0], copies[i % n][1]), None, s), 2 * n), kv_bytes)
         add(ph, "  retention alone", _device_us(lambda i: ops.mixer_decode(pr, ac, None, (ret, off, H * D, copies[i % n][2]), s), 2 * n), st_bytes)
         try:
             from flash_attn import flash_attn_with_kvcache

@@ -109,10 +109,19 @@ int nqb200_retention(const void* proj, int64_t stride, int64_t q_off, int64_t k_
                      const float* log_decay, float* state, float* o, int64_t heads, int64_t dim, int64_t vdim, const nqb200_batch* b, int dtype,
                      void* stream);
 
+/* Retention, or gated linear attention where rank > 0: then decay is not read, and the decays of channel c are
+ * sigmoid(a2[c] . low + a2_bias[c])^(1 / tau), low the rank columns behind the gate. */
 typedef struct {
   int32_t heads, dim, vdim;
   float eps, out_scale;
   const float* decay;     /* [heads] */
+  const float* norm;      /* [vdim] weight of the norm over a head's output, or NULL */
+  const float* inv_freq;  /* [rot / 2]; q and k turn in pairs (i, i + rot/2) inside nqb200_mixer_decode; other calls take */
+  int32_t rot;            /* them turned (nqb200_norm_rope) */
+  int32_t rank;
+  float tau;
+  const void* a2;         /* [heads * dim, rank] of dtype */
+  const float* a2_bias;   /* [heads * dim] */
 } nqb200_retention_desc;
 
 /* Prompts (bf16): retention in chunkwise form with norm and gate.  proj holds q | k | v | gate from column off; the
@@ -163,11 +172,11 @@ int nqb200_dense_decode_glu(const void* x, const void* w, void* out, int64_t M, 
 int nqb200_dense_decode_mingru(const void* x, const void* w, const float* z_bias, const float* x_bias, float* state, void* out,
                                int64_t width, int64_t K, const nqb200_batch* b, void* stream);
 
-/* One token per sequence: rotary embedding, K/V store and attention (columns q | k | v of proj from a_off, output
- * from column a_col of act), and retention with norm and gate (columns q | k | v | g from r_off, output from r_col),
- * in one launch.  a or r may be NULL.  Sizes as nqb200_mixer_decode_supported says. */
+/* One token per sequence: norm and rotation of the heads, K/V store and attention (columns q | k of proj from a_off, v from
+ * v_off, output from column a_col of act), and retention or gated linear attention with norm and gate (columns q | k | v | g
+ * [| low] from r_off, output from r_col), in one launch.  a or r may be NULL.  Sizes as nqb200_mixer_decode_supported says. */
 int nqb200_mixer_decode(const void* proj, int64_t stride, void* act, int64_t act_stride, const nqb200_attention* a,
-                        const float* inv_freq, int64_t rot, int64_t a_off, int64_t a_col, void* k_cache, void* v_cache,
+                        const nqb200_rope* rope, int64_t a_off, int64_t v_off, int64_t a_col, void* k_cache, void* v_cache,
                         const nqb200_retention_desc* r, int64_t r_off, int64_t r_col, float* state, const nqb200_batch* b, void* stream);
 int nqb200_mixer_decode_supported(const nqb200_attention* a, const nqb200_retention_desc* r);
 

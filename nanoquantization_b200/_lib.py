@@ -90,7 +90,8 @@ class RopeDesc(ctypes.Structure):
 class RetentionDesc(ctypes.Structure):
     """nqb200_retention_desc of include/nqb200_mixers.h."""
     _fields_ = [("heads", ctypes.c_int32), ("dim", ctypes.c_int32), ("vdim", ctypes.c_int32), ("eps", ctypes.c_float),
-                ("out_scale", ctypes.c_float), ("decay", _vp)]
+                ("out_scale", ctypes.c_float), ("decay", _vp), ("norm", _vp), ("inv_freq", _vp), ("rot", ctypes.c_int32),
+                ("rank", ctypes.c_int32), ("tau", ctypes.c_float), ("a2", _vp), ("a2_bias", _vp)]
 
 
 class RouterDesc(ctypes.Structure):
@@ -135,7 +136,7 @@ MIXER_SIGNATURES = {
     "nqb200_dense_decode_glu": (_int, [_vp, _vp, _vp, _i64, _i64, _i64, _f32, _vp]),
     "nqb200_dense_decode_mingru": (_int, [_vp] * 6 + [_i64, _i64, _step, _vp]),
     "nqb200_mixer_decode_supported": (_int, [_att, _ret]),
-    "nqb200_mixer_decode": (_int, [_vp, _i64, _vp, _i64, _att, _vp, _i64, _i64, _i64, _vp, _vp, _ret, _i64, _i64, _vp, _step, _vp]),
+    "nqb200_mixer_decode": (_int, [_vp, _i64, _vp, _i64, _att, _rope, _i64, _i64, _i64, _vp, _vp, _ret, _i64, _i64, _vp, _step, _vp]),
 }
 
 # mirrors include/nqb200_moe.h one to one

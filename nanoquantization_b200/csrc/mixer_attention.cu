@@ -1,4 +1,4 @@
-// Rotary embedding + paged K/V store, and chunk-masked attention with a score cap and a sink.  The kernels in
+// Rotary embedding + paged K/V store, and attention (chunks, score cap and sink, or sigmoid weights).  The kernels in
 // this file take any head sizes and both element types; the tensor-core kernels take over where they apply.
 #include "mixers.cuh"
 
@@ -207,9 +207,9 @@ extern "C" int nqb200_chunk_attention(const void* q, int64_t q_stride, const voi
   if (!mixer_dtype(dtype)) return NQB200_ERR_BAD_DTYPE;
   if (b->tokens == 0) return NQB200_OK;
   if (!q || !k_cache || !v_cache || !out) return NQB200_ERR_NULL_POINTER;
-  if (dtype == NQB200_BF16 && !a->sigmoid && attention_umma_supports(q, q_stride, k_cache, v_cache, out, out_stride, cache_rows, a, b))
+  if (dtype == NQB200_BF16 && attention_umma_supports(q, q_stride, k_cache, v_cache, out, out_stride, cache_rows, a, b))
     return attention_umma(q, q_stride, k_cache, v_cache, out, out_stride, cache_rows, a, b, status, (cudaStream_t)stream);
-  if (dtype == NQB200_BF16 && !a->sigmoid && b->max_len > 1 && attention_prefill_supports(q, q_stride, k_cache, v_cache, out, out_stride, a))
+  if (dtype == NQB200_BF16 && b->max_len > 1 && attention_prefill_supports(q, q_stride, k_cache, v_cache, out, out_stride, a))
     return attention_prefill(q, q_stride, k_cache, v_cache, out, out_stride, a, b, (cudaStream_t)stream);
   const dim3 grid((unsigned)b->max_len, (unsigned)a->heads, (unsigned)b->batch), block(kSimpleKeys);
   const size_t smem = (size_t)a->dim * sizeof(float);

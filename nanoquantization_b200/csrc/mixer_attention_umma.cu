@@ -14,6 +14,9 @@
 // twice the cap it is the seventh convergent of Lambert's continued fraction (one reciprocal more per score); a warp
 // whose tile has a larger score, or needs a mask, takes the general path.
 //
+// Sigmoid weights (nqb200_attention.sigmoid) need no maximum and no sum: a weight is 1 / (1 + 2^x), two weights share one
+// reciprocal, 1 / a = b / (a b), with x clamped to 60 so that a b stays finite (weights below 2^-60 are 2^-60).
+//
 // Every wait is bounded; on expiry NQB200_ERR_WAIT_TIMEOUT goes to the status word, all roles drain and tensor memory is
 // released.
 #include "mixers.cuh"
@@ -33,6 +36,7 @@ struct Params {
   int heads, kv_heads, chunk;
   float scale, softcap, out_scale;
   const float* sink;
+  int sigmoid; const float* temp; const float* bias;
   int* status;
 };
 
@@ -277,6 +281,17 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
       __syncwarp();
       if (lane == 0) mbar_arrive(smem_u32(&bar_p[q][half]));
     };
+    const float sg_scale = -p.scale * (p.temp ? p.temp[h] : 1.f) * kLog2e, sg_shift = p.bias ? -p.bias[h] * kLog2e : 0.f;
+    const uint64_t sg_scale2 = pair2(sg_scale, sg_scale), sg_shift2 = pair2(sg_shift, sg_shift), one2 = pair2(1.f, 1.f);
+    auto sigmoid2 = [&](uint32_t s0, uint32_t s1, float& w0, float& w1) {
+      float x0, x1;
+      unpair2(fma2(pair2(__uint_as_float(s0), __uint_as_float(s1)), sg_scale2, sg_shift2), x0, x1);
+      float d0, d1;
+      unpair2(add2(pair2(ex2(fminf(x0, 60.f)), ex2(fminf(x1, 60.f))), one2), d0, d1);
+      const float r = rcp_fast(d0 * d1);
+      w0 = r * d1;
+      w1 = r * d0;
+    };
     const float sink = p.sink ? p.sink[h] * kLog2e : -INFINITY;
     float m = sink, l = 0.f;
     uint64_t lsum = pair2(0.f, 0.f);
@@ -291,6 +306,40 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
 #pragma unroll
       for (int c = 0; c < 4; ++c) tmem_ld32(tS + c * 32, r[c]);
       tc_wait_ld();
+      if (p.sigmoid) {
+        if (!masked) {
+#pragma unroll
+          for (int c = 0; c < 4; ++c) {
+            uint32_t w[16];
+#pragma unroll
+            for (int e = 0; e < 16; ++e) {
+              float x0, x1;
+              sigmoid2(r[c][2 * e], r[c][2 * e + 1], x0, x1);
+              w[e] = pack_bf16(x0, x1);
+            }
+            tmem_st16(tS + c * 16, w);
+            if (c == 1) half_done(0);
+          }
+        } else {
+#pragma unroll 1
+          for (int c = 0; c < 8; ++c) {
+            uint32_t v[16], w[8];
+            tmem_ld_32x32b_x16(tS + c * 16, v);
+            tc_wait_ld();
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+              const int key = key0 + c * 16 + 2 * e;
+              float x0, x1;
+              sigmoid2(v[2 * e], v[2 * e + 1], x0, x1);
+              w[e] = pack_bf16(key <= pos && key >= lo ? x0 : 0.f, key + 1 <= pos && key + 1 >= lo ? x1 : 0.f);
+            }
+            tmem_st8(tS + c * 8, w);      // lies behind what has been read of S
+            if (c == 3) half_done(0);
+          }
+        }
+        half_done(1);
+        continue;
+      }
       float mx = -INFINITY, ab = 0.f;
       if (!masked) {
         float hi[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY}, lw[4] = {INFINITY, INFINITY, INFINITY, INFINITY};
@@ -421,7 +470,7 @@ attention_umma_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_con
         tc_fence_after();
         float a, c2;
         unpair2(lsum, a, c2);
-        const float f = p.out_scale / (l + a + c2);
+        const float f = p.sigmoid ? p.out_scale : p.out_scale / (l + a + c2);
         bf16* dst = p.out + (size_t)(t0 + i) * p.out_stride + (size_t)h * V;
 #pragma unroll
         for (int c = 0; c < V / 32; ++c) {
@@ -490,7 +539,8 @@ int attention_umma(const void* q, int64_t q_stride, const void* k_cache, const v
     return NQB200_ERR_LAUNCH;
   att::Params p = {};
   p.bt = *b; p.out = (bf16*)out; p.out_stride = out_stride; p.heads = a->heads; p.kv_heads = a->kv_heads; p.chunk = a->chunk;
-  p.scale = a->scale; p.softcap = a->softcap; p.out_scale = a->out_scale; p.sink = a->sink; p.status = status;
+  p.scale = a->scale; p.softcap = a->softcap; p.out_scale = a->out_scale; p.sink = a->sink; p.sigmoid = a->sigmoid; p.temp = a->temp; p.bias = a->bias;
+  p.status = status;
   if (a->dim == 64) return a->vdim == 64 ? att::launch<64, 64>(tq, tk, tv, p, st) : att::launch<64, 128>(tq, tk, tv, p, st);
   return a->vdim == 64 ? att::launch<128, 64>(tq, tk, tv, p, st) : att::launch<128, 128>(tq, tk, tv, p, st);
 }

@@ -1,5 +1,6 @@
-// One decode step (one token per sequence) of the mixers that stand side by side in a layer, in one launch: chunked
-// attention with its rotary embedding and K/V store, and retention with its norm and gate.
+// One decode step (one token per sequence) of the mixers that stand side by side in a layer, in one launch: attention
+// (softmax in chunks, or sigmoid weights) with its head norms, rotary embedding and K/V store, and retention or gated linear
+// attention with its decays, norm and gate.
 //
 // Work is dealt to thread-block clusters: a cluster takes one (sequence, key/value head, group of query heads) of the
 // attention and splits the visible keys over its CTAs, or one (sequence, head) of the retention and splits the value
@@ -24,13 +25,13 @@ struct DecodeArgs {
   nqb200_batch bt;
   // attention; att_clusters = kv_heads * head_groups per sequence (0: none)
   nqb200_attention at;
-  const float* inv_freq; int rot;
+  nqb200_rope rope;
   int q_off, k_off, v_off, a_col, att_clusters, head_groups;
   bf16* k_cache; bf16* v_cache;
   // retention (ret_heads 0: none)
-  int ret_heads, rdim, rvdim, rq_off, rk_off, rv_off, rg_off, r_col;
-  const float* decay; float* rstate;
-  float eps, r_scale;
+  int ret_heads, rdim, rvdim, rq_off, rk_off, rv_off, rg_off, rl_off, r_col;
+  nqb200_retention_desc rd;
+  float* rstate;
 };
 
 // Fixed part of the attention's shared memory; the key / value ring follows it.
@@ -43,10 +44,13 @@ struct AttSmem {
   int rows[4][kDecMaxTile];                   // cache rows of the keys of four successive tiles
   float m[kDecHeads], l[kDecHeads], corr[kDecHeads];
   float out[kDecHeads][kDecMaxDim];           // this CTA's share, read by the cluster
+  float inv[kDecHeads + 1];                   // 1 / rms of the query heads and the new key
 };
 
+constexpr int kDecMaxRank = 512;
 struct RetSmem {
-  float q[1024], k[1024];
+  float q[1024], k[1024], d[1024];
+  float low[kDecMaxRank];
   float red[kDecThreads * 4];
   float o[1024];
   float ss, wsum[kDecThreads / 32];
@@ -87,7 +91,7 @@ __device__ void attention_decode(const DecodeArgs& a, uint8_t* smem, int b, int 
   const int lo = at.chunk > 0 ? pos / at.chunk * at.chunk : 0, nk = pos - lo + 1;
   const int per = (nk + csize - 1) / csize, k0 = lo + rank * per, k1 = min(lo + nk, k0 + per);   // this CTA's keys
   const int tiles = k1 > k0 ? (k1 - k0 + TILE - 1) / TILE : 0;
-  const int KS = att_ks(D), D8 = D / 8, V8 = V / 8, half = a.rot / 2;
+  const int KS = att_ks(D), D8 = D / 8, V8 = V / 8, half = a.rope.rot / 2;
   constexpr int VS = VP + 8, NT = VP / 32;       // n-tiles of 8 columns per warp
   const bf16* row = a.proj + (size_t)b * a.stride;
   const bool newest = k0 <= pos && pos < k1;
@@ -135,21 +139,43 @@ __device__ void attention_decode(const DecodeArgs& a, uint8_t* smem, int b, int 
   }
   for (int e = tid; e < kDecHeads * (KS - 8); e += kDecThreads) sm.q[e / (KS - 8)][e % (KS - 8)] = __float2bfloat16_rn(0.f);
   for (int e = tid; e < 16 * kDecPS; e += kDecThreads) sm.p[e / kDecPS][e % kDecPS] = __float2bfloat16_rn(0.f);
-  for (int f = tid; f < half; f += kDecThreads) sincosf((float)pos * a.inv_freq[f], &sm.cs[half + f], &sm.cs[f]);
+  for (int f = tid; f < half; f += kDecThreads) sincosf((float)pos * a.rope.inv_freq[f], &sm.cs[half + f], &sm.cs[f]);
   if (tid < kDecHeads) { sm.m[tid] = -INFINITY; sm.l[tid] = 0.f; }
+  const int pairs = half + (D - a.rope.rot), nvec = R + (newest ? 1 : 0);
+  auto vec = [&](int r) { return r < R ? row + a.q_off + (size_t)(h0 + r) * D : row + a.k_off + (size_t)kvh * D; };
+  if (a.rope.q_norm) {
+    for (int r = warp; r < nvec; r += kDecThreads / 32) {
+      const bf16* src = vec(r);
+      float ss = 0.f;
+      for (int d = lane; d < D; d += 32) { const float x = to_f(src[d]); ss += x * x; }
+      ss = warp_sum(ss);
+      if (lane == 0) sm.inv[r] = 1.f / sqrtf(ss / (float)D + a.rope.eps);
+    }
+  }
   __syncthreads();
-  const int pairs = half + (D - a.rot), nvec = R + (newest ? 1 : 0);
   for (int e = tid; e < nvec * pairs; e += kDecThreads) {
     const int r = e / pairs, j = e % pairs;
-    const bf16* src = r < R ? row + a.q_off + (size_t)(h0 + r) * D : row + a.k_off + (size_t)kvh * D;
+    const bf16* src = vec(r);
     bf16* dst = r < R ? sm.q[r] : sm.knew;
+    const float* w = r < R ? a.rope.q_norm : a.rope.k_norm;
+    const float inv = w ? sm.inv[r] : 1.f;
     if (j < half) {
-      const float u = to_f(src[j]), v = to_f(src[j + half]), c = sm.cs[j], s = sm.cs[half + j];
-      dst[j] = __float2bfloat16_rn(u * c - v * s);
-      dst[j + half] = __float2bfloat16_rn(v * c + u * s);
+      const int x = a.rope.interleaved ? 2 * j : j, y = a.rope.interleaved ? x + 1 : j + half;
+      float u = to_f(src[x]), v = to_f(src[y]);
+      const float c = sm.cs[j], s = sm.cs[half + j];
+      if (w) { u = u * inv * w[x]; v = v * inv * w[y]; }
+      dst[x] = __float2bfloat16_rn(u * c - v * s);
+      dst[y] = __float2bfloat16_rn(v * c + u * s);
     } else {
-      dst[j + half] = src[j + half];
+      dst[j + half] = w ? __float2bfloat16_rn(to_f(src[j + half]) * inv * w[j + half]) : src[j + half];
     }
+  }
+  float factor[2], shift[2];   // of this lane's two query heads in the score product
+#pragma unroll
+  for (int u = 0; u < 2; ++u) {
+    const int r = (lane & 3) * 2 + u;
+    factor[u] = at.scale * (at.temp && r < R ? at.temp[h0 + r] : 1.f);
+    shift[u] = at.bias && r < R ? at.bias[h0 + r] : 0.f;
   }
   const float inv_cap = at.softcap > 0.f ? 1.f / at.softcap : 0.f;
   const uint32_t k_lane = (uint32_t)((warp * 16 + (lane & 15)) * KS + (lane >> 4) * 8) * 2;
@@ -199,14 +225,18 @@ __device__ void attention_decode(const DecodeArgs& a, uint8_t* smem, int b, int 
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int key = warp * 16 + g + 8 * (e >> 1), r = t * 2 + (e & 1);
-        float s = c[e] * at.scale;
+        float s = c[e] * factor[e & 1] + shift[e & 1];
+        if (at.sigmoid) {
+          sm.p[r][key] = __float2bfloat16_rn(key < cnt ? sigmoid_fast(s) : 0.f);
+          continue;
+        }
         if (at.softcap > 0.f) s = at.softcap * tanh_fast(s * inv_cap);
         sm.s[r][key] = key < cnt ? s : -INFINITY;
       }
     }
     __syncthreads();
     // softmax of the tile: a head per warp, TILE / 32 keys per lane
-    if (warp < R) {
+    if (warp < R && !at.sigmoid) {
       float x[TILE / 32], mx = -INFINITY, sum = 0.f;
 #pragma unroll
       for (int k = 0; k < TILE / 32; ++k) { x[k] = sm.s[warp][lane + 32 * k]; mx = fmaxf(mx, x[k]); }
@@ -225,10 +255,12 @@ __device__ void attention_decode(const DecodeArgs& a, uint8_t* smem, int b, int 
         sm.l[warp] = sm.l[warp] * corr + sum;
       }
     }
-    __syncthreads();
-    const float corr = g < R ? sm.corr[g] : 0.f;
+    if (!at.sigmoid) {
+      __syncthreads();
+      const float corr = g < R ? sm.corr[g] : 0.f;
 #pragma unroll
-    for (int n = 0; n < NT; ++n) { O[n][0] *= corr; O[n][1] *= corr; }
+      for (int n = 0; n < NT; ++n) { O[n][0] *= corr; O[n][1] *= corr; }
+    }
     const uint32_t va = dec_smem(vt) + v_lane;
 #pragma unroll
     for (int kk = 0; kk < TILE / 32; ++kk) {
@@ -267,6 +299,13 @@ __device__ void attention_decode(const DecodeArgs& a, uint8_t* smem, int b, int 
       pl[k] = s->l[r];
       po[k] = s->out[r][c];
     }
+    if (at.sigmoid) {
+      float o = 0.f;
+#pragma unroll
+      for (int k = 0; k < 8; ++k) o += k < csize ? po[k] : 0.f;
+      a.act[(size_t)b * a.act_stride + a.a_col + (size_t)(h0 + r) * V + c] = __float2bfloat16_rn(o * at.out_scale);
+      continue;
+    }
 #pragma unroll
     for (int k = 0; k < 8; ++k) m = fmaxf(m, pm[k]);
     float l = at.sink ? expf(sink - m) : 0.f, o = 0.f;
@@ -289,11 +328,34 @@ __device__ void retention_decode(const DecodeArgs& a, RetSmem& sm, int b, int h,
   const int quads = V / VEC, per = (quads + csize - 1) / csize;                 // column groups of one CTA
   const int c0 = min(rank * per, quads), ncol = min(per, quads - c0);
   const bf16* row = a.proj + (size_t)b * a.stride;
-  const float kscale = 1.f / sqrtf((float)D), d = a.decay[h];
-  const bool fresh = a.bt.pos0[b] == 0;
-  for (int e = tid; e < D; e += kDecThreads) {
-    sm.q[e] = to_f(row[a.rq_off + (size_t)h * D + e]);
-    sm.k[e] = to_f(row[a.rk_off + (size_t)h * D + e]) * kscale;
+  const float kscale = 1.f / sqrtf((float)D);
+  const int pos = a.bt.pos0[b], half = a.rd.rot / 2;
+  const bool fresh = pos == 0;
+  const bf16 *qr = row + a.rq_off + (size_t)h * D, *kr = row + a.rk_off + (size_t)h * D;
+  for (int e = tid; e < half; e += kDecThreads) {
+    float s, c;
+    sincosf((float)pos * a.rd.inv_freq[e], &s, &c);
+    const float qu = to_f(qr[e]), qv = to_f(qr[e + half]), ku = to_f(kr[e]), kv = to_f(kr[e + half]);
+    sm.q[e] = qu * c - qv * s;
+    sm.q[e + half] = qv * c + qu * s;
+    sm.k[e] = (ku * c - kv * s) * kscale;
+    sm.k[e + half] = (kv * c + ku * s) * kscale;
+  }
+  for (int e = 2 * half + tid; e < D; e += kDecThreads) {
+    sm.q[e] = to_f(qr[e]);
+    sm.k[e] = to_f(kr[e]) * kscale;
+  }
+  if (a.rd.rank > 0) {
+    for (int e = tid; e < a.rd.rank; e += kDecThreads) sm.low[e] = to_f(row[a.rl_off + e]);
+    __syncthreads();
+    const bf16* a2 = reinterpret_cast<const bf16*>(a.rd.a2) + (size_t)h * D * a.rd.rank;
+    for (int e = tid; e < D; e += kDecThreads) {
+      float z = 0.f;
+      for (int r = 0; r < a.rd.rank; ++r) z += sm.low[r] * to_f(a2[(size_t)e * a.rd.rank + r]);
+      sm.d[e] = expf(log_sigmoid_f(z + a.rd.a2_bias[h * D + e]) / a.rd.tau);
+    }
+  } else {
+    for (int e = tid; e < D; e += kDecThreads) sm.d[e] = a.rd.decay[h];
   }
   __syncthreads();
   float* st = a.rstate + ((size_t)a.bt.slot[b] * a.ret_heads + h) * D * V;
@@ -325,7 +387,7 @@ __device__ void retention_decode(const DecodeArgs& a, RetSmem& sm, int b, int h,
         for (int u = 0; u < U; ++u) {
           const int r = r0 + u * RG;
           if (r >= D) break;
-          const float kr = sm.k[r], qr = sm.q[r];
+          const float kr = sm.k[r], qr = sm.q[r], d = sm.d[r];
 #pragma unroll
           for (int i = 0; i < VEC; ++i) { S[u][i] = d * S[u][i] + kr * v[i]; acc[i] += S[u][i] * qr; }
           float* sp = st + (size_t)r * V + col;
@@ -357,11 +419,11 @@ __device__ void retention_decode(const DecodeArgs& a, RetSmem& sm, int b, int h,
   cl.sync();
   float tot = 0.f;
   for (int k = 0; k < csize; ++k) tot += cl.map_shared_rank(&sm, k)->ss;
-  const float inv = a.r_scale / sqrtf(tot / (float)V + a.eps);
+  const float inv = a.rd.out_scale / sqrtf(tot / (float)V + a.rd.eps);
   for (int e = tid; e < ncol * VEC; e += kDecThreads) {
     const int c = c0 * VEC + e;
     const float gt = to_f(row[a.rg_off + (size_t)h * V + c]);
-    a.act[(size_t)b * a.act_stride + a.r_col + (size_t)h * V + c] = __float2bfloat16_rn(sm.o[e] * inv * (gt * sigmoid_f(gt)));
+    a.act[(size_t)b * a.act_stride + a.r_col + (size_t)h * V + c] = __float2bfloat16_rn(sm.o[e] * inv * (a.rd.norm ? a.rd.norm[c] : 1.f) * (gt * sigmoid_f(gt)));
   }
   cl.sync();
 }
@@ -415,12 +477,12 @@ extern "C" int nqb200_mixer_decode_supported(const nqb200_attention* a, const nq
   if (a && (a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads != 0 || a->dim <= 0 || a->dim % 8 != 0 || a->dim > kDecMaxDim ||
             a->vdim <= 0 || a->vdim % 8 != 0 || a->vdim > kDecMaxDim))
     return 0;
-  if (r && (r->heads <= 0 || r->dim <= 0 || r->dim > 1024 || r->vdim <= 0 || r->vdim > 1024)) return 0;
+  if (r && (r->heads <= 0 || r->dim <= 0 || r->dim > 1024 || r->vdim <= 0 || r->vdim > 1024 || r->rank > kDecMaxRank || r->rot < 0 || r->rot % 2 != 0 || r->rot > r->dim)) return 0;
   return a || r ? 1 : 0;
 }
 
 extern "C" int nqb200_mixer_decode(const void* proj, int64_t stride, void* act, int64_t act_stride, const nqb200_attention* a,
-                                   const float* inv_freq, int64_t rot, int64_t a_off, int64_t a_col, void* k_cache, void* v_cache,
+                                   const nqb200_rope* rope, int64_t a_off, int64_t v_off, int64_t a_col, void* k_cache, void* v_cache,
                                    const nqb200_retention_desc* r, int64_t r_off, int64_t r_col, float* state, const nqb200_batch* b,
                                    void* stream) {
   int s = a ? check_batch(b, true) : NQB200_OK;
@@ -429,13 +491,16 @@ extern "C" int nqb200_mixer_decode(const void* proj, int64_t stride, void* act, 
   if (!b) return NQB200_ERR_NULL_POINTER;
   if (!nqb200_mixer_decode_supported(a, r) || b->max_len > 1 || b->tokens != b->batch) return NQB200_ERR_BAD_SHAPE;
   if (b->tokens == 0) return NQB200_OK;
-  if (!proj || !act || (a && (!k_cache || !v_cache || (rot > 0 && !inv_freq))) || (r && (!state || !r->decay))) return NQB200_ERR_NULL_POINTER;
-  if (a && (rot < 0 || rot % 2 != 0 || rot > a->dim)) return NQB200_ERR_BAD_SHAPE;
+  if (!proj || !act || (a && (!k_cache || !v_cache || !rope || (rope->rot > 0 && !rope->inv_freq) || (rope->q_norm && !rope->k_norm))) ||
+      (r && (!state || (r->rot > 0 && !r->inv_freq) || (r->rank > 0 ? !r->a2 || !r->a2_bias : !r->decay))))
+    return NQB200_ERR_NULL_POINTER;
+  if (a && (rope->rot < 0 || rope->rot % 2 != 0 || rope->rot > a->dim || (a->sigmoid && (a->sink || a->softcap > 0.f)))) return NQB200_ERR_BAD_SHAPE;
+  if (r && r->rank > 0 && !(r->tau > 0.f)) return NQB200_ERR_BAD_SHAPE;
   if (a && (!aligned16(k_cache) || !aligned16(v_cache))) return NQB200_ERR_MISALIGNED;
   if (r && !aligned16(state)) return NQB200_ERR_MISALIGNED;
   if (a && r && (int64_t)(a->kv_heads + r->heads) * b->batch > kNumSMs) {
     // more than one wave: each with the shared memory and the cluster size that suit it
-    const int rc = nqb200_mixer_decode(proj, stride, act, act_stride, a, inv_freq, rot, a_off, a_col, k_cache, v_cache, nullptr, 0, 0, nullptr, b, stream);
+    const int rc = nqb200_mixer_decode(proj, stride, act, act_stride, a, rope, a_off, v_off, a_col, k_cache, v_cache, nullptr, 0, 0, nullptr, b, stream);
     return rc != NQB200_OK ? rc
                            : nqb200_mixer_decode(proj, stride, act, act_stride, nullptr, nullptr, 0, 0, 0, nullptr, nullptr, r, r_off, r_col, state, b, stream);
   }
@@ -446,8 +511,8 @@ extern "C" int nqb200_mixer_decode(const void* proj, int64_t stride, void* act, 
   if (a) {
     const int per_kv = a->heads / a->kv_heads;
     p.at = *a;
-    p.inv_freq = inv_freq; p.rot = (int)rot;
-    p.q_off = (int)a_off; p.k_off = (int)(a_off + (int64_t)a->heads * a->dim); p.v_off = p.k_off + a->kv_heads * a->dim;
+    p.rope = *rope;
+    p.q_off = (int)a_off; p.k_off = (int)(a_off + (int64_t)a->heads * a->dim); p.v_off = (int)v_off;
     p.a_col = (int)a_col; p.k_cache = (bf16*)k_cache; p.v_cache = (bf16*)v_cache;
     p.head_groups = (per_kv + kDecHeads - 1) / kDecHeads;
     p.att_clusters = a->kv_heads * p.head_groups;
@@ -459,8 +524,8 @@ extern "C" int nqb200_mixer_decode(const void* proj, int64_t stride, void* act, 
   if (r) {
     p.ret_heads = r->heads; p.rdim = r->dim; p.rvdim = r->vdim;
     p.rq_off = (int)r_off; p.rk_off = p.rq_off + r->heads * r->dim; p.rv_off = p.rk_off + r->heads * r->dim;
-    p.rg_off = p.rv_off + r->heads * r->vdim; p.r_col = (int)r_col;
-    p.decay = r->decay; p.rstate = state; p.eps = r->eps; p.r_scale = r->out_scale;
+    p.rg_off = p.rv_off + r->heads * r->vdim; p.rl_off = p.rg_off + r->heads * r->vdim; p.r_col = (int)r_col;
+    p.rd = *r; p.rstate = state;
     units += r->heads;
     while (want < 8 && (int64_t)r->dim * r->vdim * 4 > (int64_t)want * 16384 && want * 8 <= r->vdim) want *= 2;
   }

@@ -3,7 +3,7 @@
 //
 // One CTA takes 128 query tokens of one head: 8 warps of 16 rows, key tiles of 64 through a two-stage cp.async ring,
 // mma.m16n8k16 with float accumulators, scores and weights in float.  Both mixers share the loop.  Attention: scaled,
-// capped scores, online softmax that starts from the sink.  Retention: keys are those of the query's own chunk of 256
+// capped scores, online softmax that starts from the sink; or sigmoid weights, summed as they are.  Retention: keys are those of the query's own chunk of 256
 // tokens (counted from the step's first token), a score is weighted by decay^(i-j), and what lies before the chunk
 // comes as decay^(i+1) q S with S the state at the chunk's start; the head's norm and gate close the row.
 //
@@ -62,10 +62,11 @@ struct PrefillArgs {
   int kv_heads, chunk;
   float scale, softcap;
   const float* sink;
+  int sigmoid; const float* temp; const float* bias;
   // retention: k, v, gate in the same buffer as q
   const bf16* k; const bf16* v; const bf16* gate;
   const float* decay; const bf16* states;    // states [chunk id][heads][high part, rest][dim][vdim]
-  float eps;
+  float eps; const float* norm;
 };
 
 // Chunk c of sequence b has id cu[b] / 256 + b + c: distinct, and below tokens / 256 + batch.
@@ -137,6 +138,7 @@ __global__ void __launch_bounds__(kThreads, 1) prefill_kernel(const PrefillArgs 
   const uint32_t k_lane = ((lane & 7) + ((lane >> 4) << 3)) * QS + ((lane >> 3) & 1) * 8;
   const uint32_t v_lane = ((lane & 7) + (((lane >> 3) & 1) << 3)) * VS + (lane >> 4) * 8;
   const float log2d = RET ? log2f(a.decay[h]) : 0.f;
+  const float factor = !RET && a.temp ? a.scale * a.temp[h] : a.scale, shift = !RET && a.bias ? a.bias[h] : 0.f;
 
   if (RET) {
     for (int e = tid; e <= kRetChunk; e += kThreads) pw[e] = decay_pow(log2d, e);
@@ -224,6 +226,15 @@ __global__ void __launch_bounds__(kThreads, 1) prefill_kernel(const PrefillArgs 
             const int j = j0 + i * 8 + 2 * t + (e & 1), dist = pr[e >> 1] - j;
             s[i][e] = (dist >= 0 && j >= lor[e >> 1]) ? s[i][e] * (ksc * pw[min(dist, kRetChunk)]) : 0.f;
           }
+      } else if (a.sigmoid) {
+#pragma unroll
+        for (int i = 0; i < kKeys / 8; ++i)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const int j = j0 + i * 8 + 2 * t + (e & 1);
+            const float w = sigmoid_fast(s[i][e] * factor + shift);
+            s[i][e] = (mask && (j > pr[e >> 1] || j < lor[e >> 1])) ? 0.f : w;
+          }
       } else {
         float mx[2] = {m[0], m[1]};
 #pragma unroll
@@ -282,7 +293,8 @@ __global__ void __launch_bounds__(kThreads, 1) prefill_kernel(const PrefillArgs 
       for (int i = 0; i < VP / 8; ++i) ss += O[i][2 * r] * O[i][2 * r] + O[i][2 * r + 1] * O[i][2 * r + 1];
       f = a.out_scale / sqrtf(quad_sum(ss) / (float)a.vdim + a.eps);
     } else {
-      f = a.out_scale / quad_sum(l[r]);
+      const float sum = quad_sum(l[r]);
+      f = a.sigmoid ? a.out_scale : a.out_scale / sum;
     }
     if (pr[r] > plast) continue;
     const size_t tok = (size_t)(t0 + pr[r] - pos0);
@@ -294,6 +306,7 @@ __global__ void __launch_bounds__(kThreads, 1) prefill_kernel(const PrefillArgs 
       if (c >= a.vdim) break;
       float x = O[i][2 * r] * f, y = O[i][2 * r + 1] * f;
       if (RET) {
+        if (a.norm) { x *= a.norm[c]; y *= a.norm[c + 1]; }
         const uint32_t gw = *reinterpret_cast<const uint32_t*>(gp + c);
         const float gx = __uint_as_float(gw << 16), gy = __uint_as_float(gw & 0xFFFF0000u);
         x *= gx * sigmoid_fast(gx);
@@ -457,7 +470,7 @@ int attention_prefill(const void* q, int64_t q_stride, const void* k_cache, cons
   p.q = (const bf16*)q; p.q_stride = q_stride; p.out = (bf16*)out; p.out_stride = out_stride; p.bt = *b;
   p.heads = a->heads; p.dim = a->dim; p.vdim = a->vdim; p.out_scale = a->out_scale;
   p.k_cache = (const bf16*)k_cache; p.v_cache = (const bf16*)v_cache; p.kv_heads = a->kv_heads; p.chunk = a->chunk;
-  p.scale = a->scale; p.softcap = a->softcap; p.sink = a->sink;
+  p.scale = a->scale; p.softcap = a->softcap; p.sink = a->sink; p.sigmoid = a->sigmoid; p.temp = a->temp; p.bias = a->bias;
   return dispatch_prefill<false>(p, st);
 }
 
@@ -468,7 +481,7 @@ using namespace nqb200;
 extern "C" int64_t nqb200_retention_chunks(int64_t tokens, int64_t batch) { return tokens / kRetChunk + batch; }
 
 extern "C" int nqb200_retention_prefill_supported(const nqb200_retention_desc* r, int64_t stride, int64_t off, int64_t act_stride, int64_t act_col) {
-  return r && r->heads > 0 && r->dim > 0 && r->dim % 8 == 0 && r->dim <= 256 && r->vdim > 0 && r->vdim % 8 == 0 && r->vdim <= 256 &&
+  return r && r->rank <= 0 && r->heads > 0 && r->dim > 0 && r->dim % 8 == 0 && r->dim <= 256 && r->vdim > 0 && r->vdim % 8 == 0 && r->vdim <= 256 &&
                  (int64_t)r->heads * ((r->dim + 63) / 64) * ((r->vdim + 63) / 64) <= 65535 && stride % 8 == 0 && off % 8 == 0 && act_stride % 2 == 0 &&
                  act_col % 2 == 0
              ? 1
@@ -501,6 +514,6 @@ extern "C" int nqb200_retention_prefill(const void* proj, int64_t stride, int64_
   p.q = q; p.q_stride = stride; p.out = (bf16*)act + act_col; p.out_stride = act_stride; p.bt = *b;
   p.heads = r->heads; p.dim = r->dim; p.vdim = r->vdim; p.out_scale = r->out_scale; p.kv_heads = r->heads;
   p.k = q + qk; p.v = q + 2 * qk; p.gate = q + 2 * qk + vv;
-  p.decay = r->decay; p.states = starts; p.eps = r->eps; p.scale = 1.f / sqrtf((float)r->dim);
+  p.decay = r->decay; p.states = starts; p.eps = r->eps; p.norm = r->norm; p.scale = 1.f / sqrtf((float)r->dim);
   return dispatch_prefill<true>(p, st);
 }

@@ -245,10 +245,10 @@ def mixer_decode_supported(att: Optional[_lib.AttentionDesc], ret: Optional[_lib
 
 
 def mixer_decode(proj: torch.Tensor, act: torch.Tensor, att, ret, step) -> None:
-    """One token per sequence, attention and retention in one launch.  ``att = (desc, inv_freq, first projection
-    column, first output column, k_cache, v_cache)``, ``ret = (desc, first projection column, first output column,
-    state)``; either may be None."""
+    """One token per sequence, attention and retention (or gated linear attention) in one launch.  ``att = (desc, rope desc,
+    first projection column, column of the values, first output column, k_cache, v_cache)``, ``ret = (desc, first
+    projection column, first output column, state)``; either may be None."""
     a = (None, None, 0, 0, 0, None, None) if att is None else (
-        ctypes.byref(att[0]), _ptr(att[1]), 2 * att[1].numel(), att[2], att[3], att[4].data_ptr(), att[5].data_ptr())
+        ctypes.byref(att[0]), ctypes.byref(att[1]), att[2], att[3], att[4], att[5].data_ptr(), att[6].data_ptr())
     r = (None, 0, 0, None) if ret is None else (ctypes.byref(ret[0]), ret[1], ret[2], ret[3].data_ptr())
     _call("nqb200_mixer_decode", proj.data_ptr(), proj.stride(0), act.data_ptr(), act.stride(0), *a, *r, ctypes.byref(step.desc))

@@ -59,6 +59,12 @@ class AttentionMixer(nn.Module):
         return _lib.AttentionDesc(self.heads, self.kv_heads, self.dim, self.vdim, self.chunk, self.scale, self.softcap,
                                   self.sink.data_ptr(), self.out_scale, None, None, 0)
 
+    def rope_desc(self) -> _lib.RopeDesc:
+        return _lib.RopeDesc(self.heads, self.kv_heads, self.dim, self.vdim, 2 * self.inv_freq.numel(), 0, self.inv_freq.data_ptr(), None, None, 0.0)
+
+    def value_column(self, col):
+        return col + (self.heads + self.kv_heads) * self.dim
+
     def mix(self, proj, col, act, act_col, layer_step):
         q_off, k_off, v_off = col, col + self.heads * self.dim, col + (self.heads + self.kv_heads) * self.dim
         ops.rope_store(proj, layer_step.k_cache, layer_step.v_cache, self.inv_freq, layer_step.batch, q_off, k_off, v_off, self.heads)
@@ -99,6 +105,9 @@ class SigmoidAttentionMixer(nn.Module):
         return _lib.RopeDesc(self.heads, self.kv_heads, self.dim, self.vdim, self.rot, int(self.interleaved), self.inv_freq.data_ptr(),
                              self.q_norm.data_ptr(), self.k_norm.data_ptr(), self.eps)
 
+    def value_column(self, col):
+        return col + self.heads * self.dim
+
     def mix(self, proj, col, act, act_col, layer_step):
         q_off, k_off = col, col + self.heads * self.dim
         ops.norm_rope(proj, layer_step.k_cache, layer_step.v_cache, self.rope_desc(), layer_step.batch, q_off, k_off, k_off)
@@ -109,6 +118,8 @@ class SigmoidAttentionMixer(nn.Module):
 class RetentionMixer(nn.Module):
     """Linear attention with one fixed decay per head, queries and keys rotated where ``rot_dims`` says so (pairs i, i +
     rot_dims / 2); each head's output is RMS-normalised and gated."""
+
+    state_name = "retention"
 
     def __init__(self, *, heads, dim, vdim, decay, eps, out_scale=1.0, rot_base=1.0, rot_dims=0, device="cpu"):
         super().__init__()
@@ -127,13 +138,14 @@ class RetentionMixer(nn.Module):
         return None
 
     def state_shapes(self):
-        return {"retention": (self.heads, self.dim, self.vdim)}
+        return {self.state_name: (self.heads, self.dim, self.vdim)}
 
     def checkpoint(self, prefix):
         return {}
 
     def desc(self) -> _lib.RetentionDesc:
-        return _lib.RetentionDesc(self.heads, self.dim, self.vdim, self.eps, self.out_scale, self.decay.data_ptr())
+        return _lib.RetentionDesc(self.heads, self.dim, self.vdim, self.eps, self.out_scale, self.decay.data_ptr(), None,
+                                  self.inv_freq.data_ptr(), self.rot)
 
     def rope_desc(self) -> _lib.RopeDesc:
         return _lib.RopeDesc(self.heads, self.heads, self.dim, self.vdim, self.rot, 0, self.inv_freq.data_ptr(), None, None, 0.0)
@@ -147,6 +159,8 @@ class RetentionMixer(nn.Module):
 class GatedLinearMixer(nn.Module):
     """Gated linear attention: a decay per key channel and token, sigmoid(z)^(1 / tau) with z a low-rank projection of the
     input; each head's output is RMS-normalised with a weight and gated."""
+
+    state_name = "gla"
 
     def __init__(self, *, heads, dim, vdim, rank, tau, eps, out_scale=1.0, dtype=torch.bfloat16, device="cpu"):
         super().__init__()
@@ -164,7 +178,11 @@ class GatedLinearMixer(nn.Module):
         return None
 
     def state_shapes(self):
-        return {"gla": (self.heads, self.dim, self.vdim)}
+        return {self.state_name: (self.heads, self.dim, self.vdim)}
+
+    def desc(self) -> _lib.RetentionDesc:
+        return _lib.RetentionDesc(self.heads, self.dim, self.vdim, self.eps, self.out_scale, None, self.norm.data_ptr(), None, 0, self.rank,
+                                  self.tau, self.a2.data_ptr(), self.a2_bias.data_ptr())
 
     def checkpoint(self, prefix):
         return {prefix + "a2": self.a2, prefix + "a2.b": self.a2_bias, prefix + "norm": self.norm}
@@ -189,9 +207,9 @@ class ParallelMixer(nn.Module):
         self._at_once = None
         row = col = 0
         for m in parts.values():
-            if isinstance(m, AttentionMixer):
+            if isinstance(m, (AttentionMixer, SigmoidAttentionMixer)):
                 self._attention = (m, row, col)
-            elif isinstance(m, RetentionMixer):
+            elif isinstance(m, (RetentionMixer, GatedLinearMixer)):
                 self._retention = (m, row, col)
             row += sum(n for _, n in m.in_parts)
             col += m.out_columns
@@ -201,7 +219,6 @@ class ParallelMixer(nn.Module):
             return False
         if self._at_once is None:
             self._at_once = (len(self.parts) == (self._attention is not None) + (self._retention is not None)
-                             and not (self._retention and self._retention[0].rot)
                              and ops.mixer_decode_supported(self._attention and self._attention[0].desc(),
                                                             self._retention and self._retention[0].desc()))
         return self._at_once
@@ -231,8 +248,9 @@ class ParallelMixer(nn.Module):
         """The input product -> the operand of the output product; a decode step in one launch where its kernel takes the sizes."""
         if self._decodes_at_once(proj, layer_step.batch):
             att, ret = self._attention, self._retention
-            ops.mixer_decode(proj, act, att and (att[0].desc(), att[0].inv_freq, att[1], att[2], layer_step.k_cache, layer_step.v_cache),
-                             ret and (ret[0].desc(), ret[1], ret[2], layer_step.state["retention"]), layer_step.batch)
+            ops.mixer_decode(proj, act, att and (att[0].desc(), att[0].rope_desc(), att[1], att[0].value_column(att[1]), att[2], layer_step.k_cache,
+                                                 layer_step.v_cache),
+                             ret and (ret[0].desc(), ret[1], ret[2], layer_step.state[ret[0].state_name]), layer_step.batch)
             return
         row = col = 0
         for m in self.parts.values():

@@ -474,7 +474,7 @@ def test_one_launch_decode_step(att, ret):
         act = torch.full((rows.shape[0], r_col + RH * RV + 2), 7.0, dtype=dtype, device=DEV)
         rows = rows.contiguous()
         if b.max_len == 1:
-            ops.mixer_decode(rows, act, att and (m.desc(), m.inv_freq, a_off, a_col, kc, vc), ret and (rdesc, r_off, r_col, state), b)
+            ops.mixer_decode(rows, act, att and (m.desc(), m.rope_desc(), a_off, m.value_column(a_off), a_col, kc, vc), ret and (rdesc, r_off, r_col, state), b)
             assert (act[:, :a_col] == 7).all() and (act[:, a_col + H * V:r_col] == 7).all() and (act[:, -2:] == 7).all()
             return act
         Step.batch = b

@@ -68,6 +68,8 @@ def weights(c, seed=0):
             w = 0.3 * w              # some choices are negative
         elif name.endswith("router"):
             w = 2.0 * w * shape[-1] ** -0.5
+        elif name.endswith(".down"):
+            w = 0.6 * w * shape[-1] ** -0.5   # where rounding sends a token to another expert, it is not thrown far
         elif "embed" not in name:
             w = 1.3 * w * shape[-1] ** -0.5
         out[name] = w.to(torch.bfloat16)
