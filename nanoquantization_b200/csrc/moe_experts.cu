@@ -179,6 +179,6 @@ extern "C" int nqb200_moe_linear(const void* x, const void* w, void* out, int ki
   a.x = x; a.w = w; a.out = out; a.kind = kind; a.tokens = (int)tokens; a.N = (int)N; a.K = (int)K; a.experts = r->experts; a.top = r->top;
   a.plan = *plan; a.dtype = dtype; a.out_dtype = out_dtype; a.status = status; a.stream = (cudaStream_t)stream;
   if (dtype == NQB200_BF16 && moe_decode_supports(tokens, N, K)) return moe_decode(a);
-  if (dtype == NQB200_BF16 && moe_umma_supports(tokens, N, K, r->top)) return moe_umma(a);
+  if (dtype == NQB200_BF16 && out_dtype == NQB200_BF16 && a.experts <= 1024 && a.experts * N >= 128 && moe_umma_supports(tokens, N, K, r->top)) return moe_umma(a);
   return moe_simple(a);
 }
