@@ -137,6 +137,13 @@ int64_t nqb200_retention_chunks(int64_t tokens, int64_t batch);
 int nqb200_gla_log_decay(const void* low, int64_t low_stride, const void* a2, const float* bias, float* log_decay,
                          int64_t tokens, int64_t channels, int64_t rank, float tau, int dtype, void* stream);
 
+/* Prompts (bf16): gated linear attention (rank > 0) in chunkwise form with norm and gate.  proj holds q | k | v | gate | low
+ * from column off; the result goes to act from column act_col.  scratch: nqb200_gla_scratch() floats. */
+int nqb200_gla_prefill(const void* proj, int64_t stride, int64_t off, void* act, int64_t act_stride, int64_t act_col,
+                       const nqb200_retention_desc* r, float* state, float* scratch, const nqb200_batch* b, void* stream);
+int nqb200_gla_prefill_supported(const nqb200_retention_desc* r, int64_t stride, int64_t off, int64_t act_stride, int64_t act_col);
+int64_t nqb200_gla_scratch(const nqb200_retention_desc* r, int64_t tokens, int64_t batch);
+
 /* out[t * out_stride + h * vdim + c] = out_scale * o / rms(o over the head) * weight[c] * silu(gate[t * gate_stride + h *
  * vdim + c]); weight [vdim] or NULL. */
 int nqb200_head_norm_gate(const float* o, const void* gate, int64_t gate_stride, const float* weight, void* out, int64_t out_stride,

@@ -131,6 +131,9 @@ MIXER_SIGNATURES = {
     "nqb200_retention_prefill": (_int, [_vp, _i64, _i64, _vp, _i64, _i64, _ret, _vp, _vp, _step, _vp]),
     "nqb200_retention_prefill_supported": (_int, [_ret, _i64, _i64, _i64, _i64]),
     "nqb200_retention_chunks": (_i64, [_i64, _i64]),
+    "nqb200_gla_prefill": (_int, [_vp, _i64, _i64, _vp, _i64, _i64, _ret, _vp, _vp, _step, _vp]),
+    "nqb200_gla_prefill_supported": (_int, [_ret, _i64, _i64, _i64, _i64]),
+    "nqb200_gla_scratch": (_i64, [_ret, _i64, _i64]),
     "nqb200_dense_decode": (_int, [_vp, _vp, _vp, _i64, _i64, _i64, _int, _f32, _vp]),
     "nqb200_dense_decode_gelu_table": (_int, [_vp, _vp, _vp, _vp, _i64, _i64, _vp, _i64, _i64, _i64, _vp]),
     "nqb200_dense_decode_glu": (_int, [_vp, _vp, _vp, _i64, _i64, _i64, _f32, _vp]),

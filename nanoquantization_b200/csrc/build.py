@@ -19,8 +19,8 @@ MIXERS_PATH = os.path.join(LIB_DIR, "libnqb200_mixers.so")
 MOE_PATH = os.path.join(LIB_DIR, "libnqb200_moe.so")
 SOURCES = ["api.cu", "unpack_dequant.cu", "gemm_decode.cu", "gemm_stream.cu", "gemm_umma_prefill.cu", "gemm_umma_pair.cu", "quantize_pack.cu", "fused_elementwise.cu", "peer_allreduce.cu"]
 HEADERS = ["common.cuh", "tma_utils.cuh", "umma_utils.cuh", os.path.join(ROOT, "include", "nqb200.h")]
-MIXER_SOURCES = ["mixer_norm.cu", "mixer_attention.cu", "mixer_recurrent.cu", "mixer_dense.cu", "mixer_decode.cu", "mixer_prefill.cu", "mixer_attention_umma.cu"]
-MIXER_HEADERS = ["common.cuh", "mixers.cuh", "tma_utils.cuh", "umma_utils.cuh", os.path.join(ROOT, "include", "nqb200.h"), os.path.join(ROOT, "include", "nqb200_mixers.h")]
+MIXER_SOURCES = ["mixer_norm.cu", "mixer_attention.cu", "mixer_recurrent.cu", "mixer_dense.cu", "mixer_decode.cu", "mixer_prefill.cu", "mixer_attention_umma.cu", "mixer_gla.cu"]
+MIXER_HEADERS = ["common.cuh", "mixers.cuh", "mma_utils.cuh", "tma_utils.cuh", "umma_utils.cuh", os.path.join(ROOT, "include", "nqb200.h"), os.path.join(ROOT, "include", "nqb200_mixers.h")]
 MOE_SOURCES = ["moe_route.cu", "moe_experts.cu", "moe_umma.cu"]
 MOE_HEADERS = MIXER_HEADERS + ["moe.cuh", os.path.join(ROOT, "include", "nqb200_moe.h")]
 LIBRARIES = {LIB_PATH: (SOURCES, HEADERS), MIXERS_PATH: (MIXER_SOURCES, MIXER_HEADERS), MOE_PATH: (MOE_SOURCES, MOE_HEADERS)}

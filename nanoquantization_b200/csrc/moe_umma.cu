@@ -8,11 +8,13 @@
 // tile costs what it holds and a step of few tokens streams the weights past a narrow tile.  The tiles of all experts are
 // numbered, feature tiles fastest (they share the pairs' rows), and dealt to the persistent clusters in turn.
 //
-//   warp 0        TMA: the weight tile, and the pairs' rows: gathered by token for the first linear (tile::gather4, a lane
-//                 fetches four rows), contiguous for the second.  A ring of five stages of 64 k.
+//   warp 0        TMA: the weight tile, and for the second linear the pairs' rows, which are contiguous.  A ring of five
+//                 stages of 64 k.
 //   warp 1        the leader's: one thread issues the MMAs; the other CTA's: reports its landed stages to the leader.
 //   warps 2-9     epilogue: accumulator (two of them take turns) -> gelu or the pair's weight -> 16 bits in shared memory,
 //                 [pair][feature] -> rows of 256 bytes to their places in the output.
+//   warps 10-13   first linear: the pairs' rows, gathered by token with cp.async into the swizzled layout, two stages ahead
+//                 of what they report (TMA's gather of four rows per instruction took 1.4 us per stage of 128 rows).
 //
 // Every wait is bounded; on expiry NQB200_ERR_WAIT_TIMEOUT goes to the status word, all roles drain and tensor memory is
 // released.
@@ -23,17 +25,18 @@
 namespace nqb200 {
 namespace moe {
 
-constexpr int kStages = 5, kEpiWarps = 8, kThreads = (2 + kEpiWarps) * 32, kMaxExperts = 1024;
+constexpr int kStages = 5, kEpiWarps = 8, kLoadWarps = 4, kMaxExperts = 1024;
 constexpr int kTile = 256, kStepK = 64;
 constexpr int kABytes = 128 * kStepK * 2, kStageBytes = 2 * kABytes;
 constexpr int kOffOut = kStages * kStageBytes, kRound = 128, kOutBytes = kRound * 128 * 2;
 constexpr int kSmem = kOffOut + kOutBytes + 1024;
 constexpr int kTmemCols = 512;
+constexpr int kAhead = 2;   // stages between a gather and its report
 
 struct Params {
   const int32_t* offsets; const int32_t* order; const float* weight;
-  bf16* out;
-  int kind, N, K, experts, top, ntn, steps, clusters;
+  const bf16* x; bf16* out;
+  int N, K, experts, top, ntn, steps, clusters;
   int* status;
 };
 
@@ -63,9 +66,9 @@ __device__ __forceinline__ void umma_ss_pair(uint32_t d_tmem, uint32_t a_lo, uin
                " tcgen05.mma.cta_group::2.kind::f16 [%0], a, b, %4, p;\n}"
                ::"r"(d_tmem), "r"(a_lo), "r"(b_lo), "r"(hi), "r"(idesc), "r"(accumulate) : "memory");
 }
-__device__ __forceinline__ void tma_gather4(uint32_t dst, const CUtensorMap* map, int col, int r0, int r1, int r2, int r3, uint32_t bar) {
-  asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.tile::gather4.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5, %6, %7}], [%2];"
-               ::"r"(dst), "l"(map), "r"(bar), "r"(col), "r"(r0), "r"(r1), "r"(r2), "r"(r3) : "memory");
+__device__ __forceinline__ void copy16(uint32_t dst, const void* src, bool ok) {   // zeros where not ok
+  const int n = ok ? 16 : 0;
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(n));
 }
 // Barrier of the epilogue's threads that tells all of them whether all of them are well.
 __device__ __forceinline__ bool epi_all(bool ok) {
@@ -94,7 +97,10 @@ __device__ __forceinline__ Item locate(const Params& p, const int* tiles, int it
   return it;
 }
 
-__global__ void __launch_bounds__(kThreads, 1) moe_umma_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__ CUtensorMap tm_x, const Params p) {
+template <bool UP>
+__global__ void __launch_bounds__((2 + kEpiWarps + (UP ? kLoadWarps : 0)) * 32, 1) moe_umma_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__ CUtensorMap tm_x, const __grid_constant__ CUtensorMap tm_x128,
+                const Params p) {
+  constexpr int kThreads = (2 + kEpiWarps + (UP ? kLoadWarps : 0)) * 32, kLocal = 1 + (UP ? kLoadWarps : 0);
   extern __shared__ uint8_t smem_raw[];
   __shared__ __align__(8) uint64_t bar_full[kStages], bar_free[kStages], bar_dfull[2], bar_dempty[2], bar_drain;
   __shared__ int tiles[kMaxExperts], s_rows[2][kTile];
@@ -110,7 +116,7 @@ __global__ void __launch_bounds__(kThreads, 1) moe_umma_kernel(const __grid_cons
   if (threadIdx.x == 0) {
     for (int s = 0; s < kStages; ++s) {
       // the leader's stage is complete when its own copies have landed and the other CTA has reported its own
-      mbar_init(smem_u32(&bar_full[s]), rank == 0 ? 2 : 1);
+      mbar_init(smem_u32(&bar_full[s]), kLocal + (rank == 0 ? 1 : 0));
       mbar_init(smem_u32(&bar_free[s]), 1);
     }
     for (int d = 0; d < 2; ++d) { mbar_init(smem_u32(&bar_dfull[d]), 1); mbar_init(smem_u32(&bar_dempty[d]), 2 * kEpiWarps); }
@@ -144,16 +150,15 @@ __global__ void __launch_bounds__(kThreads, 1) moe_umma_kernel(const __grid_cons
 
   if (warp == 0) {
     // ------------------------------------------------------------------ TMA
-    if (lane == 0) { prefetch_tmap(&tm_w); prefetch_tmap(&tm_x); }
+    if (lane == 0) { prefetch_tmap(&tm_w); prefetch_tmap(&tm_x); prefetch_tmap(&tm_x128); }
     int n = 0;            // stages filled so far
     bool ok = true;
     for (int item = cluster; ok && item < items; item += p.clusters) {
       const Item it = locate(p, tiles, item);
       const int th = it.nt / 2, w_row = it.expert * p.N + it.feature + (int)rank * 128, first = (int)rank * th;
-      int rows[4];
-#pragma unroll
-      for (int i = 0; i < 4; ++i) rows[i] = p.kind == NQB200_MOE_UP ? p.order[it.lo + min(first + 4 * lane + i, it.cnt - 1)] / p.top : 0;
-      const uint32_t bytes = (uint32_t)kABytes + (uint32_t)th * 128u;
+      // one box of 128 rows where that is not far too many (what lies behind the tile is not used): boxes cost by the piece
+      const bool one = th > 48;
+      const uint32_t bytes = (uint32_t)kABytes + (UP ? 0u : one ? 128u * 128u : (uint32_t)th * 128u);
       for (int k = 0; k < p.steps; ++k, ++n) {
         const int s = n % kStages;
         const uint32_t st = smem + s * kStageBytes, bar = smem_u32(&bar_full[s]);
@@ -164,11 +169,8 @@ __global__ void __launch_bounds__(kThreads, 1) moe_umma_kernel(const __grid_cons
         ok = __shfl_sync(0xFFFFFFFFu, (int)ok, 0) != 0;
         if (!ok) break;
         if (lane == 0) tma_load_2d(st, &tm_w, k * kStepK, w_row, bar);
-        if (p.kind == NQB200_MOE_UP) {
-          if (4 * lane < th) tma_gather4(st + kABytes + lane * 512, &tm_x, k * kStepK, rows[0], rows[1], rows[2], rows[3], bar);
-        } else {
-          if (16 * lane < th) tma_load_2d(st + kABytes + lane * 2048, &tm_x, k * kStepK, it.lo + first + 16 * lane, bar);
-        }
+        if (!UP && one && lane == 0) tma_load_2d(st + kABytes, &tm_x128, k * kStepK, it.lo + first, bar);
+        if (!UP && !one && 16 * lane < th) tma_load_2d(st + kABytes + lane * 2048, &tm_x, k * kStepK, it.lo + first + 16 * lane, bar);
       }
     }
     // do not leave while a copy may still be landing
@@ -214,6 +216,42 @@ __global__ void __launch_bounds__(kThreads, 1) moe_umma_kernel(const __grid_cons
           if (++s == kStages) { s = 0; phase ^= 1u; }
         }
     }
+  } else if (UP && warp >= 2 + kEpiWarps) {
+    // ------------------------------------------------------------ gathered rows
+    const int t = threadIdx.x - (2 + kEpiWarps) * 32, chunk = t & 7, row0 = t >> 3;
+    const uint32_t dst0 = smem + kABytes + row0 * 128 + ((chunk ^ (row0 & 7)) << 4);   // rows 16 apart keep the same swizzle
+    int n = 0;
+    bool ok = true;
+    auto report = [&](int m) {   // copies of stage m have landed: the tensor core reads them through the async proxy
+      asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+      __syncwarp();
+      if (lane == 0) mbar_arrive(smem_u32(&bar_full[m % kStages]));
+    };
+    for (int item = cluster; ok && item < items; item += p.clusters) {
+      const Item it = locate(p, tiles, item);
+      const int th = it.nt / 2, first = (int)rank * th;
+      const bf16* src[8];
+#pragma unroll
+      for (int i = 0; i < 8; ++i)
+        src[i] = p.x + (size_t)(p.order[it.lo + min(first + row0 + 16 * i, it.cnt - 1)] / p.top) * p.K + chunk * 8;
+      for (int k = 0; k < p.steps; ++k, ++n) {
+        const int s = n % kStages;
+        if (n >= kStages) ok = wait_bar(&bar_free[s], ((n / kStages) - 1) & 1, s_abort, p.status);
+        ok = __all_sync(0xFFFFFFFFu, ok) != 0;
+        if (!ok) break;
+        const bool in = k * kStepK + chunk * 8 < p.K;   // K is a multiple of 8
+#pragma unroll
+        for (int i = 0; i < 8; ++i)
+          if (16 * i < th) copy16(dst0 + s * kStageBytes + i * 2048, in ? src[i] + k * kStepK : src[i], in);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        if (n >= kAhead) {
+          asm volatile("cp.async.wait_group %0;" ::"n"(kAhead) : "memory");
+          report(n - kAhead);
+        }
+      }
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    for (int m = n > kAhead ? n - kAhead : 0; m < n; ++m) report(m);
   } else {
     // -------------------------------------------------------------- epilogue
     const int quarter = warp & 3, half = (warp - 2) >> 2, tid = threadIdx.x - 64;
@@ -224,9 +262,9 @@ __global__ void __launch_bounds__(kThreads, 1) moe_umma_kernel(const __grid_cons
       const Item it = locate(p, tiles, item);
       const int buf = li & 1;
       if (tid < it.cnt) {   // where pair `tid` of the tile goes, and its weight
-        const int pair = p.kind == NQB200_MOE_DOWN ? p.order[it.lo + tid] : it.lo + tid;
+        const int pair = UP ? it.lo + tid : p.order[it.lo + tid];
         s_rows[buf][tid] = pair;
-        s_weight[buf][tid] = p.kind == NQB200_MOE_DOWN ? p.weight[pair] : 1.f;
+        s_weight[buf][tid] = UP ? 1.f : p.weight[pair];
       }
       const bool ok = wait_bar(&bar_dfull[buf], (li >> 1) & 1, s_abort, p.status);
       if (!epi_all(ok)) break;
@@ -240,7 +278,7 @@ __global__ void __launch_bounds__(kThreads, 1) moe_umma_kernel(const __grid_cons
           tmem_ld_32x32b_x16(lanes + buf * 256 + c, d);
           tc_wait_ld();
           uint8_t* dst = stage + (size_t)(c - c0) * 256 + (quarter * 32 + lane) * 2;
-          if (p.kind == NQB200_MOE_UP) {
+          if (UP) {
 #pragma unroll
             for (int i = 0; i < 16; ++i) *reinterpret_cast<bf16*>(dst + i * 256) = __float2bfloat16_rn(gelu_erf_f(__uint_as_float(d[i])));
           } else {
@@ -279,28 +317,30 @@ bool moe_umma_supports(int64_t tokens, int64_t N, int64_t K, int64_t top) {
 int moe_umma(const MoeArgs& a) {
   using namespace moe;
   if (a.experts > kMaxExperts) return NQB200_ERR_TOO_LARGE;
-  alignas(64) CUtensorMap tw, tx;
+  alignas(64) CUtensorMap tw, tx, txl;
   const int64_t pairs = (int64_t)a.tokens * a.top;
   const bool up = a.kind == NQB200_MOE_UP;
   bool ok = encode_2d(&tw, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.w, (uint64_t)a.experts * a.N, a.K, 128, kStepK, CU_TENSOR_MAP_SWIZZLE_128B);
-  ok = ok && encode_2d(&tx, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.x, up ? a.tokens : pairs, a.K, up ? 1 : 16, kStepK, CU_TENSOR_MAP_SWIZZLE_128B);
+  ok = ok && encode_2d(&tx, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.x, up ? a.tokens : pairs, a.K, 16, kStepK, CU_TENSOR_MAP_SWIZZLE_128B);   // second linear
+  ok = ok && encode_2d(&txl, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.x, up ? a.tokens : pairs, a.K, 128, kStepK, CU_TENSOR_MAP_SWIZZLE_128B);
   if (!ok) return NQB200_ERR_LAUNCH;
   Params p = {};
-  p.offsets = a.plan.offsets; p.order = a.plan.order; p.weight = a.plan.weight; p.out = (bf16*)a.out;
-  p.kind = a.kind; p.N = a.N; p.K = a.K; p.experts = a.experts; p.top = a.top;
+  p.offsets = a.plan.offsets; p.order = a.plan.order; p.weight = a.plan.weight; p.x = (const bf16*)a.x; p.out = (bf16*)a.out;
+  p.N = a.N; p.K = a.K; p.experts = a.experts; p.top = a.top;
   p.ntn = (a.N + kTile - 1) / kTile; p.steps = (a.K + kStepK - 1) / kStepK; p.status = a.status;
   const int64_t most = ((pairs < a.experts ? pairs : a.experts) + pairs / kTile) * p.ntn;
   p.clusters = (int)(most < kNumSMs / 2 ? most : kNumSMs / 2);
-  if (cudaFuncSetAttribute(moe_umma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem) != cudaSuccess) { cudaGetLastError(); return NQB200_ERR_LAUNCH; }
+  auto kernel = up ? moe_umma_kernel<true> : moe_umma_kernel<false>;
+  if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem) != cudaSuccess) { cudaGetLastError(); return NQB200_ERR_LAUNCH; }
   cudaLaunchConfig_t cfg = {};
-  cfg.gridDim = dim3((unsigned)(2 * p.clusters)); cfg.blockDim = dim3(kThreads); cfg.dynamicSmemBytes = kSmem; cfg.stream = a.stream;
+  cfg.gridDim = dim3((unsigned)(2 * p.clusters)); cfg.blockDim = dim3((2 + kEpiWarps + (up ? kLoadWarps : 0)) * 32); cfg.dynamicSmemBytes = kSmem; cfg.stream = a.stream;
   cudaLaunchAttribute attr[2];
   attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
   attr[0].val.programmaticStreamSerializationAllowed = 1;
   attr[1].id = cudaLaunchAttributeClusterDimension;
   attr[1].val.clusterDim.x = 2; attr[1].val.clusterDim.y = 1; attr[1].val.clusterDim.z = 1;
   cfg.attrs = attr; cfg.numAttrs = 2;
-  if (cudaLaunchKernelEx(&cfg, moe_umma_kernel, tw, tx, p) != cudaSuccess) { cudaGetLastError(); return NQB200_ERR_LAUNCH; }
+  if (cudaLaunchKernelEx(&cfg, kernel, tw, tx, txl, p) != cudaSuccess) { cudaGetLastError(); return NQB200_ERR_LAUNCH; }
   return NQB200_OK;
 }
 

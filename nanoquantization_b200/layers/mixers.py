@@ -163,11 +163,19 @@ def retention_gated(proj: torch.Tensor, off: int, desc: _lib.RetentionDesc, deca
 
 def gla_gated(proj: torch.Tensor, off: int, m, state: torch.Tensor, act: torch.Tensor, act_col: int, step) -> None:
     """Gated linear attention with norm and gate of mixer ``m``: ``proj`` holds q | k | v | gate | low-rank decay input from
-    column ``off``, the result goes to ``act`` from column ``act_col``."""
+    column ``off``, the result goes to ``act`` from column ``act_col``.  Prompts in bfloat16 run chunkwise on the tensor cores,
+    the rest token by token."""
     _, heads, dim, vdim = state.shape
     k_off, v_off = off + heads * dim, off + 2 * heads * dim
     g_off = v_off + heads * vdim
     a_off = g_off + heads * vdim
+    lib, desc = _lib.load_mixers(), m.desc()
+    if (proj.dtype == torch.bfloat16 and step.max_len >= RETENTION_PREFILL_TOKENS
+            and lib.nqb200_gla_prefill_supported(ctypes.byref(desc), proj.stride(0), off, act.stride(0), act_col)):
+        scratch = torch.empty(lib.nqb200_gla_scratch(ctypes.byref(desc), step.num_tokens, step.batch), dtype=torch.float32, device=proj.device)
+        _call("nqb200_gla_prefill", proj.data_ptr(), proj.stride(0), off, act.data_ptr(), act.stride(0), act_col, ctypes.byref(desc),
+              state.data_ptr(), scratch.data_ptr(), ctypes.byref(step.desc))
+        return
     log_decay = gla_log_decay(proj[:, a_off:a_off + m.rank], m.a2, m.a2_bias, m.tau)
     o = retention(proj, off, k_off, v_off, None, state, step, log_decay)
     head_norm_gate(o, proj[:, g_off:a_off], act[:, act_col:act_col + heads * vdim], m.eps, m.out_scale, m.norm)

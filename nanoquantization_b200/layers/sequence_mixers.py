@@ -198,7 +198,8 @@ class ParallelMixer(nn.Module):
     def __init__(self, width: int, parts: dict, *, dtype, device="cpu", beta=1.0, prefixes=None):
         super().__init__()
         self.parts, self.beta, self.prefixes = nn.ModuleDict(parts), float(beta), prefixes or {k: k + "." for k in parts}
-        self.rows = sum(n for m in parts.values() for _, n in m.in_parts)
+        # rows of zeros fill up to a multiple of 8: rows of the product then start on 16-byte boundaries
+        self.rows = -(-sum(n for m in parts.values() for _, n in m.in_parts) // 8) * 8
         self.columns = sum(m.out_columns for m in parts.values())
         _buffer(self, "w_in", self.rows, width, dtype=dtype, device=device)
         _buffer(self, "w_out", width, self.columns, dtype=dtype, device=device)

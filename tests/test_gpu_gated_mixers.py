@@ -75,8 +75,7 @@ def mix(r, mixer, inputs, dtype, state=None, width_out=None, col=8):
     def fn(b, rows):
         Step.batch = b
         act = torch.full((rows.shape[0], mixer.out_columns), 7.0, dtype=dtype, device=DEV)
-        proj = rows.contiguous()
-        assert proj.shape[1] == width
+        proj = torch.nn.functional.pad(rows, (0, layer.rows - width)).contiguous()
         layer.mix(proj, act, Step)
         return act
     return r.run([p.to(dtype) for p in inputs], fn)
