@@ -40,14 +40,15 @@ __device__ __forceinline__ size_t chunk_id(const nqb200_batch& bt, int b, int c)
 
 constexpr int kDecayChannels = 128, kDecayStep = 16;
 __global__ void __launch_bounds__(kDecayChannels) gla_decay_kernel(const Args a) {
-  extern __shared__ float low_s[];   // [chunk][rank]
+  extern __shared__ float4 low_smem[];
+  float* low_s = reinterpret_cast<float*>(low_smem);   // [rank][chunk]
   grid_launch_dependents();
   grid_dependency_wait();
   const int b = blockIdx.z, t0 = a.bt.cu[b], n = a.bt.cu[b + 1] - t0, first = blockIdx.y * kChunk, rank = a.r.rank;
   if (first >= n) return;
   const int len = min(kChunk, n - first), channels = a.r.heads * a.r.dim;
-  for (int e = threadIdx.x; e < len * rank; e += kDecayChannels)
-    low_s[e] = to_f(a.proj[(size_t)(t0 + first + e / rank) * a.stride + a.l_off + e % rank]);
+  for (int e = threadIdx.x; e < kChunk * rank; e += kDecayChannels)
+    low_s[e % rank * kChunk + e / rank] = to_f(a.proj[(size_t)(t0 + first + min(e / rank, len - 1)) * a.stride + a.l_off + e % rank]);
   __syncthreads();
   const int c = blockIdx.x * kDecayChannels + threadIdx.x;
   if (c >= channels) return;
@@ -60,13 +61,17 @@ __global__ void __launch_bounds__(kDecayChannels) gla_decay_kernel(const Args a)
     for (int i = 0; i < kDecayStep; ++i) z[i] = bias;
     for (int r = 0; r < rank; ++r) {
       const float wr = to_f(w[r]);
+      const float4* lr = reinterpret_cast<const float4*>(low_s + r * kChunk + i0);
 #pragma unroll
-      for (int i = 0; i < kDecayStep; ++i) z[i] += wr * low_s[min(i0 + i, len - 1) * rank + r];
+      for (int i = 0; i < kDecayStep / 4; ++i) {
+        const float4 l = lr[i];
+        z[4 * i] += wr * l.x; z[4 * i + 1] += wr * l.y; z[4 * i + 2] += wr * l.z; z[4 * i + 3] += wr * l.w;
+      }
     }
 #pragma unroll
     for (int i = 0; i < kDecayStep; ++i) {
       if (i0 + i >= len) break;
-      run += log_sigmoid_f(z[i]) * inv_tau;
+      run += (fminf(z[i], 0.f) - log1pf(exp_fast(-fabsf(z[i])))) * inv_tau;
       a.cum[(size_t)(t0 + first + i0 + i) * channels + c] = run;
     }
   }
@@ -228,38 +233,69 @@ __global__ void __launch_bounds__(kThreads, 1) gla_output_kernel(const Args a) {
     ends[e] = d < D ? cum[(size_t)min(w * kBlock + kBlock - 1, len - 1) * channels + d] : 0.f;
   }
   __syncthreads();
-  for (int e = tid; e < kChunk * (DP / 2); e += kThreads) {
-    const int j = e / (DP / 2), d = e % (DP / 2) * 2;
-    float x = 0.f, y = 0.f;
-    if (j < len && d < D) {
-      const float2 bj = *reinterpret_cast<const float2*>(cum + (size_t)j * channels + d);
-      const uint32_t kv = *reinterpret_cast<const uint32_t*>(rows + (size_t)j * a.stride + a.k_off + (size_t)h * D + d);
-      const float* en = ends + (j / kBlock) * DP + d;
-      x = __uint_as_float(kv << 16) * kscale * exp_fast(en[0] - bj.x);
-      y = __uint_as_float(kv & 0xFFFF0000u) * kscale * exp_fast(en[1] - bj.y);
+  {
+    // a thread weighs two neighbouring channels of every RT-th token, 8 tokens' loads under way at once (from places that exist)
+    constexpr int RT = kThreads / (DP / 2);
+    const int d = tid % (DP / 2) * 2, dd = d < D ? d : 0;
+    const float* cb = cum + dd;
+    const bf16* kb = rows + a.k_off + (size_t)h * D + dd;
+    for (int j0 = tid / (DP / 2); j0 < kChunk; j0 += 8 * RT) {
+      float2 bj[8];
+      uint32_t kv[8];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        const int j = min(j0 + i * RT, len - 1);
+        bj[i] = *reinterpret_cast<const float2*>(cb + (size_t)j * channels);
+        kv[i] = *reinterpret_cast<const uint32_t*>(kb + (size_t)j * a.stride);
+      }
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        const int j = j0 + i * RT;
+        const float* en = ends + (j / kBlock) * DP + d;
+        const bool ok = j < len && d < D;
+        const float x = __uint_as_float(kv[i] << 16) * kscale * exp_fast(en[0] - bj[i].x);
+        const float y = __uint_as_float(kv[i] & 0xFFFF0000u) * kscale * exp_fast(en[1] - bj[i].y);
+        *reinterpret_cast<uint32_t*>(ks + j * KS + d) = ok ? pack2(x, y) : 0u;
+      }
     }
-    *reinterpret_cast<uint32_t*>(ks + j * KS + d) = pack2(x, y);
   }
   // this warp's queries: rows g and g + 8 of block `warp`, times exp(b_i - b at the end of the block before)
   const int i0 = warp * kBlock;
   const bool busy = i0 < len;
   const float* ref = warp > 0 ? ends + (warp - 1) * DP : nullptr;
   float q[DP / 16][8];   // [k-step][row g: 2t, 2t + 1; row g + 8; the same 8 channels on]
+  {
+    const float* cb[2];
+    const bf16* qb[2];
 #pragma unroll
-  for (int kt = 0; kt < DP / 16; ++kt)
-#pragma unroll
-    for (int u = 0; u < 4; ++u) {
-      const int row = i0 + g + 8 * (u & 1), d = kt * 16 + 2 * t + 8 * (u >> 1);
-      float x = 0.f, y = 0.f;
-      if (row < len && d < D) {
-        const float2 bi = *reinterpret_cast<const float2*>(cum + (size_t)row * channels + d);
-        const uint32_t qv = *reinterpret_cast<const uint32_t*>(rows + (size_t)row * a.stride + a.q_off + (size_t)h * D + d);
-        x = __uint_as_float(qv << 16) * exp_fast(bi.x - (ref ? ref[d] : 0.f));
-        y = __uint_as_float(qv & 0xFFFF0000u) * exp_fast(bi.y - (ref ? ref[d + 1] : 0.f));
-      }
-      q[kt][2 * u] = x;
-      q[kt][2 * u + 1] = y;
+    for (int r = 0; r < 2; ++r) {
+      const int row = min(i0 + g + 8 * r, len - 1);
+      cb[r] = cum + (size_t)row * channels;
+      qb[r] = rows + (size_t)row * a.stride + a.q_off + (size_t)h * D;
     }
+#pragma unroll
+    for (int k0 = 0; k0 < DP / 16; k0 += 2) {
+      float2 bi[2][4];
+      uint32_t qv[2][4];
+#pragma unroll
+      for (int k = 0; k < 2; ++k)
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+          const int d = (k0 + k) * 16 + 2 * t + 8 * (u >> 1), dd = d < D ? d : 0;
+          bi[k][u] = *reinterpret_cast<const float2*>(cb[u & 1] + dd);
+          qv[k][u] = *reinterpret_cast<const uint32_t*>(qb[u & 1] + dd);
+        }
+#pragma unroll
+      for (int k = 0; k < 2; ++k)
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+          const int d = (k0 + k) * 16 + 2 * t + 8 * (u >> 1);
+          const bool ok = d < D && i0 + g + 8 * (u & 1) < len;
+          q[k0 + k][2 * u] = ok ? __uint_as_float(qv[k][u] << 16) * exp_fast(bi[k][u].x - (ref ? ref[d] : 0.f)) : 0.f;
+          q[k0 + k][2 * u + 1] = ok ? __uint_as_float(qv[k][u] & 0xFFFF0000u) * exp_fast(bi[k][u].y - (ref ? ref[d + 1] : 0.f)) : 0.f;
+        }
+    }
+  }
   bool steep = false;
   if (busy)
     for (int d = lane; d < D; d += 32) steep |= (ref ? ref[d] : 0.f) - ends[warp * DP + d] > kMaxSpan;
@@ -387,14 +423,24 @@ __global__ void __launch_bounds__(kThreads, 1) gla_output_kernel(const Args a) {
     if (row >= len) continue;
     bf16* dst = a.act + (size_t)(t0 + first + row) * a.act_stride + (size_t)h * V;
     const bf16* gp = rows + (size_t)row * a.stride + a.g_off + (size_t)h * V;
+    constexpr int U = VP / 8 < 16 ? VP / 8 : 16;   // loads under way at once (from places that exist)
 #pragma unroll
-    for (int i = 0; i < VP / 8; ++i) {
-      const int c = i * 8 + 2 * t;
-      if (c >= V) break;
-      const uint32_t gw = *reinterpret_cast<const uint32_t*>(gp + c);
-      const float gx = __uint_as_float(gw << 16), gy = __uint_as_float(gw & 0xFFFF0000u);
-      const float wx = a.r.norm ? a.r.norm[c] : 1.f, wy = a.r.norm ? a.r.norm[c + 1] : 1.f;
-      *reinterpret_cast<uint32_t*>(dst + c) = pack2(O[i][2 * r] * f * wx * (gx * sigmoid_fast(gx)), O[i][2 * r + 1] * f * wy * (gy * sigmoid_fast(gy)));
+    for (int i1 = 0; i1 < VP / 8; i1 += U) {
+      uint32_t gw[U];
+      float2 nw[U];
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const int c = (i1 + u) * 8 + 2 * t, cc = c < V ? c : 0;
+        gw[u] = *reinterpret_cast<const uint32_t*>(gp + cc);
+        nw[u] = a.r.norm ? *reinterpret_cast<const float2*>(a.r.norm + cc) : make_float2(1.f, 1.f);
+      }
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const int i = i1 + u, c = i * 8 + 2 * t;
+        const float gx = __uint_as_float(gw[u] << 16), gy = __uint_as_float(gw[u] & 0xFFFF0000u);
+        if (c < V)
+          *reinterpret_cast<uint32_t*>(dst + c) = pack2(O[i][2 * r] * f * nw[u].x * (gx * sigmoid_fast(gx)), O[i][2 * r + 1] * f * nw[u].y * (gy * sigmoid_fast(gy)));
+      }
     }
   }
 }

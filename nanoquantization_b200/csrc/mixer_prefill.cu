@@ -272,19 +272,30 @@ __global__ void __launch_bounds__(kThreads, 1) prefill_kernel(const PrefillArgs 
     const size_t tok = (size_t)(t0 + pr[r] - pos0);
     bf16* dst = a.out + tok * a.out_stride + (size_t)h * a.vdim;
     const bf16* gp = RET ? a.gate + tok * a.q_stride + (size_t)h * a.vdim : nullptr;
+    constexpr int U = VP / 8 < 16 ? VP / 8 : 16;   // loads under way at once (from places that exist)
 #pragma unroll
-    for (int i = 0; i < VP / 8; ++i) {
-      const int c = i * 8 + 2 * t;
-      if (c >= a.vdim) break;
-      float x = O[i][2 * r] * f, y = O[i][2 * r + 1] * f;
+    for (int i1 = 0; i1 < VP / 8; i1 += U) {
+      uint32_t gw[U];
+      float2 nw[U];
       if (RET) {
-        if (a.norm) { x *= a.norm[c]; y *= a.norm[c + 1]; }
-        const uint32_t gw = *reinterpret_cast<const uint32_t*>(gp + c);
-        const float gx = __uint_as_float(gw << 16), gy = __uint_as_float(gw & 0xFFFF0000u);
-        x *= gx * sigmoid_fast(gx);
-        y *= gy * sigmoid_fast(gy);
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+          const int c = (i1 + u) * 8 + 2 * t, cc = c < a.vdim ? c : 0;
+          gw[u] = *reinterpret_cast<const uint32_t*>(gp + cc);
+          nw[u] = a.norm ? *reinterpret_cast<const float2*>(a.norm + cc) : make_float2(1.f, 1.f);
+        }
       }
-      *reinterpret_cast<uint32_t*>(dst + c) = pack2(x, y);
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const int i = i1 + u, c = i * 8 + 2 * t;
+        float x = O[i][2 * r] * f, y = O[i][2 * r + 1] * f;
+        if (RET) {
+          const float gx = __uint_as_float(gw[u] << 16), gy = __uint_as_float(gw[u] & 0xFFFF0000u);
+          x *= nw[u].x * (gx * sigmoid_fast(gx));
+          y *= nw[u].y * (gy * sigmoid_fast(gy));
+        }
+        if (c < a.vdim) *reinterpret_cast<uint32_t*>(dst + c) = pack2(x, y);
+      }
     }
   }
 }
