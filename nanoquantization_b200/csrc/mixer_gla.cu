@@ -94,7 +94,6 @@ __global__ void __launch_bounds__(kThreads) gla_chunk_kernel(const Args a) {
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3, wd = warp & 3, wv = warp >> 2;
   const float kscale = 1.f / sqrtf((float)D);
   const float* cum = a.cum + (size_t)(t0 + first) * channels + h * D;
-  for (int e = tid; e < 64 * (VP - V); e += kThreads) vs[(e / (VP - V)) * VS + V + e % (VP - V)] = __float2bfloat16_rn(0.f);
   float acc[NT][4];
 #pragma unroll
   for (int i = 0; i < NT; ++i)
@@ -109,10 +108,10 @@ __global__ void __launch_bounds__(kThreads) gla_chunk_kernel(const Args a) {
   if (live) last = *reinterpret_cast<const float2*>(cum + (size_t)(len - 1) * channels + d0 + c2);
   for (int j0 = 0; j0 < len; j0 += 64) {
     __syncthreads();
-    for (int e = tid; e < 64 * V8; e += kThreads) {
-      const int r = e / V8, c = e % V8;
-      const bool ok = j0 + r < len;
-      cp16(smem_addr(vs + r * VS + c * 8), a.proj + (size_t)(t0 + first + (ok ? j0 + r : 0)) * a.stride + a.v_off + (size_t)h * V + c * 8, ok);
+    for (int e = tid; e < 64 * (VP / 8); e += kThreads) {   // columns past V become zeros
+      const int r = e / (VP / 8), c = e % (VP / 8);
+      const bool ok = j0 + r < len && c < V8;
+      cp16(smem_addr(vs + r * VS + c * 8), a.proj + (size_t)(t0 + first + (ok ? j0 + r : 0)) * a.stride + a.v_off + (size_t)h * V + (ok ? c * 8 : 0), ok);
     }
     cp_commit();
     float2 bb[8];
@@ -194,12 +193,11 @@ __global__ void __launch_bounds__(256) gla_scan_kernel(const Args a) {
 
 template <int DP, int VP>
 __global__ void __launch_bounds__(kThreads, 1) gla_output_kernel(const Args a) {
-  constexpr int KS = DP + 8, VS = VP + 8, SR = 64;   // SR: rows of the state per pass
+  constexpr int KS = DP + 8, VS = VP + 8, SR = 64, SLICES = DP / SR;   // SR: channels of the state per pass
   extern __shared__ __align__(16) uint8_t smem_raw[];
   bf16* ks = reinterpret_cast<bf16*>(smem_raw);      // [chunk][DP] keys, weighted to the end of their block
-  bf16* vs = ks + kChunk * KS;                       // [chunk][VP]
-  bf16* ss = vs + kChunk * VS;                       // [high part, rest][SR][VP]
-  float* ends = reinterpret_cast<float*>(ss + 2 * SR * VS);   // [blocks][DP] b at the end of each block
+  bf16* buf = ks + kChunk * KS;                      // two tiles of 128 x VP, in turn: slices of the state ([high part, rest][SR][VP]), the values
+  float* ends = reinterpret_cast<float*>(buf + 2 * kChunk * VS);   // [blocks][DP] b at the end of each block
   grid_launch_dependents();
   grid_dependency_wait();
   const int b = blockIdx.z, h = blockIdx.y, chunk = blockIdx.x, t0 = a.bt.cu[b], n = a.bt.cu[b + 1] - t0, first = chunk * kChunk;
@@ -212,22 +210,27 @@ __global__ void __launch_bounds__(kThreads, 1) gla_output_kernel(const Args a) {
   const bf16* S = a.starts + (chunk_id(a.bt, b, chunk) * a.r.heads + h) * (size_t)(2 * D * V);
   const bool has_state = chunk > 0 || a.bt.pos0[b] != 0;
 
-  auto load_state = [&](int d0) {
-    for (int e = tid; e < 2 * SR * V8; e += kThreads) {
-      const int part = e / (SR * V8), r = (e / V8) % SR, c = e % V8;
-      const bool ok = d0 + r < D;
-      cp16(smem_addr(ss + (part * SR + r) * VS + c * 8), S + ((size_t)part * D + (ok ? d0 + r : 0)) * V + c * 8, ok);
+  const int slices = has_state ? SLICES : 0;
+  auto load = [&](int i) {   // tile i; columns past V and what lies outside the chunk become zeros
+    bf16* dst = buf + (i & 1) * kChunk * VS;
+    for (int e = tid; e < kChunk * (VP / 8); e += kThreads) {
+      const int r = e / (VP / 8), c = e % (VP / 8);
+      const bf16* src;
+      bool ok = c < V8;
+      if (i < slices) {
+        const int d = i * SR + r % SR;
+        ok = ok && d < D;
+        src = S + ((size_t)(r / SR) * D + (ok ? d : 0)) * V + (ok ? c * 8 : 0);
+      } else {
+        ok = ok && r < len;
+        src = rows + (size_t)(ok ? r : 0) * a.stride + a.v_off + (size_t)h * V + (ok ? c * 8 : 0);
+      }
+      cp16(smem_addr(dst + r * VS + c * 8), src, ok);
     }
     cp_commit();
   };
-  for (int e = tid; e < kChunk * V8; e += kThreads) {
-    const int r = e / V8, c = e % V8;
-    const bool ok = r < len;
-    cp16(smem_addr(vs + r * VS + c * 8), rows + (size_t)(ok ? r : 0) * a.stride + a.v_off + (size_t)h * V + c * 8, ok);
-  }
-  cp_commit();
-  if (has_state) load_state(0);
-  for (int e = tid; e < (kChunk + 2 * SR) * (VP - V); e += kThreads) vs[(e / (VP - V)) * VS + V + e % (VP - V)] = __float2bfloat16_rn(0.f);
+  load(0);
+  if (slices > 0) load(1);
   for (int e = tid; e < kBlocks * DP; e += kThreads) {
     const int w = e / DP, d = e % DP;
     ends[e] = d < D ? cum[(size_t)min(w * kBlock + kBlock - 1, len - 1) * channels + d] : 0.f;
@@ -300,27 +303,67 @@ __global__ void __launch_bounds__(kThreads, 1) gla_output_kernel(const Args a) {
   if (busy)
     for (int d = lane; d < D; d += 32) steep |= (ref ? ref[d] : 0.f) - ends[warp * DP + d] > kMaxSpan;
   steep = __any_sync(0xFFFFFFFFu, steep);
-  __syncthreads();   // the keys are in place
-
-  // scores, block by block, as operands of the product with the values
-  uint32_t P[kBlocks][4];
+  float O[VP / 8][4];
+#pragma unroll
+  for (int i = 0; i < VP / 8; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) O[i][e] = 0.f;
   const uint32_t k_lane = smem_addr(ks) + (((lane & 7) + ((lane >> 4) << 3)) * KS + ((lane >> 3) & 1) * 8) * 2;
+  const uint32_t v_lane = (((lane & 7) + (((lane >> 3) & 1) << 3)) * VS + (lane >> 4) * 8) * 2;
+  auto product = [&](const uint32_t (&pa)[4], uint32_t base) {   // O += 16 x 16 operand times 16 rows of a tile
 #pragma unroll
-  for (int J = 0; J < kBlocks; ++J) {
+    for (int nt = 0; nt < VP / 16; ++nt) {
+      uint32_t vb[4];
+      ldsm4t(vb, base + nt * 32);
+      mma(O[2 * nt], pa, vb[0], vb[1]);
+      mma(O[2 * nt + 1], pa, vb[2], vb[3]);
+    }
+  };
+  // queries against the state at the chunk's start
 #pragma unroll
-    for (int u = 0; u < 4; ++u) P[J][u] = 0;
-    if (!busy || J > warp) continue;
+  for (int sl = 0; sl < SLICES; ++sl) {
+    if (sl >= slices) break;
+    cp_wait<1>();       // the next tile may still be under way
+    __syncthreads();
+    if (busy) {
+#pragma unroll
+      for (int k = 0; k < SR / 16; ++k) {
+        const int kt = sl * (SR / 16) + k;
+        float f[4];
+#pragma unroll
+        for (int u = 0; u < 4; ++u) f[u] = ref ? exp_fast(ref[kt * 16 + 2 * t + 8 * (u >> 1) + (u & 1)]) : 1.f;
+        const uint32_t qa[4] = {pack2(q[kt][0] * f[0], q[kt][1] * f[1]), pack2(q[kt][2] * f[0], q[kt][3] * f[1]),
+                                pack2(q[kt][4] * f[2], q[kt][5] * f[3]), pack2(q[kt][6] * f[2], q[kt][7] * f[3])};
+        const uint32_t base = smem_addr(buf + (sl & 1) * kChunk * VS + k * 16 * VS) + v_lane;
+        product(qa, base);
+        product(qa, base + SR * VS * 2);
+      }
+    }
+    __syncthreads();
+    if (sl + 2 <= slices) load(sl + 2);
+  }
+  cp_wait<0>();
+  __syncthreads();   // the values (and the keys) are in place
+  if (!busy) return;
+  // scores inside the chunk, block by block, and their product with the values
+  const uint32_t values = smem_addr(buf + (slices & 1) * kChunk * VS) + v_lane;
+#pragma unroll 1
+  for (int J = 0; J <= warp; ++J) {
     float s[2][4] = {};
     if (J == warp && steep) {
       const bf16 *qg = rows + a.q_off + (size_t)h * D, *kg = rows + a.k_off + (size_t)h * D;
+#pragma unroll
       for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int i = i0 + g + 8 * (e >> 1), j = i0 + nt * 8 + 2 * t + (e & 1);
           float sum = 0.f;
-          if (i < len && j <= i)
+          if (i < len && j <= i) {
+#pragma unroll 1
             for (int d = 0; d < D; ++d)
               sum += to_f(qg[(size_t)i * a.stride + d]) * to_f(kg[(size_t)j * a.stride + d]) *
                      exp_fast(cum[(size_t)i * channels + d] - cum[(size_t)j * channels + d]);
+          }
           s[nt][e] = sum * kscale;
         }
     } else {
@@ -347,71 +390,8 @@ __global__ void __launch_bounds__(kThreads, 1) gla_output_kernel(const Args a) {
             if (nt * 8 + 2 * t + (e & 1) > g + 8 * (e >> 1)) s[nt][e] = 0.f;
       }
     }
-    P[J][0] = pack2(s[0][0], s[0][1]);
-    P[J][1] = pack2(s[0][2], s[0][3]);
-    P[J][2] = pack2(s[1][0], s[1][1]);
-    P[J][3] = pack2(s[1][2], s[1][3]);
-  }
-  // queries against the state at the chunk's start
-  uint32_t qs[DP / 16][4];
-#pragma unroll
-  for (int kt = 0; kt < DP / 16; ++kt) {
-    float f[4];
-#pragma unroll
-    for (int u = 0; u < 4; ++u) f[u] = ref ? exp_fast(ref[kt * 16 + 2 * t + 8 * (u >> 1) + (u & 1)]) : 1.f;
-    qs[kt][0] = pack2(q[kt][0] * f[0], q[kt][1] * f[1]);
-    qs[kt][1] = pack2(q[kt][2] * f[0], q[kt][3] * f[1]);
-    qs[kt][2] = pack2(q[kt][4] * f[2], q[kt][5] * f[3]);
-    qs[kt][3] = pack2(q[kt][6] * f[2], q[kt][7] * f[3]);
-  }
-  float O[VP / 8][4];
-#pragma unroll
-  for (int i = 0; i < VP / 8; ++i)
-#pragma unroll
-    for (int e = 0; e < 4; ++e) O[i][e] = 0.f;
-  const uint32_t v_lane = (((lane & 7) + (((lane >> 3) & 1) << 3)) * VS + (lane >> 4) * 8) * 2;
-  if (has_state) {
-#pragma unroll
-    for (int d0 = 0; d0 < DP; d0 += SR) {
-      if (d0 > 0) {
-        __syncthreads();
-        load_state(d0);
-      }
-      cp_wait<0>();
-      __syncthreads();
-      if (busy) {
-#pragma unroll
-        for (int kt = 0; kt < SR / 16; ++kt) {
-#pragma unroll
-          for (int part = 0; part < 2; ++part) {
-            const uint32_t base = smem_addr(ss + (part * SR + kt * 16) * VS) + v_lane;
-#pragma unroll
-            for (int nt = 0; nt < VP / 16; ++nt) {
-              uint32_t vb[4];
-              ldsm4t(vb, base + nt * 32);
-              mma(O[2 * nt], qs[d0 / 16 + kt], vb[0], vb[1]);
-              mma(O[2 * nt + 1], qs[d0 / 16 + kt], vb[2], vb[3]);
-            }
-          }
-        }
-      }
-    }
-  } else {
-    cp_wait<0>();
-    __syncthreads();
-  }
-  if (!busy) return;
-#pragma unroll
-  for (int J = 0; J < kBlocks; ++J) {
-    if (J > warp) break;
-    const uint32_t base = smem_addr(vs + J * kBlock * VS) + v_lane;
-#pragma unroll
-    for (int nt = 0; nt < VP / 16; ++nt) {
-      uint32_t vb[4];
-      ldsm4t(vb, base + nt * 32);
-      mma(O[2 * nt], P[J], vb[0], vb[1]);
-      mma(O[2 * nt + 1], P[J], vb[2], vb[3]);
-    }
+    const uint32_t pa[4] = {pack2(s[0][0], s[0][1]), pack2(s[0][2], s[0][3]), pack2(s[1][0], s[1][1]), pack2(s[1][2], s[1][3])};
+    product(pa, values + J * kBlock * VS * 2);
   }
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
@@ -463,7 +443,7 @@ static int launch_chunk(const Args& a, int chunks, cudaStream_t st) {
 }
 template <int DP, int VP>
 static int launch_output(const Args& a, int chunks, cudaStream_t st) {
-  const size_t smem = (size_t)(kChunk * (DP + 8) + (kChunk + 2 * 64) * (VP + 8)) * sizeof(bf16) + (size_t)kBlocks * DP * sizeof(float);
+  const size_t smem = (size_t)(kChunk * (DP + 8) + 2 * kChunk * (VP + 8)) * sizeof(bf16) + (size_t)kBlocks * DP * sizeof(float);
   const int rc = set_smem(gla_output_kernel<DP, VP>, smem);
   if (rc != NQB200_OK) return rc;
   return launch_overlapped(gla_output_kernel<DP, VP>, dim3((unsigned)chunks, (unsigned)a.r.heads, (unsigned)a.bt.batch), dim3(kThreads), smem, st, a);
