@@ -762,7 +762,7 @@ def _engine_throughput(eng, vocab, batches, context, prefill, steps=16):
         for i in range(B):
             s = Sequence(i, torch.randint(0, vocab, (context,), generator=g).tolist(), 10 ** 9)
             eng._hold(s, context + 8)
-            s.output.append(1)
+            s.output.append(s.prompt[0])      # unlike tokens: a router sends them to unlike experts
             seqs.append(s)
         for _ in range(3):
             eng._decode(seqs)
@@ -964,6 +964,208 @@ def run_vemedra(args):
         del eng, model
         torch.cuda.empty_cache()
     line["kernels"] = vemedra_kernels(dev, peaks)
+    line["clocks"] = sampler.stop()
+    emit(json.dumps(line))
+
+
+# --------------------------------------------------------------------------
+# Verozen: layers of a real model's size beside the Vemedra layers of the same size (--verozen)
+# --------------------------------------------------------------------------
+VEROZEN_LAYERS = 8
+VEROZEN_EXPERTS = {"experts": 64, "top": 8, "groups": {"count": 8, "keep": 4}, "scale": 2.5}
+VEROZEN_FF, VEROZEN_SIDE, VEROZEN_RANK = 1536, 256, 16     # a token's experts together have the 12288 of Vemedra's feed-forward
+
+
+def verozen_config(layers=VEROZEN_LAYERS):
+    """The widths and heads of ``vemedra_config``: of every four layers two gated linear attention, one sigmoid attention, one
+    retention."""
+    mlp = {"kind": "moe", "expert": {"ff": VEROZEN_FF}, "router": VEROZEN_EXPERTS}
+    gla = {"type": "gla", "mlp": mlp, "mixer": {"heads": 16, "dim": 128, "vdim": 256, "tau": 16.0, "rank": VEROZEN_RANK}}
+    att = {"type": "attention", "mlp": mlp, "mixer": {"heads": 32, "kv_heads": 8, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "rot": {"base": 1e6, "dims": 128}}}
+    ret = {"type": "retention", "mlp": mlp, "mixer": {"heads": 16, "dim": 128, "vdim": 256, "decay": [1 - 2.0 ** -(5 + 0.5 * h) for h in range(16)],
+                                                      "rot": {"base": 1e4, "dims": 128}}}
+    return {"architecture": "Verozen", "vocab": 151936, "width": 4096, "norm": {"eps": 1e-6, "groups": 4}, "postln_alpha": 2.0,
+            "token_side": {"dim": VEROZEN_SIDE}, "layers": [(gla, gla, att, ret)[i % 4] for i in range(layers)]}
+
+
+def verozen_kernels(dev, peaks, T=8192, context=2048):
+    """Each kernel of a Verozen layer on its own, on inputs larger than L2 (rotating copies), against its roofline, beside
+    the like kernel of a Vemedra layer."""
+    from nanoquantization_b200 import _lib
+    from nanoquantization_b200.engine import StepBatch
+    from nanoquantization_b200.layers import mixers as ops, moe
+    from nanoquantization_b200.layers.sequence_mixers import AttentionMixer, GatedLinearMixer, RetentionMixer, SigmoidAttentionMixer
+    hbm, bf16 = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    W, H, G, D, RH, RD, RV, FF, bs = 4096, 32, 8, 128, 16, 128, 256, 12288, 256
+    E, top, ff, n_side, rank = VEROZEN_EXPERTS["experts"], VEROZEN_EXPERTS["top"], VEROZEN_FF, VEROZEN_SIDE, VEROZEN_RANK
+    rows, dt, f32 = [], torch.bfloat16, torch.float32
+
+    def rnd(*shape, dtype=dt):
+        return torch.randn(*shape, device=dev, dtype=f32).to(dtype)
+
+    def add(phase, name, us, nbytes=0, flops=0):
+        tb, tf = nbytes / hbm * 1e6, flops / bf16 * 1e6
+        rows.append({"phase": phase, "kernel": name, "us": round(us, 2), "bound": "hbm" if tb >= tf else "tensor",
+                     "of_roofline": round(max(tb, tf) / us, 3)})
+
+    def step(n, B, start):
+        blocks = -(-(start + n) // bs)
+        return StepBatch.host([[0] * n] * B, [start] * B, [[b * blocks + i for i in range(blocks)] for b in range(B)], list(range(B)), blocks, bs).to(dev)
+    sig = SigmoidAttentionMixer(heads=H, kv_heads=G, dim=D, rot_base=1e6, rot_dims=D, interleaved=True, scale=D ** -0.5, eps=1e-6, device=dev)
+    for t in (sig.q_norm, sig.k_norm, sig.temp):
+        t.fill_(1.0)
+    sig.bias.fill_(-7.0)
+    cap = AttentionMixer(heads=H, kv_heads=G, dim=D, vdim=D, chunk=T, rot_base=1e6, rot_dims=D, scale=D ** -0.5, softcap=50.0, device=dev)
+    gla = GatedLinearMixer(heads=RH, dim=RD, vdim=RV, rank=rank, tau=16.0, eps=1e-6, dtype=dt, device=dev)
+    gla.a2.copy_(rnd(RH * RD, rank) * rank ** -0.5)
+    gla.a2_bias.copy_(2 + rnd(RH * RD, dtype=f32))
+    gla.norm.fill_(1.0)
+    decay = [1 - 2.0 ** -(5 + 0.5 * h) for h in range(RH)]
+    ret = RetentionMixer(heads=RH, dim=RD, vdim=RV, decay=decay, eps=1e-6, rot_base=1e4, rot_dims=RD, device=dev)
+    plain = RetentionMixer(heads=RH, dim=RD, vdim=RV, decay=decay, eps=1e-6, device=dev)
+    router = _lib.RouterDesc(E, top, VEROZEN_EXPERTS["groups"]["count"], VEROZEN_EXPERTS["groups"]["keep"], 2.5, None)
+    lin_cols = 2 * RH * RD + 2 * RH * RV
+    # prefill
+    one = step(T, 1, 0)
+    x, nw, cw = [rnd(T, W, dtype=f32) for _ in range(2)], torch.ones(W, device=dev), rnd(4, W, dtype=f32)
+    cst = torch.zeros(65, 3, W, device=dev)
+    add("prefill", "norm in 4 groups after the sum", _device_us(lambda i: ops.post_norm_(x[i % 2], None, 1.0, nw, 4, 1e-6, dt), 8), T * W * 10)
+    y8 = [rnd(T, top, W) for _ in range(2)]
+    add("prefill", "the same with the sum of 8 experts", _device_us(lambda i: ops.post_norm_(x[i % 2], y8[i % 2], 2.0, nw, 4, 1e-6, dt), 8), T * W * (10 + 2 * top))
+    del y8
+    yf = [rnd(T, W, dtype=f32) for _ in range(2)]
+    add("prefill", "side input: norm and add", _device_us(lambda i: ops.add_normed_(x[i % 2], yf[i % 2], nw, 1e-6, dt), 8), T * W * 14)
+    del yf
+    add("prefill", "Vemedra: rmsnorm + convolution", _device_us(lambda i: ops.rmsnorm_conv(x[i % 2], nw, cw, cst, one, 1e-6, dt), 8), T * W * 6)
+    pq = [rnd(T, (H + 2 * G) * D) for _ in range(3)]
+    kc, vc = rnd(T // bs + 1, bs, G, D), rnd(T // bs + 1, bs, G, D)
+    rd, rr = sig.rope_desc(), ret.rope_desc()
+    add("prefill", "head norm + rotary + K/V store", _device_us(lambda i: ops.norm_rope(pq[i % 3], kc, vc, rd, one, 0, H * D, H * D), 9), T * (2 * H * D + 3 * G * D) * 2)
+    add("prefill", "Vemedra: rotary + K/V store", _device_us(lambda i: ops.rope_store(pq[i % 3], kc, vc, cap.inv_freq, one, 0, H * D, (H + G) * D, H), 9),
+        T * (2 * H * D + 4 * G * D) * 2)
+    o = rnd(T, H * D)
+    for name, m in (("sigmoid attention", sig), ("Vemedra: capped softmax attention, one chunk of all", cap)):
+        d = m.desc()
+        us = _device_us(lambda i: ops.chunk_attention(pq[i % 3][:, :H * D], kc, vc, o, d, one), 4)
+        add("prefill", name, us, flops=T * T / 2 * 4 * D * H)
+    del pq, o
+    pl, act, st = [rnd(T, lin_cols + rank) for _ in range(2)], rnd(T, RH * RV), torch.zeros(65, RH, RD, RV, device=dev)
+    gd = plain.desc()
+    flow = T * (2 * RH * RD + 3 * RH * RV) * 2
+    add("prefill", "gated linear attention + norm + gate (4 launches)", _device_us(lambda i: ops.gla_gated(pl[i % 2], 0, gla, st, act, 0, one), 4), flow + T * rank * 2,
+        4 * T * RH * RD * RV)
+    add("prefill", "rotary of retention", _device_us(lambda i: ops.norm_rope(pl[i % 2], None, None, rr, one, 0, RH * RD, 0), 8), T * 4 * RH * RD * 2)
+    add("prefill", "retention + norm + gate (3 launches, as Vemedra's)", _device_us(lambda i: ops.retention_gated(pl[i % 2], 0, gd, plain.decay, st, act, 0, one), 4), flow,
+        4 * T * RH * RD * RV)
+    del pl, act
+    h = [rnd(T, W) for _ in range(2)]
+    up, down, wr = rnd(E, ff, W), rnd(E, W, ff), rnd(E, W)
+    plan = moe.route(rnd(T, E, dtype=f32), router)
+    u = moe.experts_up(h[0], up, plan)
+    lg = [rnd(T, E, dtype=f32) for _ in range(2)]
+    add("prefill", "router product (library)", _device_us(lambda i: ops.linear(h[i % 2], wr, f32), 8), T * (W * 2 + E * 4) + E * W * 2)
+    add("prefill", "routing and sort (3 launches)", _device_us(lambda i: moe.route(lg[i % 2], router), 8), T * (E * 4 + top * 16))
+    add("prefill", "experts' first product + gelu", _device_us(lambda i: moe.experts_up(h[i % 2], up, plan), 4), flops=2 * T * top * W * ff)
+    add("prefill", "experts' second product + weight", _device_us(lambda i: moe.experts_down(u, down, plan), 4), flops=2 * T * top * W * ff)
+    del u
+    w2, y = rnd(W, FF), rnd(T, FF)
+    add("prefill", "Vemedra: down product + residual (library)", _device_us(lambda i: ops.linear_residual_(x[i % 2], y, w2), 4), flops=2 * T * W * FF)
+    del w2, y
+    ids, table = torch.randint(0, 1000, (T,), device=dev), rnd(1000, 8 * n_side)
+    sg, sp = rnd(n_side, W), rnd(W, n_side)
+    add("prefill", "side input: gate product (library) + gelu + table", _device_us(lambda i: ops.linear_gelu_table(h[i % 2], sg, ids, table, n_side), 8),
+        T * (W + n_side) * 2, 2 * T * W * n_side)
+    gg = [rnd(T, n_side) for _ in range(2)]
+    add("prefill", "side input: product (library)", _device_us(lambda i: ops.linear(gg[i % 2], sp, f32), 8), T * (n_side * 2 + W * 4), 2 * T * W * n_side)
+    del x, h, lg, gg
+    torch.cuda.empty_cache()
+    # decode: weights and caches rotate over copies larger than L2
+    for B in (1, 16):
+        ph, s, h = f"decode, batch {B}", step(1, B, context - 1), rnd(B, W)
+        stream, nin = rnd(B, W, dtype=f32), lin_cols + rank
+        ws = [rnd(nin, W) for _ in range(3)]
+        add(ph, "merged input product (gated linear attention)", _device_us(lambda i: ops.linear(h, ws[i % 3]), 12), nin * W * 2)
+        ws = [rnd(W, RH * RV) for _ in range(8)]
+        a4 = rnd(B, RH * RV)
+        add(ph, "output product + scaled residual", _device_us(lambda i: ops.linear_residual_(stream, a4, ws[i % 8], 2.0), 16), W * RH * RV * 2)
+        # disjoint experts from call to call, as far as there are
+        plans, bytes_ = [], []
+        for c in range(4):
+            lg = rnd(B, E, dtype=f32)
+            if B == 1:
+                lg[:, 8 * c:8 * c + 8] += 20
+            plans.append(moe.route(lg, _lib.RouterDesc(E, top, 1, 1, 1.0, None)))
+            bytes_.append(int(plans[-1].active[0]) * ff * W * 2)
+        us_ = [moe.experts_up(h, up, p) for p in plans]
+        add(ph, "experts' first product + gelu", _device_us(lambda i: moe.experts_up(h, up, plans[i % 4]), 12), sum(bytes_) / 4)
+        add(ph, "experts' second product + weight", _device_us(lambda i: moe.experts_down(us_[i % 4], down, plans[i % 4]), 12), sum(bytes_) / 4)
+        ws = [rnd(2 * FF, W) for _ in range(2)]
+        add(ph, "Vemedra: gate | up product + clamped GLU", _device_us(lambda i: ops.dense_glu(h, ws[i % 2], 7.0), 8), 2 * FF * W * 2)
+        ws, f12 = [rnd(W, FF) for _ in range(3)], rnd(B, FF)
+        add(ph, "Vemedra: down product + residual", _device_us(lambda i: ops.linear_residual_(stream, f12, ws[i % 3]), 12), FF * W * 2)
+        ws = [rnd(E, W) for _ in range(2)]
+        add(ph, "router product", _device_us(lambda i: ops.linear(h, ws[i % 2], f32), 16), E * W * 2)
+        lg = rnd(B, E, dtype=f32)
+        add(ph, "routing and sort", _device_us(lambda i: moe.route(lg, router), 16), B * E * 4)
+        idb = torch.randint(0, 1000, (B,), device=dev)
+        add(ph, "side input: gate product + gelu + table", _device_us(lambda i: ops.linear_gelu_table(h, sg, idb, table, n_side), 16), n_side * W * 2)
+        gb = rnd(B, n_side)
+        add(ph, "side input: product", _device_us(lambda i: ops.linear(gb, sp, f32), 16), n_side * W * 2)
+        yb, y8 = rnd(B, W, dtype=f32), rnd(B, top, W, dtype=f32)
+        add(ph, "side input: norm and add", _device_us(lambda i: ops.add_normed_(stream, yb, nw, 1e-6, dt), 16), B * W * 14)
+        add(ph, "norm in 4 groups after the sum", _device_us(lambda i: ops.post_norm_(stream, None, 1.0, nw, 4, 1e-6, dt), 16), B * W * 10)
+        add(ph, "the same with the sum of 8 experts", _device_us(lambda i: ops.post_norm_(stream, y8, 2.0, nw, 4, 1e-6, dt), 16), B * W * (10 + 4 * top))
+        add(ph, "Vemedra: rmsnorm + convolution", _device_us(lambda i: ops.rmsnorm_conv(stream, nw, cw, cst, s, 1e-6, dt), 16), B * W * (6 + 24) + W * 20)
+        del ws
+        n = 8 if B == 1 else 2   # copies of cache and state
+        copies = []
+        for _ in range(n):
+            nb = B * (context // bs)
+            copies.append((rnd(nb, bs, G, D), rnd(nb, bs, G, D), torch.zeros(B, RH, RD, RV, device=dev)))
+        pa, pl, ac = rnd(B, (H + 2 * G) * D), rnd(B, lin_cols + rank), rnd(B, H * D)
+        kv_bytes, st_bytes = B * context * 2 * G * D * 2, 2 * B * RH * RD * RV * 4
+        for name, m in (("head norm + rotary + store + sigmoid attention", sig), ("Vemedra: rotary + store + attention", cap)):
+            d, r = m.desc(), m.rope_desc()
+            v = m.value_column(0)
+            add(ph, name, _device_us(lambda i: ops.mixer_decode(pa, ac, (d, r, 0, v, 0, copies[i % n][0], copies[i % n][1]), None, s), 2 * n), kv_bytes)
+        for name, m in (("gated linear attention + norm + gate", gla), ("rotary + retention + norm + gate", ret), ("Vemedra: retention + norm + gate", plain)):
+            d = m.desc()
+            add(ph, name, _device_us(lambda i: ops.mixer_decode(pl, ac, None, (d, 0, 0, copies[i % n][2]), s), 2 * n), st_bytes)
+        del copies
+    return rows
+
+
+def run_verozen(args):
+    """--verozen: random-init layers of real sizes through the engine, beside Vemedra layers of the same width, heads and
+    (active) feed-forward, and every kernel against its roofline."""
+    from nanoquantization_b200.engine import LLMEngine
+    from nanoquantization_b200.models import VemedraConfig, VemedraForCausalLM, VerozenConfig, VerozenForCausalLM
+    torch.cuda.set_device(0)
+    dev, dt = torch.device("cuda", 0), torch.bfloat16
+    torch.manual_seed(0)
+    with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as fh:
+        peaks = json.load(fh)
+    line = {"what": "Verozen beside Vemedra, random init, one GPU, bf16", "layers": VEROZEN_LAYERS,
+            "note": "weights and caches larger than L2; rooflines are the measured copy bandwidth and bf16 peak"}
+    sampler = ClockSampler(0)
+    sampler.start()
+    if not args.verozen_kernels_only:
+        for name, build in (("verozen", lambda: VerozenForCausalLM(VerozenConfig.from_dict(verozen_config()), device=dev, dtype=dt)),
+                            ("vemedra", lambda: VemedraForCausalLM(VemedraConfig.from_dict(vemedra_config()), device=dev, dtype=dt))):
+            model = build()
+            for key, t in model.checkpoint_tensors().items():
+                if "norm" in key or key.endswith("temp"):
+                    t.fill_(1.0)
+                elif key.endswith("pb"):
+                    t.fill_(-7.0)
+                else:
+                    t.copy_(torch.randn(t.shape, device=dev) * (t.shape[-1] ** -0.5 if t.dim() > 1 else 0.1))
+            eng = LLMEngine(model, num_blocks=64 * 9 + 40, max_batch=64)
+            line[name] = _engine_throughput(eng, 151936, (1, 16, 64), 2047, 8192)
+            line[name]["weights_gb"] = round(sum(t.numel() * t.element_size() for t in model.buffers()) / 1e9, 2)
+            del eng, model
+            torch.cuda.empty_cache()
+    line["kernels"] = verozen_kernels(dev, peaks)
     line["clocks"] = sampler.stop()
     emit(json.dumps(line))
 
@@ -1296,6 +1498,9 @@ def main():
     ap.add_argument("--vemedra", action="store_true",
                     help="instead of the sweep: Vemedra layers of real sizes beside Qwen3 layers of the same size, and every kernel against its roofline")
     ap.add_argument("--vemedra-kernels-only", action="store_true", help="with --vemedra: the kernels alone")
+    ap.add_argument("--verozen", action="store_true",
+                    help="instead of the sweep: Verozen layers of real sizes beside Vemedra layers of the same size, and every kernel against its roofline")
+    ap.add_argument("--verozen-kernels-only", action="store_true", help="with --verozen: the kernels alone")
     ap.add_argument("--requests", type=int, default=256)
     ap.add_argument("--decode-only", type=int, default=0, metavar="BATCH",
                     help="only the Qwen3-8B decode point of this batch size, 1 GPU (the case a launch list is taken of)")
@@ -1307,6 +1512,8 @@ def main():
         emit(json.dumps(decode_bench(1, 0, torch.device("cuda", 0), dtype, batches=(args.decode_only,), steps=4, prefill=False)))
     elif args.vemedra:
         run_vemedra(args)
+    elif args.verozen:
+        run_verozen(args)
     elif args.serve:
         run_serve(args)
     elif args.point:

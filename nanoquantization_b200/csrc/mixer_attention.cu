@@ -79,6 +79,119 @@ __global__ void __launch_bounds__(256) norm_rope_kernel(T* __restrict__ proj, T*
   }
 }
 
+// The same for bf16 heads of up to 256 in pieces of 8: a lane holds one piece.  A CTA takes `span` tokens, whose heads its
+// warps share; four heads of a warp are under way while four are worked on.  Pairs of neighbours lie in one lane; the other
+// layout's partners are fetched from the lane half / 8 away.
+__device__ __forceinline__ void unpack8(uint4 v, float (&x)[8]) {
+  const uint32_t w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+  for (int i = 0; i < 4; ++i) { x[2 * i] = __uint_as_float(w[i] << 16); x[2 * i + 1] = __uint_as_float(w[i] & 0xFFFF0000u); }
+}
+__device__ __forceinline__ uint4 pack8(const float (&x)[8]) {
+  uint32_t w[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const __nv_bfloat162 p = __floats2bfloat162_rn(x[2 * i], x[2 * i + 1]);
+    w[i] = *reinterpret_cast<const uint32_t*>(&p);
+  }
+  return make_uint4(w[0], w[1], w[2], w[3]);
+}
+constexpr int kRopeSpan = 4;
+template <bool NEIGHBOURS>
+__global__ void __launch_bounds__(256, 4) norm_rope_vec_kernel(bf16* proj, bf16* k_cache, bf16* v_cache, const nqb200_rope r, const nqb200_batch bt,
+                                                               int64_t stride, int q_off, int k_off, int v_off, int span) {
+  extern __shared__ __align__(16) float cs[];  // [dim] q_norm, [dim] k_norm, [span][rot/2] cos, [span][rot/2] sin
+  __shared__ size_t slot[kRopeSpan];
+  const int half = r.rot / 2, cos_at = 2 * r.dim, sin_at = cos_at + span * half;
+  grid_launch_dependents();
+  if (r.q_norm)
+    for (int e = threadIdx.x; e < r.dim; e += blockDim.x) { cs[e] = r.q_norm[e]; cs[r.dim + e] = r.k_norm[e]; }
+  grid_dependency_wait();
+  const int b = blockIdx.y, t0 = bt.cu[b], n = bt.cu[b + 1] - t0, first = blockIdx.x * span, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (first >= n) return;
+  const int tokens = min(span, n - first), heads = r.heads + r.kv_heads, items = tokens * heads;
+  bf16* rows = proj + (size_t)(t0 + first) * stride;
+  const bool live = lane * 8 < r.dim;
+  const int piece = live ? lane * 8 : 0;
+  auto token_of = [&](int it) { return (it >= heads) + (it >= 2 * heads) + (it >= 3 * heads); };
+  auto place = [&](int tk, int hd) { return rows + (size_t)tk * stride + (hd < r.heads ? q_off + hd * r.dim : k_off + (hd - r.heads) * r.dim) + piece; };
+  constexpr int U = 4;
+  uint4 in[U], next[U];
+  auto request = [&](int i0, uint4 (&v)[U]) {
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int it = min(i0 + 8 * u, items - 1), tk = token_of(it);
+      v[u] = *reinterpret_cast<const uint4*>(place(tk, it - tk * heads));
+    }
+  };
+  request(warp, next);
+  const int p0 = bt.pos0[b] + first;
+  for (int e = threadIdx.x; e < tokens * half; e += blockDim.x) {
+    const int tk = e / half, f = e - tk * half;
+    sincosf((float)(p0 + tk) * r.inv_freq[f], &cs[sin_at + e], &cs[cos_at + e]);
+  }
+  if (k_cache && (int)threadIdx.x < tokens) slot[threadIdx.x] = kv_row(bt, b, p0 + threadIdx.x);
+  __syncthreads();
+  const bool turns = live && lane * 8 < r.rot;
+  const bool upper = !NEIGHBOURS && lane * 8 >= half;
+  const int partner = NEIGHBOURS || !turns ? lane : upper ? lane - half / 8 : lane + half / 8;
+  const int angle = turns ? (NEIGHBOURS ? lane * 4 : lane * 8 - (upper ? half : 0)) : 0;   // of the piece's first element
+  for (int i0 = warp; i0 < items; i0 += 8 * U) {
+#pragma unroll
+    for (int u = 0; u < U; ++u) in[u] = next[u];
+    if (i0 + 8 * U < items) request(i0 + 8 * U, next);
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int it = i0 + 8 * u;
+      if (it >= items) break;
+      const int tk = token_of(it), hd = it - tk * heads;
+      float x[8], y[8];
+      unpack8(in[u], x);
+      if (r.q_norm) {
+        float ss = 0.f;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) ss += x[e] * x[e];
+        const float inv = 1.f / sqrtf(warp_sum(live ? ss : 0.f) / (float)r.dim + r.eps);
+        const float4* w = reinterpret_cast<const float4*>(cs + (hd < r.heads ? 0 : r.dim) + piece);
+        const float4 w0 = w[0], w1 = w[1];
+        const float wv[8] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[e] = x[e] * inv * wv[e];
+      }
+      const float4* cp = reinterpret_cast<const float4*>(cs + cos_at + tk * half + angle);
+      const float4* sp = reinterpret_cast<const float4*>(cs + sin_at + tk * half + angle);
+      if (NEIGHBOURS) {
+        const float4 c = turns ? cp[0] : make_float4(1.f, 1.f, 1.f, 1.f), s = turns ? sp[0] : make_float4(0.f, 0.f, 0.f, 0.f);
+        const float cv[4] = {c.x, c.y, c.z, c.w}, sv[4] = {s.x, s.y, s.z, s.w};
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          y[2 * e] = x[2 * e] * cv[e] - x[2 * e + 1] * sv[e];
+          y[2 * e + 1] = x[2 * e + 1] * cv[e] + x[2 * e] * sv[e];
+        }
+      } else {
+#pragma unroll
+        for (int q = 0; q < 2; ++q) {
+          const float4 c = turns ? cp[q] : make_float4(1.f, 1.f, 1.f, 1.f), s = turns ? sp[q] : make_float4(0.f, 0.f, 0.f, 0.f);
+          const float cv[4] = {c.x, c.y, c.z, c.w}, sv[4] = {s.x, s.y, s.z, s.w};
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const float other = __shfl_sync(0xFFFFFFFFu, x[4 * q + e], partner);
+            y[4 * q + e] = x[4 * q + e] * cv[e] + other * (upper ? sv[e] : -sv[e]);
+          }
+        }
+      }
+      if (live) *reinterpret_cast<uint4*>(hd < r.heads || !k_cache ? place(tk, hd) : k_cache + (slot[tk] * r.kv_heads + (hd - r.heads)) * r.dim + piece) = pack8(y);
+    }
+  }
+  if (k_cache) {
+    const int per = r.kv_heads * r.vdim / 8;
+    for (int e = threadIdx.x; e < tokens * per; e += blockDim.x) {
+      const int tk = e / per, c = e - tk * per;
+      reinterpret_cast<uint4*>(v_cache + slot[tk] * r.kv_heads * r.vdim)[c] = reinterpret_cast<const uint4*>(rows + (size_t)tk * stride + v_off)[c];
+    }
+  }
+}
+
 constexpr int kSimpleKeys = 128;   // keys per pass = threads
 constexpr int kSimpleVCols = 8;    // value columns per thread at most: vdim <= 1024
 
@@ -187,6 +300,15 @@ extern "C" int nqb200_norm_rope(void* proj, void* k_cache, void* v_cache, const 
   const dim3 grid((unsigned)b->max_len, (unsigned)b->batch), block(256);
   const size_t smem = (size_t)r->rot * sizeof(float);
   cudaStream_t s = (cudaStream_t)stream;
+  const bool pieces = dtype == NQB200_BF16 && r->dim % 8 == 0 && r->dim <= 256 && r->rot % (r->interleaved ? 8 : 16) == 0 && stride % 8 == 0 && q_off % 8 == 0 &&
+                      k_off % 8 == 0 && aligned16(proj) && (!r->q_norm || r->k_norm) && (r->q_norm || !r->k_norm) &&
+                      (!k_cache || (aligned16(k_cache) && aligned16(v_cache) && r->vdim % 8 == 0 && v_off % 8 == 0));
+  if (pieces) {
+    auto kernel = r->interleaved ? norm_rope_vec_kernel<true> : norm_rope_vec_kernel<false>;
+    const int span = b->max_len >= 4 * kNumSMs ? kRopeSpan : 1;
+    return launch_overlapped(kernel, dim3((unsigned)((b->max_len + span - 1) / span), (unsigned)b->batch), block, (size_t)(2 * r->dim + span * r->rot) * sizeof(float), s,
+                             (bf16*)proj, (bf16*)k_cache, (bf16*)v_cache, *r, *b, stride, (int)q_off, (int)k_off, (int)v_off, span);
+  }
   if (dtype == NQB200_F32)
     return launch_overlapped(norm_rope_kernel<float>, grid, block, smem, s, (float*)proj, (float*)k_cache, (float*)v_cache, *r, *b, stride,
                              (int)q_off, (int)k_off, (int)v_off);

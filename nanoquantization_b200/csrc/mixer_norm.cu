@@ -258,9 +258,10 @@ static int launch_rmsnorm_conv(const float* x, const float* weight, const float*
 // Norms after the sum.  A CTA takes a token; the row (alpha x + the terms of y) stays in shared memory between the sums of
 // squares and the use.  The groups of the row are split into about as many pieces as there are warps, a warp sums whole
 // pieces, and the group's scale is taken from its pieces.  out: the row rounded to T; x (if written): the row itself.
-constexpr int kNormThreads = 256, kNormWarps = kNormThreads / 32;
-template <typename T, typename Y>
-__global__ void __launch_bounds__(kNormThreads) group_norm_kernel(float* x, const int64_t* __restrict__ rows, const Y* __restrict__ y, int terms, float alpha,
+// Few rows: wide CTAs, so that a row's loads (of every term) are under way at once.
+constexpr int kNormThreads = 256, kNormWarps = kNormThreads / 32, kNormWide = 1024;
+template <typename T, typename Y, int THREADS>
+__global__ void __launch_bounds__(THREADS, THREADS == kNormWide ? 1 : 4) group_norm_kernel(float* x, const int64_t* __restrict__ rows, const Y* __restrict__ y, int terms, float alpha,
                                                                   const float* __restrict__ weight, T* __restrict__ out, int width, int groups, int pieces,
                                                                   float eps, int write_x) {
   extern __shared__ float4 norm_smem[];
@@ -269,22 +270,26 @@ __global__ void __launch_bounds__(kNormThreads) group_norm_kernel(float* x, cons
   grid_launch_dependents();
   grid_dependency_wait();
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  constexpr int threads = THREADS, U = THREADS == kNormWide ? 8 : 4;   // terms under way at once
   const int64_t at = rows ? rows[blockIdx.x] : blockIdx.x;
   float* xr = x + (size_t)at * width;
   const Y* yr = y + (size_t)blockIdx.x * terms * width;
   const int size = width / groups;
   const bool vec = size % 4 == 0;
   if (vec) {
-    for (int c = tid * 4; c < width; c += kNormThreads * 4) {
+    for (int c = tid * 4; c < width; c += threads * 4) {
       float4 v = scale4(ld4(xr + c), alpha);
-      for (int j = 0; j < terms; ++j) {
-        const float4 a = load4(yr + (size_t)j * width + c);
-        v.x += a.x; v.y += a.y; v.z += a.z; v.w += a.w;
+      for (int j0 = 0; j0 < terms; j0 += U) {
+        float4 a[U];
+#pragma unroll
+        for (int j = 0; j < U; ++j) a[j] = j0 + j < terms ? load4(yr + (size_t)(j0 + j) * width + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int j = 0; j < U; ++j) { v.x += a[j].x; v.y += a[j].y; v.z += a[j].z; v.w += a[j].w; }
       }
       *reinterpret_cast<float4*>(row_s + c) = v;
     }
   } else {
-    for (int c = tid; c < width; c += kNormThreads) {
+    for (int c = tid; c < width; c += threads) {
       float v = alpha * xr[c];
       for (int j = 0; j < terms; ++j) v += to_f(yr[(size_t)j * width + c]);
       row_s[c] = v;
@@ -292,7 +297,7 @@ __global__ void __launch_bounds__(kNormThreads) group_norm_kernel(float* x, cons
   }
   __syncthreads();
   const int len = (size + pieces - 1) / pieces;
-  for (int q = warp; q < groups * pieces; q += kNormWarps) {
+  for (int q = warp; q < groups * pieces; q += threads / 32) {
     const int g = q / pieces, lo = (q - g * pieces) * len, hi = min(lo + len, size);
     const float* s = row_s + g * size;
     float ss = 0.f;
@@ -301,7 +306,7 @@ __global__ void __launch_bounds__(kNormThreads) group_norm_kernel(float* x, cons
     if (lane == 0) part[q] = ss;
   }
   __syncthreads();
-  for (int g = tid; g < groups; g += kNormThreads) {   // a thread per group; its pieces' places become free for the scale
+  for (int g = tid; g < groups; g += threads) {   // a thread per group; its pieces' places become free for the scale
     float ss = 0.f;
     for (int k = 0; k < pieces; ++k) ss += part[g * pieces + k];
     part[g * pieces] = 1.f / sqrtf(ss / (float)size + eps);
@@ -309,13 +314,13 @@ __global__ void __launch_bounds__(kNormThreads) group_norm_kernel(float* x, cons
   __syncthreads();
   T* o = out + (size_t)blockIdx.x * width;
   if (vec) {
-    for (int c = tid * 4; c < width; c += kNormThreads * 4) {
+    for (int c = tid * 4; c < width; c += threads * 4) {
       const float4 v = mul4(scale4(*reinterpret_cast<const float4*>(row_s + c), part[c / size * pieces]), ld4(weight + c));
       if (write_x) *reinterpret_cast<float4*>(xr + c) = v;
       store4<T>(o + c, v);
     }
   } else {
-    for (int c = tid; c < width; c += kNormThreads) {
+    for (int c = tid; c < width; c += threads) {
       const float v = row_s[c] * part[c / size * pieces] * weight[c];
       if (write_x) xr[c] = v;
       o[c] = from_f<T>(v);
@@ -376,18 +381,27 @@ __global__ void __launch_bounds__(256) gelu_table_kernel(const T* __restrict__ g
   }
 }
 
-template <typename T, typename Y>
-static int launch_group_norm(float* x, const int64_t* rows, const void* y, int64_t terms, float alpha, const float* weight, void* out, int64_t n,
+template <typename T, typename Y, int THREADS>
+static int launch_group_norm_by(float* x, const int64_t* rows, const void* y, int64_t terms, float alpha, const float* weight, void* out, int64_t n,
                              int64_t width, int64_t groups, float eps, int write_x, cudaStream_t st) {
-  const int pieces = groups >= kNormWarps ? 1 : (int)((kNormWarps + groups - 1) / groups);
+  constexpr int warps = THREADS / 32;
+  const int pieces = groups >= warps ? 1 : (int)((warps + groups - 1) / groups);
   const size_t smem = ((size_t)(width + 3) / 4 * 4 + (size_t)groups * pieces) * sizeof(float);
   if (smem > 200 * 1024) return NQB200_ERR_TOO_LARGE;
-  if (smem > 48 * 1024 && cudaFuncSetAttribute(group_norm_kernel<T, Y>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+  if (smem > 48 * 1024 && cudaFuncSetAttribute(group_norm_kernel<T, Y, THREADS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
     cudaGetLastError();
     return NQB200_ERR_LAUNCH;
   }
-  return launch_overlapped(group_norm_kernel<T, Y>, dim3((unsigned)n), dim3(kNormThreads), smem, st, x, rows, (const Y*)y, (int)terms, alpha, weight,
+  return launch_overlapped(group_norm_kernel<T, Y, THREADS>, dim3((unsigned)n), dim3(THREADS), smem, st, x, rows, (const Y*)y, (int)terms, alpha, weight,
                            (T*)out, (int)width, (int)groups, pieces, eps, write_x);
+}
+
+template <typename T, typename Y>
+static int launch_group_norm(float* x, const int64_t* rows, const void* y, int64_t terms, float alpha, const float* weight, void* out, int64_t n,
+                             int64_t width, int64_t groups, float eps, int write_x, cudaStream_t st) {
+  if (n <= 2 * kNumSMs && width > 2 * kNormThreads)
+    return launch_group_norm_by<T, Y, kNormWide>(x, rows, y, terms, alpha, weight, out, n, width, groups, eps, write_x, st);
+  return launch_group_norm_by<T, Y, kNormThreads>(x, rows, y, terms, alpha, weight, out, n, width, groups, eps, write_x, st);
 }
 
 template <typename T>

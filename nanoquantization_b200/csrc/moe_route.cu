@@ -1,5 +1,6 @@
 // Routing: a warp per token takes the scores, the groups and the experts; then the pairs are sorted by expert.  Few tokens:
 // one CTA does all of it.  Many: the routing CTAs count, one CTA scans the counts, and the pairs are dealt to their places.
+#include <limits.h>
 #include "moe.cuh"
 
 namespace nqb200 {
@@ -7,27 +8,29 @@ namespace nqb200 {
 constexpr int kRouteMaxExperts = 1024;      // 32 per lane
 constexpr int kRouteSmallTokens = 32;
 
-// Index of the largest open value (bit i of a lane's mask: item lane + 32 i), the lowest index among equals; -1 if none is open.
-__device__ __forceinline__ int warp_argmax(const float* v, uint32_t open, int lane) {
-  float best = -INFINITY;
-  int at = -1;
+// Floats (no NaN) as integers in the same order, above 0.
+__device__ __forceinline__ uint32_t ordered(float v) {
+  const uint32_t u = __float_as_uint(v + 0.f);
+  return (u >> 31) ? ~u : u | 0x80000000u;
+}
+// Index of the largest open key (bit i of a lane's mask: item lane + 32 i), the lowest index among equals.
+__device__ __forceinline__ int warp_argmax(const uint32_t* key, uint32_t open, int lane) {
+  uint32_t best = 0;
+  int at = INT_MAX;
   while (open) {
     const int i = __ffs(open) - 1, e = lane + 32 * i;
     open &= open - 1;
-    if (at < 0 || v[e] > best) { best = v[e]; at = e; }
+    if (key[e] > best) { best = key[e]; at = e; }
   }
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) {
-    const float ov = __shfl_xor_sync(0xFFFFFFFFu, best, o);
-    const int oa = __shfl_xor_sync(0xFFFFFFFFu, at, o);
-    if (oa >= 0 && (at < 0 || ov > best || (ov == best && oa < at))) { best = ov; at = oa; }
-  }
-  return at;
+  const uint32_t top = __reduce_max_sync(0xFFFFFFFFu, best);
+  return __reduce_min_sync(0xFFFFFFFFu, best == top ? at : INT_MAX);
 }
 
 // smem: [experts] scores, [experts] choices, [groups] group scores, all this warp's own.
-__device__ void route_token(const float* __restrict__ z, const nqb200_router& r, float* smem, int lane, int32_t* expert, float* weight) {
-  float *s = smem, *choice = s + r.experts, *gs = choice + r.experts;
+__device__ void route_token(const float* __restrict__ z, const nqb200_router& r, float* smem, int lane, int32_t* expert, float* weight,
+                            int* copy = nullptr) {
+  float *s = smem, *choice = s + r.experts;
+  uint32_t *key = reinterpret_cast<uint32_t*>(choice), *gs = key + r.experts;   // the choices are keys once the groups have their scores
   for (int e = lane; e < r.experts; e += 32) {
     const float v = sigmoid_f(z[e]);
     s[e] = v;
@@ -46,23 +49,25 @@ __device__ void route_token(const float* __restrict__ z, const nqb200_router& r,
         if (v > a) { b = a; a = v; } else if (v > b) { b = v; }
       }
       const float sum = size > 1 ? a + b : a;
-      gs[g] = sum == sum ? sum : -INFINITY;
+      gs[g] = ordered(sum == sum ? sum : -INFINITY);
       gopen |= 1u << i;
     }
     __syncwarp();
     for (int k = 0; k < r.keep; ++k) {
-      const int g = warp_argmax(gs, gopen, lane);
+      const int g = warp_argmax(gs, gopen, lane), lo = g * size;
       if (lane == (g & 31)) gopen &= ~(1u << (g >> 5));
       for (int i = 0; lane + 32 * i < r.experts; ++i)
-        if ((lane + 32 * i) / size == g) open |= 1u << i;
+        if (lane + 32 * i >= lo && lane + 32 * i < lo + size) open |= 1u << i;
     }
   } else {
     for (int i = 0; lane + 32 * i < r.experts; ++i) open |= 1u << i;
   }
+  for (int e = lane; e < r.experts; e += 32) key[e] = ordered(choice[e]);
+  __syncwarp();
   float sum = 0.f;
   int mine[4] = {0, 0, 0, 0};   // of choices lane, lane + 32, ...
   for (int k = 0; k < r.top; ++k) {
-    const int e = warp_argmax(choice, open, lane);
+    const int e = warp_argmax(key, open, lane);
     if (lane == (e & 31)) open &= ~(1u << (e >> 5));
     sum += s[e];
     if (lane == (k & 31)) mine[(k >> 5) & 3] = e;
@@ -70,6 +75,7 @@ __device__ void route_token(const float* __restrict__ z, const nqb200_router& r,
   for (int k = lane; k < r.top; k += 32) {
     const int e = mine[(k >> 5) & 3];
     expert[k] = e;
+    if (copy) copy[k] = e;
     weight[k] = s[e] / (sum + 1e-20f) * r.scale;
   }
   __syncwarp();
@@ -108,17 +114,20 @@ __global__ void __launch_bounds__(1024) moe_route_small_kernel(const float* __re
   grid_launch_dependents();
   grid_dependency_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, pairs = tokens * r.top;
+  int* expert = reinterpret_cast<int*>(route_smem);     // [pairs]
+  float* scores = route_smem + pairs;
   for (int e = threadIdx.x; e < r.experts; e += blockDim.x) hist[e] = 0;
   if (warp < tokens)
-    route_token(logits + (size_t)warp * r.experts, r, route_smem + (size_t)warp * (2 * r.experts + r.groups), lane, p.expert + warp * r.top, p.weight + warp * r.top);
-  __syncthreads();   // the CTA's own global writes are visible to it
-  for (int q = threadIdx.x; q < pairs; q += blockDim.x) atomicAdd(&hist[p.expert[q]], 1);
+    route_token(logits + (size_t)warp * r.experts, r, scores + (size_t)warp * (2 * r.experts + r.groups), lane, p.expert + warp * r.top, p.weight + warp * r.top,
+                expert + warp * r.top);
+  __syncthreads();
+  for (int q = threadIdx.x; q < pairs; q += blockDim.x) atomicAdd(&hist[expert[q]], 1);
   __syncthreads();
   const int count = (int)threadIdx.x < r.experts ? hist[threadIdx.x] : 0;
   const int first = place_experts(count, r.experts, p, warp_sums);
   if ((int)threadIdx.x < r.experts) hist[threadIdx.x] = first;
   __syncthreads();
-  for (int q = threadIdx.x; q < pairs; q += blockDim.x) p.order[atomicAdd(&hist[p.expert[q]], 1)] = q;
+  for (int q = threadIdx.x; q < pairs; q += blockDim.x) p.order[atomicAdd(&hist[expert[q]], 1)] = q;
 }
 
 constexpr int kRouteWarps = 8;
@@ -190,9 +199,10 @@ extern "C" int nqb200_moe_route(const float* logits, const nqb200_router* r, con
   if (!logits || !plan->expert || !plan->weight || !plan->offsets || !plan->order || !plan->active || !plan->counters) return NQB200_ERR_NULL_POINTER;
   cudaStream_t st = (cudaStream_t)stream;
   const size_t per_warp = (size_t)(2 * r->experts + r->groups) * sizeof(float);
-  if (tokens <= kRouteSmallTokens && tokens * per_warp <= 40 * 1024) {
+  const size_t small = tokens * (per_warp + r->top * sizeof(int));
+  if (tokens <= kRouteSmallTokens && small <= 40 * 1024) {
     const int need = (int)tokens * 32 > r->experts ? (int)tokens * 32 : r->experts, threads = (need + 31) / 32 * 32;
-    return launch_overlapped(moe_route_small_kernel, dim3(1), dim3((unsigned)threads), tokens * per_warp, st, logits, *r, *plan, (int)tokens);
+    return launch_overlapped(moe_route_small_kernel, dim3(1), dim3((unsigned)threads), small, st, logits, *r, *plan, (int)tokens);
   }
   if (cudaMemsetAsync(plan->counters, 0, (size_t)r->experts * sizeof(int32_t), st) != cudaSuccess) { cudaGetLastError(); return NQB200_ERR_LAUNCH; }
   const size_t smem = kRouteWarps * per_warp;
