@@ -186,11 +186,12 @@ def test_graph_and_plain_decoding_agree_in_bf16():
     assert engine(model, num_blocks=60).generate(prompts, 20) == engine(model, num_blocks=60, use_cuda_graph=False).generate(prompts, 20)
 
 
-def test_long_decoding_keeps_to_the_prompt_path():
+@pytest.mark.parametrize("name", ["gla-only", "attention-first"])
+def test_long_decoding_keeps_to_the_prompt_path(name):
     """500 decoded tokens, against the same tokens as one prompt (float32)."""
-    c, model, _ = made("gla-only", torch.float32)
+    c, model, _ = made(name, torch.float32)
     toks = prompt(520, c["vocab"], 8)
-    eng = engine(model, num_blocks=80)
+    eng = engine(model, num_blocks=140)
     a, b = Sequence(0, [], 1), Sequence(1, [], 1)
     whole = feed(eng, a, toks, [520])
     single = feed(eng, b, toks, [20] + [1] * 500)
